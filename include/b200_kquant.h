@@ -54,7 +54,8 @@ enum {
     B200_TYPE_Q8_0 = 8,  /* KV-cache rows only: 32 elements / 34 bytes */
     B200_TYPE_Q4_K = 12, /* 256 elements / 144 bytes */
     B200_TYPE_Q6_K = 14, /* 256 elements / 210 bytes */
-    B200_TYPE_I32 = 26
+    B200_TYPE_I32 = 26,
+    B200_TYPE_BF16 = 30  /* weights of stages created with b200_stage_create_layers */
 };
 
 /* ---- ops understood by graph_compute (the subset on the hot path) -------------------------- */
@@ -320,6 +321,56 @@ typedef struct b200_stage_config {
 } b200_stage_config;
 
 B200_API b200_status b200_stage_create(const b200_stage_config *cfg, b200_stage **out);
+
+/* ---- stages whose layers are described one by one, with bf16 weights ----------------------------
+ * For decoders that are not a repetition of one attention + SwiGLU block (an addition of this library, no
+ * counterpart in the reference): every layer names its mixer and its feed-forward and brings its own sizes;
+ * a contiguous range of layers may run several times in a row with the same weights, each pass with its own
+ * cache and state.  Norms stand before and after every sub-layer: x += norm_b(f(norm(x))), RMS norms of weight
+ * norm_offset + w.  The stage is loaded, run, split by layer range (a looped range stays on one stage), captured
+ * into graphs and freed through the same calls as any other.  Tensor names: "embed", "final.norm", and per layer i
+ * "l<i>.norm1", ".norm1b", ".norm2", ".norm2b", "l<i>.mix.*", "l<i>.mlp.*"; matrices are bf16 [out][in], vectors
+ * f32 (set_tensor also takes them as bf16).
+ * Positions: a sequence slot starts at pos0 = 0, which forgets whatever it held, and continues exactly where its last
+ * call stopped; any other pos0 is refused with B200_ERR_STATE (the recurrent state cannot be rewound).        */
+enum {
+    B200_MIXER_LATENT_ATTN = 1, /* low-rank shared keys / values, one rotated key part, sliding window, output gate */
+    B200_MIXER_LINEAR_REC = 2   /* gated diagonal linear recurrence behind a short convolution, gated by a GELU branch */
+};
+enum { B200_FFN_NONE = 0, B200_FFN_CLAMPED_GLU = 1 };
+enum { B200_PRECISION_BF16 = 0, B200_PRECISION_F32 = 1 };
+typedef struct b200_layer_config {
+    int32_t mixer, ffn;
+    /* B200_MIXER_LATENT_ATTN: per head qk_dim unrotated and rot_dim rotated query / key dimensions (pairs (2i, 2i+1) of
+     * the first rot_dims of them turn by position * rope_base^(-2i / rot_dims)), v_dim values; latent of kv_rank.
+     * A query sees the last `window` positions, itself included (0: all).                        */
+    int32_t n_head, qk_dim, rot_dim, rot_dims, v_dim, kv_rank, window;
+    float rope_base, attn_scale;
+    /* B200_MIXER_LINEAR_REC: rec_width channels in rec_blocks equal blocks, log a = -rec_decay r softplus(lam) */
+    int32_t rec_width, rec_blocks, conv_taps;
+    float rec_decay;
+    /* B200_FFN_CLAMPED_GLU: g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit)   */
+    int32_t n_ff;
+    float glu_limit, glu_alpha;
+} b200_layer_config;
+typedef struct b200_stack_config {
+    int32_t loop_start, loop_stop, loop_times; /* layers [start, stop) run `times` times; times <= 1: no loop   */
+    int32_t precision;  /* BF16: matrix products on tensor cores with bf16 operands; F32: f32 throughout       */
+    float embd_scale;   /* factor on the embedding rows (not on the output head, which is the same matrix)     */
+    float norm_offset;  /* RMS norms multiply by norm_offset + w                                               */
+} b200_stack_config;
+/* cfg: n_layer, layer_begin, layer_end, n_embd, n_vocab, n_ctx, n_seq, n_ubatch, has_embd, has_output, rms_eps and
+ * device are used; layers: n_layer descriptions (of the whole model).                                */
+B200_API b200_status b200_stage_create_layers(const b200_stage_config *cfg, const b200_stack_config *stack,
+                                              const b200_layer_config *layers, b200_stage **out);
+/* Diagnostics: every following forward call also leaves the residual stream after each layer run in buf (device,
+ * f32 [layer runs][rows][n_embd]); NULL switches it off.  b200_stage_layer_runs: how many there are.        */
+B200_API b200_status b200_stage_trace_residual(b200_stage *st, float *buf);
+B200_API int32_t b200_stage_layer_runs(b200_stage *st);
+/* the position a sequence slot continues at; -1: only position 0 is possible                          */
+B200_API int32_t b200_stage_seq_pos(b200_stage *st, int32_t seq);
+/* device bytes of the caches and recurrent states of one sequence slot                                */
+B200_API size_t b200_stage_state_bytes(b200_stage *st);
 B200_API void b200_stage_free(b200_stage *st);
 /* load one tensor by its GGUF name from host memory in GGUF byte layout                        */
 B200_API b200_status b200_stage_set_tensor(b200_stage *st, const char *name, uint32_t type,
@@ -404,6 +455,27 @@ B200_API b200_status b200_gguf_stage_config(const b200_gguf *g, int32_t layer_be
 /* reads every tensor the stage owns, and nothing else, from the file and uploads it               */
 B200_API b200_status b200_stage_load_gguf(b200_stage *st, const b200_gguf *g, int64_t *n_loaded,
                                           int64_t *bytes_read);
+
+/* ---- checkpoint folders: config.json + model.safetensors ------------------------------------------
+ * The second container of this library, for models whose layers are described one by one.  The folder's config.json
+ * names an architecture; the library's table of architectures turns its keys into the descriptions
+ * b200_stage_create_layers takes.  Malformed files are rejected with B200_ERR_INVALID and a message, an unknown
+ * architecture with B200_ERR_UNSUPPORTED.                                                        */
+typedef struct b200_ckpt b200_ckpt;
+B200_API b200_status b200_ckpt_open(const char *dir, b200_ckpt **out);
+B200_API void b200_ckpt_close(b200_ckpt *ck);
+B200_API const char *b200_ckpt_architecture(const b200_ckpt *ck);
+B200_API int64_t b200_ckpt_tensor_count(const b200_ckpt *ck);
+/* name, ggml type id (BF16, F16, F32, I32), shape with ne[0] contiguous, bytes in the file       */
+B200_API b200_status b200_ckpt_tensor_info(const b200_ckpt *ck, int64_t i, b200_gguf_tensor *out);
+B200_API b200_status b200_ckpt_read_tensor(const b200_ckpt *ck, int64_t i, void *dst, size_t nbytes);
+B200_API int32_t b200_ckpt_layer_count(const b200_ckpt *ck);
+/* everything b200_stage_create_layers needs for layers [layer_begin, layer_end) (layer_end < 0: to the last);
+ * layers: room for b200_ckpt_layer_count entries                                                 */
+B200_API b200_status b200_ckpt_stage_config(const b200_ckpt *ck, int32_t layer_begin, int32_t layer_end, int32_t n_ctx,
+                                            int32_t n_seq, int32_t n_ubatch, int32_t device, int32_t precision,
+                                            b200_stage_config *cfg, b200_stack_config *stack, b200_layer_config *layers);
+B200_API b200_status b200_stage_load_ckpt(b200_stage *st, const b200_ckpt *ck, int64_t *n_loaded, int64_t *bytes_read);
 
 /* ---- expert shards of a mixture-of-experts model ----------------------------------------------
  * Which experts a node holds (mesh-llm/src/inference/moe.rs:535-636: mode 0 = shared core of the

@@ -43,7 +43,8 @@ def _deps_mtime() -> float:
     return max(os.path.getmtime(f) for f in files)
 
 
-def build(force: bool = False, verbose: bool = False) -> str:
+def build(force: bool = False, verbose: bool = False, library_only: bool = False) -> str:
+    """library_only: skip the worker executable"""
     if not force and os.path.exists(SO) and os.path.getmtime(SO) >= _deps_mtime():
         return SO
     nvcc = _nvcc()
@@ -66,7 +67,7 @@ def build(force: bool = False, verbose: bool = False) -> str:
         return obj
 
     with ThreadPoolExecutor(max_workers=8) as ex:
-        objs = list(ex.map(compile_one, sources()))
+        objs = list(ex.map(compile_one, [f for f in sources() if not (library_only and os.path.basename(f) in MAIN_SOURCES)]))
     mains = [o for o in objs if os.path.basename(o)[:-2] in MAIN_SOURCES]
     objs = [o for o in objs if o not in mains]
     cmd = [nvcc, "-shared", "-o", SO, *objs, "-gencode", "arch=compute_100a,code=sm_100a",
@@ -75,6 +76,8 @@ def build(force: bool = False, verbose: bool = False) -> str:
     if r.returncode != 0:
         sys.stderr.write(r.stdout + r.stderr)
         raise RuntimeError("link failed")
+    if library_only:
+        return SO
     # the worker executable carries the library's objects, so it runs without a library path
     cmd = [nvcc, "-o", RPC_EXE, *mains, *objs, "-gencode", "arch=compute_100a,code=sm_100a",
            "-ccbin", "/usr/bin/g++", "-cudart", "static", "-lpthread"]

@@ -11,7 +11,7 @@ import os
 _HERE = os.path.dirname(os.path.abspath(__file__))
 SO_PATH = os.environ.get("B200_KQ_LIB") or os.path.join(_HERE, "libb200kq.so")
 
-TYPE_F32, TYPE_F16, TYPE_Q4_0, TYPE_Q8_0, TYPE_Q4_K, TYPE_Q6_K, TYPE_I32 = 0, 1, 2, 8, 12, 14, 26
+TYPE_F32, TYPE_F16, TYPE_Q4_0, TYPE_Q8_0, TYPE_Q4_K, TYPE_Q6_K, TYPE_I32, TYPE_BF16 = 0, 1, 2, 8, 12, 14, 26, 30
 
 OK = 0
 STATUS_NAMES = {0: "OK", -1: "INVALID", -2: "ALLOC", -3: "CUDA", -4: "UNSUPPORTED", -5: "BOUNDS",
@@ -48,6 +48,29 @@ class StageConfig(C.Structure):
         ("rms_eps", C.c_float), ("rope_theta", C.c_float),
         ("n_ubatch", C.c_int32), ("device", C.c_int32),
         ("kv_type_k", C.c_int32), ("kv_type_v", C.c_int32),
+    ]
+
+
+MIXER_LATENT_ATTN, MIXER_LINEAR_REC = 1, 2
+FFN_NONE, FFN_CLAMPED_GLU = 0, 1
+PRECISION_BF16, PRECISION_F32 = 0, 1
+
+
+class LayerConfig(C.Structure):
+    _fields_ = [
+        ("mixer", C.c_int32), ("ffn", C.c_int32),
+        ("n_head", C.c_int32), ("qk_dim", C.c_int32), ("rot_dim", C.c_int32), ("rot_dims", C.c_int32),
+        ("v_dim", C.c_int32), ("kv_rank", C.c_int32), ("window", C.c_int32),
+        ("rope_base", C.c_float), ("attn_scale", C.c_float),
+        ("rec_width", C.c_int32), ("rec_blocks", C.c_int32), ("conv_taps", C.c_int32), ("rec_decay", C.c_float),
+        ("n_ff", C.c_int32), ("glu_limit", C.c_float), ("glu_alpha", C.c_float),
+    ]
+
+
+class StackConfig(C.Structure):
+    _fields_ = [
+        ("loop_start", C.c_int32), ("loop_stop", C.c_int32), ("loop_times", C.c_int32),
+        ("precision", C.c_int32), ("embd_scale", C.c_float), ("norm_offset", C.c_float),
     ]
 
 
@@ -167,6 +190,22 @@ SIGNATURES = {
     "b200_gguf_byte_profile": (i32, [vp, C.POINTER(GgufByteProfile)]),
     "b200_gguf_stage_config": (i32, [vp, i32, i32, i32, i32, i32, i32, C.POINTER(StageConfig)]),
     "b200_stage_load_gguf": (i32, [vp, vp, C.POINTER(i64), C.POINTER(i64)]),
+    "b200_stage_create_layers": (i32, [C.POINTER(StageConfig), C.POINTER(StackConfig), C.POINTER(LayerConfig),
+                                       C.POINTER(vp)]),
+    "b200_stage_trace_residual": (i32, [vp, vp]),
+    "b200_stage_layer_runs": (i32, [vp]),
+    "b200_stage_seq_pos": (i32, [vp, i32]),
+    "b200_stage_state_bytes": (sz, [vp]),
+    "b200_ckpt_open": (i32, [C.c_char_p, C.POINTER(vp)]),
+    "b200_ckpt_close": (None, [vp]),
+    "b200_ckpt_architecture": (C.c_char_p, [vp]),
+    "b200_ckpt_tensor_count": (i64, [vp]),
+    "b200_ckpt_tensor_info": (i32, [vp, i64, C.POINTER(GgufTensor)]),
+    "b200_ckpt_read_tensor": (i32, [vp, i64, vp, sz]),
+    "b200_ckpt_layer_count": (i32, [vp]),
+    "b200_ckpt_stage_config": (i32, [vp, i32, i32, i32, i32, i32, i32, i32, C.POINTER(StageConfig),
+                                     C.POINTER(StackConfig), C.POINTER(LayerConfig)]),
+    "b200_stage_load_ckpt": (i32, [vp, vp, C.POINTER(i64), C.POINTER(i64)]),
     "b200_rpc_server_start": (i32, [C.c_char_p, i32, C.c_char_p, C.POINTER(vp)]),
     "b200_rpc_server_port": (i32, [vp]),
     "b200_rpc_server_stop": (None, [vp]),

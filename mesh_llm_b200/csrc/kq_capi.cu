@@ -34,6 +34,12 @@ int kq_sm_count() {
     return n[dev];
 }
 
+// one code per bounded wait that gave up since the last call, 0 when none did
+int kq_device_wait_errors() {
+    return kq_stream_error_fetch() | (kq_gemm_error_fetch() << 4) | (kq_attn_tc_error_fetch() << 8) | (kq_gemm_bf16_error_fetch() << 12) |
+           (kq_latent_tc_error_fetch() << 16);
+}
+
 extern "C" {
 
 const char *b200_last_error(void) { return t_err; }
@@ -54,7 +60,7 @@ const char *b200_status_string(b200_status s) {
 
 b200_status b200_check_device_waits(void) {
     KQ_CUDA(cudaDeviceSynchronize());
-    const int werr = kq_stream_error_fetch() | (kq_gemm_error_fetch() << 4) | (kq_attn_tc_error_fetch() << 8);
+    const int werr = kq_device_wait_errors();
     if (werr) {
         kq_set_error("a bounded device-side wait gave up (code 0x%x)", werr);
         return B200_ERR_TIMEOUT;

@@ -68,7 +68,8 @@ int kq_sm_count();
 static inline __host__ __device__ int64_t kq_row_bytes(uint32_t type, int64_t k) {
     switch (type) {
     case B200_TYPE_F32: return k * 4;
-    case B200_TYPE_F16: return k * 2;
+    case B200_TYPE_F16:
+    case B200_TYPE_BF16: return k * 2;
     case B200_TYPE_Q4_K: return k / KQ_QK * KQ_Q4K_BYTES;
     case B200_TYPE_Q6_K: return k / KQ_QK * KQ_Q6K_BYTES;
     case B200_TYPE_Q4_0: return k / 32 * 18; // ggml block_q4_0: f16 d, 16 bytes of nibbles
@@ -89,6 +90,7 @@ static inline __host__ __device__ int64_t kq_q6_group_bytes(int g) {
     return g == KQ_Q6_GROUP ? KQ_Q6_GROUP_BYTES : (g ? (int64_t)g * 208 + 16 : 0);
 }
 static inline __host__ __device__ int64_t kq_device_row_bytes(uint32_t type, int64_t k) {
+    if (type == B200_TYPE_BF16) return (k + 63) / 64 * 128; // zero-padded to 64 elements
     if (type == B200_TYPE_Q6_K) {
         const int64_t nb = k / KQ_QK;
         return nb / KQ_Q6_GROUP * KQ_Q6_GROUP_BYTES + kq_q6_group_bytes((int)(nb % KQ_Q6_GROUP));
@@ -308,6 +310,9 @@ b200_status kq_launch_gemm_grouped(uint32_t type, const uint8_t *W, int64_t expe
 int kq_stream_error_fetch(); // 0 ok; nonzero = a bounded device-side wait gave up since the last call
 int kq_gemm_error_fetch();
 int kq_attn_tc_error_fetch();
+int kq_gemm_bf16_error_fetch();
+int kq_latent_tc_error_fetch();
+int kq_device_wait_errors(); // all of the above in one code
 b200_status kq_launch_gemm(uint32_t type, const uint8_t *W, const int8_t *q, const float *d,
                            const int16_t *bs, int64_t M, int64_t N, int64_t K, float *y,
                            const float *bias, const float *residual, cudaStream_t st);

@@ -1,0 +1,381 @@
+// Prefill products with bf16 weights, y[m][n] = sum_k W[n][k] x[m][k]: the tensor-core form (tcgen05.mma
+// kind::f16 on bf16 operands, f32 accumulators in TMEM) and the f32 form on CUDA cores of the 32-bit mode.
+//
+// Tensor cores: one CTA computes 128 tokens (TMEM lanes) x 128 weight rows (columns), two CTAs per SM.  K runs
+// in slices of 64 (one 128-byte-swizzled row per operand row); a producer thread brings the slices in by tiled
+// TMA copies through a ring of three stages, one thread issues the MMAs, four warps drain the accumulator.
+// A gate / up pair puts 64 rows of either matrix into a tile, so that the GLU happens where both values are.
+// An f32 operand can come as several bf16 parts (x = hi + mid + lo exactly): the K loop then passes over the
+// same weights once per part.  Block-diagonal products offset the K coordinate of x and the row of W by group.
+// Every wait is bounded; on a time-out the kernel records an error, lets its copies land, frees its TMEM and
+// returns.
+#include "kq_dense.cuh"
+
+#include <cuda.h>
+#include <string.h>
+
+#include <algorithm>
+
+b200_status kq_tmap_encode(void *map128, int elem_bytes, int rank, const void *base, const uint64_t *dims,
+                           const uint64_t *strides_bytes, const uint32_t *box, int swizzle128);
+
+namespace {
+
+constexpr int TM = 128, TN = 128, BK = 64, STAGES = 3;
+constexpr int A_BYTES = TM * BK * 2, B_BYTES = TN * BK * 2, STAGE_BYTES = A_BYTES + B_BYTES;
+constexpr int SMEM_TOTAL = STAGES * STAGE_BYTES + 1024;
+constexpr int NTHREADS = 192; // producer warp, MMA warp, four epilogue warps
+constexpr uint32_t TMEM_COLS = 128;
+constexpr uint64_t LIMIT = 5 * KQ_WAIT_LIMIT_NS;
+
+__device__ int g_gemm_bf16_error;
+
+__device__ __forceinline__ uint32_t smem_u32(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
+
+// K-major operand, rows of 128 bytes under the 128-byte swizzle, 8-row groups 1024 bytes apart; K step s of 16
+__device__ __forceinline__ uint64_t desc_k(uint32_t tile, int s) {
+    uint64_t d = 0;
+    d |= (uint64_t)(((tile + s * 32) & 0x3FFFF) >> 4);
+    d |= (uint64_t)(16 >> 4) << 16;
+    d |= (uint64_t)(1024 >> 4) << 32;
+    d |= (uint64_t)1 << 46; // descriptor version of this architecture
+    d |= (uint64_t)2 << 61; // SWIZZLE_128B
+    return d;
+}
+// kind::f16: D f32, A bf16, B bf16, both K-major, M = 128, N = 128
+constexpr uint32_t IDESC = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(TN >> 3) << 17) | ((uint32_t)(TM >> 4) << 24);
+
+__device__ __forceinline__ void mma(uint32_t d_tmem, uint64_t a, uint64_t b, uint32_t acc) {
+    asm volatile("{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
+                 "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+                 :
+                 : "r"(d_tmem), "l"(a), "l"(b), "r"(IDESC), "r"(acc)
+                 : "memory");
+}
+__device__ __forceinline__ void commit(uint32_t bar) {
+    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
+}
+
+#define TMEM_LD32(taddr, r)                                                                                             \
+    asm volatile("tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,"        \
+                 "%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"                              \
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]),      \
+                   "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), \
+                   "=r"(r[16]), "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]),            \
+                   "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]),            \
+                   "=r"(r[30]), "=r"(r[31])                                                                             \
+                 : "r"(taddr)                                                                                           \
+                 : "memory")
+
+struct GemmParams {
+    CUtensorMap a, b[3];
+    KqDense c;
+    int32_t nk, parts;      // 64-element K slices per part
+    int32_t tile_end[3];    // cumulative N tiles of the segments
+};
+
+// eight consecutive output columns of one row
+__device__ __forceinline__ void put8(const KqDense &c, const KqDenseSeg &s, int64_t m, int64_t n, int g, const float *v, int n_valid) {
+    if (n_valid == 8 && s.head_in == 0 && (s.ldy & 7) == 0 && (n & 7) == 0) {
+        float o[8];
+#pragma unroll
+        for (int j = 0; j < 8; j++) {
+            float t = v[j];
+            if (s.bias) t += s.bias[n + j];
+            if (s.act == KQ_ACT_GELU_TANH) t = kq_gelu_tanh(t);
+            if (c.head_gate) t *= kq_sigmoid(c.head_gate[m * c.ld_gate + g]);
+            o[j] = t;
+        }
+        const int64_t i = m * s.ldy + n;
+        if (s.out == KQ_OUT_F32) {
+            float *y = (float *)s.y + i;
+            *reinterpret_cast<float4 *>(y) = make_float4(o[0], o[1], o[2], o[3]);
+            *reinterpret_cast<float4 *>(y + 4) = make_float4(o[4], o[5], o[6], o[7]);
+        } else {
+            uint32_t w[4];
+#pragma unroll
+            for (int j = 0; j < 4; j++)
+                w[j] = s.out == KQ_OUT_BF16 ? (uint32_t)kq_f2bf(o[2 * j]) | ((uint32_t)kq_f2bf(o[2 * j + 1]) << 16)
+                                            : (uint32_t)kq_f2h_sat(o[2 * j]) | ((uint32_t)kq_f2h_sat(o[2 * j + 1]) << 16);
+            *reinterpret_cast<uint4 *>((uint16_t *)s.y + i) = make_uint4(w[0], w[1], w[2], w[3]);
+        }
+        return;
+    }
+#pragma unroll
+    for (int j = 0; j < 8; j++)
+        if (j < n_valid) kq_dense_store(c, s, m, n + j, g, v[j]);
+}
+
+// grid (token tiles, weight-row tiles of all segments, groups)
+__global__ void __launch_bounds__(NTHREADS, 2) gemm_bf16_kernel(const __grid_constant__ GemmParams p) {
+    extern __shared__ uint8_t sm_raw[];
+    __shared__ uint64_t full[STAGES], empty[STAGES], done;
+    __shared__ uint32_t s_tmem;
+    __shared__ int s_abort;
+    KQ_PDL_TRIGGER();
+    uint8_t *sm = (uint8_t *)(((uintptr_t)sm_raw + 1023) & ~(uintptr_t)1023);
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int m0 = blockIdx.x * TM, g = blockIdx.z;
+    int seg = 0, nt = blockIdx.y;
+    if (!p.c.glu) {
+        while (seg + 1 < p.c.nseg && nt >= p.tile_end[seg]) seg++;
+        if (seg) nt -= p.tile_end[seg - 1];
+    }
+    const int n_rows = p.c.seg[seg].n_rows, n0 = nt * (p.c.glu ? TN / 2 : TN); // first row of the tile inside the group
+    if (warp == 1) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&s_tmem)), "r"(TMEM_COLS)
+                     : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    if (tid == 0) {
+        for (int i = 0; i < STAGES; i++) {
+            asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(&full[i])), "r"(1));
+            asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(&empty[i])), "r"(1));
+        }
+        asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(&done)), "r"(1));
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        s_abort = 0;
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+    const uint32_t tmem = s_tmem;
+    const int n_it = p.nk * p.parts;
+    KQ_PDL_WAIT();
+
+    auto wait = [&](uint64_t *bar, uint32_t parity, int code) {
+        if (!*(volatile int *)&s_abort && !kq_mbar_wait(smem_u32(bar), parity, LIMIT)) {
+            *(volatile int *)&s_abort = 1;
+            atomicExch(&g_gemm_bf16_error, code);
+        }
+        return !*(volatile int *)&s_abort;
+    };
+    if (warp == 0) {
+        if (lane == 0) {
+            int posted = 0;
+            for (int it = 0; it < n_it; it++) {
+                const int s = it % STAGES;
+                if (it >= STAGES && !wait(&empty[s], (uint32_t)((it / STAGES - 1) & 1), 1)) break;
+                const uint32_t bar = smem_u32(&full[s]), dst = smem_u32(sm + s * STAGE_BYTES);
+                asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(STAGE_BYTES) : "memory");
+                const int part = it / p.nk, kk = (it % p.nk) * BK;
+                asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];" ::"r"(dst),
+                             "l"(&p.a), "r"((int)(g * p.c.xg) + kk), "r"(m0), "r"(part), "r"(bar)
+                             : "memory");
+#pragma unroll
+                for (int hb = 0; hb < 2; hb++) { // 64 weight rows each: two halves of one matrix, or gate and up
+                    const CUtensorMap *map = p.c.glu ? &p.b[hb] : &p.b[seg];
+                    const int row = g * n_rows + n0 + (p.c.glu ? 0 : hb * 64);
+                    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(
+                                     dst + A_BYTES + hb * (B_BYTES / 2)),
+                                 "l"(map), "r"(kk), "r"(row), "r"(bar)
+                                 : "memory");
+                }
+                posted = it + 1;
+            }
+            if (*(volatile int *)&s_abort) // copies that were posted must land before the CTA goes away
+                for (int it = std::max(0, posted - STAGES); it < posted; it++)
+                    kq_mbar_wait(smem_u32(&full[it % STAGES]), (uint32_t)((it / STAGES) & 1), KQ_WAIT_LIMIT_NS);
+        }
+        __syncwarp();
+    } else if (warp == 1) {
+        if (lane == 0) {
+            for (int it = 0; it < n_it; it++) {
+                const int s = it % STAGES;
+                if (!wait(&full[s], (uint32_t)((it / STAGES) & 1), 2)) break;
+                asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                const uint32_t a = smem_u32(sm + s * STAGE_BYTES), b = a + A_BYTES;
+#pragma unroll
+                for (int k = 0; k < BK / 16; k++) mma(tmem, desc_k(a, k), desc_k(b, k), (it > 0 || k > 0) ? 1u : 0u);
+                commit(smem_u32(&empty[s]));
+            }
+            commit(smem_u32(&done));
+            if (*(volatile int *)&s_abort) kq_mbar_wait(smem_u32(&done), 0, KQ_WAIT_LIMIT_NS); // MMAs in flight end before TMEM is freed
+        }
+        __syncwarp();
+    } else {
+        const bool ok = wait(&done, 0, 3);
+        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+        if (__all_sync(0xffffffffu, ok)) {
+            const int q = warp & 3, row = m0 + q * 32 + lane; // a warp reaches the TMEM lanes of its quarter
+            const uint32_t tl = tmem + ((uint32_t)(q * 32) << 16);
+            const KqDenseSeg &s = p.c.seg[seg];
+            const bool row_ok = row < p.c.M;
+            if (p.c.glu) {
+#pragma unroll 1
+                for (int c = 0; c < 2; c++) {
+                    uint32_t a[32], b[32];
+                    TMEM_LD32(tl + 32 * c, a);
+                    TMEM_LD32(tl + 64 + 32 * c, b);
+                    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+                    if (row_ok) {
+#pragma unroll
+                        for (int j = 0; j < 32; j += 8) {
+                            const int n = n0 + 32 * c + j;
+                            float v[8];
+#pragma unroll
+                            for (int e = 0; e < 8; e++)
+                                v[e] = n + e < n_rows ? kq_clamped_glu(__uint_as_float(a[j + e]), __uint_as_float(b[j + e]),
+                                                                       p.c.glu_limit, p.c.glu_alpha)
+                                                      : 0.f;
+                            const int lim = std::max(n_rows, s.pad_cols); // the padding of a staging row is written too
+                            if (n < lim) put8(p.c, s, row, n, 0, v, std::min(8, lim - n));
+                        }
+                    }
+                }
+            } else {
+#pragma unroll 1
+                for (int c = 0; c < TN / 32; c++) {
+                    uint32_t a[32];
+                    TMEM_LD32(tl + 32 * c, a);
+                    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+                    if (row_ok) {
+#pragma unroll
+                        for (int j = 0; j < 32; j += 8) {
+                            const int n = n0 + 32 * c + j;
+                            if (n < n_rows) {
+                                float v[8];
+#pragma unroll
+                                for (int e = 0; e < 8; e++) v[e] = __uint_as_float(a[j + e]);
+                                put8(p.c, s, row, (int64_t)g * n_rows + n, g, v, std::min(8, n_rows - n));
+                            }
+                        }
+                    }
+                }
+            }
+        }
+    }
+    asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+    __syncthreads();
+    if (warp == 1) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(TMEM_COLS) : "memory");
+}
+
+// ---- f32 form ------------------------------------------------------------------------------------
+constexpr int FT = 64, FK = 16;
+struct F32Params {
+    KqDense c;
+    const float *x;
+    int64_t ldx;
+    int32_t tile_end[3];
+};
+
+template <bool GLU>
+__global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ F32Params p) {
+    KQ_PDL_ENTER();
+    __shared__ float sa[FK][FT + 4], sb[GLU ? 2 : 1][FK][FT + 4];
+    const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4, g = blockIdx.z;
+    int seg = 0, nt = blockIdx.y;
+    if (!GLU) {
+        while (seg + 1 < p.c.nseg && nt >= p.tile_end[seg]) seg++;
+        if (seg) nt -= p.tile_end[seg - 1];
+    }
+    const KqDenseSeg &s = p.c.seg[seg];
+    const int m0 = blockIdx.x * FT, n0 = nt * FT, n_rows = s.n_rows, K = p.c.K;
+    float acc[GLU ? 2 : 1][4][4] = {};
+    for (int k0 = 0; k0 < K; k0 += FK) {
+        for (int i = tid; i < FT * FK; i += 256) {
+            const int r = i / FK, k = i % FK;
+            sa[k][r] = m0 + r < p.c.M && k0 + k < K ? p.x[(m0 + r) * p.ldx + g * p.c.xg + k0 + k] : 0.f;
+#pragma unroll
+            for (int h = 0; h < (GLU ? 2 : 1); h++)
+                sb[h][k][r] = n0 + r < n_rows && k0 + k < K
+                                  ? kq_bf2f(p.c.seg[GLU ? h : seg].W[((int64_t)g * n_rows + n0 + r) * p.c.ldw + k0 + k])
+                                  : 0.f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < FK; k++) {
+            const float4 a = *reinterpret_cast<const float4 *>(&sa[k][ty * 4]);
+            const float av[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+            for (int h = 0; h < (GLU ? 2 : 1); h++) {
+                const float4 b = *reinterpret_cast<const float4 *>(&sb[h][k][tx * 4]);
+                const float bv[4] = {b.x, b.y, b.z, b.w};
+#pragma unroll
+                for (int i = 0; i < 4; i++)
+#pragma unroll
+                    for (int j = 0; j < 4; j++) acc[h][i][j] = fmaf(av[i], bv[j], acc[h][i][j]);
+            }
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; i++)
+#pragma unroll
+        for (int j = 0; j < 4; j++) {
+            const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
+            if (m >= p.c.M || n >= n_rows) continue;
+            if (GLU) kq_dense_put(s, m, n, kq_clamped_glu(acc[0][i][j], acc[GLU ? 1 : 0][i][j], p.c.glu_limit, p.c.glu_alpha));
+            else kq_dense_store(p.c, s, m, (int64_t)g * n_rows + n, g, acc[0][i][j]);
+        }
+}
+
+} // namespace
+
+int kq_gemm_bf16_error_fetch() {
+    int v = 0, zero = 0;
+    if (cudaMemcpyFromSymbol(&v, g_gemm_bf16_error, sizeof(int)) != cudaSuccess) return -1;
+    if (v) cudaMemcpyToSymbol(g_gemm_bf16_error, &zero, sizeof(int));
+    return v;
+}
+
+b200_status kq_gemm_bf16(const KqDense &c, const uint16_t *a, int64_t lda, int parts, cudaStream_t st) {
+    KQ_REQUIRE(c.M >= 1 && c.nseg >= 1 && c.nseg <= 3 && c.groups >= 1 && c.K >= 1 && parts >= 1, "gemm_bf16: bad call");
+    KQ_REQUIRE(c.ldw % 64 == 0 && c.ldw >= c.K && lda % 64 == 0 && (c.groups == 1 || c.xg % 64 == 0),
+               "gemm_bf16: rows must be padded to 64 elements");
+    KQ_REQUIRE(!c.glu || (c.nseg == 2 && c.groups == 1 && c.seg[0].n_rows == c.seg[1].n_rows), "gemm_bf16: a GLU has two equal segments");
+    GemmParams p;
+    p.c = c;
+    p.parts = parts;
+    p.nk = (int)kq_div_up(c.K, BK);
+    {
+        const uint64_t dims[3] = {(uint64_t)lda, (uint64_t)c.M, (uint64_t)parts};
+        const uint64_t str[2] = {(uint64_t)lda * 2, (uint64_t)lda * 2 * c.M};
+        const uint32_t box[3] = {BK, TM, 1};
+        const b200_status rc = kq_tmap_encode(&p.a, 2, 3, a, dims, str, box, 1);
+        if (rc != B200_OK) return rc;
+    }
+    int tiles = 0;
+    for (int i = 0; i < 3; i++) {
+        const KqDenseSeg &s = c.seg[std::min(i, c.nseg - 1)];
+        const uint64_t dims[2] = {(uint64_t)c.ldw, (uint64_t)s.n_rows * c.groups}, str[1] = {(uint64_t)c.ldw * 2};
+        const uint32_t box[2] = {BK, 64};
+        const b200_status rc = kq_tmap_encode(&p.b[i], 2, 2, s.W, dims, str, box, 1);
+        if (rc != B200_OK) return rc;
+        if (i < c.nseg) tiles += (int)kq_div_up(s.n_rows, TN);
+        p.tile_end[i] = tiles;
+    }
+    if (c.glu) tiles = (int)kq_div_up(std::max(c.seg[0].n_rows, c.seg[0].pad_cols), TN / 2);
+    static bool attr[16];
+    int dev = 0;
+    KQ_CUDA(cudaGetDevice(&dev));
+    if (dev < 0 || dev >= 16 || !attr[dev]) {
+        KQ_CUDA(cudaFuncSetAttribute(gemm_bf16_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL));
+        if (dev >= 0 && dev < 16) attr[dev] = true;
+    }
+    const dim3 grid((unsigned)kq_div_up(c.M, TM), (unsigned)tiles, (unsigned)c.groups);
+    kq_launch(gemm_bf16_kernel, grid, NTHREADS, SMEM_TOTAL, st, p);
+    KQ_COUNT_LAUNCH();
+    KQ_LAUNCH_CHECK();
+    return B200_OK;
+}
+
+b200_status kq_gemm_f32(const KqDense &c, const float *x, int64_t ldx, cudaStream_t st) {
+    KQ_REQUIRE(c.M >= 1 && c.nseg >= 1 && c.nseg <= 3 && c.groups >= 1 && c.K >= 1, "gemm_f32: bad call");
+    F32Params p;
+    p.c = c;
+    p.x = x;
+    p.ldx = ldx;
+    int tiles = 0;
+    for (int i = 0; i < 3; i++) {
+        if (i < c.nseg) tiles += (int)kq_div_up(c.seg[i].n_rows, FT);
+        p.tile_end[i] = tiles;
+    }
+    if (c.glu) tiles = (int)kq_div_up(c.seg[0].n_rows, FT);
+    const dim3 grid((unsigned)kq_div_up(c.M, FT), (unsigned)tiles, (unsigned)c.groups);
+    if (c.glu) kq_launch(gemm_f32_kernel<true>, grid, 256, 0, st, p);
+    else kq_launch(gemm_f32_kernel<false>, grid, 256, 0, st, p);
+    KQ_COUNT_LAUNCH();
+    KQ_LAUNCH_CHECK();
+    return B200_OK;
+}

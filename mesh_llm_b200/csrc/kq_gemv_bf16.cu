@@ -1,0 +1,391 @@
+// Matrix-vector products for 1..8 rows of f32 activations and bf16 weights: the decode projections of a 16-bit
+// model.  The products are f32 throughout (a bf16 weight is exact in f32), so the same kernels serve the 32-bit
+// mode.
+//
+// Every CTA owns an equal share of the output rows (to within one row) and all its warps split K: a thread
+// reads the 16-byte chunks tid, tid + 256, ... of four rows at a time straight from global memory, the activations
+// sit in shared memory as two planes of float4 (elements 0..3 and 4..7 of each chunk), so that a warp's reads are
+// free of bank conflicts.  The four rows' partial sums are reduced across the warp in six shuffles, the eight
+// warps' through shared memory once per 64 rows.  The prologue can add a normed sub-layer output to the
+// residual and norm the result (every CTA does that for itself; CTA 0 also leaves the new residual), the
+// first weights are requested before the dependency wait.
+#include "kq_dense.cuh"
+
+#include <algorithm>
+#include <stdlib.h>
+
+namespace {
+
+constexpr int NT = 256, NW = NT / 32, SB = 64; // threads, warps, rows between two combines
+
+struct GemvParams {
+    KqDense c;
+    KqNormPrep p;
+    int32_t V;   // rows in all (a gate / up pair is two), in the order they are walked
+    int32_t nck; // 16-byte chunks per weight row
+};
+
+__device__ __forceinline__ float4 load4(const float *p, int k, int K, bool vec) {
+    if (vec && k + 3 < K) return *reinterpret_cast<const float4 *>(p + k);
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (k < K) v.x = p[k];
+    if (k + 1 < K) v.y = p[k + 1];
+    if (k + 2 < K) v.z = p[k + 2];
+    if (k + 3 < K) v.w = p[k + 3];
+    return v;
+}
+
+__device__ __forceinline__ float block_sum(float v, float *red) {
+    v = kq_warp_sum(v);
+    __syncthreads();
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float t = 0.f;
+#pragma unroll
+    for (int i = 0; i < NW; i++) t += red[i];
+    return t;
+}
+
+// walked row v -> (segment, row); gate / up rows alternate
+__device__ __forceinline__ void locate(const GemvParams &p, int v, int &seg, int &row) {
+    if (p.c.glu) {
+        seg = v & 1;
+        row = v >> 1;
+        return;
+    }
+    seg = 0;
+    row = v;
+    while (seg + 1 < p.c.nseg && row >= p.c.seg[seg].n_rows) row -= p.c.seg[seg++].n_rows;
+}
+
+template <int M>
+__global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __grid_constant__ GemvParams p) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float part[2][NW][SB][M];
+    __shared__ float red[NW];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int nck = p.nck, K = p.c.K, step = p.c.glu ? 2 : 1;
+    const int64_t units = p.V / step;
+    const int v0 = (int)(units * blockIdx.x / gridDim.x) * step, v1 = (int)(units * (blockIdx.x + 1) / gridDim.x) * step;
+    KQ_PDL_TRIGGER();
+
+    auto row_ptr = [&](int v) {
+        int s, r;
+        locate(p, min(v, p.V - 1), s, r);
+        return reinterpret_cast<const uint4 *>(p.c.seg[s].W + (int64_t)r * p.c.ldw);
+    };
+    // first weights of this CTA: they depend on nothing
+    uint4 w[4][2];
+    const uint4 *wp[4];
+    auto load = [&](int i) {
+#pragma unroll
+        for (int r = 0; r < 4; r++)
+#pragma unroll
+            for (int j = 0; j < 2; j++) {
+                const int c = i + j * NT;
+                w[r][j] = c < nck ? kq_ld_stream(wp[r] + c) : make_uint4(0, 0, 0, 0);
+            }
+    };
+    if (v0 < v1) {
+#pragma unroll
+        for (int r = 0; r < 4; r++) wp[r] = row_ptr(v0 + r);
+        load(tid);
+    }
+    KQ_PDL_WAIT();
+
+    // ---- activations
+    float4 *pl = reinterpret_cast<float4 *>(sm); // [M][2][nck]
+    const bool vec = (p.p.ldx & 3) == 0 && (p.p.ld_sub & 3) == 0 && (p.p.ld_out & 3) == 0 &&
+                     (((uintptr_t)p.p.x | (uintptr_t)p.p.sub | (uintptr_t)p.p.x_out) & 15) == 0;
+    const int n4 = nck * 2;
+#pragma unroll 1
+    for (int m = 0; m < M; m++) {
+        float4 *px = pl + (int64_t)m * 2 * nck;
+        const float *x = p.p.x + m * p.p.ldx;
+        float ss = 0.f;
+        if (p.p.sub) {
+            const float *sub = p.p.sub + m * p.p.ld_sub;
+            float sc = 1.f;
+            if (p.p.sub_w) {
+                float s2 = 0.f;
+                for (int i = tid; i < n4; i += NT) {
+                    const float4 v = load4(sub, 4 * i, K, vec);
+                    s2 += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+                }
+                sc = 1.0f / sqrtf(block_sum(s2, red) / (float)K + p.p.eps);
+            }
+            for (int i = tid; i < n4; i += NT) {
+                const float4 a = load4(x, 4 * i, K, vec), b = load4(sub, 4 * i, K, vec);
+                float4 g = make_float4(1.f, 1.f, 1.f, 1.f);
+                if (p.p.sub_w) {
+                    g = load4(p.p.sub_w, 4 * i, K, true);
+                    g.x += p.p.w_off, g.y += p.p.w_off, g.z += p.p.w_off, g.w += p.p.w_off;
+                }
+                float4 v = make_float4(a.x + b.x * sc * g.x, a.y + b.y * sc * g.y, a.z + b.z * sc * g.z, a.w + b.w * sc * g.w);
+                ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+                px[(i & 1) * nck + (i >> 1)] = v;
+                if (p.p.x_out && blockIdx.x == 0) {
+                    float *o = p.p.x_out + m * p.p.ld_out + 4 * i;
+                    if (vec && 4 * i + 3 < K) *reinterpret_cast<float4 *>(o) = v;
+                    else {
+                        if (4 * i < K) o[0] = v.x;
+                        if (4 * i + 1 < K) o[1] = v.y;
+                        if (4 * i + 2 < K) o[2] = v.z;
+                        if (4 * i + 3 < K) o[3] = v.w;
+                    }
+                }
+            }
+        } else {
+            for (int i = tid; i < n4; i += NT) {
+                const float4 v = load4(x, 4 * i, K, vec);
+                ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+                px[(i & 1) * nck + (i >> 1)] = v;
+            }
+        }
+        if (p.p.norm_w) {
+            const float sc = 1.0f / sqrtf(block_sum(ss, red) / (float)K + p.p.eps);
+            for (int i = tid; i < n4; i += NT) {
+                const float4 g = load4(p.p.norm_w, 4 * i, K, true);
+                float4 v = px[(i & 1) * nck + (i >> 1)];
+                v.x *= sc * (p.p.w_off + g.x), v.y *= sc * (p.p.w_off + g.y);
+                v.z *= sc * (p.p.w_off + g.z), v.w *= sc * (p.p.w_off + g.w);
+                px[(i & 1) * nck + (i >> 1)] = v;
+            }
+        }
+    }
+    __syncthreads();
+
+    // ---- rows
+    int buf = 0;
+    bool loaded = true;
+    for (int vb = v0; vb < v1; vb += SB, buf ^= 1) {
+        const int ve = min(v1, vb + SB);
+        for (int v = vb; v < ve; v += 4) {
+            if (!loaded) {
+#pragma unroll
+                for (int r = 0; r < 4; r++) wp[r] = row_ptr(v + r);
+            }
+            float acc[4][M];
+#pragma unroll
+            for (int r = 0; r < 4; r++)
+#pragma unroll
+                for (int m = 0; m < M; m++) acc[r][m] = 0.f;
+            for (int i = tid; i < nck; i += 2 * NT) {
+                if (!loaded) load(i);
+                loaded = false;
+#pragma unroll
+                for (int j = 0; j < 2; j++) {
+                    const int c = i + j * NT;
+                    if (c < nck) {
+#pragma unroll
+                        for (int m = 0; m < M; m++) {
+                            const float4 a = pl[(m * 2) * nck + c], b = pl[(m * 2 + 1) * nck + c];
+#pragma unroll
+                            for (int r = 0; r < 4; r++) {
+                                const uint4 q = w[r][j];
+                                float s = acc[r][m];
+                                s = fmaf(__uint_as_float(q.x << 16), a.x, s);
+                                s = fmaf(__uint_as_float(q.x & 0xffff0000u), a.y, s);
+                                s = fmaf(__uint_as_float(q.y << 16), a.z, s);
+                                s = fmaf(__uint_as_float(q.y & 0xffff0000u), a.w, s);
+                                s = fmaf(__uint_as_float(q.z << 16), b.x, s);
+                                s = fmaf(__uint_as_float(q.z & 0xffff0000u), b.y, s);
+                                s = fmaf(__uint_as_float(q.w << 16), b.z, s);
+                                s = fmaf(__uint_as_float(q.w & 0xffff0000u), b.w, s);
+                                acc[r][m] = s;
+                            }
+                        }
+                    }
+                }
+            }
+            loaded = false;
+            // four rows across the warp: after two exchanges a lane holds one row's sum over four lanes' worth
+#pragma unroll
+            for (int m = 0; m < M; m++) {
+                const bool h16 = lane & 16, h8 = lane & 8;
+                const float s0 = __shfl_xor_sync(0xffffffffu, h16 ? acc[0][m] : acc[2][m], 16);
+                const float s1 = __shfl_xor_sync(0xffffffffu, h16 ? acc[1][m] : acc[3][m], 16);
+                const float a0 = (h16 ? acc[2][m] : acc[0][m]) + s0, a1 = (h16 ? acc[3][m] : acc[1][m]) + s1;
+                float t = (h8 ? a1 : a0) + __shfl_xor_sync(0xffffffffu, h8 ? a0 : a1, 8);
+                t += __shfl_xor_sync(0xffffffffu, t, 4);
+                t += __shfl_xor_sync(0xffffffffu, t, 2);
+                t += __shfl_xor_sync(0xffffffffu, t, 1);
+                if ((lane & 7) == 0) part[buf][warp][v - vb + ((lane >> 4) & 1) * 2 + ((lane >> 3) & 1)][m] = t;
+            }
+        }
+        __syncthreads();
+        const int nout = (ve - vb) / step * M;
+        for (int t = tid; t < nout; t += NT) {
+            const int u = t / M, m = t % M, vl = u * step;
+            float s = 0.f, s2 = 0.f;
+#pragma unroll
+            for (int i = 0; i < NW; i++) s += part[buf][i][vl][m];
+            int sg, r;
+            locate(p, vb + vl, sg, r);
+            if (p.c.glu) {
+#pragma unroll
+                for (int i = 0; i < NW; i++) s2 += part[buf][i][vl + 1][m];
+                kq_dense_put(p.c.seg[0], m, r, kq_clamped_glu(s, s2, p.c.glu_limit, p.c.glu_alpha));
+            } else {
+                kq_dense_store(p.c, p.c.seg[sg], m, r, 0, s);
+            }
+        }
+    }
+}
+
+// Block-diagonal form: one warp per four rows of a group, activations from L1 / L2.
+struct GroupedParams {
+    KqDense c;
+    const float *x;
+    int64_t ldx;
+    int32_t quads; // four-row units per group and segment
+    int32_t vec;
+};
+
+template <int M>
+__global__ void __launch_bounds__(NT) gemv_grouped_bf16_kernel(const __grid_constant__ GroupedParams p) {
+    KQ_PDL_TRIGGER();
+    const int lane = threadIdx.x & 31;
+    const int64_t id = (int64_t)blockIdx.x * NW + (threadIdx.x >> 5), n_id = (int64_t)p.quads * p.c.groups * p.c.nseg;
+    KQ_PDL_WAIT();
+    if (id >= n_id) return;
+    const int sg = (int)(id / ((int64_t)p.quads * p.c.groups));
+    const int64_t rem = id % ((int64_t)p.quads * p.c.groups);
+    const int g = (int)(rem / p.quads), r0 = (int)(rem % p.quads) * 4;
+    const KqDenseSeg &s = p.c.seg[sg];
+    if (r0 >= s.n_rows) return;
+    const int K = p.c.K, nck = (int)((K + 7) / 8);
+    const uint4 *wp[4];
+#pragma unroll
+    for (int r = 0; r < 4; r++)
+        wp[r] = reinterpret_cast<const uint4 *>(s.W + ((int64_t)g * s.n_rows + min(r0 + r, s.n_rows - 1)) * p.c.ldw);
+    float acc[4][M];
+#pragma unroll
+    for (int r = 0; r < 4; r++)
+#pragma unroll
+        for (int m = 0; m < M; m++) acc[r][m] = 0.f;
+    for (int c = lane; c < nck; c += 32) {
+        uint4 w[4];
+#pragma unroll
+        for (int r = 0; r < 4; r++) w[r] = kq_ld_stream(wp[r] + c);
+#pragma unroll
+        for (int m = 0; m < M; m++) {
+            const float *x = p.x + m * p.ldx + g * p.c.xg;
+            const float4 a = load4(x, 8 * c, K, p.vec), b = load4(x, 8 * c + 4, K, p.vec);
+#pragma unroll
+            for (int r = 0; r < 4; r++) {
+                const uint4 q = w[r];
+                float t = acc[r][m];
+                t = fmaf(__uint_as_float(q.x << 16), a.x, t);
+                t = fmaf(__uint_as_float(q.x & 0xffff0000u), a.y, t);
+                t = fmaf(__uint_as_float(q.y << 16), a.z, t);
+                t = fmaf(__uint_as_float(q.y & 0xffff0000u), a.w, t);
+                t = fmaf(__uint_as_float(q.z << 16), b.x, t);
+                t = fmaf(__uint_as_float(q.z & 0xffff0000u), b.y, t);
+                t = fmaf(__uint_as_float(q.w << 16), b.z, t);
+                t = fmaf(__uint_as_float(q.w & 0xffff0000u), b.w, t);
+                acc[r][m] = t;
+            }
+        }
+    }
+#pragma unroll
+    for (int r = 0; r < 4; r++)
+#pragma unroll
+        for (int m = 0; m < M; m++) {
+            const float v = kq_warp_sum(acc[r][m]);
+            if (lane == 0 && r0 + r < s.n_rows) kq_dense_store(p.c, s, m, (int64_t)g * s.n_rows + r0 + r, g, v);
+        }
+}
+
+template <int M>
+b200_status launch_gemv(const GemvParams &p, size_t smem, cudaStream_t st) {
+    static bool attr[16];
+    int dev = 0;
+    KQ_CUDA(cudaGetDevice(&dev));
+    if (dev < 0 || dev >= 16 || !attr[dev]) {
+        KQ_CUDA(cudaFuncSetAttribute(gemv_bf16_kernel<M>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        if (dev >= 0 && dev < 16) attr[dev] = true;
+    }
+    static int mul = -1; // B200_GEMV16_CTAS: CTAs per SM of the decode projections
+    if (mul < 0) {
+        const char *v = getenv("B200_GEMV16_CTAS");
+        mul = v ? std::max(1, atoi(v)) : 2;
+    }
+    const int64_t units = p.V / (p.c.glu ? 2 : 1);
+    const int64_t want = std::max<int64_t>(1, kq_div_up(units * (p.c.glu ? 2 : 1), 4));
+    const unsigned grid = (unsigned)std::min<int64_t>(want, (int64_t)kq_sm_count() * mul);
+    kq_launch(gemv_bf16_kernel<M>, grid, NT, smem, st, p);
+    KQ_COUNT_LAUNCH();
+    KQ_LAUNCH_CHECK();
+    return B200_OK;
+}
+
+// the call for rows m0 .. m0 + m - 1 of a larger one
+KqDense rows_of(const KqDense &c, int m0, int m) {
+    KqDense d = c;
+    d.M = m;
+    for (int i = 0; i < d.nseg; i++)
+        d.seg[i].y = (uint8_t *)c.seg[i].y + m0 * c.seg[i].ldy * (c.seg[i].out == KQ_OUT_F32 ? 4 : 2);
+    if (d.head_gate) d.head_gate += m0 * d.ld_gate;
+    return d;
+}
+
+} // namespace
+
+b200_status kq_gemv_bf16(const KqDense &c, const KqNormPrep &pr, cudaStream_t st) {
+    KQ_REQUIRE(c.M >= 1 && c.nseg >= 1 && c.nseg <= 3 && c.groups == 1 && c.K >= 1, "gemv_bf16: bad call");
+    KQ_REQUIRE(c.ldw % 64 == 0 && c.ldw >= c.K, "gemv_bf16: weight rows must be padded to 64 elements");
+    const int nck = (int)kq_div_up(c.K, 8);
+    const int64_t row_smem = (int64_t)nck * 32;
+    const int cap = (int)std::min<int64_t>(8, 190 * 1024 / row_smem);
+    if (cap < 1) {
+        kq_set_error("gemv_bf16: rows of %d values do not fit in shared memory", c.K);
+        return B200_ERR_UNSUPPORTED;
+    }
+    for (int m0 = 0; m0 < c.M;) {
+        const int left = c.M - m0;
+        const int m = left >= 8 && cap >= 8 ? 8 : left >= 4 && cap >= 4 ? 4 : left >= 2 && cap >= 2 ? 2 : 1;
+        GemvParams p;
+        p.c = rows_of(c, m0, m);
+        p.p = pr;
+        p.p.x += m0 * pr.ldx;
+        if (pr.sub) p.p.sub += m0 * pr.ld_sub;
+        if (pr.x_out) p.p.x_out += m0 * pr.ld_out;
+        p.nck = nck;
+        p.V = 0;
+        for (int i = 0; i < c.nseg; i++) p.V += c.seg[i].n_rows;
+        b200_status rc;
+        const size_t smem = (size_t)(row_smem * m);
+        switch (m) {
+        case 1: rc = launch_gemv<1>(p, smem, st); break;
+        case 2: rc = launch_gemv<2>(p, smem, st); break;
+        case 4: rc = launch_gemv<4>(p, smem, st); break;
+        default: rc = launch_gemv<8>(p, smem, st); break;
+        }
+        if (rc != B200_OK) return rc;
+        m0 += m;
+    }
+    return B200_OK;
+}
+
+b200_status kq_gemv_grouped_bf16(const KqDense &c, const float *x, int64_t ldx, cudaStream_t st) {
+    KQ_REQUIRE(c.M >= 1 && c.nseg >= 1 && c.nseg <= 3 && c.groups >= 1 && !c.glu, "gemv_grouped_bf16: bad call");
+    for (int m0 = 0; m0 < c.M;) {
+        const int left = c.M - m0, m = left >= 4 ? 4 : left >= 2 ? 2 : 1;
+        GroupedParams p;
+        p.c = rows_of(c, m0, m);
+        p.x = x + m0 * ldx;
+        p.ldx = ldx;
+        p.quads = 0;
+        for (int i = 0; i < c.nseg; i++) p.quads = std::max<int>(p.quads, (int)kq_div_up(c.seg[i].n_rows, 4));
+        p.vec = (ldx % 4 == 0) && (c.xg % 4 == 0) && ((uintptr_t)x & 15) == 0;
+        const unsigned grid = (unsigned)kq_div_up((int64_t)p.quads * c.groups * c.nseg, NW);
+        if (m == 4) kq_launch(gemv_grouped_bf16_kernel<4>, grid, NT, 0, st, p);
+        else if (m == 2) kq_launch(gemv_grouped_bf16_kernel<2>, grid, NT, 0, st, p);
+        else kq_launch(gemv_grouped_bf16_kernel<1>, grid, NT, 0, st, p);
+        KQ_COUNT_LAUNCH();
+        KQ_LAUNCH_CHECK();
+        m0 += m;
+    }
+    return B200_OK;
+}

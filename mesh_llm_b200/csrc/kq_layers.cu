@@ -1,0 +1,664 @@
+// Stages whose layers are described one by one (b200_stage_create_layers): tensor table, caches and states, and the
+// forward pass, on top of the stage object of kq_stage.cuh (loading, decode graphs, logits, counters are shared
+// with the K-quant decoder).
+//
+// The residual stream x is f32.  A sub-layer leaves its output un-normed in `sub`; the next projection's prologue
+// forms x + norm_b(sub) and the norm in front of itself, so that no launch of its own does either in a decode step.
+// Up to 8 rows (decode) run on the matrix-vector kernels with f32 activations; more rows on the tensor-core GEMM with
+// a bf16 copy of each projection's input, or on the f32 GEMM in the 32-bit mode.
+//
+// State of one layer run and sequence slot: latent attention keeps a ring of cap rows (window + micro-batch, so
+// that a micro-batch's first row still finds its window), the recurrence its state and the convolution's last inputs.
+// A slot that starts at position 0 reads none of what it held, so nothing has to be cleared between sequences.
+#include "kq_dense.cuh"
+#include "kq_stage.cuh"
+
+#include <math.h>
+#include <stdlib.h>
+
+#include <algorithm>
+
+// expanded form of latent attention for prompts (kq_latent_prefill.cu)
+struct KqLatentPrefill {
+    const uint16_t *uk, *uv; // bf16 [n_head * dim][kq_bf16_ld(kv_rank)]
+    void *work;
+    size_t work_bytes;
+};
+size_t kq_latent_prefill_bytes(const KqLatent &l, int max_rows, int max_keys);
+b200_status kq_latent_prefill(const KqLatent &l, const KqLatentPrefill &w, const float *q, int64_t ldq, const float *gate, int64_t ldg,
+                              int T, int pos0, uint16_t *out, int64_t ldo, cudaStream_t st);
+
+struct LayerDesc {
+    b200_layer_config c;
+    const float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;
+    // recurrence
+    const uint16_t *wy = nullptr, *wx = nullptr, *wo = nullptr;
+    const float *by = nullptr, *bx = nullptr;
+    KqRecW rec = {};
+    // latent attention
+    const uint16_t *wq = nullptr, *dkv = nullptr, *uk = nullptr, *uv = nullptr, *wg = nullptr;
+    uint16_t *uk_t = nullptr; // [n_head * kv_rank][kq_bf16_ld(qk_dim)], derived
+    const float *kv_norm = nullptr;
+    double *freq = nullptr;
+    // feed-forward
+    const uint16_t *gate = nullptr, *up = nullptr, *down = nullptr;
+};
+
+struct RunState { // one pass over a layer
+    int layer;
+    float *conv = nullptr, *s = nullptr;
+    void *cache = nullptr;
+    int cap = 0;
+};
+
+struct KqLayers {
+    b200_stack_config s;
+    std::vector<LayerDesc> layers; // [layer_begin, layer_end)
+    std::vector<RunState> runs;
+    std::vector<int> seq_pos;
+    float *trace = nullptr;
+    size_t state_bytes = 0;
+    const uint16_t *embed = nullptr;
+    const float *final_norm = nullptr;
+    // activations, sized for the widest layer
+    int64_t ldx = 0;
+    float *x[2] = {}, *sub = nullptr, *h32 = nullptr;
+    uint16_t *h16 = nullptr;
+    float *f[7] = {}; // projections of a mixer
+    uint16_t *u16 = nullptr, *z16 = nullptr, *act16 = nullptr;
+    float *act32 = nullptr, *att_scratch = nullptr;
+    size_t att_scratch_bytes = 0;
+    int *counters = nullptr;
+    void *prefill_work = nullptr;
+    size_t prefill_bytes = 0;
+};
+
+void KqLayersDelete::operator()(KqLayers *p) const { delete p; }
+
+namespace {
+
+constexpr int SMALL_ROWS = 8;
+
+// uk [H * dim][ld_in] -> uk_t [H * R][ld_out]
+__global__ void transpose_heads_kernel(const uint16_t *in, int64_t ld_in, int H, int dim, int R, uint16_t *out, int64_t ld_out) {
+    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= (int64_t)H * R * ld_out) return;
+    const int64_t row = i / ld_out;
+    const int d = (int)(i % ld_out), h = (int)(row / R), r = (int)(row % R);
+    out[i] = d < dim ? in[((int64_t)h * dim + d) * ld_in + r] : 0;
+}
+
+b200_status check_layer(const b200_layer_config &l, int i) {
+    if (l.mixer == B200_MIXER_LATENT_ATTN) {
+        KQ_REQUIRE(l.n_head >= 1 && l.qk_dim >= 1 && l.rot_dim >= 0 && l.v_dim >= 1 && l.kv_rank >= 1 && l.window >= 0,
+                   "layer %d: sizes of the latent attention", i);
+        KQ_REQUIRE(l.rot_dims >= 0 && l.rot_dims % 2 == 0 && l.rot_dims <= l.rot_dim && (l.rot_dims == 0 || l.rope_base > 0.f),
+                   "layer %d: rotary dimensions %d of %d", i, l.rot_dims, l.rot_dim);
+        if (l.kv_rank > 1024) {
+            kq_set_error("layer %d: latents of up to 1024 values", i);
+            return B200_ERR_UNSUPPORTED;
+        }
+    } else if (l.mixer == B200_MIXER_LINEAR_REC) {
+        KQ_REQUIRE(l.rec_width >= 1 && l.rec_blocks >= 1 && l.rec_width % l.rec_blocks == 0 && l.conv_taps >= 1,
+                   "layer %d: sizes of the recurrence", i);
+    } else {
+        kq_set_error("layer %d: unknown mixer %d", i, l.mixer);
+        return B200_ERR_UNSUPPORTED;
+    }
+    KQ_REQUIRE(l.ffn == B200_FFN_NONE || (l.ffn == B200_FFN_CLAMPED_GLU && l.n_ff >= 1), "layer %d: feed-forward", i);
+    return B200_OK;
+}
+
+std::string lname(int i, const char *what) { return "l" + std::to_string(i) + "." + what; }
+
+int64_t max_keys(const b200_stage_config &c, const b200_layer_config &l) {
+    return l.window > 0 ? std::min<int64_t>(l.window, c.n_ctx) : c.n_ctx;
+}
+
+KqLatent latent_of(const b200_stage *st, const LayerDesc &L, const RunState &r, int seq0) {
+    const b200_layer_config &c = L.c;
+    KqLatent l = {};
+    l.n_head = c.n_head, l.qk_dim = c.qk_dim, l.rot_dim = c.rot_dim, l.rot_dims = c.rot_dims, l.v_dim = c.v_dim, l.kv_rank = c.kv_rank;
+    l.window = c.window;
+    l.scale = c.attn_scale;
+    l.freq = L.freq;
+    l.cap = r.cap;
+    l.f32 = st->layers_desc->s.precision == B200_PRECISION_F32;
+    l.rot_at = kq_latent_rot_at(c.kv_rank);
+    l.ld = kq_latent_ld(c.kv_rank, c.rot_dim);
+    l.seq_stride = (int64_t)r.cap * l.ld;
+    l.cache = (uint8_t *)r.cache + seq0 * l.seq_stride * (l.f32 ? 4 : 2);
+    return l;
+}
+
+// The residual stream of a forward pass: x, plus norm_b(sub) still to be added when sub_w is set.
+struct Stream {
+    const float *x;
+    int64_t ldx;
+    const float *sub_w; // null: nothing pending
+    int next;           // which of the two x buffers is free
+};
+
+struct Pass {
+    b200_stage *st;
+    KqLayers *k;
+    int seq0, n_seq, T, pos0, rows;
+    const int32_t *pos_dev;
+    bool small, f32;
+    unsigned classes;
+    cudaStream_t s;
+    Stream x;
+
+#define GEMV_(expr) do { if (classes & CLS_GEMV) KQ_TRY(expr); } while (0)
+#define ATTN_(expr) do { if (classes & CLS_ATTN) KQ_TRY(expr); } while (0)
+#define OTHER_(expr) do { if (classes & CLS_OTHER) KQ_TRY(expr); } while (0)
+
+    KqNormPrep prep(const float *norm_w, bool keep) {
+        KqNormPrep p;
+        p.x = x.x, p.ldx = x.ldx;
+        p.norm_w = norm_w;
+        p.eps = st->c.rms_eps;
+        p.w_off = k->s.norm_offset;
+        if (x.sub_w) {
+            p.sub = k->sub, p.ld_sub = k->ldx, p.sub_w = x.sub_w;
+            if (keep) p.x_out = k->x[x.next], p.ld_out = k->ldx;
+        }
+        return p;
+    }
+    void taken() { // the pending sub-layer output is now part of x
+        if (!x.sub_w) return;
+        x.x = k->x[x.next], x.ldx = k->ldx, x.sub_w = nullptr;
+        x.next ^= 1;
+    }
+    static KqDenseSeg seg(const uint16_t *W, int64_t n, void *y, int64_t ldy, const float *bias = nullptr, int act = KQ_ACT_NONE,
+                          int out = KQ_OUT_F32) {
+        KqDenseSeg g = {};
+        g.W = W, g.n_rows = (int32_t)n, g.y = y, g.ldy = ldy, g.bias = bias, g.act = act, g.out = out;
+        return g;
+    }
+    KqDense call(int64_t K) {
+        KqDense c;
+        c.M = rows, c.K = (int)K, c.ldw = kq_bf16_ld(K);
+        return c;
+    }
+    // projection of norm(x): the residual is brought up to date on the way
+    b200_status project(const KqDense &c, const float *norm_w) {
+        const KqNormPrep p = prep(norm_w, true);
+        const int h = st->c.n_embd;
+        if (small) {
+            GEMV_(kq_gemv_bf16(c, p, s));
+        } else if (f32) {
+            OTHER_(kq_norm_prep(p, rows, h, k->h32, k->ldx, nullptr, 0, s));
+            GEMV_(kq_gemm_f32(c, k->h32, k->ldx, s));
+        } else {
+            OTHER_(kq_norm_prep(p, rows, h, nullptr, 0, k->h16, kq_bf16_ld(h), s));
+            GEMV_(kq_gemm_bf16(c, k->h16, kq_bf16_ld(h), 1, s));
+        }
+        taken();
+        return B200_OK;
+    }
+    // output projection of a sub-layer: sub = W a, a in f32 (few rows, 32-bit mode) or bf16
+    b200_status close(const uint16_t *W, int64_t K, const float *a32, int64_t ld32, const uint16_t *a16, const float *norm_b) {
+        KqDense c = call(K);
+        c.nseg = 1;
+        c.seg[0] = seg(W, st->c.n_embd, k->sub, k->ldx);
+        if (small) {
+            KqNormPrep p;
+            p.x = a32, p.ldx = ld32;
+            GEMV_(kq_gemv_bf16(c, p, s));
+        } else if (f32) {
+            GEMV_(kq_gemm_f32(c, a32, ld32, s));
+        } else {
+            GEMV_(kq_gemm_bf16(c, a16, kq_bf16_ld(K), 1, s));
+        }
+        x.sub_w = norm_b;
+        return B200_OK;
+    }
+
+    b200_status recurrence(const LayerDesc &L, const RunState &r) {
+        const int W = L.c.rec_width, B = L.c.rec_blocks, m = W / B;
+        const int64_t ld = kq_f32_ld(W);
+        float *y = k->f[0], *xi = k->f[1], *u = k->f[2], *gr = k->f[3], *gi = k->f[4], *z = k->f[5];
+        KqDense c = call(st->c.n_embd);
+        c.nseg = 2;
+        c.seg[0] = seg(L.wy, W, y, ld, L.by, KQ_ACT_GELU_TANH);
+        c.seg[1] = seg(L.wx, W, xi, ld, L.bx);
+        KQ_TRY(project(c, L.norm1));
+        KqRecState rs;
+        rs.conv = r.conv + (int64_t)seq0 * L.c.conv_taps * W;
+        rs.s = r.s + (int64_t)seq0 * W;
+        if (T == 1 && small) {
+            OTHER_(kq_recurrence_step(L.rec, rs, xi, ld, y, ld, n_seq, pos_dev, pos0, z, ld, s));
+            return close(L.wo, W, z, ld, nullptr, L.norm1b);
+        }
+        const bool tc = !small && !f32;
+        const int64_t ldu = (int64_t)B * kq_bf16_ld(m);
+        OTHER_(kq_causal_conv(L.rec, rs, xi, ld, n_seq, T, pos_dev, pos0, u, ld, tc ? k->u16 : nullptr, s));
+        KqDense g = call(m);
+        g.nseg = 2;
+        g.groups = B;
+        g.seg[0] = seg(L.rec.ra, m, gr, ld, L.rec.ra_b);
+        g.seg[1] = seg(L.rec.ri, m, gi, ld, L.rec.ri_b);
+        g.xg = tc ? kq_bf16_ld(m) : m;
+        if (small) OTHER_(kq_gemv_grouped_bf16(g, u, ld, s));
+        else if (f32) OTHER_(kq_gemm_f32(g, u, ld, s));
+        else OTHER_(kq_gemm_bf16(g, k->u16, ldu, 3, s)); // the gates see u in full f32
+        OTHER_(kq_linear_recurrence(L.rec, rs, gr, gi, ld, u, ld, xi, ld, y, ld, n_seq, T, pos_dev, pos0, tc ? nullptr : z, ld,
+                                    tc ? k->z16 : nullptr, kq_bf16_ld(W), s));
+        return close(L.wo, W, z, ld, k->z16, L.norm1b);
+    }
+
+    b200_status latent(const LayerDesc &L, const RunState &r) {
+        const b200_layer_config &c = L.c;
+        const int H = c.n_head, hd = c.qk_dim + c.rot_dim;
+        const int64_t ldq = kq_f32_ld((int64_t)H * hd), ldkv = kq_f32_ld(c.kv_rank + c.rot_dim), ldg = kq_f32_ld(H), rp = kq_f32_ld(c.kv_rank);
+        const int64_t lda = kq_f32_ld((int64_t)H * c.v_dim);
+        float *q = k->f[0], *kv = k->f[1], *g = k->f[2], *q_lat = k->f[3], *o_lat = k->f[4], *att = k->f[5];
+        KqDense p = call(st->c.n_embd);
+        p.nseg = 3;
+        p.seg[0] = seg(L.wq, (int64_t)H * hd, q, ldq);
+        p.seg[1] = seg(L.dkv, c.kv_rank + c.rot_dim, kv, ldkv);
+        p.seg[2] = seg(L.wg, H, g, ldg);
+        KQ_TRY(project(p, L.norm1));
+        const KqLatent l = latent_of(st, L, r, seq0);
+        const bool tc = !small && !f32;
+        // prompts on tensor cores: keys and values of the visible rows are worked out per head
+        if (tc && T > SMALL_ROWS && !pos_dev && k->prefill_work) {
+            OTHER_(kq_latent_store(l, L.kv_norm, st->c.rms_eps, q, ldq, kv, ldkv, n_seq, T, pos_dev, pos0, nullptr, 0, s));
+            const KqLatentPrefill w = {L.uk, L.uv, k->prefill_work, k->prefill_bytes};
+            b200_status rc = B200_OK;
+            for (int i = 0; i < n_seq && rc == B200_OK; i++) {
+                KqLatent li = l;
+                li.cache = (uint8_t *)l.cache + i * l.seq_stride * 2;
+                if (classes & CLS_ATTN)
+                    rc = kq_latent_prefill(li, w, q + (int64_t)i * T * ldq, ldq, g + (int64_t)i * T * ldg, ldg, T, pos0,
+                                           k->z16 + (int64_t)i * T * kq_bf16_ld((int64_t)H * c.v_dim), kq_bf16_ld((int64_t)H * c.v_dim), s);
+            }
+            if (rc == B200_OK) return close(L.wo, (int64_t)H * c.v_dim, nullptr, 0, k->z16, L.norm1b);
+            if (rc != B200_ERR_UNSUPPORTED) return rc;
+            // q is rotated already: only its copy into the latent layout is missing
+            KQ_TRY(absorb(L, l, q, ldq, hd, q_lat, true));
+        } else {
+            OTHER_(kq_latent_store(l, L.kv_norm, st->c.rms_eps, q, ldq, kv, ldkv, n_seq, T, pos_dev, pos0, q_lat, (int64_t)H * l.ld, s));
+            KQ_TRY(absorb(L, l, q, ldq, hd, q_lat, false));
+        }
+        ATTN_(kq_latent_attention(l, q_lat, n_seq, T, pos_dev, pos0, (int)max_keys(st->c, c), o_lat, k->att_scratch, k->att_scratch_bytes,
+                                  k->counters, s));
+        KqDense v = call(c.kv_rank);
+        v.nseg = 1;
+        v.groups = H;
+        v.xg = rp;
+        v.head_gate = g;
+        v.ld_gate = ldg;
+        v.seg[0] = tc ? seg(L.uv, c.v_dim, k->z16, kq_bf16_ld((int64_t)H * c.v_dim), nullptr, KQ_ACT_NONE, KQ_OUT_BF16)
+                      : seg(L.uv, c.v_dim, att, lda);
+        if (small) ATTN_(kq_gemv_grouped_bf16(v, o_lat, H * rp, s));
+        else ATTN_(kq_gemm_f32(v, o_lat, H * rp, s));
+        return close(L.wo, (int64_t)H * c.v_dim, att, lda, k->z16, L.norm1b);
+    }
+    // q_lat[h] = [W_uk[h]^T q_unrot | q_rot]
+    b200_status absorb(const LayerDesc &L, const KqLatent &l, const float *q, int64_t ldq, int hd, float *q_lat, bool copy_rot) {
+        KqDense a = call(L.c.qk_dim);
+        a.nseg = 1;
+        a.groups = L.c.n_head;
+        a.xg = hd;
+        a.seg[0] = seg(L.uk_t, L.c.kv_rank, q_lat, (int64_t)L.c.n_head * l.ld);
+        a.seg[0].head_in = L.c.kv_rank;
+        a.seg[0].head_out = l.ld;
+        if (copy_rot) {
+            KQ_CUDA(cudaMemsetAsync(q_lat, 0, (size_t)rows * L.c.n_head * l.ld * 4, s));
+            for (int i = 0; i < rows && L.c.rot_dim; i++)
+                KQ_CUDA(cudaMemcpy2DAsync(q_lat + (int64_t)i * L.c.n_head * l.ld + l.rot_at, (size_t)l.ld * 4, q + i * ldq + L.c.qk_dim, (size_t)hd * 4,
+                                          (size_t)L.c.rot_dim * 4, (size_t)L.c.n_head, cudaMemcpyDeviceToDevice, s));
+        }
+        if (small) ATTN_(kq_gemv_grouped_bf16(a, q, ldq, s));
+        else ATTN_(kq_gemm_f32(a, q, ldq, s));
+        return B200_OK;
+    }
+
+    b200_status feed_forward(const LayerDesc &L) {
+        const int ff = L.c.n_ff;
+        const bool tc = !small && !f32;
+        KqDense c = call(st->c.n_embd);
+        c.nseg = 2;
+        c.glu = 1;
+        c.glu_limit = L.c.glu_limit;
+        c.glu_alpha = L.c.glu_alpha;
+        c.seg[0] = tc ? seg(L.gate, ff, k->act16, kq_bf16_ld(ff), nullptr, KQ_ACT_NONE, KQ_OUT_BF16) : seg(L.gate, ff, k->act32, kq_f32_ld(ff));
+        if (tc) c.seg[0].pad_cols = (int32_t)kq_bf16_ld(ff);
+        c.seg[1] = seg(L.up, ff, nullptr, 0);
+        KQ_TRY(project(c, L.norm2));
+        return close(L.down, ff, k->act32, kq_f32_ld(ff), k->act16, L.norm2b);
+    }
+
+    b200_status head(float *logits, int all_logits, int32_t *next_tokens) {
+        const b200_stage_config &c = st->c;
+        const int out_rows = all_logits ? rows : n_seq, h = c.n_embd;
+        float *lg = logits ? logits : st->logits_int;
+        if (!lg || !(logits || next_tokens)) return B200_OK;
+        KQ_REQUIRE(logits || out_rows <= c.n_seq, "stage: internal logits hold one row per sequence");
+        KqNormPrep p = prep(k->final_norm, false);
+        if (!all_logits) { // last token of each sequence
+            p.x += (int64_t)(T - 1) * p.ldx, p.ldx *= T;
+            if (p.sub) p.sub += (int64_t)(T - 1) * p.ld_sub, p.ld_sub *= T;
+        }
+        KqDense d = call(h);
+        d.M = out_rows;
+        d.nseg = 1;
+        d.seg[0] = seg(k->embed, c.n_vocab, lg, c.n_vocab);
+        if (out_rows <= SMALL_ROWS) {
+            GEMV_(kq_gemv_bf16(d, p, s));
+        } else if (f32) {
+            OTHER_(kq_norm_prep(p, out_rows, h, k->h32, k->ldx, nullptr, 0, s));
+            GEMV_(kq_gemm_f32(d, k->h32, k->ldx, s));
+        } else {
+            OTHER_(kq_norm_prep(p, out_rows, h, nullptr, 0, k->h16, kq_bf16_ld(h), s));
+            GEMV_(kq_gemm_bf16(d, k->h16, kq_bf16_ld(h), 1, s));
+        }
+        if (next_tokens)
+            OTHER_(b200_logit_signals(lg, out_rows, c.n_vocab, nullptr, nullptr, next_tokens, st->scan_scratch, st->scan_scratch_bytes, s));
+        return B200_OK;
+    }
+    // the residual stream as it stands, into a buffer of n_embd-wide rows
+    b200_status residual_to(float *out) {
+        KqNormPrep p = prep(nullptr, false);
+        p.x_out = out;
+        p.ld_out = st->c.n_embd;
+        OTHER_(kq_norm_prep(p, rows, st->c.n_embd, nullptr, 0, nullptr, 0, s));
+        return B200_OK;
+    }
+};
+
+} // namespace
+
+b200_status kq_layers_forward(b200_stage *st, const int32_t *tokens, const float *hidden_in, int seq0, int n_seq, int T, int pos0,
+                              bool pos_from_dev, float *hidden_out, float *logits, int all_logits, int32_t *next_tokens, cudaStream_t s,
+                              unsigned classes) {
+    KqLayers *k = st->layers_desc.get();
+    const b200_stage_config &c = st->c;
+    Pass P;
+    P.st = st, P.k = k, P.seq0 = seq0, P.n_seq = n_seq, P.T = T, P.pos0 = pos0, P.rows = n_seq * T;
+    P.pos_dev = pos_from_dev ? st->pos0_dev : nullptr;
+    P.small = P.rows <= SMALL_ROWS;
+    P.f32 = k->s.precision == B200_PRECISION_F32;
+    P.classes = classes;
+    P.s = s;
+    P.x = {hidden_in, c.n_embd, nullptr, 0};
+    if (c.has_embd) {
+        if (classes & CLS_OTHER) KQ_TRY(kq_embed_bf16(k->embed, kq_bf16_ld(c.n_embd), tokens, P.rows, c.n_embd, k->s.embd_scale, k->x[0], k->ldx, s));
+        P.x = {k->x[0], k->ldx, nullptr, 1};
+    }
+    int run = 0;
+    for (const RunState &r : k->runs) {
+        const LayerDesc &L = k->layers[r.layer - c.layer_begin];
+        KQ_TRY(L.c.mixer == B200_MIXER_LATENT_ATTN ? P.latent(L, r) : P.recurrence(L, r));
+        if (L.c.ffn != B200_FFN_NONE) KQ_TRY(P.feed_forward(L));
+        if (k->trace) KQ_TRY(P.residual_to(k->trace + (int64_t)run * P.rows * c.n_embd));
+        run++;
+    }
+    if (hidden_out) KQ_TRY(P.residual_to(hidden_out));
+    if (c.has_output) KQ_TRY(P.head(logits, all_logits, next_tokens));
+    return B200_OK;
+}
+
+b200_status kq_layers_resolve(b200_stage *st) {
+    KqLayers *k = st->layers_desc.get();
+    const b200_stage_config &c = st->c;
+    auto f32 = [&](const std::string &n) { return (const float *)kq_stage_find(st, n)->dev; };
+    auto b16 = [&](const std::string &n) { return (const uint16_t *)kq_stage_find(st, n)->dev; };
+    for (int i = c.layer_begin; i < c.layer_end; i++) {
+        LayerDesc &L = k->layers[i - c.layer_begin];
+        L.norm1 = f32(lname(i, "norm1"));
+        L.norm1b = f32(lname(i, "norm1b"));
+        L.wo = b16(lname(i, "mix.o"));
+        if (L.c.mixer == B200_MIXER_LINEAR_REC) {
+            L.wy = b16(lname(i, "mix.y")), L.by = f32(lname(i, "mix.y.b"));
+            L.wx = b16(lname(i, "mix.x")), L.bx = f32(lname(i, "mix.x.b"));
+            L.rec.conv_w = f32(lname(i, "mix.conv")), L.rec.conv_b = f32(lname(i, "mix.conv.b"));
+            L.rec.ra = b16(lname(i, "mix.ra")), L.rec.ra_b = f32(lname(i, "mix.ra.b"));
+            L.rec.ri = b16(lname(i, "mix.ri")), L.rec.ri_b = f32(lname(i, "mix.ri.b"));
+            L.rec.lam = f32(lname(i, "mix.lam"));
+            L.rec.decay = L.c.rec_decay;
+            L.rec.width = L.c.rec_width, L.rec.blocks = L.c.rec_blocks, L.rec.taps = L.c.conv_taps;
+        } else {
+            L.wq = b16(lname(i, "mix.q")), L.dkv = b16(lname(i, "mix.dkv")), L.kv_norm = f32(lname(i, "mix.dkv.norm"));
+            L.uk = b16(lname(i, "mix.uk")), L.uv = b16(lname(i, "mix.uv")), L.wg = b16(lname(i, "mix.g"));
+            const int64_t ld = kq_bf16_ld(L.c.qk_dim), n = (int64_t)L.c.n_head * L.c.kv_rank * ld;
+            transpose_heads_kernel<<<(unsigned)kq_div_up(n, 256), 256>>>(L.uk, kq_bf16_ld(L.c.kv_rank), L.c.n_head, L.c.qk_dim, L.c.kv_rank, L.uk_t, ld);
+            KQ_LAUNCH_CHECK();
+        }
+        if (L.c.ffn != B200_FFN_NONE) {
+            L.norm2 = f32(lname(i, "norm2")), L.norm2b = f32(lname(i, "norm2b"));
+            L.gate = b16(lname(i, "mlp.gate")), L.up = b16(lname(i, "mlp.up")), L.down = b16(lname(i, "mlp.down"));
+        }
+    }
+    if (c.has_embd || c.has_output) k->embed = b16("embed");
+    if (c.has_output) k->final_norm = f32("final.norm");
+    KQ_CUDA(cudaDeviceSynchronize());
+    return B200_OK;
+}
+
+b200_status kq_layers_check_pos(b200_stage *st, int seq0, int n_seq, int T, int pos0) {
+    const KqLayers *k = st->layers_desc.get();
+    (void)T;
+    for (int i = seq0; i < seq0 + n_seq; i++)
+        if (pos0 != 0 && pos0 != k->seq_pos[i]) {
+            kq_set_error("stage_forward: sequence %d stands at position %d, the call starts at %d", i, k->seq_pos[i], pos0);
+            return B200_ERR_STATE;
+        }
+    return B200_OK;
+}
+
+void kq_layers_advance(b200_stage *st, int seq0, int n_seq, int pos) {
+    if (!st->layers_desc) return;
+    for (int i = seq0; i < seq0 + n_seq; i++) st->layers_desc->seq_pos[i] = pos;
+}
+
+bool kq_layers_tracing(const b200_stage *st) { return st->layers_desc && st->layers_desc->trace; }
+
+b200_status kq_layers_peek(b200_stage *st, const char *which, float *host_out, size_t n_floats) {
+    KqLayers *k = st->layers_desc.get();
+    KQ_REQUIRE(std::string(which) == "sub", "stage_peek: no buffer named %s (sub: the last sub-layer's output)", which);
+    KQ_REQUIRE(n_floats <= (size_t)st->rows_max * k->ldx, "stage_peek: %s holds %zu floats", which, (size_t)st->rows_max * k->ldx);
+    KqDevGuard dev_guard(st->c.device);
+    KQ_CUDA(cudaDeviceSynchronize());
+    KQ_CUDA(cudaMemcpy(host_out, k->sub, n_floats * 4, cudaMemcpyDeviceToHost));
+    return B200_OK;
+}
+
+extern "C" {
+
+b200_status b200_stage_create_layers(const b200_stage_config *cfg, const b200_stack_config *stack, const b200_layer_config *layers,
+                                     b200_stage **out) {
+    KQ_REQUIRE(cfg && stack && layers && out, "stage_create_layers: null argument");
+    b200_stage_config c = *cfg;
+    KQ_REQUIRE(c.n_embd > 0 && c.n_layer > 0 && c.layer_begin >= 0 && c.layer_begin <= c.layer_end && c.layer_end <= c.n_layer,
+               "stage: bad layer range [%d,%d) of %d", c.layer_begin, c.layer_end, c.n_layer);
+    KQ_REQUIRE(c.n_ctx > 0 && c.n_seq > 0 && c.n_ubatch > 0, "stage: n_ctx, n_seq, n_ubatch");
+    KQ_REQUIRE(!(c.has_embd || c.has_output) || c.n_vocab > 0, "stage: n_vocab");
+    KQ_REQUIRE(stack->precision == B200_PRECISION_BF16 || stack->precision == B200_PRECISION_F32, "stage: precision %d", stack->precision);
+    const bool loop = stack->loop_times > 1 && stack->loop_stop > stack->loop_start;
+    if (loop) {
+        KQ_REQUIRE(stack->loop_start >= 0 && stack->loop_stop <= c.n_layer, "stage: looped layers [%d,%d) of %d", stack->loop_start,
+                   stack->loop_stop, c.n_layer);
+        const bool outside = c.layer_end <= stack->loop_start || c.layer_begin >= stack->loop_stop;
+        const bool inside = c.layer_begin <= stack->loop_start && c.layer_end >= stack->loop_stop;
+        KQ_REQUIRE(outside || inside, "stage: the looped layers [%d,%d) cannot be split between stages", stack->loop_start, stack->loop_stop);
+    }
+    for (int i = 0; i < c.n_layer; i++) KQ_TRY(check_layer(layers[i], i));
+    KqDevGuard dev_guard(c.device);
+    b200_stage *st = new b200_stage();
+    c.n_head = c.n_head_kv = c.head_dim = c.n_ff = c.n_expert = 0;
+    st->c = c;
+    st->layers_desc.reset(new KqLayers());
+    KqLayers *k = st->layers_desc.get();
+    k->s = *stack;
+    k->seq_pos.assign(c.n_seq, -1);
+    for (int i = c.layer_begin; i < c.layer_end; i++) {
+        LayerDesc L;
+        L.c = layers[i];
+        k->layers.push_back(L);
+        const int times = loop && i == stack->loop_start ? stack->loop_times : 1;
+        const int last = loop && i == stack->loop_start ? stack->loop_stop : i + 1;
+        for (int t = 0; t < times; t++)
+            for (int j = i; j < last; j++)
+                if (times > 1 || !loop || j < stack->loop_start || j >= stack->loop_stop) {
+                    RunState r;
+                    r.layer = j;
+                    k->runs.push_back(r);
+                }
+    }
+    const int64_t h = c.n_embd, R = c.n_ubatch;
+    if (c.has_embd || c.has_output) kq_stage_add_tensor(st, "embed", B200_TYPE_BF16, h, c.n_vocab, 1);
+    int64_t fmax[6] = {}, wmax16 = 0, u16max = 0, ffmax = 0, scratch = 0, counters = 256, prefill = 0;
+    const bool f32 = stack->precision == B200_PRECISION_F32;
+    auto grow = [](int64_t &a, int64_t b) { a = std::max(a, b); };
+    for (int i = c.layer_begin; i < c.layer_end; i++) {
+        const b200_layer_config &l = layers[i];
+        auto mat = [&](const char *w, int64_t in, int64_t rows, int64_t n = 1) { kq_stage_add_tensor(st, lname(i, w), B200_TYPE_BF16, in, rows, n); };
+        auto vec = [&](const char *w, int64_t a, int64_t b = 1) { kq_stage_add_tensor(st, lname(i, w), B200_TYPE_F32, a, b, 1); };
+        vec("norm1", h);
+        vec("norm1b", h);
+        if (l.mixer == B200_MIXER_LINEAR_REC) {
+            const int64_t W = l.rec_width, m = W / l.rec_blocks;
+            mat("mix.y", h, W);
+            vec("mix.y.b", W);
+            mat("mix.x", h, W);
+            vec("mix.x.b", W);
+            vec("mix.conv", l.conv_taps, W);
+            vec("mix.conv.b", W);
+            mat("mix.ra", m, m, l.rec_blocks);
+            vec("mix.ra.b", m, l.rec_blocks);
+            mat("mix.ri", m, m, l.rec_blocks);
+            vec("mix.ri.b", m, l.rec_blocks);
+            vec("mix.lam", W);
+            mat("mix.o", W, h);
+            for (int f = 0; f < 6; f++) grow(fmax[f], kq_f32_ld(W));
+            grow(wmax16, kq_bf16_ld(W));
+            grow(u16max, 3 * l.rec_blocks * kq_bf16_ld(m));
+        } else {
+            const int64_t H = l.n_head, hd = l.qk_dim + l.rot_dim;
+            mat("mix.q", h, H * hd);
+            mat("mix.dkv", h, l.kv_rank + l.rot_dim);
+            vec("mix.dkv.norm", l.kv_rank);
+            mat("mix.uk", l.kv_rank, H * l.qk_dim);
+            mat("mix.uv", l.kv_rank, H * l.v_dim);
+            mat("mix.g", h, H);
+            mat("mix.o", H * l.v_dim, h);
+            grow(fmax[0], kq_f32_ld(H * hd));
+            grow(fmax[1], kq_f32_ld(l.kv_rank + l.rot_dim));
+            grow(fmax[2], kq_f32_ld(H));
+            grow(fmax[3], H * kq_latent_ld(l.kv_rank, l.rot_dim));
+            grow(fmax[4], H * kq_f32_ld(l.kv_rank));
+            grow(fmax[5], kq_f32_ld(H * l.v_dim));
+            grow(wmax16, kq_bf16_ld(H * l.v_dim));
+            grow(scratch, (int64_t)kq_latent_scratch_bytes(l.n_head, l.kv_rank, (int)max_keys(c, l)));
+            grow(counters, (int64_t)kq_latent_counter_bytes(l.n_head));
+            KqLatent q = {};
+            q.n_head = l.n_head, q.qk_dim = l.qk_dim, q.rot_dim = l.rot_dim, q.v_dim = l.v_dim, q.kv_rank = l.kv_rank, q.window = l.window;
+            if (!f32) grow(prefill, (int64_t)kq_latent_prefill_bytes(q, (int)R, (int)std::min<int64_t>(c.n_ctx, max_keys(c, l) - 1 + R)));
+        }
+        if (l.ffn != B200_FFN_NONE) {
+            vec("norm2", h);
+            vec("norm2b", h);
+            mat("mlp.gate", h, l.n_ff);
+            mat("mlp.up", h, l.n_ff);
+            mat("mlp.down", l.n_ff, h);
+            grow(ffmax, l.n_ff);
+        }
+    }
+    if (c.has_output) kq_stage_add_tensor(st, "final.norm", B200_TYPE_F32, h, 1, 1);
+    b200_status rc = B200_OK;
+    auto A = [&](void *p, size_t bytes) { // zeroed: padding is read (times zero weights), so it must not hold NaNs
+        void **pp = (void **)p;
+        if (rc == B200_OK) rc = kq_stage_alloc(st, pp, bytes);
+        if (rc == B200_OK && bytes && cudaMemset(*pp, 0, bytes) != cudaSuccess) rc = B200_ERR_CUDA;
+    };
+    for (auto &t : st->tensors) A(&t.dev, t.dev_bytes + 16);
+    for (size_t i = 0; i < k->layers.size(); i++) {
+        LayerDesc &L = k->layers[i];
+        if (L.c.mixer != B200_MIXER_LATENT_ATTN) continue;
+        A(&L.uk_t, (size_t)L.c.n_head * L.c.kv_rank * kq_bf16_ld(L.c.qk_dim) * 2);
+        std::vector<double> fr(L.c.rot_dims / 2 + 1, 0.0);
+        for (int j = 0; j < L.c.rot_dims / 2; j++) fr[j] = pow((double)L.c.rope_base, -2.0 * j / L.c.rot_dims);
+        A(&L.freq, fr.size() * 8);
+        if (rc == B200_OK && cudaMemcpy(L.freq, fr.data(), fr.size() * 8, cudaMemcpyHostToDevice) != cudaSuccess) rc = B200_ERR_CUDA;
+    }
+    for (RunState &r : k->runs) {
+        const b200_layer_config &l = k->layers[r.layer - c.layer_begin].c;
+        size_t b;
+        if (l.mixer == B200_MIXER_LINEAR_REC) {
+            A(&r.conv, b = (size_t)c.n_seq * l.conv_taps * l.rec_width * 4);
+            k->state_bytes += b;
+            A(&r.s, b = (size_t)c.n_seq * l.rec_width * 4);
+        } else {
+            r.cap = (int)std::min<int64_t>(c.n_ctx, max_keys(c, l) - 1 + R);
+            A(&r.cache, b = (size_t)c.n_seq * r.cap * kq_latent_ld(l.kv_rank, l.rot_dim) * (f32 ? 4 : 2));
+        }
+        k->state_bytes += b;
+    }
+    st->rows_max = (int)R;
+    k->ldx = kq_f32_ld(h);
+    for (int i = 0; i < 2; i++) A(&k->x[i], (size_t)(R * k->ldx * 4));
+    A(&k->sub, (size_t)(R * k->ldx * 4));
+    const bool wide = R > SMALL_ROWS || c.n_seq > SMALL_ROWS;
+    if (wide) A(&k->h32, (size_t)(R * k->ldx * 4));
+    if (wide) A(&k->h16, (size_t)(R * kq_bf16_ld(h) * 2));
+    for (int f = 0; f < 6; f++)
+        if (fmax[f]) A(&k->f[f], (size_t)(R * fmax[f] * 4));
+    if (wide) A(&k->z16, (size_t)(R * wmax16 * 2));
+    if (wide) A(&k->u16, (size_t)(R * u16max * 2));
+    if (ffmax) A(&k->act32, (size_t)((f32 ? R : std::min<int64_t>(R, SMALL_ROWS)) * kq_f32_ld(ffmax) * 4));
+    if (ffmax && wide) A(&k->act16, (size_t)(R * kq_bf16_ld(ffmax) * 2));
+    k->att_scratch_bytes = (size_t)scratch;
+    A(&k->att_scratch, (size_t)scratch);
+    A(&k->counters, (size_t)counters);
+    k->prefill_bytes = wide ? (size_t)prefill : 0;
+    if (k->prefill_bytes) A(&k->prefill_work, k->prefill_bytes);
+    A(&st->pos0_dev, 256);
+    A(&st->rid_scratch, 1024);
+    A(&st->xn, (size_t)(c.n_seq * h * 4));
+    A(&st->att, (size_t)(c.n_seq * h * 4));
+    if (c.has_output) {
+        A(&st->logits_int, (size_t)c.n_seq * c.n_vocab * 4);
+        st->scan_scratch_bytes = b200_logit_signals_scratch_bytes(std::max<int64_t>(R, c.n_seq));
+        A(&st->scan_scratch, st->scan_scratch_bytes);
+    }
+    if (rc == B200_OK && cudaStreamCreateWithFlags(&st->cap_stream, cudaStreamNonBlocking) != cudaSuccess) {
+        kq_set_error("stage: cudaStreamCreate failed");
+        rc = B200_ERR_CUDA;
+    }
+    if (rc == B200_OK && cudaDeviceSynchronize() != cudaSuccess) rc = B200_ERR_CUDA;
+    if (rc != B200_OK) {
+        b200_stage_free(st);
+        return rc;
+    }
+    const char *ng = getenv("B200_NO_GRAPH");
+    st->use_graph = !(ng && ng[0] == '1');
+    *out = st;
+    return B200_OK;
+}
+
+b200_status b200_stage_trace_residual(b200_stage *st, float *buf) {
+    KQ_REQUIRE(st && st->layers_desc, "stage_trace_residual: a stage with described layers");
+    st->layers_desc->trace = buf;
+    return B200_OK;
+}
+
+int32_t b200_stage_layer_runs(b200_stage *st) {
+    if (!st) return -1;
+    return st->layers_desc ? (int32_t)st->layers_desc->runs.size() : st->c.layer_end - st->c.layer_begin;
+}
+
+int32_t b200_stage_seq_pos(b200_stage *st, int32_t seq) {
+    if (!st || !st->layers_desc || seq < 0 || seq >= st->c.n_seq) return -1;
+    return st->layers_desc->seq_pos[seq];
+}
+
+size_t b200_stage_state_bytes(b200_stage *st) {
+    if (!st) return 0;
+    if (st->layers_desc) return st->layers_desc->state_bytes / (size_t)st->c.n_seq;
+    return (size_t)(st->c.layer_end - st->c.layer_begin) * st->c.n_ctx * st->c.n_head_kv * (st->k_row + st->v_row);
+}
+
+} // extern "C"

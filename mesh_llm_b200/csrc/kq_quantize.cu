@@ -2,6 +2,8 @@
 // device repack, and the on-device generator of synthetic Q4_K_M weights.
 #include "kq_common.cuh"
 
+#include <cuda_bf16.h>
+
 namespace {
 
 __global__ void __launch_bounds__(128) quantize_act_kernel(const float *x, int64_t nblocks,
@@ -237,6 +239,15 @@ __global__ void synth_f32_kernel(float *w, int64_t n, uint64_t key, float mean, 
     if (i < n) w[i] = mean + sigma * gauss_at(key, (uint64_t)i);
 }
 
+// bf16 rows of K values padded with zeros to ld
+__global__ void synth_bf16_kernel(uint16_t *w, int64_t n_rows, int64_t K, int64_t ld, uint64_t key, float mean, float sigma) {
+    KQ_PDL_ENTER();
+    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= n_rows * ld) return;
+    const int64_t r = i / ld, k = i % ld;
+    w[i] = k < K ? __bfloat16_as_ushort(__float2bfloat16_rn(mean + sigma * gauss_at(key, (uint64_t)(r * K + k)))) : 0;
+}
+
 } // namespace
 
 b200_status kq_synth_weights(uint32_t type, void *W, int64_t n_rows, int64_t K, uint64_t key,
@@ -244,6 +255,9 @@ b200_status kq_synth_weights(uint32_t type, void *W, int64_t n_rows, int64_t K, 
     if (type == B200_TYPE_F32) {
         const int64_t n = n_rows * K;
         kq_launch(synth_f32_kernel, (unsigned)kq_div_up(n, 256), 256, 0, st, (float *)W, n, key, mean, sigma);
+    } else if (type == B200_TYPE_BF16) {
+        const int64_t ld = kq_device_row_bytes(type, K) / 2, n = n_rows * ld;
+        kq_launch(synth_bf16_kernel, (unsigned)kq_div_up(n, 256), 256, 0, st, (uint16_t *)W, n_rows, K, ld, key, mean, sigma);
     } else {
         KQ_REQUIRE(type == B200_TYPE_Q4_K || type == B200_TYPE_Q6_K, "synth: type %u", type);
         KQ_REQUIRE(K % 256 == 0, "synth: K %% 256");

@@ -6,14 +6,11 @@
 // pass below is the graph llama.cpp builds for these architectures, expressed as launches of the
 // kernels in this directory; decode steps (T == 1) are captured once into a CUDA graph and
 // replayed, since at batch 1 the step is a chain of ~10 short kernels per layer.
-#include "kq_common.cuh"
-#include "kq_kvq.cuh"
+#include "kq_stage.cuh"
 
 #include <stdlib.h>
 
-#include <map>
-#include <string>
-#include <vector>
+#include <algorithm>
 
 b200_status kq_synth_weights(uint32_t type, void *W, int64_t n_rows, int64_t K, uint64_t key, float mean,
                              float sigma, cudaStream_t st);
@@ -46,36 +43,6 @@ b200_status kq_rope_store(float *q, const float *k, const float *v, const int32_
                           KqKvTypes kvt, cudaStream_t st);
 
 namespace {
-
-struct StTensor {
-    std::string name;
-    uint32_t type = 0;
-    int64_t ne[3] = {0, 0, 0};
-    void *dev = nullptr;
-    size_t dev_bytes = 0;
-    bool loaded = false;
-};
-
-struct LayerW {
-    const float *attn_norm = nullptr, *ffn_norm = nullptr, *bq = nullptr, *bk = nullptr, *bv = nullptr,
-                *q_norm = nullptr, *k_norm = nullptr, *router = nullptr;
-    StTensor *wq = nullptr, *wk = nullptr, *wv = nullptr, *wo = nullptr, *gate = nullptr, *up = nullptr,
-             *down = nullptr, *gate_e = nullptr, *up_e = nullptr, *down_e = nullptr;
-};
-
-struct GraphKey {
-    int n_seq, n_split, seq0, pad_;
-    const void *tokens, *hidden_in, *hidden_out, *logits, *next;
-    bool operator<(const GraphKey &o) const {
-        return memcmp(this, &o, sizeof(GraphKey)) < 0;
-    }
-};
-
-struct GraphEntry {
-    int n_split = 0; // attention slices the instantiated graph was last captured / updated for
-    cudaGraphExec_t exec = nullptr;
-    long long launches = 0;
-};
 
 // f32 matvec for the router: one warp per (token, expert)
 __global__ void __launch_bounds__(128) router_logits_kernel(const float *W, const float *x, int T, int E,
@@ -133,46 +100,7 @@ uint64_t name_hash(const char *s) {
 
 } // namespace
 
-struct b200_stage {
-    b200_stage_config c;
-    std::vector<StTensor> tensors;
-    std::map<std::string, int> index;
-    std::vector<LayerW> layers;
-    StTensor *tok_embd = nullptr, *out_w = nullptr;
-    const float *out_norm = nullptr;
-    bool resolved = false;
-    // KV cache [layer_local][seq][ctx][n_kv][hd] f16
-    uint16_t *kc = nullptr, *vc = nullptr;
-    KqKvTypes kvt;
-    int k_row = 0, v_row = 0; // bytes of one (position, kv head) row of each cache
-    // activations
-    int rows_max = 0;
-    float *x = nullptr, *xn = nullptr, *q = nullptr, *k = nullptr, *v = nullptr, *att = nullptr, *g = nullptr,
-          *u = nullptr, *last = nullptr, *logits_int = nullptr, *att_scratch = nullptr, *rl = nullptr,
-          *rw = nullptr, *hp = nullptr, *hp2 = nullptr, *yp = nullptr;
-    int32_t *moe_sorted = nullptr; // expert-major order of the routed pairs of a batch
-    size_t moe_sorted_bytes = 0;
-    uint8_t *expert_mask = nullptr; // one byte per expert, 1 = allowed (all ones when no mask is set)
-    int32_t *rid = nullptr, *pos0_dev = nullptr, *rid_scratch = nullptr, *attn_counters = nullptr;
-    unsigned int *moe_counters = nullptr; // one word per token row, zero between launches (moe_router_fused_kernel)
-    int32_t *emit_counters = nullptr;     // one word per 256 rows of the feed-forward width, zero between launches (KqEmitQ8)
-    size_t att_scratch_bytes = 0;
-    void *scan_scratch = nullptr; // slices and counters of the vocabulary scan
-    size_t scan_scratch_bytes = 0;
-    int8_t *aq = nullptr;
-    float *ad = nullptr;
-    int16_t *abs16 = nullptr;
-    int64_t kmax = 0;
-    std::map<GraphKey, GraphEntry> graphs;
-    cudaStream_t cap_stream = nullptr;
-    long long launches = 0;
-    bool use_graph = true;
-    std::vector<void *> allocs;
-};
-
-namespace {
-
-b200_status dev_alloc(b200_stage *st, void **p, size_t bytes) {
+b200_status kq_stage_alloc(b200_stage *st, void **p, size_t bytes) {
     *p = nullptr;
     if (bytes == 0) bytes = 256;
     cudaError_t e = cudaMalloc(p, bytes);
@@ -185,7 +113,7 @@ b200_status dev_alloc(b200_stage *st, void **p, size_t bytes) {
     return B200_OK;
 }
 
-void add_tensor(b200_stage *st, const std::string &name, uint32_t type, int64_t ne0, int64_t ne1,
+void kq_stage_add_tensor(b200_stage *st, const std::string &name, uint32_t type, int64_t ne0, int64_t ne1,
                 int64_t ne2) {
     StTensor t;
     t.name = name;
@@ -198,22 +126,18 @@ void add_tensor(b200_stage *st, const std::string &name, uint32_t type, int64_t 
     st->tensors.push_back(t);
 }
 
-StTensor *find(b200_stage *st, const std::string &name) {
+StTensor *kq_stage_find(b200_stage *st, const std::string &name) {
     auto it = st->index.find(name);
     return it == st->index.end() ? nullptr : &st->tensors[it->second];
 }
 
+namespace {
+
 StTensor *lt(b200_stage *st, int l, const char *what) {
     char buf[96];
     snprintf(buf, sizeof(buf), "blk.%d.%s", l, what);
-    return find(st, buf);
+    return kq_stage_find(st, buf);
 }
-
-#define KQ_TRY(expr)                      \
-    do {                                  \
-        b200_status rc__ = (expr);        \
-        if (rc__ != B200_OK) return rc__; \
-    } while (0)
 
 // MUL_MAT on quantised activations already sitting in st->aq/ad/abs16
 b200_status mm(b200_stage *st, const StTensor *w, int rows, float *y, const float *bias,
@@ -221,8 +145,6 @@ b200_status mm(b200_stage *st, const StTensor *w, int rows, float *y, const floa
     return b200_mul_mat_q8(w->type, w->dev, st->aq, st->ad, st->abs16, rows, w->ne[1], w->ne[0], y, bias,
                            residual, s);
 }
-
-enum { CLS_GEMV = 1, CLS_ATTN = 2, CLS_OTHER = 4, CLS_ALL = 7 };
 
 // `classes` selects which kernel classes are launched; anything but CLS_ALL is timing
 // instrumentation (the outputs are then meaningless).
@@ -232,6 +154,9 @@ b200_status forward_body(b200_stage *st, const int32_t *tokens, const float *hid
 #define GEMV_(expr) do { if (classes & CLS_GEMV) KQ_TRY(expr); } while (0)
 #define ATTN_(expr) do { if (classes & CLS_ATTN) KQ_TRY(expr); } while (0)
 #define OTHER_(expr) do { if (classes & CLS_OTHER) KQ_TRY(expr); } while (0)
+    if (st->layers_desc)
+        return kq_layers_forward(st, tokens, hidden_in, seq0, n_seq, T, pos0, pos_from_dev, hidden_out, logits, all_logits, next_tokens, s,
+                                 classes);
     const b200_stage_config &c = st->c;
     const int rows = n_seq * T;
     const int h = c.n_embd, hd = c.head_dim, nq = c.n_head * hd, nkv = c.n_head_kv * hd;
@@ -491,6 +416,11 @@ b200_status resolve(b200_stage *st) {
             kq_set_error("stage: tensor %s has not been loaded", t.name.c_str());
             return B200_ERR_STATE;
         }
+    if (st->layers_desc) {
+        KQ_TRY(kq_layers_resolve(st));
+        st->resolved = true;
+        return B200_OK;
+    }
     const b200_stage_config &c = st->c;
     st->layers.assign(c.layer_end - c.layer_begin, LayerW());
     for (int l = c.layer_begin; l < c.layer_end; l++) {
@@ -518,9 +448,9 @@ b200_status resolve(b200_stage *st) {
         L.up_e = lt(st, l, "ffn_up_exps.weight");
         L.down_e = lt(st, l, "ffn_down_exps.weight");
     }
-    st->tok_embd = find(st, "token_embd.weight");
-    st->out_w = find(st, "output.weight");
-    StTensor *on = find(st, "output_norm.weight");
+    st->tok_embd = kq_stage_find(st, "token_embd.weight");
+    st->out_w = kq_stage_find(st, "output.weight");
+    StTensor *on = kq_stage_find(st, "output_norm.weight");
     st->out_norm = on ? (const float *)on->dev : nullptr;
     st->resolved = true;
     return B200_OK;
@@ -564,13 +494,13 @@ b200_status b200_stage_create(const b200_stage_config *cfg, b200_stage **out) {
     st->k_row = kq_kv_row_bytes(kvt.k, c.head_dim);
     st->v_row = kq_kv_row_bytes(kvt.v, c.head_dim);
     const int64_t h = c.n_embd, hd = c.head_dim, nq = (int64_t)c.n_head * hd, nkv = (int64_t)c.n_head_kv * hd;
-    if (c.has_embd) add_tensor(st, "token_embd.weight", B200_TYPE_Q4_K, h, c.n_vocab, 1);
+    if (c.has_embd) kq_stage_add_tensor(st, "token_embd.weight", B200_TYPE_Q4_K, h, c.n_vocab, 1);
     for (int l = c.layer_begin; l < c.layer_end; l++) {
         const uint32_t alt = (l & 1) ? B200_TYPE_Q6_K : B200_TYPE_Q4_K;
         auto add = [&](const char *w, uint32_t ty, int64_t a, int64_t b, int64_t cc) {
             char buf[96];
             snprintf(buf, sizeof(buf), "blk.%d.%s", l, w);
-            add_tensor(st, buf, ty, a, b, cc);
+            kq_stage_add_tensor(st, buf, ty, a, b, cc);
         };
         add("attn_norm.weight", B200_TYPE_F32, h, 1, 1);
         add("attn_q.weight", B200_TYPE_Q4_K, h, nq, 1);
@@ -599,12 +529,12 @@ b200_status b200_stage_create(const b200_stage_config *cfg, b200_stage **out) {
         }
     }
     if (c.has_output) {
-        add_tensor(st, "output_norm.weight", B200_TYPE_F32, h, 1, 1);
-        add_tensor(st, "output.weight", B200_TYPE_Q6_K, h, c.n_vocab, 1);
+        kq_stage_add_tensor(st, "output_norm.weight", B200_TYPE_F32, h, 1, 1);
+        kq_stage_add_tensor(st, "output.weight", B200_TYPE_Q6_K, h, c.n_vocab, 1);
     }
     b200_status rc = B200_OK;
     auto A = [&](void **p, size_t bytes) {
-        if (rc == B200_OK) rc = dev_alloc(st, p, bytes);
+        if (rc == B200_OK) rc = kq_stage_alloc(st, p, bytes);
     };
     for (auto &t : st->tensors) A(&t.dev, t.dev_bytes + 16);
     const int64_t n_local = c.layer_end - c.layer_begin;
@@ -707,14 +637,15 @@ b200_status b200_stage_tensor_info(b200_stage *st, int64_t i, char *name, size_t
 b200_status b200_stage_set_tensor(b200_stage *st, const char *name, uint32_t type, const void *host_data,
                                   size_t nbytes) {
     KQ_REQUIRE(st && name && host_data, "stage_set_tensor: null argument");
-    StTensor *t = find(st, name);
+    StTensor *t = kq_stage_find(st, name);
     if (!t) {
         kq_set_error("stage_set_tensor: %s is not a tensor of this stage", name);
         return B200_ERR_INVALID;
     }
     const int64_t rows = t->ne[1] * t->ne[2];
-    KQ_REQUIRE(type == B200_TYPE_F32 ? t->type == B200_TYPE_F32
-                                     : (type == B200_TYPE_Q4_K || type == B200_TYPE_Q6_K) &&
+    KQ_REQUIRE(type == B200_TYPE_BF16  ? t->type == B200_TYPE_BF16 || (st->layers_desc && t->type == B200_TYPE_F32)
+               : type == B200_TYPE_F32 ? t->type == B200_TYPE_F32
+                                       : t->type != B200_TYPE_BF16 && (type == B200_TYPE_Q4_K || type == B200_TYPE_Q6_K) &&
                                            t->type != B200_TYPE_F32,
                "stage_set_tensor: %s cannot take type %u", name, type);
     const size_t want = (size_t)(kq_row_bytes(type, t->ne[0]) * rows);
@@ -723,10 +654,28 @@ b200_status b200_stage_set_tensor(b200_stage *st, const char *name, uint32_t typ
         return B200_ERR_BOUNDS;
     }
     KqDevGuard dev_guard(st->c.device);
+    if (type == B200_TYPE_BF16) {
+        const size_t n = (size_t)(t->ne[0] * rows), row = (size_t)t->ne[0] * 2;
+        if (t->type == B200_TYPE_F32) { // vectors are kept in f32
+            std::vector<float> wide(n);
+            for (size_t i = 0; i < n; i++) {
+                const uint32_t b = (uint32_t)((const uint16_t *)host_data)[i] << 16;
+                memcpy(&wide[i], &b, 4);
+            }
+            KQ_CUDA(cudaMemcpy(t->dev, wide.data(), n * 4, cudaMemcpyHostToDevice));
+        } else { // rows padded with zeros
+            const size_t ld = (size_t)kq_device_row_bytes(B200_TYPE_BF16, t->ne[0]);
+            KQ_CUDA(cudaMemset(t->dev, 0, t->dev_bytes));
+            KQ_CUDA(cudaMemcpy2D(t->dev, ld, host_data, row, row, (size_t)rows, cudaMemcpyHostToDevice));
+        }
+        t->loaded = true;
+        st->resolved = false; // derived copies
+        return B200_OK;
+    }
     if (type != t->type) { // same shape, other K-quant: reallocate the device rows
         void *p = nullptr;
         const size_t nb = (size_t)(kq_device_row_bytes(type, t->ne[0]) * rows);
-        KQ_TRY(dev_alloc(st, &p, nb + 16));
+        KQ_TRY(kq_stage_alloc(st, &p, nb + 16));
         t->dev = p;
         t->dev_bytes = nb;
         t->type = type;
@@ -759,7 +708,7 @@ b200_status b200_stage_set_tensor(b200_stage *st, const char *name, uint32_t typ
 
 b200_status b200_stage_get_tensor(b200_stage *st, const char *name, void *host_data, size_t nbytes) {
     KQ_REQUIRE(st && name && host_data, "stage_get_tensor: null argument");
-    StTensor *t = find(st, name);
+    StTensor *t = kq_stage_find(st, name);
     if (!t) {
         kq_set_error("stage_get_tensor: %s is not a tensor of this stage", name);
         return B200_ERR_INVALID;
@@ -783,6 +732,11 @@ b200_status b200_stage_get_tensor(b200_stage *st, const char *name, void *host_d
         cudaFree(tmp);
         return rc;
     }
+    if (t->type == B200_TYPE_BF16) {
+        const size_t row = (size_t)t->ne[0] * 2;
+        KQ_CUDA(cudaMemcpy2D(host_data, row, t->dev, (size_t)kq_device_row_bytes(B200_TYPE_BF16, t->ne[0]), row, (size_t)rows, cudaMemcpyDeviceToHost));
+        return B200_OK;
+    }
     KQ_CUDA(cudaMemcpy(host_data, t->dev, nbytes, cudaMemcpyDeviceToHost));
     return B200_OK;
 }
@@ -792,11 +746,13 @@ b200_status b200_stage_generate(b200_stage *st, uint64_t seed) {
     KqDevGuard dev_guard(st->c.device);
     for (auto &t : st->tensors) {
         const uint64_t key = mix64_host(seed ^ name_hash(t.name.c_str()));
-        const bool is_norm = t.name.find("norm.weight") != std::string::npos;
+        // plain norm weights around one, everything else (zero-centred norm weights included) around zero
+        const bool is_norm = t.name.find("norm.weight") != std::string::npos || t.name.find("dkv.norm") != std::string::npos;
         KQ_TRY(kq_synth_weights(t.type, t.dev, t.ne[1] * t.ne[2], t.ne[0], key, is_norm ? 1.0f : 0.0f, 0.02f,
                                 nullptr));
         t.loaded = true;
     }
+    if (st->layers_desc) st->resolved = false;
     KQ_CUDA(cudaDeviceSynchronize());
     return B200_OK;
 }
@@ -823,11 +779,12 @@ b200_status b200_stage_forward(b200_stage *st, const int32_t *tokens, const floa
     KQ_REQUIRE(c.has_output || hidden_out, "stage_forward: missing hidden_out");
     KqDevGuard dev_guard(c.device);
     KQ_TRY(resolve(st));
+    if (st->layers_desc) KQ_TRY(kq_layers_check_pos(st, seq0, n_seq, T, pos0));
     cudaStream_t s = (cudaStream_t)stream;
     const long long before = g_kq_launches;
-    if (T == 1 && st->use_graph) {
+    if (T == 1 && st->use_graph && !kq_layers_tracing(st)) {
         // decode step: positions come from device memory so one captured graph serves every step
-        const int n_split = kq_attention_decode_splits(pos0 + 1, n_seq * st->c.n_head_kv);
+        const int n_split = st->layers_desc ? 0 : kq_attention_decode_splits(pos0 + 1, n_seq * st->c.n_head_kv);
         GraphKey key;
         memset(&key, 0, sizeof(key));
         key.n_seq = n_seq;
@@ -880,11 +837,13 @@ b200_status b200_stage_forward(b200_stage *st, const int32_t *tokens, const floa
         KQ_CUDA(cudaGraphLaunch(it->second.exec, s));
         st->launches += it->second.launches + 1;
         g_kq_launches = before + it->second.launches + 1;
+        kq_layers_advance(st, seq0, n_seq, pos0 + 1);
         return B200_OK;
     }
     b200_status rc = forward_body(st, tokens, hidden_in, seq0, n_seq, T, pos0, false, 0, hidden_out, logits,
                                   all_logits, next_tokens, s);
     st->launches += g_kq_launches - before;
+    kq_layers_advance(st, seq0, n_seq, rc == B200_OK ? pos0 + T : -1);
     return rc;
 }
 
@@ -900,6 +859,7 @@ b200_status b200_stage_profile_decode(b200_stage *st, int32_t n_seq, int32_t pos
     // inputs of the replayed step live in the stage's own scratch (their values do not matter)
     int32_t *tok = (int32_t *)st->rid_scratch;
     float *hin = st->xn, *hout = st->att;
+    kq_layers_advance(st, 0, n_seq, -1); // the replays move the recurrent states
     cudaStream_t s = st->cap_stream;
     KQ_CUDA(cudaMemsetAsync(tok, 0, 256, s));
     kq_launch(set_pos_kernel, 1, 1, 0, s, st->pos0_dev, pos0);
@@ -909,7 +869,7 @@ b200_status b200_stage_profile_decode(b200_stage *st, int32_t n_seq, int32_t pos
     cudaGraphExec_t exec = nullptr;
     KQ_CUDA(cudaStreamBeginCapture(s, cudaStreamCaptureModeThreadLocal));
     b200_status rc = forward_body(st, tok, hin, 0, n_seq, 1, pos0, true,
-                                  kq_attention_splits(n_seq, c.n_head_kv, pos0 + 1),
+                                  st->layers_desc ? 0 : kq_attention_splits(n_seq, c.n_head_kv, pos0 + 1),
                                   c.has_output ? nullptr : hout, nullptr, 0,
                                   c.has_output ? (int32_t *)st->rid_scratch + 32 : nullptr, s, classes);
     cudaError_t e = cudaStreamEndCapture(s, &graph);
@@ -944,6 +904,7 @@ b200_status b200_stage_profile_decode(b200_stage *st, int32_t n_seq, int32_t pos
 
 b200_status b200_stage_peek(b200_stage *st, const char *which, float *host_out, size_t n_floats) {
     KQ_REQUIRE(st && which && host_out, "stage_peek: null argument");
+    if (st->layers_desc) return kq_layers_peek(st, which, host_out, n_floats);
     const b200_stage_config &c = st->c;
     const size_t R = (size_t)st->rows_max, nq = (size_t)c.n_head * c.head_dim, nkv = (size_t)c.n_head_kv * c.head_dim;
     const float *src = nullptr;
@@ -986,7 +947,7 @@ b200_status b200_stage_synchronize(b200_stage *st) {
     KQ_REQUIRE(st, "stage_synchronize: null stage");
     KqDevGuard dev_guard(st->c.device);
     KQ_CUDA(cudaDeviceSynchronize());
-    const int werr = kq_stream_error_fetch() | (kq_gemm_error_fetch() << 4) | (kq_attn_tc_error_fetch() << 8);
+    const int werr = kq_device_wait_errors();
     if (werr) {
         kq_set_error("stage_synchronize: a bounded device-side wait gave up (code %d)", werr);
         return B200_ERR_TIMEOUT;

@@ -12,7 +12,7 @@ import numpy as np
 import torch
 
 from . import capi
-from .capi import StageConfig, check, lib, ptr, cur_stream
+from .capi import LayerConfig, StackConfig, StageConfig, check, lib, ptr, cur_stream
 
 _DEFAULTS = dict(n_expert=0, n_expert_used=0, n_ff_exp=0, n_ff=0, n_seq=1, rope_neox=1, qkv_bias=0,
                  qk_norm=0, has_embd=1, has_output=1, rms_eps=1e-6, rope_theta=1e6, layer_begin=0,
@@ -20,15 +20,32 @@ _DEFAULTS = dict(n_expert=0, n_expert_used=0, n_ff_exp=0, n_ff=0, n_seq=1, rope_
 
 
 class Stage:
-    def __init__(self, **kw):
+    def __init__(self, stack=None, layers=None, **kw):
+        """A stage of the K-quant decoder; with `layers` (one LayerConfig per layer of the model) and `stack` (a
+        StackConfig) one whose layers are described one by one."""
         cfg = dict(_DEFAULTS)
         cfg.update(kw)
         cfg.setdefault("layer_end", cfg["n_layer"])
         self.cfg = StageConfig(**cfg)
+        self.described = layers is not None
         self.device = torch.device("cuda", self.cfg.device)
         h = C.c_void_p()
-        check(lib().b200_stage_create(C.byref(self.cfg), C.byref(h)))
+        if self.described:
+            arr = (LayerConfig * len(layers))(*layers)
+            check(lib().b200_stage_create_layers(C.byref(self.cfg), C.byref(stack), arr, C.byref(h)))
+        else:
+            check(lib().b200_stage_create(C.byref(self.cfg), C.byref(h)))
         self.h = h
+
+    @classmethod
+    def from_checkpoint(cls, ckpt, layer_begin=0, layer_end=-1, n_ctx=4096, n_seq=1, n_ubatch=512, device=0, precision=0):
+        """Stage for layers [layer_begin, layer_end) of an open Checkpoint, with exactly its own tensors read.
+        Returns (stage, tensors loaded, bytes read)."""
+        cfg, stack, layers = ckpt.stage_config(layer_begin, layer_end, n_ctx, n_seq, n_ubatch, device, precision)
+        st = cls(stack=stack, layers=layers, **{name: getattr(cfg, name) for name, _ in StageConfig._fields_})
+        n, nbytes = C.c_int64(), C.c_int64()
+        check(lib().b200_stage_load_ckpt(st.h, ckpt.h, C.byref(n), C.byref(nbytes)))
+        return st, n.value, nbytes.value
 
     @classmethod
     def from_gguf(cls, gguf_file, layer_begin=0, layer_end=-1, n_ctx=4096, n_seq=1, n_ubatch=512, device=0):
@@ -80,6 +97,22 @@ class Stage:
 
     def weight_bytes(self):
         return lib().b200_stage_weight_bytes(self.h)
+
+    def layer_runs(self):
+        """how many layers a forward pass runs, every pass over a looped layer counted"""
+        return lib().b200_stage_layer_runs(self.h)
+
+    def trace_residual(self, buf):
+        """diagnostics of a stage with described layers: following forward calls leave the residual stream after
+        every layer run in buf (device f32 [layer_runs, rows, n_embd]); None switches it off"""
+        check(lib().b200_stage_trace_residual(self.h, ptr(buf)))
+
+    def seq_pos(self, seq):
+        return lib().b200_stage_seq_pos(self.h, seq)
+
+    def state_bytes(self):
+        """device bytes of the caches and states of one sequence slot"""
+        return lib().b200_stage_state_bytes(self.h)
 
     def kernel_launches(self):
         return lib().b200_stage_kernel_launches(self.h)
