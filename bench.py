@@ -294,6 +294,138 @@ def run_sweep(args):
                 print(json.dumps(micro_one(N, K, M, tname, max(4, args.micro_iters // (1 + M // 64)))), flush=True)
 
 
+# Gonetar-shaped models (gated linear recurrence, windowed latent attention every third layer) at layer sizes of real
+# recurrent models, each next to a K-quant decoder of the same width, depth, feed-forward and vocabulary
+ARCH_SIZES = {
+    "gonetar-2b": dict(width=2560, rec=2560, blocks=10, ff=7680, heads=20, kv=4, n_layer=26),
+    "gonetar-4b": dict(width=3072, rec=3072, blocks=12, ff=9216, heads=24, kv=8, n_layer=32),
+    "gonetar-9b": dict(width=4096, rec=4096, blocks=16, ff=12288, heads=32, kv=8, n_layer=38),
+}
+ARCH_VOCAB, ARCH_WINDOW, ARCH_RANK, ARCH_DIM, ARCH_ROT, ARCH_VDIM = 128256, 2048, 512, 128, 64, 128
+
+
+def arch_stage(z, n_layer, n_ctx, ubatch, local, precision=0):
+    """a stage of that size with random weights; pattern: two recurrent layers, one of attention"""
+    from mesh_llm_b200 import capi
+    from mesh_llm_b200.stage import Stage
+
+    layers = []
+    for i in range(n_layer):
+        l = capi.LayerConfig(ffn=capi.FFN_CLAMPED_GLU, n_ff=z["ff"], glu_limit=7.0, glu_alpha=1.702)
+        if i % 3 == 2:
+            l.mixer, l.n_head, l.qk_dim, l.rot_dim, l.rot_dims = capi.MIXER_LATENT_ATTN, z["heads"], ARCH_DIM, ARCH_ROT, ARCH_ROT
+            l.v_dim, l.kv_rank, l.window = ARCH_VDIM, ARCH_RANK, ARCH_WINDOW
+            l.rope_base, l.attn_scale = 1e4, (ARCH_DIM + ARCH_ROT) ** -0.5
+        else:
+            l.mixer, l.rec_width, l.rec_blocks, l.conv_taps, l.rec_decay = capi.MIXER_LINEAR_REC, z["rec"], z["blocks"], 4, 8.0
+        layers.append(l)
+    stack = capi.StackConfig(loop_times=1, precision=precision, embd_scale=z["width"] ** 0.5, norm_offset=1.0)
+    st = Stage(stack=stack, layers=layers, n_layer=n_layer, n_embd=z["width"], n_vocab=ARCH_VOCAB, n_ctx=n_ctx, n_seq=1,
+               n_ubatch=ubatch, device=local)
+    st.generate(20251125)
+    return st
+
+
+def arch_work(z, n_layer):
+    """per token: (bytes of projection weights, bytes of gate weights, flops of a prompt's matrix products)"""
+    h, W, H = z["width"], z["rec"], z["heads"]
+    n_att = sum(1 for i in range(n_layer) if i % 3 == 2)
+    n_rec = n_layer - n_att
+    rec = 3 * h * W
+    att = h * (H * (ARCH_DIM + ARCH_ROT) + ARCH_RANK + ARCH_ROT + H) + H * ARCH_VDIM * h
+    lat = ARCH_RANK * H * (ARCH_DIM + ARCH_VDIM)
+    ff = 3 * h * z["ff"]
+    proj = n_rec * rec + n_att * att + n_layer * ff + ARCH_VOCAB * h
+    gates = n_rec * 2 * W * (W // z["blocks"])
+    return 2 * proj, 2 * gates, 2 * n_att * lat, 2 * (n_rec * rec + n_att * att + n_layer * ff) + 3 * 2 * gates // 2 + 2 * n_att * lat
+
+
+def run_arch(args):
+    """--arch: prefill and decode of Gonetar-shaped models and of the K-quant decoder of equal size; one JSON line each"""
+    import ctypes as C
+
+    import torch
+
+    from mesh_llm_b200.capi import check, lib
+    from mesh_llm_b200.stage import Stage
+
+    local = 0
+    torch.cuda.set_device(local)
+    dev = torch.device("cuda", local)
+    hbm, hbm_src = hbm_peak()
+    try:
+        tf = float(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops_sustained"])
+    except Exception:
+        tf = 1400.0
+    prompt, steps = 4096, max(16, args.steps)
+    names = sorted(ARCH_SIZES) if args.arch == "all" else [args.arch]
+    for name in names:
+        z = ARCH_SIZES[name]
+        L = args.layers or z["n_layer"]
+        for kind in ("gonetar", "kquant"):
+            n_ctx = prompt + 4 * steps + 64
+            if kind == "gonetar":
+                st = arch_stage(z, L, n_ctx, 2048, local)
+            else:
+                st = Stage(n_layer=L, n_embd=z["width"], n_head=z["heads"], n_head_kv=z["kv"], head_dim=128, n_ff=z["ff"],
+                           n_vocab=ARCH_VOCAB, n_ctx=n_ctx, n_seq=1, n_ubatch=2048, device=local)
+                st.generate(20251125)
+            out = {"arch": kind, "size": name, "layers": L, "weight_bytes": st.weight_bytes(), "data": "synthetic, random weights",
+                   "prompt": prompt, "window": ARCH_WINDOW if kind == "gonetar" else None}
+            toks = torch.from_numpy(np.random.default_rng(1).integers(0, ARCH_VOCAB, prompt).astype(np.int32)).to(dev)
+            logits = torch.empty((1, ARCH_VOCAB), dtype=torch.float32, device=dev)
+            nxt = torch.zeros(1, dtype=torch.int32, device=dev)
+            sampler = ClockSampler(local)
+            sampler.start()
+            t0 = time.time()
+            for ub in (512, 2048):
+                best = 0.0
+                for _ in range(4):  # the first pass is the warm-up
+                    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                    torch.cuda.synchronize()
+                    e0.record()
+                    for p in range(0, prompt, ub):
+                        st.forward(tokens=toks[p:p + ub], n_seq=1, T=ub, pos0=p, logits=logits, next_tokens=nxt)
+                    e1.record()
+                    torch.cuda.synchronize()
+                    best = max(best, prompt / (e0.elapsed_time(e1) * 1e-3))
+                out[f"prefill_ubatch{ub}_tok_s"] = best
+            pos = prompt
+            for timed in (False, True):
+                e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+                torch.cuda.synchronize()
+                e0.record()
+                for _ in range(steps):
+                    st.forward(tokens=nxt, n_seq=1, T=1, pos0=pos, logits=logits, next_tokens=nxt)
+                    pos += 1
+                e1.record()
+                torch.cuda.synchronize()
+                out["decode_tok_s"] = steps / (e0.elapsed_time(e1) * 1e-3)
+            for cls, label in ((1, "gemv"), (2, "attention"), (4, "other"), (7, "step")):
+                ms, n = C.c_float(), C.c_int64()
+                check(lib().b200_stage_profile_decode(st.h, 1, pos, cls, 10, C.byref(ms), C.byref(n)))
+                out[f"{label}_ms"], out[f"{label}_launches"] = ms.value, int(n.value)
+            out["clocks"] = sampler.stop(t0, time.time())
+            st.synchronize()
+            if kind == "gonetar":
+                proj, gates, lat, flops = arch_work(z, L)
+                out["gemv_frac_of_hbm_peak"] = proj / (out["gemv_ms"] * 1e-3) / 1e9 / hbm
+                out["step_frac_of_hbm_peak"] = (proj + gates + lat) / (out["step_ms"] * 1e-3) / 1e9 / hbm
+                out["prefill_frac_of_bf16_peak"] = out["prefill_ubatch2048_tok_s"] * flops / 1e12 / tf
+            else:
+                w = dict(n_embd=z["width"], n_head=z["heads"], n_head_kv=z["kv"], head_dim=128, n_ff=z["ff"], n_vocab=ARCH_VOCAB)
+                b = step_gemv_bytes(w, 0, L, True)
+                out["gemv_frac_of_hbm_peak"] = b / (out["gemv_ms"] * 1e-3) / 1e9 / hbm
+                out["step_frac_of_hbm_peak"] = b / (out["step_ms"] * 1e-3) / 1e9 / hbm
+                flops = 2 * sum(N * K for l in range(L) for (N, K, _) in matmuls(w, l))
+                out["prefill_frac_of_bf16_peak"] = out["prefill_ubatch2048_tok_s"] * flops / 1e12 / tf
+            out["hbm_peak_source"] = hbm_src
+            print(json.dumps(out), flush=True)
+            st.close()
+            del st
+            torch.cuda.empty_cache()
+
+
 # ------------------------------------------------------------------------------------------------
 def main():
     ap = argparse.ArgumentParser()
@@ -323,7 +455,11 @@ def main():
     ap.add_argument("--no-extras", action="store_true", help="N = 1: skip the cfg3 / cfg4 / cfg1-against-CPU measurements "
                     "that follow the headline workload in the same run")
     ap.add_argument("--sweep", action="store_true", help="the isolated matmul sweep: all shapes x types x M")
+    ap.add_argument("--arch", default="", choices=["", "all"] + sorted(ARCH_SIZES), help="prefill and decode of a Gonetar-shaped "
+                    "model (random weights) next to the K-quant decoder of equal size; one JSON line each")
     args = ap.parse_args()
+    if args.arch:
+        return run_arch(args)
     if args.micro:
         return run_micro(args)
     if args.micro_attn:

@@ -193,6 +193,9 @@ B200_API size_t b200_mul_mat_scratch_bytes(int64_t M, int64_t K);
 B200_API b200_status b200_mul_mat(uint32_t type, const void *W, const float *x, int64_t M,
                                   int64_t N, int64_t K, float *y, void *scratch,
                                   size_t scratch_bytes, void *stream);
+/* b200_mul_mat also takes B200_TYPE_BF16 rows (zero-padded to 64 elements: b200_device_row_bytes), any K: f32
+ * products for M <= 8, bf16 operands on tensor cores above; scratch of at least this many bytes.       */
+B200_API size_t b200_mul_mat_bf16_scratch_bytes(int64_t M, int64_t K);
 /* same contraction on already-quantised activations, with optional fused epilogue:
  * y = W.x (+ bias[N]) (+ residual[M][N])                                                       */
 B200_API b200_status b200_mul_mat_q8(uint32_t type, const void *W, const int8_t *q, const float *d,

@@ -190,6 +190,7 @@ SIGNATURES = {
     "b200_gguf_byte_profile": (i32, [vp, C.POINTER(GgufByteProfile)]),
     "b200_gguf_stage_config": (i32, [vp, i32, i32, i32, i32, i32, i32, C.POINTER(StageConfig)]),
     "b200_stage_load_gguf": (i32, [vp, vp, C.POINTER(i64), C.POINTER(i64)]),
+    "b200_mul_mat_bf16_scratch_bytes": (sz, [i64, i64]),
     "b200_stage_create_layers": (i32, [C.POINTER(StageConfig), C.POINTER(StackConfig), C.POINTER(LayerConfig),
                                        C.POINTER(vp)]),
     "b200_stage_trace_residual": (i32, [vp, vp]),

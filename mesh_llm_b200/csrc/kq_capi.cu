@@ -1,6 +1,6 @@
 // C ABI plumbing: error strings, registry / device queries, and the MUL_MAT entry points that pick
 // between the decode GEMV (M <= 8) and the prefill GEMM.
-#include "kq_common.cuh"
+#include "kq_dense.cuh"
 
 #include <stdarg.h>
 #include <stdlib.h>
@@ -163,8 +163,27 @@ b200_status b200_mul_mat_q8(uint32_t type, const void *W, const int8_t *q, const
     return kq_launch_gemm(type, (const uint8_t *)W, q, d, bsum16, M, N, K, y, bias, residual, st);
 }
 
+size_t b200_mul_mat_bf16_scratch_bytes(int64_t M, int64_t K) { return M <= 8 ? 256 : (size_t)(M * kq_bf16_ld(K) * 2 + 256); }
+
+static b200_status mul_mat_bf16(const void *W, const float *x, int64_t M, int64_t N, int64_t K, float *y, void *scratch,
+                                size_t scratch_bytes, cudaStream_t st) {
+    KQ_REQUIRE(M > 0 && N > 0 && K > 0, "mul_mat: bad shape");
+    KqDense c;
+    c.M = (int32_t)M, c.K = (int32_t)K, c.ldw = kq_bf16_ld(K), c.nseg = 1;
+    c.seg[0] = {};
+    c.seg[0].W = (const uint16_t *)W, c.seg[0].n_rows = (int32_t)N, c.seg[0].y = y, c.seg[0].ldy = N;
+    KqNormPrep p;
+    p.x = x, p.ldx = K;
+    if (M <= 8) return kq_gemv_bf16(c, p, st);
+    KQ_REQUIRE(scratch && scratch_bytes >= b200_mul_mat_bf16_scratch_bytes(M, K) && ((uintptr_t)scratch & 255) == 0,
+               "mul_mat: scratch of %zu bytes, 256-byte aligned", b200_mul_mat_bf16_scratch_bytes(M, K));
+    const b200_status rc = kq_norm_prep(p, M, (int)K, nullptr, 0, (uint16_t *)scratch, kq_bf16_ld(K), st);
+    return rc == B200_OK ? kq_gemm_bf16(c, (const uint16_t *)scratch, kq_bf16_ld(K), 1, st) : rc;
+}
+
 b200_status b200_mul_mat(uint32_t type, const void *W, const float *x, int64_t M, int64_t N, int64_t K,
                          float *y, void *scratch, size_t scratch_bytes, void *stream) {
+    if (type == B200_TYPE_BF16) return mul_mat_bf16(W, x, M, N, K, y, scratch, scratch_bytes, (cudaStream_t)stream);
     KQ_REQUIRE(M > 0 && K > 0 && K % 256 == 0, "mul_mat: bad shape");
     KQ_REQUIRE(scratch && scratch_bytes >= b200_mul_mat_scratch_bytes(M, K),
                "mul_mat: scratch too small (%zu < %zu)", scratch_bytes, b200_mul_mat_scratch_bytes(M, K));

@@ -160,3 +160,15 @@ size_t kq_latent_scratch_bytes(int n_head, int kv_rank, int max_keys);
 size_t kq_latent_counter_bytes(int n_head);
 b200_status kq_latent_attention(const KqLatent &l, const float *q_lat, int n_seq, int T, const int32_t *pos0_dev, int pos0,
                                 int max_keys, float *o_lat, float *scratch, size_t scratch_bytes, int *counters, cudaStream_t st);
+
+// ---- kq_latent_prefill.cu: the expanded form for prompts of one sequence, bf16 cache
+struct KqLatentPrefill {
+    const uint16_t *uk, *uv; // bf16 [n_head * dim][kq_bf16_ld(kv_rank)]
+    void *work;              // kq_latent_prefill_bytes, zeroed once
+    size_t work_bytes;
+};
+size_t kq_latent_prefill_bytes(const KqLatent &l, int max_rows, int max_keys);
+// q [T][n_head * (qk_dim + rot_dim)] f32, rotated; out bf16 [T][ldo]: head h's output times sigmoid(gate[t][h]).  The new
+// rows are in the cache already.  B200_ERR_UNSUPPORTED: shapes the kernel is not built for.
+b200_status kq_latent_prefill(const KqLatent &l, const KqLatentPrefill &w, const float *q, int64_t ldq, const float *gate, int64_t ldg,
+                              int T, int pos0, uint16_t *out, int64_t ldo, cudaStream_t st);

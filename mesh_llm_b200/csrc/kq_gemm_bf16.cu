@@ -10,14 +10,11 @@
 // Every wait is bounded; on a time-out the kernel records an error, lets its copies land, frees its TMEM and
 // returns.
 #include "kq_dense.cuh"
+#include "kq_tc.cuh"
 
-#include <cuda.h>
 #include <string.h>
 
 #include <algorithm>
-
-b200_status kq_tmap_encode(void *map128, int elem_bytes, int rank, const void *base, const uint64_t *dims,
-                           const uint64_t *strides_bytes, const uint32_t *box, int swizzle128);
 
 namespace {
 
@@ -30,42 +27,8 @@ constexpr uint64_t LIMIT = 5 * KQ_WAIT_LIMIT_NS;
 
 __device__ int g_gemm_bf16_error;
 
-__device__ __forceinline__ uint32_t smem_u32(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
-
-// K-major operand, rows of 128 bytes under the 128-byte swizzle, 8-row groups 1024 bytes apart; K step s of 16
-__device__ __forceinline__ uint64_t desc_k(uint32_t tile, int s) {
-    uint64_t d = 0;
-    d |= (uint64_t)(((tile + s * 32) & 0x3FFFF) >> 4);
-    d |= (uint64_t)(16 >> 4) << 16;
-    d |= (uint64_t)(1024 >> 4) << 32;
-    d |= (uint64_t)1 << 46; // descriptor version of this architecture
-    d |= (uint64_t)2 << 61; // SWIZZLE_128B
-    return d;
-}
 // kind::f16: D f32, A bf16, B bf16, both K-major, M = 128, N = 128
-constexpr uint32_t IDESC = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(TN >> 3) << 17) | ((uint32_t)(TM >> 4) << 24);
-
-__device__ __forceinline__ void mma(uint32_t d_tmem, uint64_t a, uint64_t b, uint32_t acc) {
-    asm volatile("{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
-                 "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}"
-                 :
-                 : "r"(d_tmem), "l"(a), "l"(b), "r"(IDESC), "r"(acc)
-                 : "memory");
-}
-__device__ __forceinline__ void commit(uint32_t bar) {
-    asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
-}
-
-#define TMEM_LD32(taddr, r)                                                                                             \
-    asm volatile("tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,"        \
-                 "%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"                              \
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]),      \
-                   "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), \
-                   "=r"(r[16]), "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]),            \
-                   "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]),            \
-                   "=r"(r[30]), "=r"(r[31])                                                                             \
-                 : "r"(taddr)                                                                                           \
-                 : "memory")
+constexpr uint32_t IDESC = tc_idesc(TM, TN, true, false);
 
 struct GemmParams {
     CUtensorMap a, b[3];
@@ -76,7 +39,7 @@ struct GemmParams {
 
 // eight consecutive output columns of one row
 __device__ __forceinline__ void put8(const KqDense &c, const KqDenseSeg &s, int64_t m, int64_t n, int g, const float *v, int n_valid) {
-    if (n_valid == 8 && s.head_in == 0 && (s.ldy & 7) == 0 && (n & 7) == 0) {
+    if (n_valid == 8 && ((s.ldy | n | s.head_in | s.head_out) & 7) == 0) { // all eight in one head, 16-byte aligned
         float o[8];
 #pragma unroll
         for (int j = 0; j < 8; j++) {
@@ -86,7 +49,7 @@ __device__ __forceinline__ void put8(const KqDense &c, const KqDenseSeg &s, int6
             if (c.head_gate) t *= kq_sigmoid(c.head_gate[m * c.ld_gate + g]);
             o[j] = t;
         }
-        const int64_t i = m * s.ldy + n;
+        const int64_t i = m * s.ldy + kq_dense_col(s, n);
         if (s.out == KQ_OUT_F32) {
             float *y = (float *)s.y + i;
             *reinterpret_cast<float4 *>(y) = make_float4(o[0], o[1], o[2], o[3]);
@@ -112,7 +75,8 @@ __global__ void __launch_bounds__(NTHREADS, 2) gemm_bf16_kernel(const __grid_con
     __shared__ uint64_t full[STAGES], empty[STAGES], done;
     __shared__ uint32_t s_tmem;
     __shared__ int s_abort;
-    KQ_PDL_TRIGGER();
+    // the wait comes before the TMEM allocation: a CTA that started early must not hold columns its predecessor needs
+    KQ_PDL_ENTER();
     uint8_t *sm = (uint8_t *)(((uintptr_t)sm_raw + 1023) & ~(uintptr_t)1023);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int m0 = blockIdx.x * TM, g = blockIdx.z;
@@ -141,7 +105,6 @@ __global__ void __launch_bounds__(NTHREADS, 2) gemm_bf16_kernel(const __grid_con
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t tmem = s_tmem;
     const int n_it = p.nk * p.parts;
-    KQ_PDL_WAIT();
 
     auto wait = [&](uint64_t *bar, uint32_t parity, int code) {
         if (!*(volatile int *)&s_abort && !kq_mbar_wait(smem_u32(bar), parity, LIMIT)) {
@@ -186,10 +149,10 @@ __global__ void __launch_bounds__(NTHREADS, 2) gemm_bf16_kernel(const __grid_con
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 const uint32_t a = smem_u32(sm + s * STAGE_BYTES), b = a + A_BYTES;
 #pragma unroll
-                for (int k = 0; k < BK / 16; k++) mma(tmem, desc_k(a, k), desc_k(b, k), (it > 0 || k > 0) ? 1u : 0u);
-                commit(smem_u32(&empty[s]));
+                for (int k = 0; k < BK / 16; k++) tc_mma_ss(tmem, tc_desc_k(a, k), tc_desc_k(b, k), IDESC, (it > 0 || k > 0) ? 1u : 0u);
+                tc_commit(smem_u32(&empty[s]));
             }
-            commit(smem_u32(&done));
+            tc_commit(smem_u32(&done));
             if (*(volatile int *)&s_abort) kq_mbar_wait(smem_u32(&done), 0, KQ_WAIT_LIMIT_NS); // MMAs in flight end before TMEM is freed
         }
         __syncwarp();

@@ -17,6 +17,7 @@
 namespace {
 
 constexpr int NT = 256, NW = NT / 32, SB = 64; // threads, warps, rows between two combines
+constexpr int MAX_X_BYTES = 192 * 1024;       // activations in shared memory, next to 32 KB of partial sums at 8 rows
 
 struct GemvParams {
     KqDense c;
@@ -303,7 +304,7 @@ b200_status launch_gemv(const GemvParams &p, size_t smem, cudaStream_t st) {
     int dev = 0;
     KQ_CUDA(cudaGetDevice(&dev));
     if (dev < 0 || dev >= 16 || !attr[dev]) {
-        KQ_CUDA(cudaFuncSetAttribute(gemv_bf16_kernel<M>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+        KQ_CUDA(cudaFuncSetAttribute(gemv_bf16_kernel<M>, cudaFuncAttributeMaxDynamicSharedMemorySize, MAX_X_BYTES));
         if (dev >= 0 && dev < 16) attr[dev] = true;
     }
     static int mul = -1; // B200_GEMV16_CTAS: CTAs per SM of the decode projections
@@ -337,7 +338,7 @@ b200_status kq_gemv_bf16(const KqDense &c, const KqNormPrep &pr, cudaStream_t st
     KQ_REQUIRE(c.ldw % 64 == 0 && c.ldw >= c.K, "gemv_bf16: weight rows must be padded to 64 elements");
     const int nck = (int)kq_div_up(c.K, 8);
     const int64_t row_smem = (int64_t)nck * 32;
-    const int cap = (int)std::min<int64_t>(8, 190 * 1024 / row_smem);
+    const int cap = (int)std::min<int64_t>(8, MAX_X_BYTES / row_smem);
     if (cap < 1) {
         kq_set_error("gemv_bf16: rows of %d values do not fit in shared memory", c.K);
         return B200_ERR_UNSUPPORTED;

@@ -18,16 +18,6 @@
 
 #include <algorithm>
 
-// expanded form of latent attention for prompts (kq_latent_prefill.cu)
-struct KqLatentPrefill {
-    const uint16_t *uk, *uv; // bf16 [n_head * dim][kq_bf16_ld(kv_rank)]
-    void *work;
-    size_t work_bytes;
-};
-size_t kq_latent_prefill_bytes(const KqLatent &l, int max_rows, int max_keys);
-b200_status kq_latent_prefill(const KqLatent &l, const KqLatentPrefill &w, const float *q, int64_t ldq, const float *gate, int64_t ldg,
-                              int T, int pos0, uint16_t *out, int64_t ldo, cudaStream_t st);
-
 struct LayerDesc {
     b200_layer_config c;
     const float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;

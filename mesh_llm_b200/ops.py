@@ -11,7 +11,7 @@ import ctypes as C
 import torch
 
 from . import capi
-from .capi import TYPE_F32, TYPE_Q4_K, TYPE_Q6_K, check, lib, ptr, cur_stream
+from .capi import TYPE_BF16, TYPE_F32, TYPE_Q4_K, TYPE_Q6_K, check, lib, ptr, cur_stream
 
 Q4K_BYTES, Q6K_BYTES = 144, 210
 
@@ -49,6 +49,26 @@ def download_weights(type_, dev_rows, n_rows, k):
     out = torch.empty(n_rows * row_bytes(type_, k), dtype=torch.uint8, device=dev_rows.device)
     check(lib().b200_unpack_q6k(ptr(dev_rows), ptr(out), n_rows, k, cur_stream()))
     return out
+
+
+def upload_bf16(w, device="cuda"):
+    """[N, K] float matrix -> device-layout bf16 rows (zero-padded to a multiple of 64 elements)"""
+    w = torch.as_tensor(w).to(device=device, dtype=torch.bfloat16)
+    ld = device_row_bytes(TYPE_BF16, w.shape[1]) // 2
+    out = torch.zeros((w.shape[0], ld), dtype=torch.bfloat16, device=device)
+    out[:, :w.shape[1]] = w
+    return out
+
+
+def mul_mat_bf16(W, x, N, K):
+    """W from upload_bf16, x [M, K] f32 -> y [M, N] f32"""
+    x = _dev(x).contiguous().float().reshape(-1, K)
+    M = x.shape[0]
+    need = lib().b200_mul_mat_bf16_scratch_bytes(M, K)
+    scratch = torch.empty(need, dtype=torch.uint8, device=x.device)
+    y = torch.empty((M, N), dtype=torch.float32, device=x.device)
+    check(lib().b200_mul_mat(TYPE_BF16, ptr(W), ptr(x), M, N, K, ptr(y), ptr(scratch), need, cur_stream()))
+    return y
 
 
 def quantize_act(x):
