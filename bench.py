@@ -298,7 +298,7 @@ def run_sweep(args):
 # recurrent models, each next to a K-quant decoder of the same width, depth, feed-forward and vocabulary
 ARCH_SIZES = {
     "gonetar-2b": dict(width=2560, rec=2560, blocks=10, ff=7680, heads=20, kv=4, n_layer=26),
-    "gonetar-4b": dict(width=3072, rec=3072, blocks=12, ff=9216, heads=24, kv=8, n_layer=32),
+    "gonetar-4b": dict(width=3072, rec=3072, blocks=12, ff=9216, heads=24, kv=6, n_layer=32),
     "gonetar-9b": dict(width=4096, rec=4096, blocks=16, ff=12288, heads=32, kv=8, n_layer=38),
 }
 ARCH_VOCAB, ARCH_WINDOW, ARCH_RANK, ARCH_DIM, ARCH_ROT, ARCH_VDIM = 128256, 2048, 512, 128, 64, 128

@@ -153,13 +153,19 @@ static inline int kq_latent_ld(int kv_rank, int rot_dim) { return (int)(kq_pad(k
 b200_status kq_latent_store(const KqLatent &l, const float *norm_w, float eps, float *q, int64_t ldq, const float *kv,
                             int64_t ldkv, int n_seq, int T, const int32_t *pos0_dev, int pos0, float *q_lat, int64_t ldql,
                             cudaStream_t st);
-// attention over the latent rows: q_lat [rows][n_head][ld] (absorbed queries, same layout as a cache row) ->
-// o_lat [rows][n_head][kq_f32_ld(kv_rank)]
-// (max_keys: the most keys a row can see; counters: zero between launches)
-size_t kq_latent_scratch_bytes(int n_head, int kv_rank, int max_keys);
-size_t kq_latent_counter_bytes(int n_head);
-b200_status kq_latent_attention(const KqLatent &l, const float *q_lat, int n_seq, int T, const int32_t *pos0_dev, int pos0,
-                                int max_keys, float *o_lat, float *scratch, size_t scratch_bytes, int *counters, cudaStream_t st);
+// Few rows: the store, and in the same launch the absorbed queries q_lat[row][h] = [W_uk[h]^T q_unrot | q_rot]
+// (rows laid out like a cache row; `absorb` is that block-diagonal product)
+constexpr int KQ_LATENT_ROWS = 8;
+b200_status kq_latent_query(const KqLatent &l, const float *norm_w, float eps, float *q, int64_t ldq, const float *kv, int64_t ldkv, int n_seq,
+                            int T, const int32_t *pos0_dev, int pos0, float *q_lat, int64_t ldql, const KqDense &absorb, cudaStream_t st);
+// Attention over the latent rows.  o_lat given: o_lat [rows][n_head][kq_f32_ld(kv_rank)].  Otherwise (up to KQ_LATENT_ROWS
+// rows) partial results of key ranges in scratch, for kq_latent_output: out[row][h * v_dim ..] = sigmoid(gate[row][h]) W_uv[h] o.
+// max_keys: the most keys a row can see.
+size_t kq_latent_scratch_bytes(const KqLatent &l, int max_keys);
+b200_status kq_latent_attention(const KqLatent &l, const float *q_lat, int n_seq, int T, const int32_t *pos0_dev, int pos0, int max_keys,
+                                float *o_lat, float *scratch, size_t scratch_bytes, cudaStream_t st);
+b200_status kq_latent_output(const KqLatent &l, const float *scratch, int n_seq, int T, const int32_t *pos0_dev, int pos0, int max_keys,
+                             const uint16_t *uv, const float *gate, int64_t ldg, float *out, int64_t ldo, cudaStream_t st);
 
 // ---- kq_latent_prefill.cu: the expanded form for prompts of one sequence, bf16 cache
 struct KqLatentPrefill {

@@ -9,7 +9,7 @@
 // warps' through shared memory once per 64 rows.  The prologue can add a normed sub-layer output to the
 // residual and norm the result (every CTA does that for itself; CTA 0 also leaves the new residual), the
 // first weights are requested before the dependency wait.
-#include "kq_dense.cuh"
+#include "kq_gemv_grouped.cuh"
 
 #include <algorithm>
 #include <stdlib.h>
@@ -25,16 +25,6 @@ struct GemvParams {
     int32_t V;   // rows in all (a gate / up pair is two), in the order they are walked
     int32_t nck; // 16-byte chunks per weight row
 };
-
-__device__ __forceinline__ float4 load4(const float *p, int k, int K, bool vec) {
-    if (vec && k + 3 < K) return *reinterpret_cast<const float4 *>(p + k);
-    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (k < K) v.x = p[k];
-    if (k + 1 < K) v.y = p[k + 1];
-    if (k + 2 < K) v.z = p[k + 2];
-    if (k + 3 < K) v.w = p[k + 3];
-    return v;
-}
 
 __device__ __forceinline__ float block_sum(float v, float *red) {
     v = kq_warp_sum(v);
@@ -110,16 +100,16 @@ __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __g
             if (p.p.sub_w) {
                 float s2 = 0.f;
                 for (int i = tid; i < n4; i += NT) {
-                    const float4 v = load4(sub, 4 * i, K, vec);
+                    const float4 v = kq_load4(sub, 4 * i, K, vec);
                     s2 += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
                 }
                 sc = 1.0f / sqrtf(block_sum(s2, red) / (float)K + p.p.eps);
             }
             for (int i = tid; i < n4; i += NT) {
-                const float4 a = load4(x, 4 * i, K, vec), b = load4(sub, 4 * i, K, vec);
+                const float4 a = kq_load4(x, 4 * i, K, vec), b = kq_load4(sub, 4 * i, K, vec);
                 float4 g = make_float4(1.f, 1.f, 1.f, 1.f);
                 if (p.p.sub_w) {
-                    g = load4(p.p.sub_w, 4 * i, K, true);
+                    g = kq_load4(p.p.sub_w, 4 * i, K, true);
                     g.x += p.p.w_off, g.y += p.p.w_off, g.z += p.p.w_off, g.w += p.p.w_off;
                 }
                 float4 v = make_float4(a.x + b.x * sc * g.x, a.y + b.y * sc * g.y, a.z + b.z * sc * g.z, a.w + b.w * sc * g.w);
@@ -138,7 +128,7 @@ __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __g
             }
         } else {
             for (int i = tid; i < n4; i += NT) {
-                const float4 v = load4(x, 4 * i, K, vec);
+                const float4 v = kq_load4(x, 4 * i, K, vec);
                 ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
                 px[(i & 1) * nck + (i >> 1)] = v;
             }
@@ -146,7 +136,7 @@ __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __g
         if (p.p.norm_w) {
             const float sc = 1.0f / sqrtf(block_sum(ss, red) / (float)K + p.p.eps);
             for (int i = tid; i < n4; i += NT) {
-                const float4 g = load4(p.p.norm_w, 4 * i, K, true);
+                const float4 g = kq_load4(p.p.norm_w, 4 * i, K, true);
                 float4 v = px[(i & 1) * nck + (i >> 1)];
                 v.x *= sc * (p.p.w_off + g.x), v.y *= sc * (p.p.w_off + g.y);
                 v.z *= sc * (p.p.w_off + g.z), v.w *= sc * (p.p.w_off + g.w);
@@ -183,17 +173,7 @@ __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __g
                             const float4 a = pl[(m * 2) * nck + c], b = pl[(m * 2 + 1) * nck + c];
 #pragma unroll
                             for (int r = 0; r < 4; r++) {
-                                const uint4 q = w[r][j];
-                                float s = acc[r][m];
-                                s = fmaf(__uint_as_float(q.x << 16), a.x, s);
-                                s = fmaf(__uint_as_float(q.x & 0xffff0000u), a.y, s);
-                                s = fmaf(__uint_as_float(q.y << 16), a.z, s);
-                                s = fmaf(__uint_as_float(q.y & 0xffff0000u), a.w, s);
-                                s = fmaf(__uint_as_float(q.z << 16), b.x, s);
-                                s = fmaf(__uint_as_float(q.z & 0xffff0000u), b.y, s);
-                                s = fmaf(__uint_as_float(q.w << 16), b.z, s);
-                                s = fmaf(__uint_as_float(q.w & 0xffff0000u), b.w, s);
-                                acc[r][m] = s;
+                                acc[r][m] = kq_dot8(w[r][j], a, b, acc[r][m]);
                             }
                         }
                     }
@@ -234,68 +214,10 @@ __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __g
     }
 }
 
-// Block-diagonal form: one warp per four rows of a group, activations from L1 / L2.
-struct GroupedParams {
-    KqDense c;
-    const float *x;
-    int64_t ldx;
-    int32_t quads; // four-row units per group and segment
-    int32_t vec;
-};
-
 template <int M>
-__global__ void __launch_bounds__(NT) gemv_grouped_bf16_kernel(const __grid_constant__ GroupedParams p) {
+__global__ void __launch_bounds__(NT) gemv_grouped_bf16_kernel(const __grid_constant__ KqGrouped p) {
     KQ_PDL_TRIGGER();
-    const int lane = threadIdx.x & 31;
-    const int64_t id = (int64_t)blockIdx.x * NW + (threadIdx.x >> 5), n_id = (int64_t)p.quads * p.c.groups * p.c.nseg;
-    KQ_PDL_WAIT();
-    if (id >= n_id) return;
-    const int sg = (int)(id / ((int64_t)p.quads * p.c.groups));
-    const int64_t rem = id % ((int64_t)p.quads * p.c.groups);
-    const int g = (int)(rem / p.quads), r0 = (int)(rem % p.quads) * 4;
-    const KqDenseSeg &s = p.c.seg[sg];
-    if (r0 >= s.n_rows) return;
-    const int K = p.c.K, nck = (int)((K + 7) / 8);
-    const uint4 *wp[4];
-#pragma unroll
-    for (int r = 0; r < 4; r++)
-        wp[r] = reinterpret_cast<const uint4 *>(s.W + ((int64_t)g * s.n_rows + min(r0 + r, s.n_rows - 1)) * p.c.ldw);
-    float acc[4][M];
-#pragma unroll
-    for (int r = 0; r < 4; r++)
-#pragma unroll
-        for (int m = 0; m < M; m++) acc[r][m] = 0.f;
-    for (int c = lane; c < nck; c += 32) {
-        uint4 w[4];
-#pragma unroll
-        for (int r = 0; r < 4; r++) w[r] = kq_ld_stream(wp[r] + c);
-#pragma unroll
-        for (int m = 0; m < M; m++) {
-            const float *x = p.x + m * p.ldx + g * p.c.xg;
-            const float4 a = load4(x, 8 * c, K, p.vec), b = load4(x, 8 * c + 4, K, p.vec);
-#pragma unroll
-            for (int r = 0; r < 4; r++) {
-                const uint4 q = w[r];
-                float t = acc[r][m];
-                t = fmaf(__uint_as_float(q.x << 16), a.x, t);
-                t = fmaf(__uint_as_float(q.x & 0xffff0000u), a.y, t);
-                t = fmaf(__uint_as_float(q.y << 16), a.z, t);
-                t = fmaf(__uint_as_float(q.y & 0xffff0000u), a.w, t);
-                t = fmaf(__uint_as_float(q.z << 16), b.x, t);
-                t = fmaf(__uint_as_float(q.z & 0xffff0000u), b.y, t);
-                t = fmaf(__uint_as_float(q.w << 16), b.z, t);
-                t = fmaf(__uint_as_float(q.w & 0xffff0000u), b.w, t);
-                acc[r][m] = t;
-            }
-        }
-    }
-#pragma unroll
-    for (int r = 0; r < 4; r++)
-#pragma unroll
-        for (int m = 0; m < M; m++) {
-            const float v = kq_warp_sum(acc[r][m]);
-            if (lane == 0 && r0 + r < s.n_rows) kq_dense_store(p.c, s, m, (int64_t)g * s.n_rows + r0 + r, g, v);
-        }
+    kq_grouped_rows<M>(p, (int64_t)blockIdx.x * NW + (threadIdx.x >> 5), threadIdx.x & 31);
 }
 
 template <int M>
@@ -321,16 +243,6 @@ b200_status launch_gemv(const GemvParams &p, size_t smem, cudaStream_t st) {
     return B200_OK;
 }
 
-// the call for rows m0 .. m0 + m - 1 of a larger one
-KqDense rows_of(const KqDense &c, int m0, int m) {
-    KqDense d = c;
-    d.M = m;
-    for (int i = 0; i < d.nseg; i++)
-        d.seg[i].y = (uint8_t *)c.seg[i].y + m0 * c.seg[i].ldy * (c.seg[i].out == KQ_OUT_F32 ? 4 : 2);
-    if (d.head_gate) d.head_gate += m0 * d.ld_gate;
-    return d;
-}
-
 } // namespace
 
 b200_status kq_gemv_bf16(const KqDense &c, const KqNormPrep &pr, cudaStream_t st) {
@@ -347,7 +259,7 @@ b200_status kq_gemv_bf16(const KqDense &c, const KqNormPrep &pr, cudaStream_t st
         const int left = c.M - m0;
         const int m = left >= 8 && cap >= 8 ? 8 : left >= 4 && cap >= 4 ? 4 : left >= 2 && cap >= 2 ? 2 : 1;
         GemvParams p;
-        p.c = rows_of(c, m0, m);
+        p.c = kq_rows_of(c, m0, m);
         p.p = pr;
         p.p.x += m0 * pr.ldx;
         if (pr.sub) p.p.sub += m0 * pr.ld_sub;
@@ -373,13 +285,7 @@ b200_status kq_gemv_grouped_bf16(const KqDense &c, const float *x, int64_t ldx, 
     KQ_REQUIRE(c.M >= 1 && c.nseg >= 1 && c.nseg <= 3 && c.groups >= 1 && !c.glu, "gemv_grouped_bf16: bad call");
     for (int m0 = 0; m0 < c.M;) {
         const int left = c.M - m0, m = left >= 4 ? 4 : left >= 2 ? 2 : 1;
-        GroupedParams p;
-        p.c = rows_of(c, m0, m);
-        p.x = x + m0 * ldx;
-        p.ldx = ldx;
-        p.quads = 0;
-        for (int i = 0; i < c.nseg; i++) p.quads = std::max<int>(p.quads, (int)kq_div_up(c.seg[i].n_rows, 4));
-        p.vec = (ldx % 4 == 0) && (c.xg % 4 == 0) && ((uintptr_t)x & 15) == 0;
+        const KqGrouped p = kq_grouped_params(kq_rows_of(c, m0, m), x + m0 * ldx, ldx);
         const unsigned grid = (unsigned)kq_div_up((int64_t)p.quads * c.groups * c.nseg, NW);
         if (m == 4) kq_launch(gemv_grouped_bf16_kernel<4>, grid, NT, 0, st, p);
         else if (m == 2) kq_launch(gemv_grouped_bf16_kernel<2>, grid, NT, 0, st, p);

@@ -58,7 +58,6 @@ struct KqLayers {
     uint16_t *u16 = nullptr, *z16 = nullptr, *act16 = nullptr;
     float *act32 = nullptr, *att_scratch = nullptr;
     size_t att_scratch_bytes = 0;
-    int *counters = nullptr;
     void *prefill_work = nullptr;
     size_t prefill_bytes = 0;
 };
@@ -67,7 +66,7 @@ void KqLayersDelete::operator()(KqLayers *p) const { delete p; }
 
 namespace {
 
-constexpr int SMALL_ROWS = 8;
+constexpr int SMALL_ROWS = KQ_LATENT_ROWS;
 
 // uk [H * dim][ld_in] -> uk_t [H * R][ld_out]
 __global__ void transpose_heads_kernel(const uint16_t *in, int64_t ld_in, int H, int dim, int R, uint16_t *out, int64_t ld_out) {
@@ -267,13 +266,19 @@ struct Pass {
             if (rc == B200_OK) return close(L.wo, (int64_t)H * c.v_dim, nullptr, 0, k->z16, L.norm1b);
             if (rc != B200_ERR_UNSUPPORTED) return rc;
             // q is rotated already: only its copy into the latent layout is missing
-            KQ_TRY(absorb(L, l, q, ldq, hd, q_lat, true));
+            KQ_TRY(copy_rotated(L, l, q, ldq, hd, q_lat));
+        } else if (small) {
+            const int keys = (int)max_keys(st->c, c);
+            ATTN_(kq_latent_query(l, L.kv_norm, st->c.rms_eps, q, ldq, kv, ldkv, n_seq, T, pos_dev, pos0, q_lat, (int64_t)H * l.ld,
+                                  absorb(L, l, hd, q_lat), s));
+            ATTN_(kq_latent_attention(l, q_lat, n_seq, T, pos_dev, pos0, keys, nullptr, k->att_scratch, k->att_scratch_bytes, s));
+            ATTN_(kq_latent_output(l, k->att_scratch, n_seq, T, pos_dev, pos0, keys, L.uv, g, ldg, att, lda, s));
+            return close(L.wo, (int64_t)H * c.v_dim, att, lda, nullptr, L.norm1b);
         } else {
             OTHER_(kq_latent_store(l, L.kv_norm, st->c.rms_eps, q, ldq, kv, ldkv, n_seq, T, pos_dev, pos0, q_lat, (int64_t)H * l.ld, s));
-            KQ_TRY(absorb(L, l, q, ldq, hd, q_lat, false));
         }
-        ATTN_(kq_latent_attention(l, q_lat, n_seq, T, pos_dev, pos0, (int)max_keys(st->c, c), o_lat, k->att_scratch, k->att_scratch_bytes,
-                                  k->counters, s));
+        ATTN_(kq_gemm_f32(absorb(L, l, hd, q_lat), q, ldq, s));
+        ATTN_(kq_latent_attention(l, q_lat, n_seq, T, pos_dev, pos0, (int)max_keys(st->c, c), o_lat, nullptr, 0, s));
         KqDense v = call(c.kv_rank);
         v.nseg = 1;
         v.groups = H;
@@ -282,12 +287,11 @@ struct Pass {
         v.ld_gate = ldg;
         v.seg[0] = tc ? seg(L.uv, c.v_dim, k->z16, kq_bf16_ld((int64_t)H * c.v_dim), nullptr, KQ_ACT_NONE, KQ_OUT_BF16)
                       : seg(L.uv, c.v_dim, att, lda);
-        if (small) ATTN_(kq_gemv_grouped_bf16(v, o_lat, H * rp, s));
-        else ATTN_(kq_gemm_f32(v, o_lat, H * rp, s));
+        ATTN_(kq_gemm_f32(v, o_lat, H * rp, s));
         return close(L.wo, (int64_t)H * c.v_dim, att, lda, k->z16, L.norm1b);
     }
-    // q_lat[h] = [W_uk[h]^T q_unrot | q_rot]
-    b200_status absorb(const LayerDesc &L, const KqLatent &l, const float *q, int64_t ldq, int hd, float *q_lat, bool copy_rot) {
+    // q_lat[h] = W_uk[h]^T q_unrot, into rows laid out like a cache row
+    KqDense absorb(const LayerDesc &L, const KqLatent &l, int hd, float *q_lat) {
         KqDense a = call(L.c.qk_dim);
         a.nseg = 1;
         a.groups = L.c.n_head;
@@ -295,14 +299,13 @@ struct Pass {
         a.seg[0] = seg(L.uk_t, L.c.kv_rank, q_lat, (int64_t)L.c.n_head * l.ld);
         a.seg[0].head_in = L.c.kv_rank;
         a.seg[0].head_out = l.ld;
-        if (copy_rot) {
-            KQ_CUDA(cudaMemsetAsync(q_lat, 0, (size_t)rows * L.c.n_head * l.ld * 4, s));
-            for (int i = 0; i < rows && L.c.rot_dim; i++)
-                KQ_CUDA(cudaMemcpy2DAsync(q_lat + (int64_t)i * L.c.n_head * l.ld + l.rot_at, (size_t)l.ld * 4, q + i * ldq + L.c.qk_dim, (size_t)hd * 4,
-                                          (size_t)L.c.rot_dim * 4, (size_t)L.c.n_head, cudaMemcpyDeviceToDevice, s));
-        }
-        if (small) ATTN_(kq_gemv_grouped_bf16(a, q, ldq, s));
-        else ATTN_(kq_gemm_f32(a, q, ldq, s));
+        return a;
+    }
+    b200_status copy_rotated(const LayerDesc &L, const KqLatent &l, const float *q, int64_t ldq, int hd, float *q_lat) {
+        KQ_CUDA(cudaMemsetAsync(q_lat, 0, (size_t)rows * L.c.n_head * l.ld * 4, s));
+        for (int i = 0; i < rows && L.c.rot_dim; i++)
+            KQ_CUDA(cudaMemcpy2DAsync(q_lat + (int64_t)i * L.c.n_head * l.ld + l.rot_at, (size_t)l.ld * 4, q + i * ldq + L.c.qk_dim, (size_t)hd * 4,
+                                      (size_t)L.c.rot_dim * 4, (size_t)L.c.n_head, cudaMemcpyDeviceToDevice, s));
         return B200_OK;
     }
 
@@ -500,7 +503,7 @@ b200_status b200_stage_create_layers(const b200_stage_config *cfg, const b200_st
     }
     const int64_t h = c.n_embd, R = c.n_ubatch;
     if (c.has_embd || c.has_output) kq_stage_add_tensor(st, "embed", B200_TYPE_BF16, h, c.n_vocab, 1);
-    int64_t fmax[6] = {}, wmax16 = 0, u16max = 0, ffmax = 0, scratch = 0, counters = 256, prefill = 0;
+    int64_t fmax[6] = {}, wmax16 = 0, u16max = 0, ffmax = 0, scratch = 0, prefill = 0;
     const bool f32 = stack->precision == B200_PRECISION_F32;
     auto grow = [](int64_t &a, int64_t b) { a = std::max(a, b); };
     for (int i = c.layer_begin; i < c.layer_end; i++) {
@@ -542,10 +545,10 @@ b200_status b200_stage_create_layers(const b200_stage_config *cfg, const b200_st
             grow(fmax[4], H * kq_f32_ld(l.kv_rank));
             grow(fmax[5], kq_f32_ld(H * l.v_dim));
             grow(wmax16, kq_bf16_ld(H * l.v_dim));
-            grow(scratch, (int64_t)kq_latent_scratch_bytes(l.n_head, l.kv_rank, (int)max_keys(c, l)));
-            grow(counters, (int64_t)kq_latent_counter_bytes(l.n_head));
             KqLatent q = {};
             q.n_head = l.n_head, q.qk_dim = l.qk_dim, q.rot_dim = l.rot_dim, q.v_dim = l.v_dim, q.kv_rank = l.kv_rank, q.window = l.window;
+            q.f32 = f32, q.ld = kq_latent_ld(l.kv_rank, l.rot_dim);
+            grow(scratch, (int64_t)kq_latent_scratch_bytes(q, (int)max_keys(c, l)));
             if (!f32) grow(prefill, (int64_t)kq_latent_prefill_bytes(q, (int)R, (int)std::min<int64_t>(c.n_ctx, max_keys(c, l) - 1 + R)));
         }
         if (l.ffn != B200_FFN_NONE) {
@@ -602,7 +605,6 @@ b200_status b200_stage_create_layers(const b200_stage_config *cfg, const b200_st
     if (ffmax && wide) A(&k->act16, (size_t)(R * kq_bf16_ld(ffmax) * 2));
     k->att_scratch_bytes = (size_t)scratch;
     A(&k->att_scratch, (size_t)scratch);
-    A(&k->counters, (size_t)counters);
     k->prefill_bytes = wide ? (size_t)prefill : 0;
     if (k->prefill_bytes) A(&k->prefill_work, k->prefill_bytes);
     A(&st->pos0_dev, 256);
