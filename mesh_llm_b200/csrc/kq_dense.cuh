@@ -130,7 +130,8 @@ b200_status kq_causal_conv(const KqRecW &w, const KqRecState &s, const float *x,
 b200_status kq_linear_recurrence(const KqRecW &w, const KqRecState &s, float *r, float *i, int64_t ldr, const float *u,
                                  int64_t ldu, const float *x, int64_t ldx, const float *y, int64_t ldy, int n_seq, int T,
                                  const int32_t *pos0_dev, int pos0, float *z32, int64_t ld32, uint16_t *z16, int64_t ld16,
-                                 cudaStream_t st);
+                                 float *scratch, size_t scratch_bytes, cudaStream_t st);
+size_t kq_recurrence_scratch_bytes(int width, int rows, int n_seq); // calls of up to `rows` rows
 // one token per sequence: convolution, gates, recurrence and the product with y in one launch
 b200_status kq_recurrence_step(const KqRecW &w, const KqRecState &s, const float *x, int64_t ldx, const float *y,
                                int64_t ldy, int n_seq, const int32_t *pos_dev, int pos, float *z, int64_t ldz, cudaStream_t st);

@@ -68,19 +68,19 @@ __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __g
     // first weights of this CTA: they depend on nothing
     uint4 w[4][2];
     const uint4 *wp[4];
-    auto load = [&](int i) {
+    auto load = [&](int i, int n) { // n: rows of the batch that are this CTA's
 #pragma unroll
         for (int r = 0; r < 4; r++)
 #pragma unroll
             for (int j = 0; j < 2; j++) {
                 const int c = i + j * NT;
-                w[r][j] = c < nck ? kq_ld_stream(wp[r] + c) : make_uint4(0, 0, 0, 0);
+                w[r][j] = c < nck && r < n ? kq_ld_stream(wp[r] + c) : make_uint4(0, 0, 0, 0);
             }
     };
     if (v0 < v1) {
 #pragma unroll
         for (int r = 0; r < 4; r++) wp[r] = row_ptr(v0 + r);
-        load(tid);
+        load(tid, v1 - v0);
     }
     KQ_PDL_WAIT();
 
@@ -162,7 +162,7 @@ __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __g
 #pragma unroll
                 for (int m = 0; m < M; m++) acc[r][m] = 0.f;
             for (int i = tid; i < nck; i += 2 * NT) {
-                if (!loaded) load(i);
+                if (!loaded) load(i, v1 - v);
                 loaded = false;
 #pragma unroll
                 for (int j = 0; j < 2; j++) {
@@ -232,7 +232,7 @@ b200_status launch_gemv(const GemvParams &p, size_t smem, cudaStream_t st) {
     static int mul = -1; // B200_GEMV16_CTAS: CTAs per SM of the decode projections
     if (mul < 0) {
         const char *v = getenv("B200_GEMV16_CTAS");
-        mul = v ? std::max(1, atoi(v)) : 2;
+        mul = v ? std::max(1, atoi(v)) : 4;
     }
     const int64_t units = p.V / (p.c.glu ? 2 : 1);
     const int64_t want = std::max<int64_t>(1, kq_div_up(units * (p.c.glu ? 2 : 1), 4));

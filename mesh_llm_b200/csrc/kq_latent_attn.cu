@@ -330,16 +330,23 @@ __global__ void __launch_bounds__(NT) latent_attn_mma_kernel(const __grid_consta
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     load_tile(k0);
-    for (int i = tid; i < HG * ld16 / 2; i += NT) { // queries, scaled, as hi + lo
-        const int hl = i / (ld16 / 2), d = i % (ld16 / 2) * 2, h = hg * HG + hl;
-        float2 v = make_float2(0.f, 0.f);
-        if (h < l.n_head && d < l.ld) v = *reinterpret_cast<const float2 *>(q_lat + (row * l.n_head + h) * l.ld + d);
-        const float f = l.scale * 1.4426950408889634f;
-        v.x *= f, v.y *= f;
-        const uint16_t hx = kq_f2bf(v.x), hy = kq_f2bf(v.y);
-        *reinterpret_cast<uint32_t *>(q_hi + hl * pitch + 2 * d) = (uint32_t)hx | ((uint32_t)hy << 16);
-        *reinterpret_cast<uint32_t *>(q_lo + hl * pitch + 2 * d) =
-            (uint32_t)kq_f2bf(v.x - kq_bf2f(hx)) | ((uint32_t)kq_f2bf(v.y - kq_bf2f(hy)) << 16);
+    const int nq = HG * ld16 / 2;
+    for (int i0 = tid; i0 < nq; i0 += 6 * NT) { // queries, scaled, as hi + lo; six loads in flight
+        float2 v[6];
+#pragma unroll
+        for (int e = 0; e < 6; e++) {
+            const int i = i0 + e * NT, hl = i / (ld16 / 2), d = i % (ld16 / 2) * 2, h = hg * HG + hl;
+            v[e] = i < nq && h < l.n_head && d < l.ld ? *reinterpret_cast<const float2 *>(q_lat + (row * l.n_head + h) * l.ld + d) : make_float2(0.f, 0.f);
+        }
+#pragma unroll
+        for (int e = 0; e < 6; e++) {
+            const int i = i0 + e * NT, hl = i / (ld16 / 2), d = i % (ld16 / 2) * 2;
+            if (i >= nq) break;
+            const float f = l.scale * 1.4426950408889634f, x = v[e].x * f, y = v[e].y * f;
+            const uint16_t hx = kq_f2bf(x), hy = kq_f2bf(y);
+            *reinterpret_cast<uint32_t *>(q_hi + hl * pitch + 2 * d) = (uint32_t)hx | ((uint32_t)hy << 16);
+            *reinterpret_cast<uint32_t *>(q_lo + hl * pitch + 2 * d) = (uint32_t)kq_f2bf(x - kq_bf2f(hx)) | ((uint32_t)kq_f2bf(y - kq_bf2f(hy)) << 16);
+        }
     }
     float m[NH] = {-INFINITY, -INFINITY}, sum[NH] = {}, o[NP][2][4];
 #pragma unroll
@@ -475,7 +482,7 @@ __global__ void __launch_bounds__(NT) latent_output_kernel(const __grid_constant
     __syncthreads();
     for (int d = 2 * tid; d < 8 * nck; d += 2 * NT) {
         float2 acc = make_float2(0.f, 0.f);
-#pragma unroll 8
+#pragma unroll 16
         for (int s = 0; s < n_split; s++) {
             const float2 v = *reinterpret_cast<const float2 *>(src + s * ps + d);
             acc.x = fmaf(s_w[s], v.x, acc.x);

@@ -18,11 +18,11 @@
 
 namespace {
 
-constexpr int BK = 128, BOX = BK * 64 * 2; // keys per tile, bytes of a box of 128 rows x 64 dims
-constexpr uint32_t COL_S = 0, COL_O = 128;
+constexpr int QBOX = 128 * 64 * 2; // bytes of a box of 128 query rows x 64 dims
+constexpr uint32_t COL_S = 0;
 constexpr int NSOFT = 256, NTHREADS = NSOFT + 32; // eight softmax warps and the issuing warp
 constexpr uint64_t LIMIT = 5 * KQ_WAIT_LIMIT_NS;
-constexpr int MAX_BOXES = 13; // operand boxes that fit in shared memory
+constexpr int MAX_SMEM = 13 * QBOX; // operands in shared memory
 
 __device__ int g_latent_tc_error;
 
@@ -50,8 +50,11 @@ __device__ __forceinline__ uint32_t pack_h2(float a, float b) {
 __device__ __forceinline__ uint32_t pack_h2_sat(float a, float b) { return (uint32_t)kq_f2h_sat(a) | ((uint32_t)kq_f2h_sat(b) << 16); }
 __device__ __forceinline__ void softmax_barrier() { asm volatile("bar.sync 1, %0;" ::"n"(NSOFT) : "memory"); }
 
-// grid (query tiles, heads)
+// grid (query tiles, heads); BK keys per tile: 128, or 64 where the operands would leave room for one CTA per SM only
+template <int BK>
 __global__ void __launch_bounds__(NTHREADS, 2) latent_prefill_tc_kernel(const __grid_constant__ AttnParams p) {
+    constexpr int BOX = BK * 128, HK = BK / 2; // bytes of a box of BK rows x 64 dims, keys of a half row
+    constexpr uint32_t COL_O = BK;
     KQ_PDL_ENTER();
     extern __shared__ uint8_t sm_raw[];
     __shared__ uint64_t full_k, full_v, s_ready, p_ready, pv_done;
@@ -65,7 +68,7 @@ __global__ void __launch_bounds__(NTHREADS, 2) latent_prefill_tc_kernel(const __
     const int t_base = blockIdx.x * 128, p_base = p.pos0 + t_base, p_last = min(p.pos0 + p.T, p_base + 128) - 1;
     const int first = p.window > 0 ? max(p.lo, p_base - p.window + 1) : p.lo; // first key (absolute) any row sees
     const int n_tiles = (p_last - first) / BK + 1;
-    uint8_t *sm_q = sm, *sm_k = sm + nk * BOX, *sm_v = sm_k + nk * BOX;
+    uint8_t *sm_q = sm, *sm_k = sm + nk * QBOX, *sm_v = sm_k + nk * BOX;
     const uint32_t bar_k = smem_u32(&full_k), bar_v = smem_u32(&full_v), bar_s = smem_u32(&s_ready), bar_p = smem_u32(&p_ready),
                    bar_pv = smem_u32(&pv_done);
     if (warp == 8) {
@@ -90,7 +93,7 @@ __global__ void __launch_bounds__(NTHREADS, 2) latent_prefill_tc_kernel(const __
         for (int b = half; b < nk; b += 2) {
             const float *src = b < p.nu ? qr + b * 64 : qr + p.dim + (b - p.nu) * 64;
             const int n = b < p.nu ? p.dim - b * 64 : p.rot - (b - p.nu) * 64;
-            uint8_t *dst = sm_q + b * BOX + row * 128;
+            uint8_t *dst = sm_q + b * QBOX + row * 128;
 #pragma unroll 2
             for (int c = 0; c < 8; c++) {
                 float v[8];
@@ -158,9 +161,9 @@ __global__ void __launch_bounds__(NTHREADS, 2) latent_prefill_tc_kernel(const __
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 if (!s_abort) {
                     for (int s = 0; s < su; s++)
-                        tc_mma_ss(tmem + COL_S, tc_desc_k(q_addr + (s >> 2) * BOX, s & 3), tc_desc_k(k_addr + (s >> 2) * BOX, s & 3), id_s, s > 0);
+                        tc_mma_ss(tmem + COL_S, tc_desc_k(q_addr + (s >> 2) * QBOX, s & 3), tc_desc_k(k_addr + (s >> 2) * BOX, s & 3), id_s, s > 0);
                     for (int s = 0; s < sr; s++)
-                        tc_mma_ss(tmem + COL_S, tc_desc_k(q_addr + (p.nu + (s >> 2)) * BOX, s & 3),
+                        tc_mma_ss(tmem + COL_S, tc_desc_k(q_addr + (p.nu + (s >> 2)) * QBOX, s & 3),
                                   tc_desc_k(k_addr + (p.nu + (s >> 2)) * BOX, s & 3), id_s, 1);
                 }
                 tc_commit(bar_s);
@@ -171,8 +174,8 @@ __global__ void __launch_bounds__(NTHREADS, 2) latent_prefill_tc_kernel(const __
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
                 if (!s_abort) {
 #pragma unroll
-                    for (int s = 0; s < 8; s++) // 16 keys per instruction: eight packed columns of P at the start of each half's columns of S
-                        tc_mma_ts(tmem + COL_O, tmem + COL_S + 64 * (s >> 2) + 8 * (s & 3), tc_desc_mn(v_addr, BOX, s), id_o,
+                    for (int s = 0; s < BK / 16; s++) // 16 keys per instruction: eight packed columns of P at the start of each half's columns of S
+                        tc_mma_ts(tmem + COL_O, tmem + COL_S + HK * (s / (HK / 16)) + 8 * (s % (HK / 16)), tc_desc_mn(v_addr, BOX, s), id_o,
                                   (i > 0 || s > 0) ? 1u : 0u);
                 }
                 tc_commit(bar_pv);
@@ -184,7 +187,7 @@ __global__ void __launch_bounds__(NTHREADS, 2) latent_prefill_tc_kernel(const __
     } else {
         // online softmax, half a row per thread
         const uint32_t tl = tmem + ((uint32_t)((warp & 3) * 32) << 16);
-        const int c0 = 64 * half;
+        const int c0 = HK * half;
         float m = -INFINITY, l = 0.f;
         for (int i = 0; i < n_tiles; i++) {
             if (!s_abort && !kq_mbar_wait(bar_s, (uint32_t)(i & 1), LIMIT)) {
@@ -197,7 +200,7 @@ __global__ void __launch_bounds__(NTHREADS, 2) latent_prefill_tc_kernel(const __
             const bool edge = t0 + BK - 1 > p_base || (p.window > 0 && t0 <= p_last - p.window);
             float t4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-            for (int c = 0; c < 2; c++) {
+            for (int c = 0; c < HK / 32; c++) {
                 uint32_t s[32];
                 TMEM_LD32(tl + COL_S + c0 + 32 * c, s);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -232,7 +235,7 @@ __global__ void __launch_bounds__(NTHREADS, 2) latent_prefill_tc_kernel(const __
             m = m_new;
             float l4[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll
-            for (int c = 0; c < 2; c++) {
+            for (int c = 0; c < HK / 32; c++) {
                 uint32_t s[32], pk[16];
                 TMEM_LD32(tl + COL_S + c0 + 32 * c, s);
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -335,7 +338,7 @@ Work layout(const KqLatent &l, int64_t keys) {
 }
 bool supported(const KqLatent &l) {
     const int nk = (int)(kq_pad(l.qk_dim, 64) + kq_pad(l.rot_dim, 64)) / 64, nv = (int)kq_pad(l.v_dim, 64) / 64;
-    return 2 * nk + nv <= MAX_BOXES && nv <= 4;
+    return nk * QBOX + (nk + nv) * QBOX / 2 <= MAX_SMEM && nv <= 4; // with 64 keys per tile
 }
 
 } // namespace
@@ -375,38 +378,41 @@ b200_status kq_latent_prefill(const KqLatent &l, const KqLatentPrefill &w, const
     b200_status rc = kq_gemm_bf16(d, c, k.ldc, 1, st);
     if (rc != B200_OK) return rc;
     AttnParams p = {};
+    const int nk = (int)(kq_pad(l.qk_dim, 64) + kq_pad(l.rot_dim, 64)) / 64, nv = (int)kq_pad(l.v_dim, 64) / 64;
+    const int bk = 2 * nk + nv <= 6 ? 128 : 64; // two CTAs per SM where that is possible
     const uint64_t H = (uint64_t)l.n_head, up = (uint64_t)kq_pad(l.qk_dim, 64), rp = (uint64_t)k.ldr, vp = (uint64_t)kq_pad(l.v_dim, 64);
     {
         const uint64_t dims[3] = {up, H, (uint64_t)keys}, str[2] = {up * 2, H * up * 2};
-        const uint32_t box[3] = {64, 1, BK};
+        const uint32_t box[3] = {64, 1, (uint32_t)bk};
         if ((rc = kq_tmap_encode(&p.ku, 2, 3, ku, dims, str, box, 1)) != B200_OK) return rc;
     }
     {
         const uint64_t dims[3] = {vp, H, (uint64_t)keys}, str[2] = {vp * 2, H * vp * 2};
-        const uint32_t box[3] = {64, 1, BK};
+        const uint32_t box[3] = {64, 1, (uint32_t)bk};
         if ((rc = kq_tmap_encode(&p.v, 2, 3, v, dims, str, box, 1)) != B200_OK) return rc;
     }
     if (rp) {
         const uint64_t dims[2] = {rp, (uint64_t)keys}, str[1] = {rp * 2};
-        const uint32_t box[2] = {64, BK};
+        const uint32_t box[2] = {64, (uint32_t)bk};
         if ((rc = kq_tmap_encode(&p.kr, 2, 2, kr, dims, str, box, 1)) != B200_OK) return rc;
     }
     p.q = q, p.gate = gate, p.out = out, p.ldq = ldq, p.ldg = ldg, p.ldo = ldo;
     p.T = T, p.pos0 = pos0, p.lo = lo, p.window = l.window;
     p.dim = l.qk_dim, p.rot = l.rot_dim, p.vdim = l.v_dim;
     p.nu = (int)(up / 64), p.nr = (int)(rp / 64), p.nv = (int)(vp / 64);
-    p.tmem_cols = 128 + p.nv * 64 <= 256 ? 256 : 512;
+    p.tmem_cols = bk + p.nv * 64 <= 256 ? 256 : 512;
     p.scale_log2 = l.scale * 1.4426950408889634f;
     p.vec = l.qk_dim % 4 == 0 && l.rot_dim % 4 == 0 && ldq % 4 == 0 && ((uintptr_t)q & 15) == 0;
-    const size_t smem = (size_t)(2 * (p.nu + p.nr) + p.nv) * BOX + 1024;
-    static size_t attr[16];
+    const size_t smem = (size_t)nk * QBOX + (size_t)(nk + nv) * bk * 128 + 1024;
+    static size_t attr[16][2];
     int dev = 0;
     KQ_CUDA(cudaGetDevice(&dev));
-    if (dev < 0 || dev >= 16 || attr[dev] < smem) {
-        KQ_CUDA(cudaFuncSetAttribute(latent_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-        if (dev >= 0 && dev < 16) attr[dev] = smem;
+    auto kern = bk == 128 ? latent_prefill_tc_kernel<128> : latent_prefill_tc_kernel<64>;
+    if (dev < 0 || dev >= 16 || attr[dev][bk == 128] < smem) {
+        KQ_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        if (dev >= 0 && dev < 16) attr[dev][bk == 128] = smem;
     }
-    kq_launch(latent_prefill_tc_kernel, dim3((unsigned)kq_div_up(T, 128), (unsigned)l.n_head), NTHREADS, smem, st, p);
+    kq_launch(kern, dim3((unsigned)kq_div_up(T, 128), (unsigned)l.n_head), NTHREADS, smem, st, p);
     KQ_COUNT_LAUNCH();
     KQ_LAUNCH_CHECK();
     return B200_OK;

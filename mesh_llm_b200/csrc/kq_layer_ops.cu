@@ -8,14 +8,30 @@
 
 namespace {
 
+// a thread per eight values of a row
 __global__ void embed_bf16_kernel(const uint16_t *W, int64_t ldw, const int32_t *ids, int64_t rows, int K, float scale, float *y,
                                   int64_t ldy) {
     KQ_PDL_ENTER();
-    const int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
-    if (i >= rows * K) return;
-    const int64_t r = i / K;
-    const int k = (int)(i % K);
-    y[r * ldy + k] = kq_bf2f(W[(int64_t)ids[r] * ldw + k]) * scale;
+    const int k = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+    const int64_t r = blockIdx.y;
+    if (k >= K) return;
+    const uint4 q = *reinterpret_cast<const uint4 *>(W + (int64_t)ids[r] * ldw + k);
+    const uint32_t w[4] = {q.x, q.y, q.z, q.w};
+    float v[8];
+#pragma unroll
+    for (int e = 0; e < 4; e++) {
+        v[2 * e] = __uint_as_float(w[e] << 16) * scale;
+        v[2 * e + 1] = __uint_as_float(w[e] & 0xffff0000u) * scale;
+    }
+    float *o = y + r * ldy + k;
+    if (k + 8 <= K && (ldy & 3) == 0) {
+        *reinterpret_cast<float4 *>(o) = make_float4(v[0], v[1], v[2], v[3]);
+        *reinterpret_cast<float4 *>(o + 4) = make_float4(v[4], v[5], v[6], v[7]);
+    } else {
+#pragma unroll
+        for (int e = 0; e < 8; e++)
+            if (k + e < K) o[e] = v[e];
+    }
 }
 
 constexpr int NT = 256;
@@ -140,32 +156,66 @@ __device__ __forceinline__ float conv_in(const float *x, int64_t ldx, const floa
     return pos >= 0 ? ring[(int64_t)(pos % taps) * width + c] : 0.f;
 }
 
+// v = hi + mid + lo exactly
+__device__ __forceinline__ void split3(float v, uint16_t *o, int64_t plane) {
+    const uint16_t hi = kq_f2bf(v);
+    float rest = v - kq_bf2f(hi);
+    const uint16_t mid = kq_f2bf(rest);
+    rest -= kq_bf2f(mid);
+    o[0] = hi;
+    o[plane] = mid;
+    o[2 * plane] = kq_f2bf(rest);
+}
+
+// grid (channels, runs of CT positions, sequences); a thread keeps the last inputs of its channel in registers.  TAPS:
+// 0 = any number of taps, read again for every position
+constexpr int CT = 16;
+template <int TAPS>
 __global__ void __launch_bounds__(NT) causal_conv_kernel(const __grid_constant__ KqRecW w, KqRecState st, const float *x, int64_t ldx,
                                                          int T, const int32_t *pos0_dev, int pos0_val, float *u, int64_t ldu,
                                                          uint16_t *u16, int64_t rows, int m, int mp) {
     KQ_PDL_ENTER();
-    const int64_t row = blockIdx.y;
     const int cp = blockIdx.x * NT + threadIdx.x; // channel in the block-padded layout
     if (cp >= w.blocks * mp) return;
-    const int b = cp / mp, j = cp % mp, c = b * m + j;
-    const int pos0 = pos0_dev ? *pos0_dev : pos0_val, seq = (int)(row / T), t = (int)(row % T);
-    float v = 0.f;
-    if (j < m) {
-        const float *ring = st.conv + (int64_t)seq * w.taps * w.width;
-        for (int k = 0; k < w.taps; k++)
-            v = fmaf(w.conv_w[(int64_t)c * w.taps + k], conv_in(x, ldx, ring, w.width, w.taps, (int64_t)seq * T, t - (w.taps - 1) + k, pos0, c), v);
-        v += w.conv_b[c];
-        u[row * ldu + c] = v;
+    const int seq = blockIdx.z, b = cp / mp, j = cp % mp, c = b * m + j, t0 = blockIdx.y * CT, t1 = min(T, t0 + CT);
+    const int64_t row0 = (int64_t)seq * T, ld16 = (int64_t)w.blocks * mp, plane = rows * ld16;
+    if (j >= m) {
+        for (int t = t0; t < t1; t++)
+            for (int q = 0; q < 3; q++) u16[q * plane + (row0 + t) * ld16 + cp] = 0;
+        return;
     }
-    if (u16) { // v = hi + mid + lo exactly
-        const int64_t ld = (int64_t)w.blocks * mp, i = row * ld + cp;
-        const uint16_t hi = kq_f2bf(v);
-        float rest = v - kq_bf2f(hi);
-        const uint16_t mid = kq_f2bf(rest);
-        rest -= kq_bf2f(mid);
-        u16[i] = hi;
-        u16[rows * ld + i] = mid;
-        u16[2 * rows * ld + i] = kq_f2bf(rest);
+    const int pos0 = pos0_dev ? *pos0_dev : pos0_val, taps = TAPS ? TAPS : w.taps;
+    const float *ring = st.conv + (int64_t)seq * w.taps * w.width;
+    const float bias = w.conv_b[c];
+    if (TAPS) {
+        constexpr int N = TAPS ? TAPS : 1;
+        float cw[N], in[N + CT - 1];
+#pragma unroll
+        for (int k = 0; k < N; k++) cw[k] = w.conv_w[(int64_t)c * N + k];
+#pragma unroll
+        for (int i = 0; i < N + CT - 1; i++) {
+            const int t = t0 - (N - 1) + i;
+            in[i] = t < t1 ? conv_in(x, ldx, ring, w.width, N, row0, t, pos0, c) : 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < CT; i++) {
+            if (t0 + i >= t1) break;
+            float v = 0.f;
+#pragma unroll
+            for (int k = 0; k < N; k++) v = fmaf(cw[k], in[i + k], v);
+            v += bias;
+            u[(row0 + t0 + i) * ldu + c] = v;
+            if (u16) split3(v, u16 + (row0 + t0 + i) * ld16 + cp, plane);
+        }
+    } else {
+        for (int t = t0; t < t1; t++) {
+            float v = 0.f;
+            for (int k = 0; k < taps; k++)
+                v = fmaf(w.conv_w[(int64_t)c * taps + k], conv_in(x, ldx, ring, w.width, taps, row0, t - (taps - 1) + k, pos0, c), v);
+            v += bias;
+            u[(row0 + t) * ldu + c] = v;
+            if (u16) split3(v, u16 + (row0 + t) * ld16 + cp, plane);
+        }
     }
 }
 
@@ -177,53 +227,69 @@ __device__ __forceinline__ void rec_coeff(float r, float i, float u, float decay
     b = sqrtf(-expm1f(2.f * la)) * kq_sigmoid(i) * u;
 }
 
-constexpr int SC = 32, SW = 16; // channels per CTA, time chunks (one warp each)
-__global__ void __launch_bounds__(SC * SW) linear_recurrence_kernel(const __grid_constant__ KqRecW w, KqRecState st, float *r, float *ig,
-                                                                    int64_t ldr, const float *u, int64_t ldu, const float *x,
-                                                                    int64_t ldx, const float *y, int64_t ldy, int T,
-                                                                    const int32_t *pos0_dev, int pos0_val, float *z32, int64_t ld32,
-                                                                    uint16_t *z16, int64_t ld16) {
+// Prefill in two passes over chunks of `chunk` positions, a thread per channel.  First: coefficients (over the gates, in
+// place) and each chunk's map of the state, s -> A s + B.  Second: the state in front of a chunk from the maps of the
+// chunks before it, then the recurrence inside the chunk.
+constexpr int RC = 128, RCHUNK = 64; // channels per CTA, positions per chunk
+__global__ void __launch_bounds__(RC) recurrence_chunks_kernel(const __grid_constant__ KqRecW w, KqRecState st, float *r, float *ig, int64_t ldr, const float *u,
+                                                               int64_t ldu, int T, const int32_t *pos0_dev, int pos0_val, int chunk, float *maps) {
     KQ_PDL_ENTER();
-    __shared__ float sa[SW][SC], sb[SW][SC];
-    const int lane = threadIdx.x & 31, k = threadIdx.x >> 5, seq = blockIdx.y;
-    const int c = blockIdx.x * SC + lane;
-    const int pos0 = pos0_dev ? *pos0_dev : pos0_val;
-    const bool ok = c < w.width;
-    const int chunk = (T + SW - 1) / SW, t0 = min(T, k * chunk), t1 = min(T, t0 + chunk);
+    const int c = blockIdx.x * RC + threadIdx.x, k = blockIdx.y, seq = blockIdx.z;
+    if (c >= w.width) return;
+    const int t0 = k * chunk, t1 = min(T, t0 + chunk);
     const int64_t row0 = (int64_t)seq * T;
-    const float dsp = ok ? w.decay * softplus(w.lam[c]) : 0.f;
+    const float dsp = w.decay * softplus(w.lam[c]);
     float A = 1.f, B = 0.f;
-    if (ok)
-        for (int t = t0; t < t1; t++) {
-            const int64_t o = (row0 + t) * ldr + c;
-            float a, b;
-            rec_coeff(r[o], ig[o], u[(row0 + t) * ldu + c], dsp, a, b);
-            r[o] = a;
-            ig[o] = b;
-            A *= a;
-            B = fmaf(a, B, b);
-        }
-    sa[k][lane] = A;
-    sb[k][lane] = B;
-    // the conv ring: its old entries were last read by the convolution of this call
-    if (ok)
-        for (int t = max(0, T - w.taps) + k; t < T; t += SW)
-            st.conv[((int64_t)seq * w.taps + (pos0 + t) % w.taps) * w.width + c] = x[(row0 + t) * ldx + c];
-    float s = ok && pos0 > 0 ? st.s[(int64_t)seq * w.width + c] : 0.f;
-    __syncthreads();
-    for (int j = 0; j < k; j++) s = fmaf(sa[j][lane], s, sb[j][lane]);
-    if (ok) {
-        for (int t = t0; t < t1; t++) {
-            const int64_t o = (row0 + t) * ldr + c;
-            s = fmaf(r[o], s, ig[o]);
-            const float v = s * y[(row0 + t) * ldy + c];
-            if (z32) z32[(row0 + t) * ld32 + c] = v;
-            if (z16) z16[(row0 + t) * ld16 + c] = kq_f2bf(v);
-        }
-    } else if (z16 && c < ld16) {
-        for (int t = t0; t < t1; t++) z16[(row0 + t) * ld16 + c] = 0;
+#pragma unroll 4
+    for (int t = t0; t < t1; t++) {
+        const int64_t o = (row0 + t) * ldr + c;
+        float a, b;
+        rec_coeff(r[o], ig[o], u[(row0 + t) * ldu + c], dsp, a, b);
+        r[o] = a;
+        ig[o] = b;
+        A *= a;
+        B = fmaf(a, B, b);
     }
-    if (ok && t1 == T && t0 < T) st.s[(int64_t)seq * w.width + c] = s;
+    float *d = maps + ((int64_t)seq * (gridDim.y + 1) + k + 1) * 2 * w.width + c;
+    d[0] = A;
+    d[w.width] = B;
+    if (k == 0) { // entry 0: the state in front of the call, which the second pass may already be replacing when others need it
+        const int pos0 = pos0_dev ? *pos0_dev : pos0_val;
+        maps[(int64_t)seq * (gridDim.y + 1) * 2 * w.width + c] = pos0 > 0 ? st.s[(int64_t)seq * w.width + c] : 0.f;
+    }
+}
+
+__global__ void __launch_bounds__(RC) recurrence_scan_kernel(const __grid_constant__ KqRecW w, KqRecState st, const float *a, const float *b, int64_t ldr,
+                                                             const float *x, int64_t ldx, const float *y, int64_t ldy, int T,
+                                                             const int32_t *pos0_dev, int pos0_val, int chunk, const float *maps, float *z32,
+                                                             int64_t ld32, uint16_t *z16, int64_t ld16) {
+    KQ_PDL_ENTER();
+    const int c = blockIdx.x * RC + threadIdx.x, k = blockIdx.y, seq = blockIdx.z;
+    const int t0 = k * chunk, t1 = min(T, t0 + chunk);
+    const int64_t row0 = (int64_t)seq * T;
+    if (c >= w.width) {
+        if (z16 && c < ld16)
+            for (int t = t0; t < t1; t++) z16[(row0 + t) * ld16 + c] = 0;
+        return;
+    }
+    const int pos0 = pos0_dev ? *pos0_dev : pos0_val;
+    const bool last = k == (int)gridDim.y - 1;
+    if (last) // the conv ring: its old entries were last read by the convolution of this call
+        for (int t = max(0, T - w.taps); t < T; t++)
+            st.conv[((int64_t)seq * w.taps + (pos0 + t) % w.taps) * w.width + c] = x[(row0 + t) * ldx + c];
+    const float *d = maps + (int64_t)seq * (gridDim.y + 1) * 2 * w.width + c;
+    float s = d[0];
+#pragma unroll 8
+    for (int j = 1; j <= k; j++) s = fmaf(d[(int64_t)j * 2 * w.width], s, d[((int64_t)j * 2 + 1) * w.width]);
+#pragma unroll 8
+    for (int t = t0; t < t1; t++) {
+        const int64_t o = (row0 + t) * ldr + c;
+        s = fmaf(a[o], s, b[o]);
+        const float v = s * y[(row0 + t) * ldy + c];
+        if (z32) z32[(row0 + t) * ld32 + c] = v;
+        if (z16) z16[(row0 + t) * ld16 + c] = kq_f2bf(v);
+    }
+    if (last) st.s[(int64_t)seq * w.width + c] = s;
 }
 
 // ---- one token: grid (row slices of all blocks, sequences); a CTA convolves its block's channels, then each warp
@@ -305,7 +371,8 @@ __global__ void __launch_bounds__(NT) recurrence_step_kernel(const __grid_consta
 b200_status kq_embed_bf16(const uint16_t *W, int64_t ldw, const int32_t *ids, int64_t rows, int K, float scale, float *y,
                           int64_t ldy, cudaStream_t st) {
     KQ_REQUIRE(W && ids && y && rows >= 1 && K >= 1, "embed_bf16: bad call");
-    kq_launch(embed_bf16_kernel, (unsigned)kq_div_up(rows * K, 256), 256, 0, st, W, ldw, ids, rows, K, scale, y, ldy);
+    KQ_REQUIRE(rows <= 65535 && ((uintptr_t)y & 15) == 0, "embed_bf16: %lld rows", (long long)rows);
+    kq_launch(embed_bf16_kernel, dim3((unsigned)kq_div_up(K, 8 * 128), (unsigned)rows), 128, 0, st, W, ldw, ids, rows, K, scale, y, ldy);
     KQ_COUNT_LAUNCH();
     KQ_LAUNCH_CHECK();
     return B200_OK;
@@ -335,22 +402,38 @@ b200_status kq_causal_conv(const KqRecW &w, const KqRecState &s, const float *x,
     const b200_status rc = check_rec(w, n_seq, T);
     if (rc != B200_OK) return rc;
     const int m = w.width / w.blocks, mp = u16 ? (int)kq_bf16_ld(m) : m;
-    kq_launch(causal_conv_kernel, dim3((unsigned)kq_div_up((int64_t)w.blocks * mp, NT), (unsigned)(n_seq * T)), NT, 0, st, w, s, x, ldx, T, pos0_dev,
-              pos0, u, ldu, u16, (int64_t)n_seq * T, m, mp);
+    const dim3 grid((unsigned)kq_div_up((int64_t)w.blocks * mp, NT), (unsigned)kq_div_up(T, CT), (unsigned)n_seq);
+    const int64_t rows = (int64_t)n_seq * T;
+#define GO(N) kq_launch(causal_conv_kernel<N>, grid, NT, 0, st, w, s, x, ldx, T, pos0_dev, pos0, u, ldu, u16, rows, m, mp)
+    if (w.taps == 4) GO(4);
+    else if (w.taps == 3) GO(3);
+    else if (w.taps == 2) GO(2);
+    else GO(0);
+#undef GO
     KQ_COUNT_LAUNCH();
     KQ_LAUNCH_CHECK();
     return B200_OK;
 }
 
+size_t kq_recurrence_scratch_bytes(int width, int rows, int n_seq) {
+    return (size_t)(rows / RCHUNK + 2 * std::min(n_seq, rows) + 1) * 2 * width * 4;
+}
+
 b200_status kq_linear_recurrence(const KqRecW &w, const KqRecState &s, float *r, float *i, int64_t ldr, const float *u,
                                  int64_t ldu, const float *x, int64_t ldx, const float *y, int64_t ldy, int n_seq, int T,
                                  const int32_t *pos0_dev, int pos0, float *z32, int64_t ld32, uint16_t *z16, int64_t ld16,
-                                 cudaStream_t st) {
+                                 float *scratch, size_t scratch_bytes, cudaStream_t st) {
     const b200_status rc = check_rec(w, n_seq, T);
     if (rc != B200_OK) return rc;
+    const unsigned chunks = (unsigned)kq_div_up(T, RCHUNK);
+    KQ_REQUIRE(scratch && scratch_bytes >= (size_t)n_seq * (chunks + 1) * 2 * w.width * 4, "recurrence: scratch");
     const int64_t cols = z16 ? std::max<int64_t>(w.width, ld16) : w.width;
-    kq_launch(linear_recurrence_kernel, dim3((unsigned)kq_div_up(cols, SC), (unsigned)n_seq), SC * SW, 0, st, w, s, r, i, ldr, u, ldu, x, ldx, y, ldy,
-              T, pos0_dev, pos0, z32, ld32, z16, ld16);
+    kq_launch(recurrence_chunks_kernel, dim3((unsigned)kq_div_up(w.width, RC), chunks, (unsigned)n_seq), RC, 0, st, w, s, r, i, ldr, u, ldu, T, pos0_dev,
+              pos0, RCHUNK, scratch);
+    KQ_COUNT_LAUNCH();
+    KQ_LAUNCH_CHECK();
+    kq_launch(recurrence_scan_kernel, dim3((unsigned)kq_div_up(cols, RC), chunks, (unsigned)n_seq), RC, 0, st, w, s, r, i, ldr, x, ldx, y, ldy, T,
+              pos0_dev, pos0, RCHUNK, scratch, z32, ld32, z16, ld16);
     KQ_COUNT_LAUNCH();
     KQ_LAUNCH_CHECK();
     return B200_OK;

@@ -56,8 +56,8 @@ struct KqLayers {
     uint16_t *h16 = nullptr;
     float *f[7] = {}; // projections of a mixer
     uint16_t *u16 = nullptr, *z16 = nullptr, *act16 = nullptr;
-    float *act32 = nullptr, *att_scratch = nullptr;
-    size_t att_scratch_bytes = 0;
+    float *act32 = nullptr, *att_scratch = nullptr, *rec_scratch = nullptr;
+    size_t att_scratch_bytes = 0, rec_scratch_bytes = 0;
     void *prefill_work = nullptr;
     size_t prefill_bytes = 0;
 };
@@ -233,7 +233,7 @@ struct Pass {
         else if (f32) OTHER_(kq_gemm_f32(g, u, ld, s));
         else OTHER_(kq_gemm_bf16(g, k->u16, ldu, 3, s)); // the gates see u in full f32
         OTHER_(kq_linear_recurrence(L.rec, rs, gr, gi, ld, u, ld, xi, ld, y, ld, n_seq, T, pos_dev, pos0, tc ? nullptr : z, ld,
-                                    tc ? k->z16 : nullptr, kq_bf16_ld(W), s));
+                                    tc ? k->z16 : nullptr, kq_bf16_ld(W), k->rec_scratch, k->rec_scratch_bytes, s));
         return close(L.wo, W, z, ld, k->z16, L.norm1b);
     }
 
@@ -503,7 +503,7 @@ b200_status b200_stage_create_layers(const b200_stage_config *cfg, const b200_st
     }
     const int64_t h = c.n_embd, R = c.n_ubatch;
     if (c.has_embd || c.has_output) kq_stage_add_tensor(st, "embed", B200_TYPE_BF16, h, c.n_vocab, 1);
-    int64_t fmax[6] = {}, wmax16 = 0, u16max = 0, ffmax = 0, scratch = 0, prefill = 0;
+    int64_t fmax[6] = {}, wmax16 = 0, u16max = 0, ffmax = 0, scratch = 0, rec_scratch = 0, prefill = 0;
     const bool f32 = stack->precision == B200_PRECISION_F32;
     auto grow = [](int64_t &a, int64_t b) { a = std::max(a, b); };
     for (int i = c.layer_begin; i < c.layer_end; i++) {
@@ -528,6 +528,7 @@ b200_status b200_stage_create_layers(const b200_stage_config *cfg, const b200_st
             mat("mix.o", W, h);
             for (int f = 0; f < 6; f++) grow(fmax[f], kq_f32_ld(W));
             grow(wmax16, kq_bf16_ld(W));
+            grow(rec_scratch, (int64_t)kq_recurrence_scratch_bytes(l.rec_width, (int)R, c.n_seq));
             grow(u16max, 3 * l.rec_blocks * kq_bf16_ld(m));
         } else {
             const int64_t H = l.n_head, hd = l.qk_dim + l.rot_dim;
@@ -603,6 +604,8 @@ b200_status b200_stage_create_layers(const b200_stage_config *cfg, const b200_st
     if (wide) A(&k->u16, (size_t)(R * u16max * 2));
     if (ffmax) A(&k->act32, (size_t)((f32 ? R : std::min<int64_t>(R, SMALL_ROWS)) * kq_f32_ld(ffmax) * 4));
     if (ffmax && wide) A(&k->act16, (size_t)(R * kq_bf16_ld(ffmax) * 2));
+    k->rec_scratch_bytes = (size_t)rec_scratch;
+    A(&k->rec_scratch, (size_t)rec_scratch);
     k->att_scratch_bytes = (size_t)scratch;
     A(&k->att_scratch, (size_t)scratch);
     k->prefill_bytes = wide ? (size_t)prefill : 0;
