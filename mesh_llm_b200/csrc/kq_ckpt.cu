@@ -175,7 +175,7 @@ bool read_all(int fd, uint64_t pos, void *dst, uint64_t n) {
 struct Cfg {
     b200_status rc = B200_OK;
     void bad(const std::string &where, const char *key, const char *what) {
-        if (rc == B200_OK) kq_set_error("config.json: %s.%s %s", where.c_str(), key, what);
+        if (rc == B200_OK) kq_set_error("config.json: %s%s%s %s", where.c_str(), where.empty() ? "" : ".", key, what);
         rc = B200_ERR_INVALID;
     }
     const Json *need(const Json *o, const std::string &where, const char *key) {
