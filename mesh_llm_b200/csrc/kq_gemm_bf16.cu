@@ -1,10 +1,11 @@
 // Prefill products with bf16 weights, y[m][n] = sum_k W[n][k] x[m][k]: the tensor-core form (tcgen05.mma
 // kind::f16 on bf16 operands, f32 accumulators in TMEM) and the f32 form on CUDA cores of the 32-bit mode.
 //
-// Tensor cores: one CTA computes 128 tokens (TMEM lanes) x 128 weight rows (columns), two CTAs per SM.  K runs
-// in slices of 64 (one 128-byte-swizzled row per operand row); a producer thread brings the slices in by tiled
-// TMA copies through a ring of three stages, one thread issues the MMAs, four warps drain the accumulator.
-// A gate / up pair puts 64 rows of either matrix into a tile, so that the GLU happens where both values are.
+// Tensor cores: a persistent CTA per SM walks tiles of 128 tokens (TMEM lanes) x 256 or 128 weight rows (columns), token
+// tiles innermost, so that the CTAs at work share the weight rows they read.  K runs in slices of 64 (one
+// 128-byte-swizzled row per operand row); a producer thread brings the slices in by tiled TMA copies through a ring
+// of stages, one thread issues the MMAs into one of two accumulators in TMEM, four warps drain the other one meanwhile.
+// A gate / up pair shares a tile half and half, so that the GLU happens where both values are.
 // An f32 operand can come as several bf16 parts (x = hi + mid + lo exactly): the K loop then passes over the
 // same weights once per part.  Block-diagonal products offset the K coordinate of x and the row of W by group.
 // Every wait is bounded; on a time-out the kernel records an error, lets its copies land, frees its TMEM and
@@ -18,33 +19,42 @@
 
 namespace {
 
-constexpr int TM = 128, TN = 128, BK = 64, STAGES = 3;
-constexpr int A_BYTES = TM * BK * 2, B_BYTES = TN * BK * 2, STAGE_BYTES = A_BYTES + B_BYTES;
-constexpr int SMEM_TOTAL = STAGES * STAGE_BYTES + 1024;
-constexpr int NTHREADS = 192; // producer warp, MMA warp, four epilogue warps
-constexpr uint32_t TMEM_COLS = 128;
+constexpr int TM = 128, BK = 64, A_BYTES = TM * BK * 2;
+template <int TN>
+struct Tile {
+    static constexpr int B_BYTES = TN * BK * 2, STAGE_BYTES = A_BYTES + B_BYTES, STAGES = 192 * 1024 / STAGE_BYTES;
+    static constexpr int SMEM_TOTAL = STAGES * STAGE_BYTES + 1024;
+    static constexpr uint32_t TMEM_COLS = 2 * TN; // two accumulators
+};
+constexpr int NTHREADS = 192, NEPI = 128; // producer warp, MMA warp, four epilogue warps
 constexpr uint64_t LIMIT = 5 * KQ_WAIT_LIMIT_NS;
 
 __device__ int g_gemm_bf16_error;
-
-// kind::f16: D f32, A bf16, B bf16, both K-major, M = 128, N = 128
-constexpr uint32_t IDESC = tc_idesc(TM, TN, true, false);
 
 struct GemmParams {
     CUtensorMap a, b[3];
     KqDense c;
     int32_t nk, parts;      // 64-element K slices per part
     int32_t tile_end[3];    // cumulative N tiles of the segments
+    int32_t mt, nt;         // tiles of tokens and of weight rows (all segments)
 };
 
 // eight consecutive output columns of one row
 __device__ __forceinline__ void put8(const KqDense &c, const KqDenseSeg &s, int64_t m, int64_t n, int g, const float *v, int n_valid) {
     if (n_valid == 8 && ((s.ldy | n | s.head_in | s.head_out) & 7) == 0) { // all eight in one head, 16-byte aligned
-        float o[8];
+        float o[8], bias[8] = {};
+        if (s.bias) {
+            if (((uintptr_t)(s.bias + n) & 15) == 0) {
+                *reinterpret_cast<float4 *>(bias) = *reinterpret_cast<const float4 *>(s.bias + n);
+                *reinterpret_cast<float4 *>(bias + 4) = *reinterpret_cast<const float4 *>(s.bias + n + 4);
+            } else {
+#pragma unroll
+                for (int j = 0; j < 8; j++) bias[j] = s.bias[n + j];
+            }
+        }
 #pragma unroll
         for (int j = 0; j < 8; j++) {
-            float t = v[j];
-            if (s.bias) t += s.bias[n + j];
+            float t = v[j] + bias[j];
             if (s.act == KQ_ACT_GELU_TANH) t = kq_gelu_tanh(t);
             if (c.head_gate) t *= kq_sigmoid(c.head_gate[m * c.ld_gate + g]);
             o[j] = t;
@@ -52,8 +62,14 @@ __device__ __forceinline__ void put8(const KqDense &c, const KqDenseSeg &s, int6
         const int64_t i = m * s.ldy + kq_dense_col(s, n);
         if (s.out == KQ_OUT_F32) {
             float *y = (float *)s.y + i;
-            *reinterpret_cast<float4 *>(y) = make_float4(o[0], o[1], o[2], o[3]);
-            *reinterpret_cast<float4 *>(y + 4) = make_float4(o[4], o[5], o[6], o[7]);
+            if (((uintptr_t)y & 31) == 0) { // a whole sector at once
+                asm volatile("st.global.v8.f32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(y), "f"(o[0]), "f"(o[1]), "f"(o[2]), "f"(o[3]),
+                             "f"(o[4]), "f"(o[5]), "f"(o[6]), "f"(o[7])
+                             : "memory");
+            } else {
+                *reinterpret_cast<float4 *>(y) = make_float4(o[0], o[1], o[2], o[3]);
+                *reinterpret_cast<float4 *>(y + 4) = make_float4(o[4], o[5], o[6], o[7]);
+            }
         } else {
             uint32_t w[4];
 #pragma unroll
@@ -69,34 +85,32 @@ __device__ __forceinline__ void put8(const KqDense &c, const KqDenseSeg &s, int6
         if (j < n_valid) kq_dense_store(c, s, m, n + j, g, v[j]);
 }
 
-// grid (token tiles, weight-row tiles of all segments, groups)
-__global__ void __launch_bounds__(NTHREADS, 2) gemm_bf16_kernel(const __grid_constant__ GemmParams p) {
+template <int TN>
+__global__ void __launch_bounds__(NTHREADS, 1) gemm_bf16_kernel(const __grid_constant__ GemmParams p) {
+    using S = Tile<TN>;
+    constexpr uint32_t IDESC = tc_idesc(TM, TN, true, false);
     extern __shared__ uint8_t sm_raw[];
-    __shared__ uint64_t full[STAGES], empty[STAGES], done;
+    __shared__ uint64_t full[S::STAGES], empty[S::STAGES], acc_full[2], acc_empty[2];
     __shared__ uint32_t s_tmem;
     __shared__ int s_abort;
     // the wait comes before the TMEM allocation: a CTA that started early must not hold columns its predecessor needs
     KQ_PDL_ENTER();
     uint8_t *sm = (uint8_t *)(((uintptr_t)sm_raw + 1023) & ~(uintptr_t)1023);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int m0 = blockIdx.x * TM, g = blockIdx.z;
-    int seg = 0, nt = blockIdx.y;
-    if (!p.c.glu) {
-        while (seg + 1 < p.c.nseg && nt >= p.tile_end[seg]) seg++;
-        if (seg) nt -= p.tile_end[seg - 1];
-    }
-    const int n_rows = p.c.seg[seg].n_rows, n0 = nt * (p.c.glu ? TN / 2 : TN); // first row of the tile inside the group
     if (warp == 1) {
-        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&s_tmem)), "r"(TMEM_COLS)
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&s_tmem)), "r"(S::TMEM_COLS)
                      : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
     if (tid == 0) {
-        for (int i = 0; i < STAGES; i++) {
+        for (int i = 0; i < S::STAGES; i++) {
             asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(&full[i])), "r"(1));
             asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(&empty[i])), "r"(1));
         }
-        asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(&done)), "r"(1));
+        for (int i = 0; i < 2; i++) {
+            asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(&acc_full[i])), "r"(1));
+            asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(&acc_empty[i])), "r"(NEPI));
+        }
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
         s_abort = 0;
     }
@@ -104,10 +118,28 @@ __global__ void __launch_bounds__(NTHREADS, 2) gemm_bf16_kernel(const __grid_con
     __syncthreads();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t tmem = s_tmem;
-    const int n_it = p.nk * p.parts;
+    const int n_it = p.nk * p.parts, n_tiles = p.mt * p.nt * p.c.groups;
 
+    struct Where {
+        int m0, g, seg, n0, n_rows;
+    };
+    auto locate = [&](int tile) {
+        Where w;
+        w.m0 = tile % p.mt * TM;
+        const int rest = tile / p.mt;
+        int nt = rest % p.nt;
+        w.g = rest / p.nt;
+        w.seg = 0;
+        if (!p.c.glu) {
+            while (w.seg + 1 < p.c.nseg && nt >= p.tile_end[w.seg]) w.seg++;
+            if (w.seg) nt -= p.tile_end[w.seg - 1];
+        }
+        w.n_rows = p.c.seg[w.seg].n_rows;
+        w.n0 = nt * (p.c.glu ? TN / 2 : TN); // first row of the tile inside the group
+        return w;
+    };
     auto wait = [&](uint64_t *bar, uint32_t parity, int code) {
-        if (!*(volatile int *)&s_abort && !kq_mbar_wait(smem_u32(bar), parity, LIMIT)) {
+        if (!*(volatile int *)&s_abort && !kq_mbar_wait_hot(smem_u32(bar), parity, LIMIT)) {
             *(volatile int *)&s_abort = 1;
             atomicExch(&g_gemm_bf16_error, code);
         }
@@ -115,61 +147,78 @@ __global__ void __launch_bounds__(NTHREADS, 2) gemm_bf16_kernel(const __grid_con
     };
     if (warp == 0) {
         if (lane == 0) {
-            int posted = 0;
-            for (int it = 0; it < n_it; it++) {
-                const int s = it % STAGES;
-                if (it >= STAGES && !wait(&empty[s], (uint32_t)((it / STAGES - 1) & 1), 1)) break;
-                const uint32_t bar = smem_u32(&full[s]), dst = smem_u32(sm + s * STAGE_BYTES);
-                asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(STAGE_BYTES) : "memory");
-                const int part = it / p.nk, kk = (it % p.nk) * BK;
-                asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];" ::"r"(dst),
-                             "l"(&p.a), "r"((int)(g * p.c.xg) + kk), "r"(m0), "r"(part), "r"(bar)
-                             : "memory");
-#pragma unroll
-                for (int hb = 0; hb < 2; hb++) { // 64 weight rows each: two halves of one matrix, or gate and up
-                    const CUtensorMap *map = p.c.glu ? &p.b[hb] : &p.b[seg];
-                    const int row = g * n_rows + n0 + (p.c.glu ? 0 : hb * 64);
-                    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(
-                                     dst + A_BYTES + hb * (B_BYTES / 2)),
-                                 "l"(map), "r"(kk), "r"(row), "r"(bar)
+            int it = 0; // slices over all tiles
+            bool ok = true;
+            for (int tile = blockIdx.x; ok && tile < n_tiles; tile += gridDim.x) {
+                const Where w = locate(tile);
+                for (int i = 0; i < n_it; i++, it++) {
+                    const int s = it % S::STAGES;
+                    if (it >= S::STAGES && !(ok = wait(&empty[s], (uint32_t)((it / S::STAGES - 1) & 1), 1))) break;
+                    const uint32_t bar = smem_u32(&full[s]), dst = smem_u32(sm + s * S::STAGE_BYTES);
+                    asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(S::STAGE_BYTES) : "memory");
+                    const int part = i / p.nk, kk = (i % p.nk) * BK;
+                    asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];" ::"r"(dst),
+                                 "l"(&p.a), "r"((int)(w.g * p.c.xg) + kk), "r"(w.m0), "r"(part), "r"(bar)
                                  : "memory");
+#pragma unroll
+                    for (int hb = 0; hb < 2; hb++) { // half a tile of weight rows each: of one matrix, or gate and up
+                        const CUtensorMap *map = p.c.glu ? &p.b[hb] : &p.b[w.seg];
+                        const int row = w.g * w.n_rows + w.n0 + (p.c.glu ? 0 : hb * (TN / 2));
+                        asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(
+                                         dst + A_BYTES + hb * (S::B_BYTES / 2)),
+                                     "l"(map), "r"(kk), "r"(row), "r"(bar)
+                                     : "memory");
+                    }
                 }
-                posted = it + 1;
             }
-            if (*(volatile int *)&s_abort) // copies that were posted must land before the CTA goes away
-                for (int it = std::max(0, posted - STAGES); it < posted; it++)
-                    kq_mbar_wait(smem_u32(&full[it % STAGES]), (uint32_t)((it / STAGES) & 1), KQ_WAIT_LIMIT_NS);
+            if (!ok) // copies that were posted must land before the CTA goes away
+                for (int i = std::max(0, it - S::STAGES); i < it; i++)
+                    kq_mbar_wait(smem_u32(&full[i % S::STAGES]), (uint32_t)((i / S::STAGES) & 1), KQ_WAIT_LIMIT_NS);
         }
         __syncwarp();
     } else if (warp == 1) {
         if (lane == 0) {
-            for (int it = 0; it < n_it; it++) {
-                const int s = it % STAGES;
-                if (!wait(&full[s], (uint32_t)((it / STAGES) & 1), 2)) break;
+            int it = 0, t = 0;
+            bool ok = true;
+            for (int tile = blockIdx.x; ok && tile < n_tiles; tile += gridDim.x, t++) {
+                const int buf = t & 1;
+                if (t >= 2 && !(ok = wait(&acc_empty[buf], (uint32_t)((t / 2 - 1) & 1), 4))) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                const uint32_t a = smem_u32(sm + s * STAGE_BYTES), b = a + A_BYTES;
+                for (int i = 0; i < n_it; i++, it++) {
+                    const int s = it % S::STAGES;
+                    if (!(ok = wait(&full[s], (uint32_t)((it / S::STAGES) & 1), 2))) break;
+                    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                    const uint32_t a = smem_u32(sm + s * S::STAGE_BYTES), b = a + A_BYTES;
 #pragma unroll
-                for (int k = 0; k < BK / 16; k++) tc_mma_ss(tmem, tc_desc_k(a, k), tc_desc_k(b, k), IDESC, (it > 0 || k > 0) ? 1u : 0u);
-                tc_commit(smem_u32(&empty[s]));
+                    for (int k = 0; k < BK / 16; k++)
+                        tc_mma_ss(tmem + buf * TN, tc_desc_k(a, k), tc_desc_k(b, k), IDESC, (i > 0 || k > 0) ? 1u : 0u);
+                    tc_commit(smem_u32(&empty[s]));
+                }
+                tc_commit(smem_u32(&acc_full[buf]));
             }
-            tc_commit(smem_u32(&done));
-            if (*(volatile int *)&s_abort) kq_mbar_wait(smem_u32(&done), 0, KQ_WAIT_LIMIT_NS); // MMAs in flight end before TMEM is freed
+            if (!ok) // MMAs in flight end before TMEM is freed
+                for (int i = std::max(0, t - 2); i < t; i++) kq_mbar_wait(smem_u32(&acc_full[i & 1]), (uint32_t)((i / 2) & 1), KQ_WAIT_LIMIT_NS);
         }
         __syncwarp();
     } else {
-        const bool ok = wait(&done, 0, 3);
-        asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        if (__all_sync(0xffffffffu, ok)) {
-            const int q = warp & 3, row = m0 + q * 32 + lane; // a warp reaches the TMEM lanes of its quarter
-            const uint32_t tl = tmem + ((uint32_t)(q * 32) << 16);
-            const KqDenseSeg &s = p.c.seg[seg];
+        const int q = warp & 3; // a warp reaches the TMEM lanes of its quarter
+        int t = 0;
+        for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x, t++) {
+            const int buf = t & 1;
+            const bool ok = wait(&acc_full[buf], (uint32_t)((t / 2) & 1), 3);
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            if (!__all_sync(0xffffffffu, ok)) break;
+            const Where w = locate(tile);
+            const int row = w.m0 + q * 32 + lane, n0 = w.n0, n_rows = w.n_rows;
+            const uint32_t tl = tmem + ((uint32_t)(q * 32) << 16) + buf * TN;
+            const KqDenseSeg &s = p.c.seg[w.seg];
             const bool row_ok = row < p.c.M;
             if (p.c.glu) {
 #pragma unroll 1
-                for (int c = 0; c < 2; c++) {
+                for (int c = 0; c < TN / 64; c++) {
                     uint32_t a[32], b[32];
                     TMEM_LD32(tl + 32 * c, a);
-                    TMEM_LD32(tl + 64 + 32 * c, b);
+                    TMEM_LD32(tl + TN / 2 + 32 * c, b);
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
                     if (row_ok) {
 #pragma unroll
@@ -189,6 +238,7 @@ __global__ void __launch_bounds__(NTHREADS, 2) gemm_bf16_kernel(const __grid_con
             } else {
 #pragma unroll 1
                 for (int c = 0; c < TN / 32; c++) {
+                    if (n0 + 32 * c >= n_rows) break;
                     uint32_t a[32];
                     TMEM_LD32(tl + 32 * c, a);
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
@@ -200,17 +250,19 @@ __global__ void __launch_bounds__(NTHREADS, 2) gemm_bf16_kernel(const __grid_con
                                 float v[8];
 #pragma unroll
                                 for (int e = 0; e < 8; e++) v[e] = __uint_as_float(a[j + e]);
-                                put8(p.c, s, row, (int64_t)g * n_rows + n, g, v, std::min(8, n_rows - n));
+                                put8(p.c, s, row, (int64_t)w.g * n_rows + n, w.g, v, std::min(8, n_rows - n));
                             }
                         }
                     }
                 }
             }
+            asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
+            asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(&acc_empty[buf])) : "memory");
         }
     }
     asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
     __syncthreads();
-    if (warp == 1) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(TMEM_COLS) : "memory");
+    if (warp == 1) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(S::TMEM_COLS) : "memory");
 }
 
 // ---- f32 form ------------------------------------------------------------------------------------
@@ -291,6 +343,19 @@ b200_status kq_gemm_bf16(const KqDense &c, const uint16_t *a, int64_t lda, int p
     p.c = c;
     p.parts = parts;
     p.nk = (int)kq_div_up(c.K, BK);
+    p.mt = (int)kq_div_up(c.M, TM);
+    // 256-row tiles read less per product, 128-row tiles fill the last wave of CTAs better
+    auto n_tiles = [&](int tn) {
+        int t = 0;
+        if (c.glu) t = (int)kq_div_up(std::max(c.seg[0].n_rows, c.seg[0].pad_cols), tn / 2);
+        else
+            for (int i = 0; i < c.nseg; i++) t += (int)kq_div_up(c.seg[i].n_rows, tn);
+        return t;
+    };
+    const int64_t sms = kq_sm_count();
+    const int64_t w256 = kq_div_up((int64_t)p.mt * n_tiles(256) * c.groups, sms) * 20, w128 = kq_div_up((int64_t)p.mt * n_tiles(128) * c.groups, sms) * 13;
+    const int tn = w256 <= w128 ? 256 : 128;
+    p.nt = n_tiles(tn);
     {
         const uint64_t dims[3] = {(uint64_t)lda, (uint64_t)c.M, (uint64_t)parts};
         const uint64_t str[2] = {(uint64_t)lda * 2, (uint64_t)lda * 2 * c.M};
@@ -302,22 +367,23 @@ b200_status kq_gemm_bf16(const KqDense &c, const uint16_t *a, int64_t lda, int p
     for (int i = 0; i < 3; i++) {
         const KqDenseSeg &s = c.seg[std::min(i, c.nseg - 1)];
         const uint64_t dims[2] = {(uint64_t)c.ldw, (uint64_t)s.n_rows * c.groups}, str[1] = {(uint64_t)c.ldw * 2};
-        const uint32_t box[2] = {BK, 64};
+        const uint32_t box[2] = {BK, (uint32_t)tn / 2};
         const b200_status rc = kq_tmap_encode(&p.b[i], 2, 2, s.W, dims, str, box, 1);
         if (rc != B200_OK) return rc;
-        if (i < c.nseg) tiles += (int)kq_div_up(s.n_rows, TN);
+        if (i < c.nseg) tiles += (int)kq_div_up(s.n_rows, tn);
         p.tile_end[i] = tiles;
     }
-    if (c.glu) tiles = (int)kq_div_up(std::max(c.seg[0].n_rows, c.seg[0].pad_cols), TN / 2);
+    const unsigned grid = (unsigned)std::min<int64_t>((int64_t)p.mt * p.nt * c.groups, sms);
     static bool attr[16];
     int dev = 0;
     KQ_CUDA(cudaGetDevice(&dev));
     if (dev < 0 || dev >= 16 || !attr[dev]) {
-        KQ_CUDA(cudaFuncSetAttribute(gemm_bf16_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_TOTAL));
+        KQ_CUDA(cudaFuncSetAttribute(gemm_bf16_kernel<256>, cudaFuncAttributeMaxDynamicSharedMemorySize, Tile<256>::SMEM_TOTAL));
+        KQ_CUDA(cudaFuncSetAttribute(gemm_bf16_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, Tile<128>::SMEM_TOTAL));
         if (dev >= 0 && dev < 16) attr[dev] = true;
     }
-    const dim3 grid((unsigned)kq_div_up(c.M, TM), (unsigned)tiles, (unsigned)c.groups);
-    kq_launch(gemm_bf16_kernel, grid, NTHREADS, SMEM_TOTAL, st, p);
+    if (tn == 256) kq_launch(gemm_bf16_kernel<256>, grid, NTHREADS, Tile<256>::SMEM_TOTAL, st, p);
+    else kq_launch(gemm_bf16_kernel<128>, grid, NTHREADS, Tile<128>::SMEM_TOTAL, st, p);
     KQ_COUNT_LAUNCH();
     KQ_LAUNCH_CHECK();
     return B200_OK;
