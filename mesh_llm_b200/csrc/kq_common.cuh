@@ -203,14 +203,6 @@ __device__ __forceinline__ bool kq_mbar_wait(uint32_t bar, uint32_t parity, uint
         if (kq_globaltimer_ns() - t0 > limit_ns) return false;
     return true;
 }
-// The same for waits that are on the critical path of a pipeline: reading %globaltimer costs more than such a wait
-// usually takes, so the clock starts only after a number of tries.
-__device__ __forceinline__ bool kq_mbar_wait_hot(uint32_t bar, uint32_t parity, uint64_t limit_ns) {
-#pragma unroll 1
-    for (int i = 0; i < 64; i++)
-        if (kq_mbar_try(bar, parity)) return true;
-    return kq_mbar_wait(bar, parity, limit_ns);
-}
 #define KQ_WAIT_LIMIT_NS 20000000ull /* 20 ms: four orders of magnitude above any healthy wait */
 
 // The activation quantiser of the library (same arithmetic as the CPU oracle, operation for

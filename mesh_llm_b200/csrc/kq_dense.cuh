@@ -76,6 +76,16 @@ __device__ __forceinline__ float kq_bf2f(uint16_t v) { return __uint_as_float((u
 __device__ __forceinline__ uint16_t kq_f2h_sat(float v) {
     return __half_as_ushort(__float2half_rn(fminf(fmaxf(v, -65504.f), 65504.f)));
 }
+// Segment i of a call that is a kernel parameter.  The selects keep the parameters in the constant bank: indexed by a
+// variable they are read through generic loads, hundreds of cycles each.
+__device__ __forceinline__ KqDenseSeg kq_dense_seg(const KqDense &c, int i) {
+    KqDenseSeg s = c.seg[0];
+    if (i == 1) s = c.seg[1];
+    if (i == 2) s = c.seg[2];
+    return s;
+}
+__device__ __forceinline__ int kq_dense_rows(const KqDense &c, int i) { return i == 0 ? c.seg[0].n_rows : i == 1 ? c.seg[1].n_rows : c.seg[2].n_rows; }
+__device__ __forceinline__ const uint16_t *kq_dense_w(const KqDense &c, int i) { return i == 0 ? c.seg[0].W : i == 1 ? c.seg[1].W : c.seg[2].W; }
 __device__ __forceinline__ int64_t kq_dense_col(const KqDenseSeg &s, int64_t n) {
     return s.head_in ? n / s.head_in * s.head_out + n % s.head_in : n;
 }

@@ -4,7 +4,8 @@
 // Tensor cores: a persistent CTA per SM walks tiles of 128 tokens (TMEM lanes) x 256 or 128 weight rows (columns), token
 // tiles innermost, so that the CTAs at work share the weight rows they read.  K runs in slices of 64 (one
 // 128-byte-swizzled row per operand row); a producer thread brings the slices in by tiled TMA copies through a ring
-// of stages, one thread issues the MMAs into one of two accumulators in TMEM, four warps drain the other one meanwhile.
+// of stages, one thread issues the MMAs into one of two accumulators in TMEM, four warps drain the other one meanwhile,
+// through a transpose in shared memory: stores of one row per lane would run at a fifth of the rate.
 // A gate / up pair shares a tile half and half, so that the GLU happens where both values are.
 // An f32 operand can come as several bf16 parts (x = hi + mid + lo exactly): the K loop then passes over the
 // same weights once per part.  Block-diagonal products offset the K coordinate of x and the row of W by group.
@@ -20,10 +21,11 @@
 namespace {
 
 constexpr int TM = 128, BK = 64, A_BYTES = TM * BK * 2;
+constexpr int EC = 32, EP = EC + 4, EPI_BYTES = 4 * 32 * EP * 4; // columns an epilogue warp turns round at a time, floats per staged row
 template <int TN>
 struct Tile {
     static constexpr int B_BYTES = TN * BK * 2, STAGE_BYTES = A_BYTES + B_BYTES, STAGES = 192 * 1024 / STAGE_BYTES;
-    static constexpr int SMEM_TOTAL = STAGES * STAGE_BYTES + 1024;
+    static constexpr int SMEM_TOTAL = STAGES * STAGE_BYTES + EPI_BYTES + 1024;
     static constexpr uint32_t TMEM_COLS = 2 * TN; // two accumulators
 };
 constexpr int NTHREADS = 192, NEPI = 128; // producer warp, MMA warp, four epilogue warps
@@ -39,51 +41,48 @@ struct GemmParams {
     int32_t mt, nt;         // tiles of tokens and of weight rows (all segments)
 };
 
-// eight consecutive output columns of one row
-__device__ __forceinline__ void put8(const KqDense &c, const KqDenseSeg &s, int64_t m, int64_t n, int g, const float *v, int n_valid) {
-    if (n_valid == 8 && ((s.ldy | n | s.head_in | s.head_out) & 7) == 0) { // all eight in one head, 16-byte aligned
-        float o[8], bias[8] = {};
-        if (s.bias) {
-            if (((uintptr_t)(s.bias + n) & 15) == 0) {
-                *reinterpret_cast<float4 *>(bias) = *reinterpret_cast<const float4 *>(s.bias + n);
-                *reinterpret_cast<float4 *>(bias + 4) = *reinterpret_cast<const float4 *>(s.bias + n + 4);
-            } else {
+// four consecutive output columns n .. n + 3 (over all groups), for a number of rows
+struct Col4 {
+    float bias[4];
+    int64_t col, n;
+    int32_t valid;
+    bool vec; // all four next to one another and aligned in every row
+    __device__ __forceinline__ Col4(const KqDense &c, const KqDenseSeg &s, int64_t n_, int n_valid) : n(n_), valid(n_valid) {
+        vec = valid == 4 && ((s.ldy | n | s.head_in | s.head_out) & 3) == 0 && ((uintptr_t)s.y & 15) == 0;
+        col = kq_dense_col(s, n);
 #pragma unroll
-                for (int j = 0; j < 8; j++) bias[j] = s.bias[n + j];
-            }
-        }
+        for (int e = 0; e < 4; e++) bias[e] = s.bias && e < valid ? s.bias[n + e] : 0.f;
+    }
+    __device__ __forceinline__ void store(const KqDense &c, const KqDenseSeg &s, int64_t m, int g, const float4 &v) const {
+        float o[4] = {v.x + bias[0], v.y + bias[1], v.z + bias[2], v.w + bias[3]};
+        if (s.act == KQ_ACT_GELU_TANH) {
 #pragma unroll
-        for (int j = 0; j < 8; j++) {
-            float t = v[j] + bias[j];
-            if (s.act == KQ_ACT_GELU_TANH) t = kq_gelu_tanh(t);
-            if (c.head_gate) t *= kq_sigmoid(c.head_gate[m * c.ld_gate + g]);
-            o[j] = t;
+            for (int e = 0; e < 4; e++) o[e] = kq_gelu_tanh(o[e]);
         }
-        const int64_t i = m * s.ldy + kq_dense_col(s, n);
-        if (s.out == KQ_OUT_F32) {
-            float *y = (float *)s.y + i;
-            if (((uintptr_t)y & 31) == 0) { // a whole sector at once
-                asm volatile("st.global.v8.f32 [%0], {%1, %2, %3, %4, %5, %6, %7, %8};" ::"l"(y), "f"(o[0]), "f"(o[1]), "f"(o[2]), "f"(o[3]),
-                             "f"(o[4]), "f"(o[5]), "f"(o[6]), "f"(o[7])
-                             : "memory");
+        if (c.head_gate) {
+            const float f = kq_sigmoid(c.head_gate[m * c.ld_gate + g]);
+#pragma unroll
+            for (int e = 0; e < 4; e++) o[e] *= f;
+        }
+        if (vec) {
+            const int64_t i = m * s.ldy + col;
+            if (s.out == KQ_OUT_F32) {
+                *reinterpret_cast<float4 *>((float *)s.y + i) = make_float4(o[0], o[1], o[2], o[3]);
             } else {
-                *reinterpret_cast<float4 *>(y) = make_float4(o[0], o[1], o[2], o[3]);
-                *reinterpret_cast<float4 *>(y + 4) = make_float4(o[4], o[5], o[6], o[7]);
+                uint32_t w[2];
+#pragma unroll
+                for (int e = 0; e < 2; e++)
+                    w[e] = s.out == KQ_OUT_BF16 ? (uint32_t)kq_f2bf(o[2 * e]) | ((uint32_t)kq_f2bf(o[2 * e + 1]) << 16)
+                                                : (uint32_t)kq_f2h_sat(o[2 * e]) | ((uint32_t)kq_f2h_sat(o[2 * e + 1]) << 16);
+                *reinterpret_cast<uint2 *>((uint16_t *)s.y + i) = make_uint2(w[0], w[1]);
             }
         } else {
-            uint32_t w[4];
 #pragma unroll
-            for (int j = 0; j < 4; j++)
-                w[j] = s.out == KQ_OUT_BF16 ? (uint32_t)kq_f2bf(o[2 * j]) | ((uint32_t)kq_f2bf(o[2 * j + 1]) << 16)
-                                            : (uint32_t)kq_f2h_sat(o[2 * j]) | ((uint32_t)kq_f2h_sat(o[2 * j + 1]) << 16);
-            *reinterpret_cast<uint4 *>((uint16_t *)s.y + i) = make_uint4(w[0], w[1], w[2], w[3]);
+            for (int e = 0; e < 4; e++)
+                if (e < valid) kq_dense_put(s, m, n + e, o[e]);
         }
-        return;
     }
-#pragma unroll
-    for (int j = 0; j < 8; j++)
-        if (j < n_valid) kq_dense_store(c, s, m, n + j, g, v[j]);
-}
+};
 
 template <int TN>
 __global__ void __launch_bounds__(NTHREADS, 1) gemm_bf16_kernel(const __grid_constant__ GemmParams p) {
@@ -131,130 +130,132 @@ __global__ void __launch_bounds__(NTHREADS, 1) gemm_bf16_kernel(const __grid_con
         w.g = rest / p.nt;
         w.seg = 0;
         if (!p.c.glu) {
-            while (w.seg + 1 < p.c.nseg && nt >= p.tile_end[w.seg]) w.seg++;
-            if (w.seg) nt -= p.tile_end[w.seg - 1];
+            if (nt >= p.tile_end[1]) w.seg = 2, nt -= p.tile_end[1];
+            else if (nt >= p.tile_end[0]) w.seg = 1, nt -= p.tile_end[0];
         }
-        w.n_rows = p.c.seg[w.seg].n_rows;
+        w.n_rows = kq_dense_rows(p.c, w.seg);
         w.n0 = nt * (p.c.glu ? TN / 2 : TN); // first row of the tile inside the group
         return w;
     };
-    auto wait = [&](uint64_t *bar, uint32_t parity, int code) {
-        if (!*(volatile int *)&s_abort && !kq_mbar_wait_hot(smem_u32(bar), parity, LIMIT)) {
-            *(volatile int *)&s_abort = 1;
-            atomicExch(&g_gemm_bf16_error, code);
-        }
-        return !*(volatile int *)&s_abort;
+    auto wait = [&](uint64_t *bar, uint32_t parity, int code) { // a warp gives up as a whole
+        return __all_sync(0xffffffffu, tc_wait(smem_u32(bar), parity, &s_abort, &g_gemm_bf16_error, code, LIMIT)) != 0;
     };
+    // The producer and the MMA warp run their loops with all lanes, so that addresses and descriptors stay in uniform
+    // registers; one lane posts and issues.
     if (warp == 0) {
-        if (lane == 0) {
-            int it = 0; // slices over all tiles
-            bool ok = true;
-            for (int tile = blockIdx.x; ok && tile < n_tiles; tile += gridDim.x) {
-                const Where w = locate(tile);
-                for (int i = 0; i < n_it; i++, it++) {
-                    const int s = it % S::STAGES;
-                    if (it >= S::STAGES && !(ok = wait(&empty[s], (uint32_t)((it / S::STAGES - 1) & 1), 1))) break;
+        const bool lead = tc_elect();
+        int it = 0, s = 0; // slices over all tiles, stage
+        uint32_t round = 0; // uses of the ring so far
+        bool ok = true;
+        for (int tile = blockIdx.x; ok && tile < n_tiles; tile += gridDim.x) {
+            const Where w = locate(tile);
+            const int row = w.g * w.n_rows + w.n0, xk = (int)(w.g * p.c.xg);
+            const CUtensorMap *map0 = p.b + (p.c.glu ? 0 : w.seg), *map1 = p.b + (p.c.glu ? 1 : w.seg); // half a tile of rows each
+            const int row1 = row + (p.c.glu ? 0 : TN / 2);
+            int part = 0, kk = 0;
+            for (int i = 0; i < n_it; i++, it++) {
+                if (round > 0 && !(ok = wait(&empty[s], (round - 1) & 1, 1))) break;
+                if (lead) {
                     const uint32_t bar = smem_u32(&full[s]), dst = smem_u32(sm + s * S::STAGE_BYTES);
                     asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(S::STAGE_BYTES) : "memory");
-                    const int part = i / p.nk, kk = (i % p.nk) * BK;
                     asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];" ::"r"(dst),
-                                 "l"(&p.a), "r"((int)(w.g * p.c.xg) + kk), "r"(w.m0), "r"(part), "r"(bar)
+                                 "l"(&p.a), "r"(xk + kk), "r"(w.m0), "r"(part), "r"(bar)
                                  : "memory");
-#pragma unroll
-                    for (int hb = 0; hb < 2; hb++) { // half a tile of weight rows each: of one matrix, or gate and up
-                        const CUtensorMap *map = p.c.glu ? &p.b[hb] : &p.b[w.seg];
-                        const int row = w.g * w.n_rows + w.n0 + (p.c.glu ? 0 : hb * (TN / 2));
-                        asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(
-                                         dst + A_BYTES + hb * (S::B_BYTES / 2)),
-                                     "l"(map), "r"(kk), "r"(row), "r"(bar)
-                                     : "memory");
-                    }
+                    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(dst + A_BYTES),
+                                 "l"(map0), "r"(kk), "r"(row), "r"(bar)
+                                 : "memory");
+                    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(
+                                     dst + A_BYTES + S::B_BYTES / 2),
+                                 "l"(map1), "r"(kk), "r"(row1), "r"(bar)
+                                 : "memory");
                 }
+                __syncwarp();
+                kk += BK;
+                if (kk == p.nk * BK) kk = 0, part++;
+                if (++s == S::STAGES) s = 0, round++;
             }
-            if (!ok) // copies that were posted must land before the CTA goes away
-                for (int i = std::max(0, it - S::STAGES); i < it; i++)
-                    kq_mbar_wait(smem_u32(&full[i % S::STAGES]), (uint32_t)((i / S::STAGES) & 1), KQ_WAIT_LIMIT_NS);
         }
+        if (!ok && lead) // copies that were posted must land before the CTA goes away
+            for (int i = std::max(0, it - S::STAGES); i < it; i++)
+                kq_mbar_wait(smem_u32(&full[i % S::STAGES]), (uint32_t)((i / S::STAGES) & 1), KQ_WAIT_LIMIT_NS);
         __syncwarp();
     } else if (warp == 1) {
-        if (lane == 0) {
-            int it = 0, t = 0;
-            bool ok = true;
-            for (int tile = blockIdx.x; ok && tile < n_tiles; tile += gridDim.x, t++) {
-                const int buf = t & 1;
-                if (t >= 2 && !(ok = wait(&acc_empty[buf], (uint32_t)((t / 2 - 1) & 1), 4))) break;
+        const bool lead = tc_elect();
+        int s = 0, t = 0;
+        uint32_t round = 0;
+        bool ok = true;
+        for (int tile = blockIdx.x; ok && tile < n_tiles; tile += gridDim.x, t++) {
+            const int buf = t & 1;
+            if (t >= 2 && !(ok = wait(&acc_empty[buf], (uint32_t)((t / 2 - 1) & 1), 4))) break;
+            asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+            for (int i = 0; i < n_it; i++) {
+                if (!(ok = wait(&full[s], round & 1, 2))) break;
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                for (int i = 0; i < n_it; i++, it++) {
-                    const int s = it % S::STAGES;
-                    if (!(ok = wait(&full[s], (uint32_t)((it / S::STAGES) & 1), 2))) break;
-                    asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
+                if (lead) {
                     const uint32_t a = smem_u32(sm + s * S::STAGE_BYTES), b = a + A_BYTES;
+                    const uint64_t da = tc_desc_k(a, 0), db = tc_desc_k(b, 0);
 #pragma unroll
-                    for (int k = 0; k < BK / 16; k++)
-                        tc_mma_ss(tmem + buf * TN, tc_desc_k(a, k), tc_desc_k(b, k), IDESC, (i > 0 || k > 0) ? 1u : 0u);
+                    for (int k = 0; k < BK / 16; k++) // 32 bytes further per step: 2 in the descriptor's address field
+                        tc_mma_ss(tmem + buf * TN, da + 2 * k, db + 2 * k, IDESC, (i > 0 || k > 0) ? 1u : 0u);
                     tc_commit(smem_u32(&empty[s]));
                 }
-                tc_commit(smem_u32(&acc_full[buf]));
+                __syncwarp();
+                if (++s == S::STAGES) s = 0, round++;
             }
-            if (!ok) // MMAs in flight end before TMEM is freed
-                for (int i = std::max(0, t - 2); i < t; i++) kq_mbar_wait(smem_u32(&acc_full[i & 1]), (uint32_t)((i / 2) & 1), KQ_WAIT_LIMIT_NS);
+            if (lead) tc_commit(smem_u32(&acc_full[buf]));
+            __syncwarp();
         }
+        if (!ok && lead) // MMAs in flight end before TMEM is freed
+            for (int i = std::max(0, t - 2); i < t; i++) kq_mbar_wait(smem_u32(&acc_full[i & 1]), (uint32_t)((i / 2) & 1), KQ_WAIT_LIMIT_NS);
         __syncwarp();
     } else {
         const int q = warp & 3; // a warp reaches the TMEM lanes of its quarter
+        float *stage = reinterpret_cast<float *>(sm + S::STAGES * S::STAGE_BYTES) + q * 32 * EP;
         int t = 0;
         for (int tile = blockIdx.x; tile < n_tiles; tile += gridDim.x, t++) {
             const int buf = t & 1;
             const bool ok = wait(&acc_full[buf], (uint32_t)((t / 2) & 1), 3);
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-            if (!__all_sync(0xffffffffu, ok)) break;
+            if (!ok) break;
             const Where w = locate(tile);
-            const int row = w.m0 + q * 32 + lane, n0 = w.n0, n_rows = w.n_rows;
+            const int n0 = w.n0, n_rows = w.n_rows, m0 = w.m0 + q * 32, m_end = std::min(p.c.M, m0 + 32);
             const uint32_t tl = tmem + ((uint32_t)(q * 32) << 16) + buf * TN;
-            const KqDenseSeg &s = p.c.seg[w.seg];
-            const bool row_ok = row < p.c.M;
-            if (p.c.glu) {
+            const KqDenseSeg s = kq_dense_seg(p.c, w.seg);
+            // EC columns at a time: a lane takes its row out of TMEM into shared memory, then eight lanes write a row's columns, four
+            // rows per store.  The loops stay loops: unrolled, the four warps would spend their time fetching code.
+            const int lim = p.c.glu ? std::max(n_rows, s.pad_cols) : n_rows; // the padding of a staging row is written too
+            const int n_cols = std::min(p.c.glu ? TN / 2 : TN, lim - n0);
+            const int r4 = lane >> 3, c4 = (lane & 7) * 4;
 #pragma unroll 1
-                for (int c = 0; c < TN / 64; c++) {
-                    uint32_t a[32], b[32];
-                    TMEM_LD32(tl + 32 * c, a);
-                    TMEM_LD32(tl + TN / 2 + 32 * c, b);
+            for (int j = 0; j < n_cols; j += EC) {
+#pragma unroll
+                for (int h = 0; h < EC; h += 16) {
+                    uint32_t a[16], b[16];
+                    TMEM_LD16(tl + j + h, a);
+                    if (p.c.glu) TMEM_LD16(tl + TN / 2 + j + h, b);
                     asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-                    if (row_ok) {
+                    if (p.c.glu) {
 #pragma unroll
-                        for (int j = 0; j < 32; j += 8) {
-                            const int n = n0 + 32 * c + j;
-                            float v[8];
+                        for (int e = 0; e < 16; e++)
+                            a[e] = n0 + j + h + e < n_rows ? __float_as_uint(kq_clamped_glu(__uint_as_float(a[e]), __uint_as_float(b[e]),
+                                                                                            p.c.glu_limit, p.c.glu_alpha))
+                                                           : 0u;
+                    }
 #pragma unroll
-                            for (int e = 0; e < 8; e++)
-                                v[e] = n + e < n_rows ? kq_clamped_glu(__uint_as_float(a[j + e]), __uint_as_float(b[j + e]),
-                                                                       p.c.glu_limit, p.c.glu_alpha)
-                                                      : 0.f;
-                            const int lim = std::max(n_rows, s.pad_cols); // the padding of a staging row is written too
-                            if (n < lim) put8(p.c, s, row, n, 0, v, std::min(8, lim - n));
-                        }
+                    for (int e = 0; e < 16; e += 4)
+                        *reinterpret_cast<uint4 *>(stage + lane * EP + h + e) = make_uint4(a[e], a[e + 1], a[e + 2], a[e + 3]);
+                }
+                __syncwarp();
+                const int n = n0 + j + c4, n_valid = std::min(4, lim - n);
+                if (n_valid > 0) {
+                    const Col4 col(p.c, s, (int64_t)w.g * n_rows + n, n_valid);
+#pragma unroll 2
+                    for (int r = r4; m0 + r < m_end; r += 4) {
+                        const float4 v = *reinterpret_cast<const float4 *>(stage + r * EP + c4);
+                        col.store(p.c, s, m0 + r, w.g, v);
                     }
                 }
-            } else {
-#pragma unroll 1
-                for (int c = 0; c < TN / 32; c++) {
-                    if (n0 + 32 * c >= n_rows) break;
-                    uint32_t a[32];
-                    TMEM_LD32(tl + 32 * c, a);
-                    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
-                    if (row_ok) {
-#pragma unroll
-                        for (int j = 0; j < 32; j += 8) {
-                            const int n = n0 + 32 * c + j;
-                            if (n < n_rows) {
-                                float v[8];
-#pragma unroll
-                                for (int e = 0; e < 8; e++) v[e] = __uint_as_float(a[j + e]);
-                                put8(p.c, s, row, (int64_t)w.g * n_rows + n, w.g, v, std::min(8, n_rows - n));
-                            }
-                        }
-                    }
-                }
+                __syncwarp();
             }
             asm volatile("tcgen05.fence::before_thread_sync;" ::: "memory");
             asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(&acc_empty[buf])) : "memory");
@@ -281,10 +282,10 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ F
     const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4, g = blockIdx.z;
     int seg = 0, nt = blockIdx.y;
     if (!GLU) {
-        while (seg + 1 < p.c.nseg && nt >= p.tile_end[seg]) seg++;
-        if (seg) nt -= p.tile_end[seg - 1];
+        if (nt >= p.tile_end[1]) seg = 2, nt -= p.tile_end[1];
+        else if (nt >= p.tile_end[0]) seg = 1, nt -= p.tile_end[0];
     }
-    const KqDenseSeg &s = p.c.seg[seg];
+    const KqDenseSeg s = kq_dense_seg(p.c, seg);
     const int m0 = blockIdx.x * FT, n0 = nt * FT, n_rows = s.n_rows, K = p.c.K;
     float acc[GLU ? 2 : 1][4][4] = {};
     for (int k0 = 0; k0 < K; k0 += FK) {
@@ -294,7 +295,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ F
 #pragma unroll
             for (int h = 0; h < (GLU ? 2 : 1); h++)
                 sb[h][k][r] = n0 + r < n_rows && k0 + k < K
-                                  ? kq_bf2f(p.c.seg[GLU ? h : seg].W[((int64_t)g * n_rows + n0 + r) * p.c.ldw + k0 + k])
+                                  ? kq_bf2f(kq_dense_w(p.c, GLU ? h : seg)[((int64_t)g * n_rows + n0 + r) * p.c.ldw + k0 + k])
                                   : 0.f;
         }
         __syncthreads();

@@ -46,7 +46,14 @@ __device__ __forceinline__ void locate(const GemvParams &p, int v, int &seg, int
     }
     seg = 0;
     row = v;
-    while (seg + 1 < p.c.nseg && row >= p.c.seg[seg].n_rows) row -= p.c.seg[seg++].n_rows;
+    if (p.c.nseg > 1 && row >= p.c.seg[0].n_rows) {
+        seg = 1;
+        row -= p.c.seg[0].n_rows;
+        if (p.c.nseg > 2 && row >= p.c.seg[1].n_rows) {
+            seg = 2;
+            row -= p.c.seg[1].n_rows;
+        }
+    }
 }
 
 template <int M>
@@ -63,7 +70,7 @@ __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __g
     auto row_ptr = [&](int v) {
         int s, r;
         locate(p, min(v, p.V - 1), s, r);
-        return reinterpret_cast<const uint4 *>(p.c.seg[s].W + (int64_t)r * p.c.ldw);
+        return reinterpret_cast<const uint4 *>(kq_dense_w(p.c, s) + (int64_t)r * p.c.ldw);
     };
     // first weights of this CTA: they depend on nothing
     uint4 w[4][2];
@@ -208,7 +215,7 @@ __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __g
                 for (int i = 0; i < NW; i++) s2 += part[buf][i][vl + 1][m];
                 kq_dense_put(p.c.seg[0], m, r, kq_clamped_glu(s, s2, p.c.glu_limit, p.c.glu_alpha));
             } else {
-                kq_dense_store(p.c, p.c.seg[sg], m, r, 0, s);
+                kq_dense_store(p.c, kq_dense_seg(p.c, sg), m, r, 0, s);
             }
         }
     }

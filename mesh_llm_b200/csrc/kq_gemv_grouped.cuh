@@ -39,7 +39,7 @@ __device__ __forceinline__ void kq_grouped_rows(const KqGrouped &p, int64_t id, 
     const bool live = id < per * p.c.nseg;
     const int sg = live ? (int)(id / per) : 0;
     const int g = live ? (int)(id % per / p.quads) : 0, r0 = (int)(id % p.quads) * 4;
-    const KqDenseSeg &s = p.c.seg[sg];
+    const KqDenseSeg s = kq_dense_seg(p.c, sg);
     const bool ok = live && r0 < s.n_rows;
     const int K = p.c.K, nck = (K + 7) / 8;
     const uint4 *wp[4];

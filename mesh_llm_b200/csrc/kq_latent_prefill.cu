@@ -150,10 +150,7 @@ __global__ void __launch_bounds__(NTHREADS, 2) latent_prefill_tc_kernel(const __
             const uint32_t id_s = tc_idesc(128, BK, false, false), id_o = tc_idesc(128, ncol, false, true);
             const int su = (p.dim + 15) / 16, sr = (p.rot + 15) / 16; // K steps of the two key parts
             auto wait = [&](uint32_t bar, uint32_t parity, int code) {
-                if (!s_abort && !kq_mbar_wait_hot(bar, parity, LIMIT)) {
-                    s_abort = 1;
-                    atomicExch(&g_latent_tc_error, code);
-                }
+                tc_wait(bar, parity, &s_abort, &g_latent_tc_error, code, LIMIT);
             };
             for (int i = 0; i < n_tiles; i++) {
                 const uint32_t ph = (uint32_t)(i & 1);
@@ -190,10 +187,7 @@ __global__ void __launch_bounds__(NTHREADS, 2) latent_prefill_tc_kernel(const __
         const int c0 = HK * half;
         float m = -INFINITY, l = 0.f;
         for (int i = 0; i < n_tiles; i++) {
-            if (!s_abort && !kq_mbar_wait_hot(bar_s, (uint32_t)(i & 1), LIMIT)) {
-                s_abort = 1;
-                atomicExch(&g_latent_tc_error, 6);
-            }
+            tc_wait(bar_s, (uint32_t)(i & 1), &s_abort, &g_latent_tc_error, 6, LIMIT);
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const int t0 = first + i * BK, k0 = t0 + c0;
             // some row of the tile sees only part of these keys: past the diagonal, or behind the last row's window
@@ -263,10 +257,7 @@ __global__ void __launch_bounds__(NTHREADS, 2) latent_prefill_tc_kernel(const __
         if (half == 0) lsum[row] = l + lsum[row];
         softmax_barrier();
         l = lsum[row];
-        if (!s_abort && !kq_mbar_wait_hot(bar_pv, (uint32_t)((n_tiles - 1) & 1), LIMIT)) {
-            s_abort = 1;
-            atomicExch(&g_latent_tc_error, 7);
-        }
+        tc_wait(bar_pv, (uint32_t)((n_tiles - 1) & 1), &s_abort, &g_latent_tc_error, 7, LIMIT);
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         const bool go = __all_sync(0xffffffffu, !s_abort);
         if (go) {

@@ -20,6 +20,29 @@ __device__ __forceinline__ uint64_t tc_desc(uint32_t saddr, uint32_t lbo, uint32
     d |= (uint64_t)2 << 61; // SWIZZLE_128B
     return d;
 }
+// Waits of a pipeline.  The common case is a few tries; only a wait that lasts looks at the clock (reading %globaltimer
+// costs more than a usual wait) and at the CTA's give-up word, and after limit_ns sets that word and the error word.
+__device__ __forceinline__ bool tc_wait(uint32_t bar, uint32_t parity, volatile int *give_up, int *error_word, int code, uint64_t limit_ns) {
+#pragma unroll 1
+    for (int i = 0; i < 32; i++)
+        if (kq_mbar_try(bar, parity)) return true;
+    const uint64_t t0 = kq_globaltimer_ns();
+    while (!kq_mbar_try(bar, parity)) {
+        if (*give_up) return false;
+        if (kq_globaltimer_ns() - t0 > limit_ns) {
+            *give_up = 1;
+            atomicExch(error_word, code);
+            return false;
+        }
+    }
+    return true;
+}
+// one lane of a converged warp
+__device__ __forceinline__ bool tc_elect() {
+    uint32_t ok;
+    asm volatile("{\n\t.reg .pred p;\n\telect.sync _|p, 0xffffffff;\n\tselp.u32 %0, 1, 0, p;\n\t}" : "=r"(ok));
+    return ok != 0;
+}
 // K-major operand: rows of 128 bytes (64 elements), 8-row groups 1024 bytes apart; K step s of 16 elements
 __device__ __forceinline__ uint64_t tc_desc_k(uint32_t tile, int s) { return tc_desc(tile + s * 32, 16, 1024); }
 // MN-major operand: 64-element atoms `atom_bytes` apart, groups of 8 K rows 1024 bytes apart; K step s of 16 rows
@@ -46,6 +69,12 @@ __device__ __forceinline__ void tc_commit(uint32_t bar) {
     asm volatile("tcgen05.commit.cta_group::1.mbarrier::arrive::one.shared::cluster.b64 [%0];" ::"r"(bar) : "memory");
 }
 
+#define TMEM_LD16(taddr, r)                                                                                             \
+    asm volatile("tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];" \
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]),      \
+                   "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]) \
+                 : "r"(taddr)                                                                                           \
+                 : "memory")
 #define TMEM_LD32(taddr, r)                                                                                             \
     asm volatile("tcgen05.ld.sync.aligned.32x32b.x32.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,"        \
                  "%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31}, [%32];"                              \
