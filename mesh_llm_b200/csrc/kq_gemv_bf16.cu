@@ -56,6 +56,11 @@ __device__ __forceinline__ void locate(const GemvParams &p, int v, int &seg, int
     }
 }
 
+// brings n floats into this SM's L1 without waiting for them
+__device__ __forceinline__ void touch(const float *p, int n) {
+    for (int i = threadIdx.x * 8; i < n; i += NT * 8) asm volatile("{\n\t.reg .f32 t;\n\tld.global.ca.f32 t, [%0];\n\t}" ::"l"(p + i));
+}
+
 template <int M>
 __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __grid_constant__ GemvParams p) {
     extern __shared__ __align__(16) float sm[];
@@ -89,6 +94,8 @@ __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __g
         for (int r = 0; r < 4; r++) wp[r] = row_ptr(v0 + r);
         load(tid, v1 - v0);
     }
+    if (p.p.sub_w) touch(p.p.sub_w, K);
+    if (p.p.norm_w) touch(p.p.norm_w, K);
     KQ_PDL_WAIT();
 
     // ---- activations
@@ -106,14 +113,15 @@ __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __g
             float sc = 1.f;
             if (p.p.sub_w) {
                 float s2 = 0.f;
-                for (int i = tid; i < n4; i += NT) {
+                for (int i = tid; i < n4; i += NT) { // x comes along: its round trip is over when it is needed
                     const float4 v = kq_load4(sub, 4 * i, K, vec);
+                    px[(i & 1) * nck + (i >> 1)] = kq_load4(x, 4 * i, K, vec);
                     s2 += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
                 }
                 sc = 1.0f / sqrtf(block_sum(s2, red) / (float)K + p.p.eps);
             }
             for (int i = tid; i < n4; i += NT) {
-                const float4 a = kq_load4(x, 4 * i, K, vec), b = kq_load4(sub, 4 * i, K, vec);
+                const float4 a = p.p.sub_w ? px[(i & 1) * nck + (i >> 1)] : kq_load4(x, 4 * i, K, vec), b = kq_load4(sub, 4 * i, K, vec);
                 float4 g = make_float4(1.f, 1.f, 1.f, 1.f);
                 if (p.p.sub_w) {
                     g = kq_load4(p.p.sub_w, 4 * i, K, true);
@@ -153,24 +161,18 @@ __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __g
     }
     __syncthreads();
 
-    // ---- rows
+    // ---- rows; the first weights of the next four are requested before this group's sums are reduced
     int buf = 0;
-    bool loaded = true;
     for (int vb = v0; vb < v1; vb += SB, buf ^= 1) {
         const int ve = min(v1, vb + SB);
         for (int v = vb; v < ve; v += 4) {
-            if (!loaded) {
-#pragma unroll
-                for (int r = 0; r < 4; r++) wp[r] = row_ptr(v + r);
-            }
             float acc[4][M];
 #pragma unroll
             for (int r = 0; r < 4; r++)
 #pragma unroll
                 for (int m = 0; m < M; m++) acc[r][m] = 0.f;
             for (int i = tid; i < nck; i += 2 * NT) {
-                if (!loaded) load(i, v1 - v);
-                loaded = false;
+                if (i != tid) load(i, v1 - v);
 #pragma unroll
                 for (int j = 0; j < 2; j++) {
                     const int c = i + j * NT;
@@ -179,14 +181,16 @@ __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __g
                         for (int m = 0; m < M; m++) {
                             const float4 a = pl[(m * 2) * nck + c], b = pl[(m * 2 + 1) * nck + c];
 #pragma unroll
-                            for (int r = 0; r < 4; r++) {
-                                acc[r][m] = kq_dot8(w[r][j], a, b, acc[r][m]);
-                            }
+                            for (int r = 0; r < 4; r++) acc[r][m] = kq_dot8(w[r][j], a, b, acc[r][m]);
                         }
                     }
                 }
             }
-            loaded = false;
+            if (v + 4 < v1) {
+#pragma unroll
+                for (int r = 0; r < 4; r++) wp[r] = row_ptr(v + 4 + r);
+                load(tid, v1 - v - 4);
+            }
             // four rows across the warp: after two exchanges a lane holds one row's sum over four lanes' worth
 #pragma unroll
             for (int m = 0; m < M; m++) {

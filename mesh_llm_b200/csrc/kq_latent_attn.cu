@@ -317,36 +317,42 @@ __global__ void __launch_bounds__(NT) latent_attn_mma_kernel(const __grid_consta
     const uint16_t *cache = (const uint16_t *)l.cache + seq * l.seq_stride;
     const int ks = (l.ld + 15) / 16, ld16 = ks * 16, n16 = ks * 2; // K steps of the scores, row length padded to them, 16-byte chunks
     auto load_tile = [&](int kb) {
-        for (int i = tid; i < MK * n16; i += NT) {
-            const int r = i / n16, c = i % n16, key = kb + r;
-            uint8_t *dst = tile + (size_t)r * pitch + 16 * c;
-            if (key < k1 && 8 * c < l.ld) {
-                const uint8_t *src = (const uint8_t *)(cache + (int64_t)(key % l.cap) * l.ld) + 16 * c;
-                asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
-            } else {
-                *reinterpret_cast<uint4 *>(dst) = make_uint4(0, 0, 0, 0);
+        for (int r = warp; r < MK; r += NW) { // a warp per row
+            const int key = kb + r;
+            const uint8_t *src = (const uint8_t *)(cache + (int64_t)(key % l.cap) * l.ld);
+            uint8_t *dst = tile + (size_t)r * pitch;
+            for (int c = lane; c < n16; c += 32) {
+                if (key < k1 && 8 * c < l.ld)
+                    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst + 16 * c)), "l"(src + 16 * c)
+                                 : "memory");
+                else
+                    *reinterpret_cast<uint4 *>(dst + 16 * c) = make_uint4(0, 0, 0, 0);
             }
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     load_tile(k0);
-    const int nq = HG * ld16 / 2;
-    for (int i0 = tid; i0 < nq; i0 += 6 * NT) { // queries, scaled, as hi + lo; six loads in flight
-        float2 v[6];
+    for (int d0 = 2 * lane; d0 < ld16; d0 += 64 * 5) { // queries of the warp's two heads, scaled, as hi + lo; ten loads in flight
+        float2 v[5][NH];
 #pragma unroll
-        for (int e = 0; e < 6; e++) {
-            const int i = i0 + e * NT, hl = i / (ld16 / 2), d = i % (ld16 / 2) * 2, h = hg * HG + hl;
-            v[e] = i < nq && h < l.n_head && d < l.ld ? *reinterpret_cast<const float2 *>(q_lat + (row * l.n_head + h) * l.ld + d) : make_float2(0.f, 0.f);
-        }
+        for (int e = 0; e < 5; e++)
 #pragma unroll
-        for (int e = 0; e < 6; e++) {
-            const int i = i0 + e * NT, hl = i / (ld16 / 2), d = i % (ld16 / 2) * 2;
-            if (i >= nq) break;
-            const float f = l.scale * 1.4426950408889634f, x = v[e].x * f, y = v[e].y * f;
-            const uint16_t hx = kq_f2bf(x), hy = kq_f2bf(y);
-            *reinterpret_cast<uint32_t *>(q_hi + hl * pitch + 2 * d) = (uint32_t)hx | ((uint32_t)hy << 16);
-            *reinterpret_cast<uint32_t *>(q_lo + hl * pitch + 2 * d) = (uint32_t)kq_f2bf(x - kq_bf2f(hx)) | ((uint32_t)kq_f2bf(y - kq_bf2f(hy)) << 16);
-        }
+            for (int a = 0; a < NH; a++) {
+                const int h = hg * HG + warp * NH + a, d = d0 + 64 * e;
+                v[e][a] = h < l.n_head && d < l.ld ? *reinterpret_cast<const float2 *>(q_lat + (row * l.n_head + h) * l.ld + d) : make_float2(0.f, 0.f);
+            }
+#pragma unroll
+        for (int e = 0; e < 5; e++)
+#pragma unroll
+            for (int a = 0; a < NH; a++) {
+                const int d = d0 + 64 * e;
+                if (d >= ld16) break;
+                const float f = l.scale * 1.4426950408889634f, x = v[e][a].x * f, y = v[e][a].y * f;
+                const uint16_t hx = kq_f2bf(x), hy = kq_f2bf(y);
+                *reinterpret_cast<uint32_t *>(q_hi + (warp * NH + a) * pitch + 2 * d) = (uint32_t)hx | ((uint32_t)hy << 16);
+                *reinterpret_cast<uint32_t *>(q_lo + (warp * NH + a) * pitch + 2 * d) =
+                    (uint32_t)kq_f2bf(x - kq_bf2f(hx)) | ((uint32_t)kq_f2bf(y - kq_bf2f(hy)) << 16);
+            }
     }
     float m[NH] = {-INFINITY, -INFINITY}, sum[NH] = {}, o[NP][2][4];
 #pragma unroll

@@ -120,8 +120,9 @@ __global__ void __launch_bounds__(NTHREADS, 2) latent_prefill_tc_kernel(const __
     const uint32_t tmem = s_tmem;
     const int ncol = p.nv * 64, nh = ncol / 2; // columns of O, and of one thread's half
 
-    if (warp == 8) {
-        if (lane == 0) {
+    if (warp == 8) { // all lanes run the loop, so that descriptors stay in uniform registers; one posts and issues
+        const bool lead = tc_elect();
+        {
             const int r0 = first - p.lo; // gathered row of the first key
             auto load_k = [&](int tile) {
                 asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar_k), "r"(nk * BOX) : "memory");
@@ -144,41 +145,54 @@ __global__ void __launch_bounds__(NTHREADS, 2) latent_prefill_tc_kernel(const __
                                  "l"(&p.v), "r"(b * 64), "r"(head), "r"(r0 + tile * BK), "r"(bar_v)
                                  : "memory");
             };
-            load_k(0);
-            load_v(0);
+            if (lead) {
+                load_k(0);
+                load_v(0);
+            }
+            __syncwarp();
             const uint32_t q_addr = smem_u32(sm_q), k_addr = smem_u32(sm_k), v_addr = smem_u32(sm_v);
             const uint32_t id_s = tc_idesc(128, BK, false, false), id_o = tc_idesc(128, ncol, false, true);
             const int su = (p.dim + 15) / 16, sr = (p.rot + 15) / 16; // K steps of the two key parts
             auto wait = [&](uint32_t bar, uint32_t parity, int code) {
-                tc_wait(bar, parity, &s_abort, &g_latent_tc_error, code, LIMIT);
+                return __all_sync(0xffffffffu, tc_wait(bar, parity, &s_abort_word, &g_latent_tc_error, code, LIMIT)) != 0; // a warp gives up as a whole
             };
+            bool go = true;
             for (int i = 0; i < n_tiles; i++) {
                 const uint32_t ph = (uint32_t)(i & 1);
-                wait(bar_k, ph, 1);
+                go = go && wait(bar_k, ph, 1);
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                if (!s_abort) {
-                    for (int s = 0; s < su; s++)
-                        tc_mma_ss(tmem + COL_S, tc_desc_k(q_addr + (s >> 2) * QBOX, s & 3), tc_desc_k(k_addr + (s >> 2) * BOX, s & 3), id_s, s > 0);
-                    for (int s = 0; s < sr; s++)
-                        tc_mma_ss(tmem + COL_S, tc_desc_k(q_addr + (p.nu + (s >> 2)) * QBOX, s & 3),
-                                  tc_desc_k(k_addr + (p.nu + (s >> 2)) * BOX, s & 3), id_s, 1);
+                if (lead) {
+                    if (go) {
+                        for (int s = 0; s < su; s++)
+                            tc_mma_ss(tmem + COL_S, tc_desc_k(q_addr + (s >> 2) * QBOX, s & 3), tc_desc_k(k_addr + (s >> 2) * BOX, s & 3), id_s, s > 0);
+                        for (int s = 0; s < sr; s++)
+                            tc_mma_ss(tmem + COL_S, tc_desc_k(q_addr + (p.nu + (s >> 2)) * QBOX, s & 3),
+                                      tc_desc_k(k_addr + (p.nu + (s >> 2)) * BOX, s & 3), id_s, 1);
+                    }
+                    tc_commit(bar_s);
                 }
-                tc_commit(bar_s);
-                wait(bar_s, ph, 2); // K has been read: the next tile's K can come in
-                if (!s_abort && i + 1 < n_tiles) load_k(i + 1);
-                wait(bar_p, ph, 3);
-                wait(bar_v, ph, 4);
+                __syncwarp();
+                go = wait(bar_s, ph, 2) && go; // K has been read: the next tile's K can come in
+                if (lead && go && i + 1 < n_tiles) load_k(i + 1);
+                __syncwarp();
+                go = go && wait(bar_p, ph, 3);
+                go = go && wait(bar_v, ph, 4);
                 asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-                if (!s_abort) {
+                if (lead) {
+                    if (go) {
 #pragma unroll
-                    for (int s = 0; s < BK / 16; s++) // 16 keys per instruction: eight packed columns of P at the start of each half's columns of S
-                        tc_mma_ts(tmem + COL_O, tmem + COL_S + HK * (s / (HK / 16)) + 8 * (s % (HK / 16)), tc_desc_mn(v_addr, BOX, s), id_o,
-                                  (i > 0 || s > 0) ? 1u : 0u);
+                        for (int s = 0; s < BK / 16; s++) // 16 keys per instruction: eight packed columns of P at the start of each half's columns of S
+                            tc_mma_ts(tmem + COL_O, tmem + COL_S + HK * (s / (HK / 16)) + 8 * (s % (HK / 16)), tc_desc_mn(v_addr, BOX, s), id_o,
+                                      (i > 0 || s > 0) ? 1u : 0u);
+                    }
+                    tc_commit(bar_pv);
                 }
-                tc_commit(bar_pv);
-                wait(bar_pv, ph, 5); // P (over S) and V have been read, O is complete up to this tile
-                if (!s_abort && i + 1 < n_tiles) load_v(i + 1);
+                __syncwarp();
+                go = wait(bar_pv, ph, 5) && go; // P (over S) and V have been read, O is complete up to this tile
+                if (lead && go && i + 1 < n_tiles) load_v(i + 1);
+                __syncwarp();
             }
+            if (!go) s_abort = 1;
         }
         __syncwarp();
     } else {
@@ -187,7 +201,7 @@ __global__ void __launch_bounds__(NTHREADS, 2) latent_prefill_tc_kernel(const __
         const int c0 = HK * half;
         float m = -INFINITY, l = 0.f;
         for (int i = 0; i < n_tiles; i++) {
-            tc_wait(bar_s, (uint32_t)(i & 1), &s_abort, &g_latent_tc_error, 6, LIMIT);
+            tc_wait(bar_s, (uint32_t)(i & 1), &s_abort_word, &g_latent_tc_error, 6, LIMIT);
             asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
             const int t0 = first + i * BK, k0 = t0 + c0;
             // some row of the tile sees only part of these keys: past the diagonal, or behind the last row's window
@@ -257,7 +271,7 @@ __global__ void __launch_bounds__(NTHREADS, 2) latent_prefill_tc_kernel(const __
         if (half == 0) lsum[row] = l + lsum[row];
         softmax_barrier();
         l = lsum[row];
-        tc_wait(bar_pv, (uint32_t)((n_tiles - 1) & 1), &s_abort, &g_latent_tc_error, 7, LIMIT);
+        tc_wait(bar_pv, (uint32_t)((n_tiles - 1) & 1), &s_abort_word, &g_latent_tc_error, 7, LIMIT);
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         const bool go = __all_sync(0xffffffffu, !s_abort);
         if (go) {
