@@ -317,9 +317,11 @@ __global__ void __launch_bounds__(NT) latent_attn_mma_kernel(const __grid_consta
     const uint16_t *cache = (const uint16_t *)l.cache + seq * l.seq_stride;
     const int ks = (l.ld + 15) / 16, ld16 = ks * 16, n16 = ks * 2; // K steps of the scores, row length padded to them, 16-byte chunks
     auto load_tile = [&](int kb) {
+        const int slot0 = kb % l.cap;
+#pragma unroll 2
         for (int r = warp; r < MK; r += NW) { // a warp per row
-            const int key = kb + r;
-            const uint8_t *src = (const uint8_t *)(cache + (int64_t)(key % l.cap) * l.ld);
+            const int key = kb + r, slot = slot0 + r < l.cap ? slot0 + r : slot0 + r - l.cap; // visible rows never wrap twice
+            const uint8_t *src = (const uint8_t *)(cache + (int64_t)slot * l.ld);
             uint8_t *dst = tile + (size_t)r * pitch;
             for (int c = lane; c < n16; c += 32) {
                 if (key < k1 && 8 * c < l.ld)
@@ -332,17 +334,18 @@ __global__ void __launch_bounds__(NT) latent_attn_mma_kernel(const __grid_consta
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     load_tile(k0);
-    for (int d0 = 2 * lane; d0 < ld16; d0 += 64 * 5) { // queries of the warp's two heads, scaled, as hi + lo; ten loads in flight
-        float2 v[5][NH];
+    constexpr int QB = 9; // loads per head in flight
+    for (int d0 = 2 * lane; d0 < ld16; d0 += 64 * QB) { // queries of the warp's two heads, scaled, as hi + lo
+        float2 v[QB][NH];
 #pragma unroll
-        for (int e = 0; e < 5; e++)
+        for (int e = 0; e < QB; e++)
 #pragma unroll
             for (int a = 0; a < NH; a++) {
                 const int h = hg * HG + warp * NH + a, d = d0 + 64 * e;
                 v[e][a] = h < l.n_head && d < l.ld ? *reinterpret_cast<const float2 *>(q_lat + (row * l.n_head + h) * l.ld + d) : make_float2(0.f, 0.f);
             }
 #pragma unroll
-        for (int e = 0; e < 5; e++)
+        for (int e = 0; e < QB; e++)
 #pragma unroll
             for (int a = 0; a < NH; a++) {
                 const int d = d0 + 64 * e;
@@ -368,21 +371,30 @@ __global__ void __launch_bounds__(NT) latent_attn_mma_kernel(const __grid_consta
         asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
         { // S: 16 heads x 8 keys
-            float sa[4] = {}, sb[4] = {};
+            float sa[2][4] = {}, sb[2][4] = {};
             const uint32_t aoff = (uint32_t)((lane & 15) * pitch + (lane >> 4) * 16);
             const uint32_t boff = t_addr + (uint32_t)((8 * warp + (lane & 7)) * pitch + ((lane >> 3) & 1) * 16);
-#pragma unroll 4
-            for (int k = 0; k < ks; k++) {
-                uint32_t a[4], b[2];
-                ldsm2(boff + 32 * k, b);
-                ldsm4(qh + aoff + 32 * k, a);
-                mma16816(sa, a, b[0], b[1]);
-                ldsm4(ql + aoff + 32 * k, a);
-                mma16816(sb, a, b[0], b[1]);
+            for (int k0 = 0; k0 < ks; k0 += 4) { // the fragments of four steps, then their products in four chains
+                uint32_t ah[4][4], al[4][4], b[4][2];
+#pragma unroll
+                for (int e = 0; e < 4; e++) {
+                    const int k = min(k0 + e, ks - 1);
+                    ldsm2(boff + 32 * k, b[e]);
+                    ldsm4(qh + aoff + 32 * k, ah[e]);
+                    ldsm4(ql + aoff + 32 * k, al[e]);
+                }
+#pragma unroll
+                for (int e = 0; e < 4; e++)
+                    if (k0 + e < ks) {
+                        mma16816(sa[e & 1], ah[e], b[e][0], b[e][1]);
+                        mma16816(sb[e & 1], al[e], b[e][0], b[e][1]);
+                    }
             }
+#pragma unroll
+            for (int e = 0; e < 4; e++) sa[0][e] += sa[1][e] + (sb[0][e] + sb[1][e]);
             const int r = lane >> 2, c = 8 * warp + (lane & 3) * 2;
-            ss[r][c] = sa[0] + sb[0], ss[r][c + 1] = sa[1] + sb[1];
-            ss[r + 8][c] = sa[2] + sb[2], ss[r + 8][c + 1] = sa[3] + sb[3];
+            ss[r][c] = sa[0][0], ss[r][c + 1] = sa[0][1];
+            ss[r + 8][c] = sa[0][2], ss[r + 8][c + 1] = sa[0][3];
         }
         __syncthreads();
 #pragma unroll
@@ -414,14 +426,16 @@ __global__ void __launch_bounds__(NT) latent_attn_mma_kernel(const __grid_consta
             if (d0 >= l.kv_rank) break;
 #pragma unroll
             for (int b = 0; b < 2; b++) o[t][b][0] *= a0, o[t][b][1] *= a0, o[t][b][2] *= a1, o[t][b][3] *= a1;
+            uint32_t v[4][4];
 #pragma unroll
-            for (int k = 0; k < 4; k++) { // 16 keys per step; lanes 0-15: keys, lanes 16-31: the next eight dimensions
-                uint32_t v[4];
-                ldsm4t(t_addr + (uint32_t)((16 * k + (lane & 15)) * pitch + 2 * d0 + (lane >> 4) * 16), v);
-                mma16816(o[t][0], fh[k], v[0], v[1]);
-                mma16816(o[t][0], fl[k], v[0], v[1]);
-                mma16816(o[t][1], fh[k], v[2], v[3]);
-                mma16816(o[t][1], fl[k], v[2], v[3]);
+            for (int k = 0; k < 4; k++) // 16 keys per step; lanes 0-15: keys, lanes 16-31: the next eight dimensions
+                ldsm4t(t_addr + (uint32_t)((16 * k + (lane & 15)) * pitch + 2 * d0 + (lane >> 4) * 16), v[k]);
+#pragma unroll
+            for (int k = 0; k < 4; k++) {
+                mma16816(o[t][0], fh[k], v[k][0], v[k][1]);
+                mma16816(o[t][1], fh[k], v[k][2], v[k][3]);
+                mma16816(o[t][0], fl[k], v[k][0], v[k][1]);
+                mma16816(o[t][1], fl[k], v[k][2], v[k][3]);
             }
         }
         if (kb + MK < k1) {
@@ -488,11 +502,16 @@ __global__ void __launch_bounds__(NT) latent_output_kernel(const __grid_constant
     __syncthreads();
     for (int d = 2 * tid; d < 8 * nck; d += 2 * NT) {
         float2 acc = make_float2(0.f, 0.f);
-#pragma unroll 16
-        for (int s = 0; s < n_split; s++) {
-            const float2 v = *reinterpret_cast<const float2 *>(src + s * ps + d);
-            acc.x = fmaf(s_w[s], v.x, acc.x);
-            acc.y = fmaf(s_w[s], v.y, acc.y);
+        for (int s0 = 0; s0 < n_split; s0 += 16) { // sixteen ranges in flight
+            float2 v[16];
+#pragma unroll
+            for (int e = 0; e < 16; e++)
+                v[e] = s0 + e < n_split ? *reinterpret_cast<const float2 *>(src + (s0 + e) * ps + d) : make_float2(0.f, 0.f);
+#pragma unroll
+            for (int e = 0; e < 16; e++) { // weights past n_split are zero
+                acc.x = fmaf(s_w[s0 + e], v[e].x, acc.x);
+                acc.y = fmaf(s_w[s0 + e], v[e].y, acc.y);
+            }
         }
         so[d] = d < l.kv_rank ? acc.x : 0.f;
         so[d + 1] = d + 1 < l.kv_rank ? acc.y : 0.f;
