@@ -43,7 +43,7 @@ def rotate_interleaved(x, pos, base, dims=None):
 
 
 def causal_conv(x, taps, bias):
-    """per-channel convolution over time, last tap on the current token, zeros before the start"""
+    """per-channel convolution over time; taps[:, -1] weighs the newest input, inputs at negative times count as zero"""
     T, n = x.shape[0], taps.shape[1]
     xp = np.concatenate([np.zeros((n - 1, x.shape[1]), x.dtype), x])
     return sum(xp[k:k + T] * taps[:, k] for k in range(n)) + bias

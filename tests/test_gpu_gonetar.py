@@ -1,7 +1,7 @@
 """Gonetar on the GPU (gated linear recurrence, windowed latent attention, sandwich norms, looped layers) against the
 plain numpy restatement in hybrid_oracle.py, on small random models, in bf16 and in 32-bit."""
-import os
 import json
+import os
 import subprocess
 import sys
 
