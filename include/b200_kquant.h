@@ -329,18 +329,26 @@ B200_API b200_status b200_stage_create(const b200_stage_config *cfg, b200_stage 
  * For decoders that are not a repetition of one attention + SwiGLU block (an addition of this library, no
  * counterpart in the reference): every layer names its mixer and its feed-forward and brings its own sizes;
  * a contiguous range of layers may run several times in a row with the same weights, each pass with its own
- * cache and state.  Norms stand before and after every sub-layer: x += norm_b(f(norm(x))), RMS norms of weight
- * norm_offset + w.  The stage is loaded, run, split by layer range (a looped range stays on one stage), captured
+ * cache and state.  Norms stand before and after every sub-layer, x += norm_b(f(norm(x))), or behind it only,
+ * x += norm(f(x)): RMS norms of weight norm_offset + w.  A layer may end with a term made from its token's own embedding
+ * for that layer (side_dim).  The stage is loaded, run, split by layer range (a looped range stays on one stage), captured
  * into graphs and freed through the same calls as any other.  Tensor names: "embed", "final.norm", and per layer i
- * "l<i>.norm1", ".norm1b", ".norm2", ".norm2b", "l<i>.mix.*", "l<i>.mlp.*"; matrices are bf16 [out][in], vectors
- * f32 (set_tensor also takes them as bf16).
+ * "l<i>.norm1", ".norm1b", ".norm2", ".norm2b" (behind only: ".norm1", ".norm2"), "l<i>.mix.*", "l<i>.mlp.*", "l<i>.side.*";
+ * matrices are bf16 [out][in], vectors f32 (set_tensor also takes them as bf16).
  * Positions: a sequence slot starts at pos0 = 0, which forgets whatever it held, and continues exactly where its last
  * call stopped; any other pos0 is refused with B200_ERR_STATE (the recurrent state cannot be rewound).        */
 enum {
     B200_MIXER_LATENT_ATTN = 1, /* low-rank shared keys / values, one rotated key part, sliding window, output gate */
-    B200_MIXER_LINEAR_REC = 2   /* gated diagonal linear recurrence behind a short convolution, gated by a GELU branch */
+    B200_MIXER_LINEAR_REC = 2,  /* gated diagonal linear recurrence behind a short convolution, gated by a GELU branch */
+    B200_MIXER_GQA = 3,         /* grouped-query attention with per-head query / key norms, window or chunks, keys and values
+                                 * of its own or another layer's */
+    B200_MIXER_DECAY_STATE = 4, /* linear attention: a matrix state per head under a fixed decay per head, output norm over
+                                 * all heads and gate */
+    B200_MIXER_DELTA_STATE = 5  /* gated delta rule: a matrix state per head, a decay per key channel, short convolutions
+                                 * and unit norms in front, output norm per head and gate */
 };
-enum { B200_FFN_NONE = 0, B200_FFN_CLAMPED_GLU = 1 };
+enum { B200_FFN_NONE = 0, B200_FFN_CLAMPED_GLU = 1, B200_FFN_MOE = 2 };
+enum { B200_NORM_SANDWICH = 0, B200_NORM_OUTPUT = 1 };
 enum { B200_PRECISION_BF16 = 0, B200_PRECISION_F32 = 1 };
 typedef struct b200_layer_config {
     int32_t mixer, ffn;
@@ -355,12 +363,27 @@ typedef struct b200_layer_config {
     /* B200_FFN_CLAMPED_GLU: g sigmoid(alpha g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit)   */
     int32_t n_ff;
     float glu_limit, glu_alpha;
+    /* B200_MIXER_GQA: n_head query heads on n_head_kv key / value heads, qk_dim and v_dim per head, attn_scale; a query sees
+     * the last `window` positions (window > 0), or those of its own run of `chunk` positions counted from 0 (chunk > 0), or
+     * all.  kv_shared: the layer has no keys and values of its own, it reads layer kv_layer's (an earlier GQA layer with its
+     * own, of equal n_head_kv, qk_dim and v_dim; both on one stage).
+     * B200_MIXER_DECAY_STATE: n_head heads of qk_dim x v_dim; tensor "mix.decay" holds the decays (f32).
+     * B200_MIXER_DELTA_STATE: n_head heads on n_head_kv query / key heads of qk_dim x v_dim, conv_taps; decay_rank and
+     * gate_rank are the inner sizes of the two low-rank projections.                             */
+    int32_t n_head_kv, chunk, kv_shared, kv_layer, decay_rank, gate_rank;
+    /* B200_FFN_MOE: n_expert_used of n_expert SiLU GLUs of n_ff_exp, weighted by a softmax over the chosen logits, plus a
+     * shared one of n_ff_shared (0: none)                                                        */
+    int32_t n_expert, n_expert_used, n_ff_exp, n_ff_shared;
 } b200_layer_config;
 typedef struct b200_stack_config {
     int32_t loop_start, loop_stop, loop_times; /* layers [start, stop) run `times` times; times <= 1: no loop   */
     int32_t precision;  /* BF16: matrix products on tensor cores with bf16 operands; F32: f32 throughout       */
     float embd_scale;   /* factor on the embedding rows (not on the output head, which is the same matrix)     */
     float norm_offset;  /* RMS norms multiply by norm_offset + w                                               */
+    int32_t norm_place; /* B200_NORM_SANDWICH or B200_NORM_OUTPUT                                              */
+    int32_t side_dim;   /* > 0: every layer ends with x += norm(proj(gelu(gate x) * e)), e the layer's side_dim values of the
+                         * token's row of "side.embed"; every stage then needs the token ids           */
+    float logit_softcap; /* > 0: logits = cap tanh(logits / cap)                                               */
 } b200_stack_config;
 /* cfg: n_layer, layer_begin, layer_end, n_embd, n_vocab, n_ctx, n_seq, n_ubatch, has_embd, has_output, rms_eps and
  * device are used; layers: n_layer descriptions (of the whole model).                                */

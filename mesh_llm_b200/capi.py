@@ -64,6 +64,9 @@ class LayerConfig(C.Structure):
         ("rope_base", C.c_float), ("attn_scale", C.c_float),
         ("rec_width", C.c_int32), ("rec_blocks", C.c_int32), ("conv_taps", C.c_int32), ("rec_decay", C.c_float),
         ("n_ff", C.c_int32), ("glu_limit", C.c_float), ("glu_alpha", C.c_float),
+        ("n_head_kv", C.c_int32), ("chunk", C.c_int32), ("kv_shared", C.c_int32), ("kv_layer", C.c_int32),
+        ("decay_rank", C.c_int32), ("gate_rank", C.c_int32),
+        ("n_expert", C.c_int32), ("n_expert_used", C.c_int32), ("n_ff_exp", C.c_int32), ("n_ff_shared", C.c_int32),
     ]
 
 
@@ -71,6 +74,7 @@ class StackConfig(C.Structure):
     _fields_ = [
         ("loop_start", C.c_int32), ("loop_stop", C.c_int32), ("loop_times", C.c_int32),
         ("precision", C.c_int32), ("embd_scale", C.c_float), ("norm_offset", C.c_float),
+        ("norm_place", C.c_int32), ("side_dim", C.c_int32), ("logit_softcap", C.c_float),
     ]
 
 

@@ -130,12 +130,6 @@ b200_status check_tensor(const b200_tensor *t) {
     return B200_OK;
 }
 
-#define KQ_TRY(expr)                      \
-    do {                                  \
-        b200_status rc__ = (expr);        \
-        if (rc__ != B200_OK) return rc__; \
-    } while (0)
-
 struct DevGuard {
     int prev = -1;
     explicit DevGuard(int dev) {

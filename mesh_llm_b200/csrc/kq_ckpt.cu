@@ -215,6 +215,7 @@ struct b200_ckpt {
     float eps = 0.f;
     b200_stack_config stack = {};
     std::vector<b200_layer_config> layers;
+    std::map<std::string, std::vector<float>> constants; // vectors that the config holds and a stage takes as tensors
     ~b200_ckpt() {
         if (fd >= 0) close(fd);
     }
@@ -290,12 +291,100 @@ b200_status read_gonetar(b200_ckpt &ck) {
     return r.rc;
 }
 
+// Lomodra: linear attention with fixed decays, chunked attention and gated delta rules in any order, norms behind the
+// sub-layers, experts with a shared one, a per-layer token input, tied output head with a soft cap.
+b200_status read_lomodra(b200_ckpt &ck) {
+    Cfg r;
+    const Json *c = &ck.cfg;
+    ck.n_embd = r.integer(c, "", "width", 1, BIG);
+    ck.n_vocab = r.integer(c, "", "vocab", 1, BIG);
+    ck.eps = r.number(r.need(c, "", "norm"), "norm", "eps");
+    ck.stack.embd_scale = 1.0f;
+    ck.stack.norm_place = B200_NORM_OUTPUT;
+    auto given = [](const Json *o, const char *key) { // absent and null are the same
+        const Json *v = o ? o->get(key) : nullptr;
+        return v && v->kind != Json::NUL ? v : nullptr;
+    };
+    if (const Json *side = given(c, "token_side")) ck.stack.side_dim = r.integer(side, "token_side", "dim", 1, BIG);
+    if (given(c, "logit_softcap")) {
+        ck.stack.logit_softcap = r.number(c, "", "logit_softcap");
+        if (!(ck.stack.logit_softcap > 0.f)) r.bad("", "logit_softcap", "is not positive");
+    }
+    const Json *layers = r.need(c, "", "layers");
+    if (layers && layers->kind != Json::ARR) r.bad("", "layers", "is not a list");
+    if (r.rc != B200_OK) return r.rc;
+    for (size_t i = 0; i < layers->arr.size(); i++) {
+        const Json *l = &layers->arr[i];
+        const std::string at = "layers[" + std::to_string(i) + "]", in = at + ".mixer", mix = "l" + std::to_string(i) + ".mix.";
+        const Json *type = r.need(l, at, "type"), *m = r.need(l, at, "mixer");
+        if (r.rc != B200_OK) return r.rc;
+        b200_layer_config d = {};
+        d.n_head = r.integer(m, in, "heads", 1, 65536);
+        d.qk_dim = r.integer(m, in, "dim", 1, 65536);
+        d.v_dim = r.integer(m, in, "vdim", 1, 65536);
+        if (type->str == "attention") {
+            d.mixer = B200_MIXER_GQA;
+            d.n_head_kv = r.integer(m, in, "kv_heads", 1, 65536);
+            d.attn_scale = r.number(m, in, "scale");
+            d.chunk = r.integer(r.need(m, in, "mask"), in + ".mask", "size", 1, BIG);
+            if (given(m, "kv_from")) {
+                d.kv_shared = 1;
+                d.kv_layer = r.integer(m, in, "kv_from", 0, (int64_t)i - 1);
+            }
+        } else if (type->str == "lightning") {
+            d.mixer = B200_MIXER_DECAY_STATE;
+            const Json *decay = r.need(m, in, "decay");
+            if (decay && (decay->kind != Json::ARR || (int64_t)decay->arr.size() != d.n_head)) r.bad(in, "decay", "is not a list of one number per head");
+            if (r.rc != B200_OK) return r.rc;
+            std::vector<float> &v = ck.constants[mix + "decay"];
+            for (const Json &x : decay->arr) {
+                if (x.kind != Json::NUM) r.bad(in, "decay", "is not a list of one number per head");
+                v.push_back((float)x.num);
+            }
+        } else if (type->str == "channel_delta") {
+            d.mixer = B200_MIXER_DELTA_STATE;
+            d.n_head_kv = r.integer(m, in, "kv_heads", 1, 65536);
+            d.conv_taps = r.integer(m, in, "conv", 1, 4096);
+            auto rank = [&](const char *leaf) { // the inner size of a low-rank projection: the rows of its first matrix
+                const auto it = ck.index.find(mix + leaf);
+                if (it != ck.index.end()) return (int32_t)ck.tensors[(size_t)it->second].ne[1];
+                kq_set_error("model.safetensors: no tensor %s%s", mix.c_str(), leaf);
+                r.rc = B200_ERR_INVALID;
+                return 0;
+            };
+            d.decay_rank = rank("a1");
+            d.gate_rank = rank("g1");
+        } else {
+            kq_set_error("config.json: %s.type \"%s\" is not a mixer of this architecture", at.c_str(), type->str.c_str());
+            return B200_ERR_UNSUPPORTED;
+        }
+        if (const Json *mlp = given(l, "mlp")) {
+            const std::string im = at + ".mlp";
+            const Json *kind = r.need(mlp, im, "kind");
+            if (kind && kind->str != "moe") {
+                kq_set_error("config.json: %s.kind \"%s\" is not a feed-forward of this architecture", im.c_str(), kind->str.c_str());
+                return B200_ERR_UNSUPPORTED;
+            }
+            d.ffn = B200_FFN_MOE;
+            const Json *router = r.need(mlp, im, "router");
+            d.n_expert = r.integer(router, im + ".router", "experts", 1, 65536);
+            d.n_expert_used = r.integer(router, im + ".router", "top", 1, d.n_expert);
+            d.n_ff_exp = r.integer(r.need(mlp, im, "expert"), im + ".expert", "ff", 1, BIG);
+            if (const Json *sh = given(mlp, "shared")) d.n_ff_shared = r.integer(sh, im + ".shared", "ff", 1, BIG);
+        }
+        if (r.rc != B200_OK) return r.rc;
+        ck.layers.push_back(d);
+    }
+    return r.rc;
+}
+
 struct Architecture {
     const char *name;
     b200_status (*read)(b200_ckpt &);
 };
 const Architecture ARCHITECTURES[] = {
     {"Gonetar", read_gonetar},
+    {"Lomodra", read_lomodra},
 };
 
 b200_status index_safetensors(b200_ckpt &ck, const std::string &path) {
@@ -373,8 +462,8 @@ b200_status open_into(b200_ckpt &ck, const std::string &dir) {
     ck.arch = a->str;
     for (const Architecture &ar : ARCHITECTURES)
         if (ck.arch == ar.name) {
-            const b200_status rc = ar.read(ck);
-            return rc == B200_OK ? index_safetensors(ck, dir + "/model.safetensors") : rc;
+            const b200_status rc = index_safetensors(ck, dir + "/model.safetensors"); // some sizes are those of the tensors
+            return rc == B200_OK ? ar.read(ck) : rc;
         }
     kq_set_error("%s: architecture %s is not one of this library", path.c_str(), ck.arch.c_str());
     return B200_ERR_UNSUPPORTED;
@@ -456,6 +545,12 @@ b200_status b200_stage_load_ckpt(b200_stage *st, const b200_ckpt *ck, int64_t *n
         b200_status rc = b200_stage_tensor_info(st, i, name, sizeof(name), &type, ne);
         if (rc != B200_OK) return rc;
         const auto it = ck->index.find(name);
+        const auto given = ck->constants.find(name);
+        if (given != ck->constants.end()) {
+            rc = b200_stage_set_tensor(st, name, B200_TYPE_F32, given->second.data(), given->second.size() * 4);
+            if (rc != B200_OK) return rc;
+            continue;
+        }
         if (it == ck->index.end()) {
             kq_set_error("stage_load_ckpt: the file has no tensor %s", name);
             return B200_ERR_STATE;

@@ -32,6 +32,12 @@ void kq_set_error(const char *fmt, ...);
         }                                \
     } while (0)
 
+#define KQ_TRY(expr)                      \
+    do {                                  \
+        b200_status rc__ = (expr);        \
+        if (rc__ != B200_OK) return rc__; \
+    } while (0)
+
 #define KQ_LAUNCH_CHECK()                                                                   \
     do {                                                                                    \
         cudaError_t e__ = cudaGetLastError();                                               \
@@ -311,7 +317,7 @@ int kq_stream_error_fetch(); // 0 ok; nonzero = a bounded device-side wait gave 
 int kq_gemm_error_fetch();
 int kq_attn_tc_error_fetch();
 int kq_gemm_bf16_error_fetch();
-int kq_latent_tc_error_fetch();
+int kq_prompt_attn_error_fetch();
 int kq_device_wait_errors(); // all of the above in one code
 b200_status kq_launch_gemm(uint32_t type, const uint8_t *W, const int8_t *q, const float *d,
                            const int16_t *bs, int64_t M, int64_t N, int64_t K, float *y,

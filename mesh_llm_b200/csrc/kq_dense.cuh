@@ -1,5 +1,6 @@
 // 16-bit dense weights: launchers of the matrix-vector and matrix-matrix kernels and of the ops of layers that
-// are described one by one (latent attention, gated linear recurrence, clamped GLU, sandwich norms).
+// are described one by one (latent and grouped-query attention, linear recurrences with a diagonal or a matrix state,
+// GLU feed-forwards, experts, norms around the sub-layers).
 //
 // Weight rows are bfloat16, padded with zeros to a multiple of 64 elements (128 bytes), so that a 64-element
 // K slice is one row of a 128-byte-swizzled TMA box and every 16-byte chunk of a row is aligned.  Activations
@@ -9,7 +10,8 @@
 
 #include <cuda_bf16.h>
 
-enum { KQ_ACT_NONE = 0, KQ_ACT_GELU_TANH = 1 };
+enum { KQ_ACT_NONE = 0, KQ_ACT_GELU_TANH = 1, KQ_ACT_SOFT_CAP = 2 }; // SOFT_CAP: cap tanh(y / cap)
+enum { KQ_GLU_NONE = 0, KQ_GLU_CLAMPED = 1, KQ_GLU_SILU = 2 };
 enum { KQ_OUT_F32 = 0, KQ_OUT_BF16 = 1, KQ_OUT_F16 = 2 };
 enum { KQ_PREC_BF16 = 0, KQ_PREC_F32 = 1 };
 
@@ -27,7 +29,7 @@ struct KqDenseSeg {
     const float *bias;
     int32_t act, out; // KQ_ACT_*, KQ_OUT_*
     int32_t head_in, head_out;
-    int32_t pad_cols; // 16-bit outputs: columns n_rows .. pad_cols-1 are written as zeros (row padding of a staging copy)
+    int32_t pad_cols; // 16-bit outputs of one group: columns n_rows .. pad_cols-1 are written as zeros (row padding of a staging copy)
 };
 
 struct KqDense {
@@ -39,17 +41,28 @@ struct KqDense {
     // g * n_rows .. of every segment and writes column range g * n_rows (through col())
     int32_t groups = 1;
     int64_t xg = 0;
-    // glu: segment 0 is the gate, segment 1 the up matrix: y = g sigmoid(alpha g) (u + 1) with g = min(gate, limit),
-    // u = clamp(up, -limit, limit); written through segment 0
+    // glu: segment 0 is the gate, segment 1 the up matrix; written through segment 0.  KQ_GLU_CLAMPED: y = g sigmoid(alpha g)
+    // (u + 1) with g = min(gate, limit), u = clamp(up, -limit, limit); KQ_GLU_SILU: y = g sigmoid(g) u
     int32_t glu = 0;
     float glu_limit = 0.f, glu_alpha = 0.f;
     // head_gate: y *= sigmoid(head_gate[m * ld_gate + group])
     const float *head_gate = nullptr;
     int64_t ld_gate = 0;
+    float cap = 0.f; // KQ_ACT_SOFT_CAP
+    // row_mul: y *= row_mul[mul_row[m] * ld_mul + n] (bf16), after the activation
+    const uint16_t *row_mul = nullptr;
+    const int32_t *mul_row = nullptr;
+    int64_t ld_mul = 0;
+    // experts > 0 (matrix products): every segment holds `experts` matrices of n_rows rows one after the other; the rows of
+    // x come in tiles of KQ_TILE_M, tile i belongs to expert tile_expert[i], *n_tiles of them (device) hold anything
+    int32_t experts = 0;
+    const int32_t *tile_expert = nullptr, *n_tiles = nullptr;
 };
+constexpr int KQ_TILE_M = 128;
 
 // Prologue of a projection: x' = x + norm(sub; sub_w) (sub null: x' = x; sub_w null: plain sum), then
-// h = norm(x'; norm_w) (norm_w null: h = x').  norm(v; w) = v / rms(v) * (w_off + w).
+// h = norm(x'; norm_w) (norm_w null: h = x') times sigmoid(gate) where a gate is given.
+// norm(v; w) = v / rms(v) * (w_off + w).
 struct KqNormPrep {
     const float *x = nullptr;
     int64_t ldx = 0;
@@ -59,6 +72,8 @@ struct KqNormPrep {
     float eps = 0.f, w_off = 0.f;
     float *x_out = nullptr; // where x' goes (null: nowhere); must not be x when several CTAs read it
     int64_t ld_out = 0;
+    const float *gate = nullptr; // [rows][ld_gate]
+    int64_t ld_gate = 0;
 };
 
 #ifdef __CUDACC__
@@ -70,6 +85,11 @@ __device__ __forceinline__ float kq_clamped_glu(float g, float u, float limit, f
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
     return g * kq_sigmoid(alpha * g) * (u + 1.0f);
+}
+__device__ __forceinline__ float kq_silu(float z) { return z * kq_sigmoid(z); }
+__device__ __forceinline__ float kq_softplus(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+__device__ __forceinline__ float kq_glu(const KqDense &c, float g, float u) {
+    return c.glu == KQ_GLU_SILU ? kq_silu(g) * u : kq_clamped_glu(g, u, c.glu_limit, c.glu_alpha);
 }
 __device__ __forceinline__ uint16_t kq_f2bf(float v) { return __bfloat16_as_ushort(__float2bfloat16_rn(v)); }
 __device__ __forceinline__ float kq_bf2f(uint16_t v) { return __uint_as_float((uint32_t)v << 16); }
@@ -98,7 +118,9 @@ __device__ __forceinline__ void kq_dense_put(const KqDenseSeg &s, int64_t m, int
 __device__ __forceinline__ void kq_dense_store(const KqDense &c, const KqDenseSeg &s, int64_t m, int64_t n, int g, float v) {
     if (s.bias) v += s.bias[n];
     if (s.act == KQ_ACT_GELU_TANH) v = kq_gelu_tanh(v);
+    if (s.act == KQ_ACT_SOFT_CAP) v = c.cap * tanhf(v / c.cap);
     if (c.head_gate) v *= kq_sigmoid(c.head_gate[m * c.ld_gate + g]);
+    if (c.row_mul) v *= kq_bf2f(c.row_mul[(int64_t)c.mul_row[m] * c.ld_mul + n]);
     kq_dense_put(s, m, n, v);
 }
 #endif
@@ -178,6 +200,30 @@ b200_status kq_latent_attention(const KqLatent &l, const float *q_lat, int n_seq
 b200_status kq_latent_output(const KqLatent &l, const float *scratch, int n_seq, int T, const int32_t *pos0_dev, int pos0, int max_keys,
                              const uint16_t *uv, const float *gate, int64_t ldg, float *out, int64_t ldo, cudaStream_t st);
 
+// ---- kq_prompt_attn.cu
+// first position that a query at `pos` sees: the start of its window (window > 0), of its chunk (chunk > 0), or 0
+static inline __host__ __device__ int kq_first_key(int pos, int window, int chunk) {
+    return window > 0 ? (pos >= window ? pos - window + 1 : 0) : chunk > 0 ? pos / chunk * chunk : 0;
+}
+// Tensor-core attention of T new positions of one sequence over f16 keys and values.  B200_ERR_UNSUPPORTED: sizes the
+// kernel is not built for (kq_prompt_attention_fits says so ahead).
+struct KqPromptAttn {
+    const float *q = nullptr; // [T][n_head * (dim + rot)], final
+    int64_t ldq = 0;
+    const uint16_t *k = nullptr, *kr = nullptr, *v = nullptr; // f16 [rows][kv_heads][dims padded to 64]; kr [rows][padded rot]: shared by all heads
+    int64_t rows = 0;
+    int32_t n_head = 0, kv_heads = 0, dim = 0, rot = 0, vdim = 0, T = 0, pos0 = 0;
+    int32_t lo = 0, ring = 0; // position of row 0; ring > 0: position p lies in row p % ring (a multiple of 128)
+    int32_t window = 0, chunk = 0;
+    float scale = 1.f;
+    const float *gate = nullptr; // [T][ldg]: head h's output times sigmoid(gate[t][h])
+    int64_t ldg = 0;
+    uint16_t *out = nullptr; // bf16 [T][ldo]
+    int64_t ldo = 0;
+};
+bool kq_prompt_attention_fits(int dim, int rot, int vdim);
+b200_status kq_prompt_attention(const KqPromptAttn &a, cudaStream_t st);
+
 // ---- kq_latent_prefill.cu: the expanded form for prompts of one sequence, bf16 cache
 struct KqLatentPrefill {
     const uint16_t *uk, *uv; // bf16 [n_head * dim][kq_bf16_ld(kv_rank)]
@@ -189,3 +235,106 @@ size_t kq_latent_prefill_bytes(const KqLatent &l, int max_rows, int max_keys);
 // rows are in the cache already.  B200_ERR_UNSUPPORTED: shapes the kernel is not built for.
 b200_status kq_latent_prefill(const KqLatent &l, const KqLatentPrefill &w, const float *q, int64_t ldq, const float *gate, int64_t ldg,
                               int T, int pos0, uint16_t *out, int64_t ldo, cudaStream_t st);
+
+// ---- kq_gqa_attn.cu: grouped-query attention over a ring of keys and values
+// Cache of one layer run: rows of [kv_heads][dims padded to 64], position p in row p % cap (cap a multiple of 128), keys
+// after their norm; f16 (saturating) or f32.
+struct KqGqa {
+    int32_t n_head, kv_heads, dim, vdim, window, chunk;
+    float scale, eps;
+    const float *q_norm, *k_norm; // [dim], plain weights
+    int32_t cap, f32;
+    void *k, *v;                  // first sequence of the call
+    bool own_kv;                  // false: the rows are another layer's, nothing is stored
+};
+static inline int64_t kq_gqa_ld(int dim) { return kq_pad(dim, 64); }
+constexpr int KQ_GQA_MAX_DIM = 512;
+// New keys and values into the cache (own_kv), q normed in place.  q, k, v: the columns of projection rows of ldp floats.
+b200_status kq_gqa_store(const KqGqa &a, float *q, const float *k, const float *v, int64_t ldp, int n_seq, int T, const int32_t *pos0_dev, int pos0,
+                         cudaStream_t st);
+// Attention of every row, split over key ranges that the last CTA of a row merges.  fused: T = 1, norms and the store
+// happen in here (q, k, v as above; otherwise q is normed and k, v are not read).  Output f32 or bf16 (either may be null).
+// scratch: kq_gqa_scratch_bytes; counters: kq_gqa_counters words, zero between launches.  max_keys: the most keys a row can see.
+int64_t kq_gqa_counters(const KqGqa &a);
+size_t kq_gqa_scratch_bytes(const KqGqa &a, int max_rows, int max_keys);
+b200_status kq_gqa_attention(const KqGqa &a, bool fused, const float *q, const float *k, const float *v, int64_t ldp, int n_seq, int T,
+                             const int32_t *pos0_dev, int pos0, int max_keys, float *out, int64_t ldo, uint16_t *out16, int64_t ldo16,
+                             float *scratch, size_t scratch_bytes, unsigned *counters, cudaStream_t st);
+
+// ---- kq_state_ops.cu: recurrences whose state is a matrix per head
+// S <- decay S + k v^T, o = S^T q, or under the delta rule S <- g S (a decay per key channel), u = beta (v - S^T k),
+// S <- S + k u^T, o = S^T q.  Query / key head floor(h / (heads / kv_heads)) serves head h.
+// State of one layer run: S transposed [seq][heads][vdim][kq_state_ld(dim)] f32, and with taps > 0 a ring of the short
+// convolution's last inputs [seq][taps][channels] (the input of position p in slot p % taps; channels: all of q, then k, then
+// v).  Position 0 starts from zero whatever they hold.
+struct KqMatState {
+    int32_t heads, kv_heads, dim, vdim, taps; // taps 0: no convolution
+    int32_t delta;                            // delta rule; else a fixed decay per head
+    const float *decay;                       // [heads]
+    const float *conv_q, *conv_k, *conv_v;    // [channels][taps]
+    const float *a_log, *dt_bias;             // delta: g = exp(-exp(a_log[h]) softplus(z + dt_bias)), z the low-rank projection
+    float *s, *conv;                          // first sequence of the call
+};
+constexpr int KQ_STATE_MAX_DIM = 256;
+static inline int kq_state_ld(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 96 ? 96 : dim <= 128 ? 128 : dim <= 192 ? 192 : 256; }
+static inline __host__ __device__ int64_t kq_state_channels(const KqMatState &m) { return 2 * (int64_t)m.kv_heads * m.dim + (int64_t)m.heads * m.vdim; }
+// Columns of the fused projection's rows
+struct KqStateIn {
+    const float *q, *k, *v, *b, *z; // z: decay projection [rows][ldz], bias not added yet; b: write strengths before the sigmoid
+    int64_t ld, ldz;
+};
+// What the token loop reads: q, k after convolution, SiLU, unit norm (delta) and scaling, v after convolution and SiLU,
+// decays g, and per head (beta, q.k).  Buffers of the caller.
+struct KqStateTok {
+    float *q, *k, *v, *g, *b; // [rows][kq_f32_ld(kv_heads dim)], same, [rows][kq_f32_ld(heads vdim)], [rows][kq_f32_ld(heads dim)], [rows][2 heads]
+};
+b200_status kq_state_tokens(const KqMatState &m, const KqStateIn &in, const KqStateTok &t, int n_seq, int T, const int32_t *pos0_dev, int pos0,
+                            cudaStream_t st);
+// the token loop over T positions: o [rows][ldo] f32; also moves the convolution's ring forward (in: its inputs)
+b200_status kq_state_scan(const KqMatState &m, const KqStateIn &in, const KqStateTok &t, int n_seq, int T, const int32_t *pos0_dev, int pos0,
+                          float *o, int64_t ldo, cudaStream_t st);
+// every head's o over its rms times norm_w [vdim] times sigmoid(gate); f32 or bf16 rows (padded with zeros)
+b200_status kq_head_norm_gate(const float *o, int64_t ldo, const float *gate, int64_t ldg, const float *norm_w, float eps, int64_t rows, int heads,
+                              int vdim, float *out32, int64_t ld32, uint16_t *out16, int64_t ld16, cudaStream_t st);
+// One token per sequence, everything between the projections in one launch.  With delta: z and the gate come out of the low-rank
+// products of a1, g1 (columns of the projection's rows) and w_a2, w_g2, and norm_w / eps give the finished rows.
+struct KqStateStep {
+    const float *a1 = nullptr, *g1 = nullptr;
+    const uint16_t *a2 = nullptr, *g2 = nullptr; // bf16 [heads dim or heads vdim][kq_bf16_ld(rank)]
+    int32_t a_rank = 0, g_rank = 0;
+    const float *norm_w = nullptr;
+    float eps = 0.f;
+};
+b200_status kq_state_step(const KqMatState &m, const KqStateIn &in, const KqStateStep &x, int n_seq, const int32_t *pos_dev, int pos, float *z,
+                          int64_t ldz, cudaStream_t st);
+// f32 columns into bf16 GEMM operands: a [rows][n] as three parts that add up, g [rows][m] rounded
+b200_status kq_rank_operands(const float *a, int n, uint16_t *a16, const float *g, int m, uint16_t *g16, int64_t ld, int64_t rows, cudaStream_t st);
+
+// ---- kq_moe_bf16.cu: SiLU-GLU experts with bf16 weights
+// Router logits z [rows][ldz] f32 (bias included); the `top` largest are chosen (ties: the lower expert), weighted by a softmax
+// over them.  A shared expert's gate and up products (before the GLU) may lie in the same rows.
+struct KqMoe {
+    int32_t experts, top, h, ff, ff_shared; // ff_shared 0: none
+    const float *z, *sh_gate, *sh_up;       // columns of rows of ldz floats
+    int64_t ldz;
+};
+constexpr int KQ_MOE_MAX_EXPERTS = 2048, KQ_MOE_MAX_TOP = 64;
+// Up to a few rows, two launches: act[row * top + s] = GLU of the s-th chosen expert (its choice goes to ids / wts), then
+// out = sum_s wts W_down act + shared.  Weights bf16 [experts][rows][kq_bf16_ld(K)].
+b200_status kq_moe_few_gate_up(const KqMoe &m, const float *x, int64_t ldx, int rows, const uint16_t *gate, const uint16_t *up, float *act,
+                               int64_t ld_act, int32_t *ids, float *wts, cudaStream_t st);
+b200_status kq_moe_few_down(const KqMoe &m, const float *act, int64_t ld_act, const int32_t *ids, const float *wts, int rows, const uint16_t *down,
+                            const uint16_t *sh_down, float *out, int64_t ldo, cudaStream_t st);
+// Many rows: choice, shared GLU (f32 or bf16 rows), order by expert in tiles of KQ_TILE_M rows, gather; after the products with
+// experts the weighted sum is added to `out` (which holds the shared expert's output, or is written when first is set).
+struct KqMoeOrder {
+    int32_t *ids, *pos;           // [rows * top]: chosen expert, place in the tiles
+    float *wts;                   // [rows * top]
+    int32_t *tile_expert, *n_tiles;
+};
+int64_t kq_moe_max_tiles(int64_t pairs, int experts);
+b200_status kq_moe_route(const KqMoe &m, int rows, const KqMoeOrder &o, float *sh32, int64_t ld32, uint16_t *sh16, int64_t ld16, cudaStream_t st);
+b200_status kq_moe_order(const KqMoe &m, int rows, const KqMoeOrder &o, cudaStream_t st);
+// rows of elem_bytes-wide elements (ld of them) to their places
+b200_status kq_moe_gather(const KqMoe &m, int rows, const KqMoeOrder &o, const void *x, void *y, int64_t ld, int elem_bytes, cudaStream_t st);
+b200_status kq_moe_combine(const KqMoe &m, int rows, const KqMoeOrder &o, const float *y, int64_t ldy, float *out, int64_t ldo, bool first, cudaStream_t st);

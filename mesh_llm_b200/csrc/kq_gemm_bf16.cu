@@ -8,7 +8,8 @@
 // through a transpose in shared memory: stores of one row per lane would run at a fifth of the rate.
 // A gate / up pair shares a tile half and half, so that the GLU happens where both values are.
 // An f32 operand can come as several bf16 parts (x = hi + mid + lo exactly): the K loop then passes over the
-// same weights once per part.  Block-diagonal products offset the K coordinate of x and the row of W by group.
+// same weights once per part.  Block-diagonal products offset the K coordinate of x and the row of W by group.  Products
+// with experts take the row of W from the expert of the token tile; how many tiles there are is read on the device.
 // Every wait is bounded; on a time-out the kernel records an error, lets its copies land, frees its TMEM and
 // returns.
 #include "kq_dense.cuh"
@@ -45,13 +46,13 @@ struct GemmParams {
 struct Col4 {
     float bias[4];
     int64_t col, n;
-    int32_t valid;
+    int32_t valid, n_mul; // columns to write; those of them that have a factor in row_mul
     bool vec; // all four next to one another and aligned in every row
-    __device__ __forceinline__ Col4(const KqDense &c, const KqDenseSeg &s, int64_t n_, int n_valid) : n(n_), valid(n_valid) {
+    __device__ __forceinline__ Col4(const KqDense &c, const KqDenseSeg &s, int64_t n_, int n_valid) : n(n_), valid(n_valid), n_mul((int)min((int64_t)n_valid, s.n_rows - n_)) {
         vec = valid == 4 && ((s.ldy | n | s.head_in | s.head_out) & 3) == 0 && ((uintptr_t)s.y & 15) == 0;
         col = kq_dense_col(s, n);
 #pragma unroll
-        for (int e = 0; e < 4; e++) bias[e] = s.bias && e < valid ? s.bias[n + e] : 0.f;
+        for (int e = 0; e < 4; e++) bias[e] = s.bias && e < valid && (c.groups > 1 || n + e < s.n_rows) ? s.bias[n + e] : 0.f;
     }
     __device__ __forceinline__ void store(const KqDense &c, const KqDenseSeg &s, int64_t m, int g, const float4 &v) const {
         float o[4] = {v.x + bias[0], v.y + bias[1], v.z + bias[2], v.w + bias[3]};
@@ -59,10 +60,20 @@ struct Col4 {
 #pragma unroll
             for (int e = 0; e < 4; e++) o[e] = kq_gelu_tanh(o[e]);
         }
+        if (s.act == KQ_ACT_SOFT_CAP) {
+#pragma unroll
+            for (int e = 0; e < 4; e++) o[e] = c.cap * tanhf(o[e] / c.cap);
+        }
         if (c.head_gate) {
             const float f = kq_sigmoid(c.head_gate[m * c.ld_gate + g]);
 #pragma unroll
             for (int e = 0; e < 4; e++) o[e] *= f;
+        }
+        if (c.row_mul) {
+            const uint16_t *f = c.row_mul + (int64_t)c.mul_row[m] * c.ld_mul + n;
+#pragma unroll
+            for (int e = 0; e < 4; e++)
+                if (e < n_mul) o[e] *= kq_bf2f(f[e]);
         }
         if (vec) {
             const int64_t i = m * s.ldy + col;
@@ -117,17 +128,18 @@ __global__ void __launch_bounds__(NTHREADS, 1) gemm_bf16_kernel(const __grid_con
     __syncthreads();
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     const uint32_t tmem = s_tmem;
-    const int n_it = p.nk * p.parts, n_tiles = p.mt * p.nt * p.c.groups;
+    const int mt = p.c.experts ? min(p.mt, *p.c.n_tiles) : p.mt;
+    const int n_it = p.nk * p.parts, n_tiles = mt * p.nt * p.c.groups;
 
     struct Where {
         int m0, g, seg, n0, n_rows;
     };
     auto locate = [&](int tile) {
         Where w;
-        w.m0 = tile % p.mt * TM;
-        const int rest = tile / p.mt;
+        const int i = tile % mt, rest = tile / mt;
+        w.m0 = i * TM;
         int nt = rest % p.nt;
-        w.g = rest / p.nt;
+        w.g = p.c.experts ? p.c.tile_expert[i] : rest / p.nt;
         w.seg = 0;
         if (!p.c.glu) {
             if (nt >= p.tile_end[1]) w.seg = 2, nt -= p.tile_end[1];
@@ -223,7 +235,7 @@ __global__ void __launch_bounds__(NTHREADS, 1) gemm_bf16_kernel(const __grid_con
             const KqDenseSeg s = kq_dense_seg(p.c, w.seg);
             // EC columns at a time: a lane takes its row out of TMEM into shared memory, then eight lanes write a row's columns, four
             // rows per store.  The loops stay loops: unrolled, the four warps would spend their time fetching code.
-            const int lim = p.c.glu ? std::max(n_rows, s.pad_cols) : n_rows; // the padding of a staging row is written too
+            const int lim = p.c.groups == 1 ? std::max(n_rows, s.pad_cols) : n_rows; // the padding of a staging row is written too
             const int n_cols = std::min(p.c.glu ? TN / 2 : TN, lim - n0);
             const int r4 = lane >> 3, c4 = (lane & 7) * 4;
 #pragma unroll 1
@@ -237,9 +249,7 @@ __global__ void __launch_bounds__(NTHREADS, 1) gemm_bf16_kernel(const __grid_con
                     if (p.c.glu) {
 #pragma unroll
                         for (int e = 0; e < 16; e++)
-                            a[e] = n0 + j + h + e < n_rows ? __float_as_uint(kq_clamped_glu(__uint_as_float(a[e]), __uint_as_float(b[e]),
-                                                                                            p.c.glu_limit, p.c.glu_alpha))
-                                                           : 0u;
+                            a[e] = n0 + j + h + e < n_rows ? __float_as_uint(kq_glu(p.c, __uint_as_float(a[e]), __uint_as_float(b[e]))) : 0u;
                     }
 #pragma unroll
                     for (int e = 0; e < 16; e += 4)
@@ -248,7 +258,7 @@ __global__ void __launch_bounds__(NTHREADS, 1) gemm_bf16_kernel(const __grid_con
                 __syncwarp();
                 const int n = n0 + j + c4, n_valid = std::min(4, lim - n);
                 if (n_valid > 0) {
-                    const Col4 col(p.c, s, (int64_t)w.g * n_rows + n, n_valid);
+                    const Col4 col(p.c, s, (p.c.experts ? 0 : (int64_t)w.g * n_rows) + n, n_valid);
 #pragma unroll 2
                     for (int r = r4; m0 + r < m_end; r += 4) {
                         const float4 v = *reinterpret_cast<const float4 *>(stage + r * EP + c4);
@@ -279,8 +289,14 @@ template <bool GLU>
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ F32Params p) {
     KQ_PDL_ENTER();
     __shared__ float sa[FK][FT + 4], sb[GLU ? 2 : 1][FK][FT + 4];
-    const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4, g = blockIdx.z;
-    int seg = 0, nt = blockIdx.y;
+    const int tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+    int seg = 0, nt = blockIdx.y, g = blockIdx.z;
+    if (p.c.experts) {
+        const int t = blockIdx.x * FT / KQ_TILE_M;
+        if (t >= *p.c.n_tiles) return;
+        g = p.c.tile_expert[t];
+    }
+    const int64_t row0 = p.c.experts ? 0 : g; // column groups of the output
     if (!GLU) {
         if (nt >= p.tile_end[1]) seg = 2, nt -= p.tile_end[1];
         else if (nt >= p.tile_end[0]) seg = 1, nt -= p.tile_end[0];
@@ -321,8 +337,8 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const __grid_constant__ F
         for (int j = 0; j < 4; j++) {
             const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
             if (m >= p.c.M || n >= n_rows) continue;
-            if (GLU) kq_dense_put(s, m, n, kq_clamped_glu(acc[0][i][j], acc[GLU ? 1 : 0][i][j], p.c.glu_limit, p.c.glu_alpha));
-            else kq_dense_store(p.c, s, m, (int64_t)g * n_rows + n, g, acc[0][i][j]);
+            if (GLU) kq_dense_put(s, m, n, kq_glu(p.c, acc[0][i][j], acc[GLU ? 1 : 0][i][j]));
+            else kq_dense_store(p.c, s, m, row0 * n_rows + n, g, acc[0][i][j]);
         }
 }
 
@@ -339,6 +355,7 @@ b200_status kq_gemm_bf16(const KqDense &c, const uint16_t *a, int64_t lda, int p
     KQ_REQUIRE(c.M >= 1 && c.nseg >= 1 && c.nseg <= 3 && c.groups >= 1 && c.K >= 1 && parts >= 1, "gemm_bf16: bad call");
     KQ_REQUIRE(c.ldw % 64 == 0 && c.ldw >= c.K && lda % 64 == 0 && (c.groups == 1 || c.xg % 64 == 0),
                "gemm_bf16: rows must be padded to 64 elements");
+    KQ_REQUIRE(!c.experts || (c.groups == 1 && c.tile_expert && c.n_tiles && c.M % TM == 0), "gemm_bf16: products with experts");
     KQ_REQUIRE(!c.glu || (c.nseg == 2 && c.groups == 1 && c.seg[0].n_rows == c.seg[1].n_rows), "gemm_bf16: a GLU has two equal segments");
     GemmParams p;
     p.c = c;
@@ -350,7 +367,7 @@ b200_status kq_gemm_bf16(const KqDense &c, const uint16_t *a, int64_t lda, int p
         int t = 0;
         if (c.glu) t = (int)kq_div_up(std::max(c.seg[0].n_rows, c.seg[0].pad_cols), tn / 2);
         else
-            for (int i = 0; i < c.nseg; i++) t += (int)kq_div_up(c.seg[i].n_rows, tn);
+            for (int i = 0; i < c.nseg; i++) t += (int)kq_div_up(std::max(c.seg[i].n_rows, c.groups == 1 ? c.seg[i].pad_cols : 0), tn);
         return t;
     };
     const int64_t sms = kq_sm_count();
@@ -367,11 +384,11 @@ b200_status kq_gemm_bf16(const KqDense &c, const uint16_t *a, int64_t lda, int p
     int tiles = 0;
     for (int i = 0; i < 3; i++) {
         const KqDenseSeg &s = c.seg[std::min(i, c.nseg - 1)];
-        const uint64_t dims[2] = {(uint64_t)c.ldw, (uint64_t)s.n_rows * c.groups}, str[1] = {(uint64_t)c.ldw * 2};
+        const uint64_t dims[2] = {(uint64_t)c.ldw, (uint64_t)s.n_rows * std::max(c.groups, c.experts)}, str[1] = {(uint64_t)c.ldw * 2};
         const uint32_t box[2] = {BK, (uint32_t)tn / 2};
         const b200_status rc = kq_tmap_encode(&p.b[i], 2, 2, s.W, dims, str, box, 1);
         if (rc != B200_OK) return rc;
-        if (i < c.nseg) tiles += (int)kq_div_up(s.n_rows, tn);
+        if (i < c.nseg) tiles += (int)kq_div_up(std::max(s.n_rows, c.groups == 1 ? s.pad_cols : 0), tn);
         p.tile_end[i] = tiles;
     }
     const unsigned grid = (unsigned)std::min<int64_t>((int64_t)p.mt * p.nt * c.groups, sms);

@@ -101,7 +101,7 @@ __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __g
     // ---- activations
     float4 *pl = reinterpret_cast<float4 *>(sm); // [M][2][nck]
     const bool vec = (p.p.ldx & 3) == 0 && (p.p.ld_sub & 3) == 0 && (p.p.ld_out & 3) == 0 &&
-                     (((uintptr_t)p.p.x | (uintptr_t)p.p.sub | (uintptr_t)p.p.x_out) & 15) == 0;
+                     (p.p.ld_gate & 3) == 0 && (((uintptr_t)p.p.x | (uintptr_t)p.p.sub | (uintptr_t)p.p.x_out | (uintptr_t)p.p.gate) & 15) == 0;
     const int n4 = nck * 2;
 #pragma unroll 1
     for (int m = 0; m < M; m++) {
@@ -155,6 +155,15 @@ __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __g
                 float4 v = px[(i & 1) * nck + (i >> 1)];
                 v.x *= sc * (p.p.w_off + g.x), v.y *= sc * (p.p.w_off + g.y);
                 v.z *= sc * (p.p.w_off + g.z), v.w *= sc * (p.p.w_off + g.w);
+                px[(i & 1) * nck + (i >> 1)] = v;
+            }
+        }
+        if (p.p.gate) {
+            const float *gate = p.p.gate + m * p.p.ld_gate;
+            for (int i = tid; i < n4; i += NT) { // the elements this thread wrote above
+                const float4 g = kq_load4(gate, 4 * i, K, vec);
+                float4 v = px[(i & 1) * nck + (i >> 1)];
+                v.x *= kq_sigmoid(g.x), v.y *= kq_sigmoid(g.y), v.z *= kq_sigmoid(g.z), v.w *= kq_sigmoid(g.w);
                 px[(i & 1) * nck + (i >> 1)] = v;
             }
         }
@@ -217,7 +226,7 @@ __global__ void __launch_bounds__(NT, M <= 2 ? 4 : 2) gemv_bf16_kernel(const __g
             if (p.c.glu) {
 #pragma unroll
                 for (int i = 0; i < NW; i++) s2 += part[buf][i][vl + 1][m];
-                kq_dense_put(p.c.seg[0], m, r, kq_clamped_glu(s, s2, p.c.glu_limit, p.c.glu_alpha));
+                kq_dense_put(p.c.seg[0], m, r, kq_glu(p.c, s, s2));
             } else {
                 kq_dense_store(p.c, kq_dense_seg(p.c, sg), m, r, 0, s);
             }
@@ -275,6 +284,7 @@ b200_status kq_gemv_bf16(const KqDense &c, const KqNormPrep &pr, cudaStream_t st
         p.p.x += m0 * pr.ldx;
         if (pr.sub) p.p.sub += m0 * pr.ld_sub;
         if (pr.x_out) p.p.x_out += m0 * pr.ld_out;
+        if (pr.gate) p.p.gate += m0 * pr.ld_gate;
         p.nck = nck;
         p.V = 0;
         for (int i = 0; i < c.nseg; i++) p.V += c.seg[i].n_rows;

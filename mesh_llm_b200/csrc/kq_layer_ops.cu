@@ -122,6 +122,12 @@ __global__ void __launch_bounds__(NT) norm_prep_kernel(const __grid_constant__ K
 #pragma unroll
             for (int e = 0; e < E; e++) v[e] *= s2 * (p.w_off + g[e]);
         }
+        if (p.gate) {
+            float g[E];
+            ld(p.gate + r * p.ld_gate, i, g);
+#pragma unroll
+            for (int e = 0; e < E; e++) v[e] *= kq_sigmoid(g[e]);
+        }
         if (h32) stf(h32 + r * ld32, i, v);
         if (h16) {
             uint16_t *o = h16 + r * ld16 + i * E;
@@ -220,7 +226,6 @@ __global__ void __launch_bounds__(NT) causal_conv_kernel(const __grid_constant__
 }
 
 // gates and step of one element: log a = -decay sigmoid(r) softplus(lam); (a, sqrt(1 - a^2) sigmoid(i) u)
-__device__ __forceinline__ float softplus(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 __device__ __forceinline__ void rec_coeff(float r, float i, float u, float decay_sp, float &a, float &b) {
     const float la = -decay_sp * kq_sigmoid(r);
     a = expf(la);
@@ -238,7 +243,7 @@ __global__ void __launch_bounds__(RC) recurrence_chunks_kernel(const __grid_cons
     if (c >= w.width) return;
     const int t0 = k * chunk, t1 = min(T, t0 + chunk);
     const int64_t row0 = (int64_t)seq * T;
-    const float dsp = w.decay * softplus(w.lam[c]);
+    const float dsp = w.decay * kq_softplus(w.lam[c]);
     float A = 1.f, B = 0.f;
 #pragma unroll 4
     for (int t = t0; t < t1; t++) {
@@ -357,7 +362,7 @@ __global__ void __launch_bounds__(NT) recurrence_step_kernel(const __grid_consta
         if (lane == 0) {
             const int c = b * m + rr;
             float a, bb;
-            rec_coeff(ar + w.ra_b[c], ai + w.ri_b[c], su[rr], w.decay * softplus(w.lam[c]), a, bb);
+            rec_coeff(ar + w.ra_b[c], ai + w.ri_b[c], su[rr], w.decay * kq_softplus(w.lam[c]), a, bb);
             float *sp = st.s + (int64_t)seq * w.width + c;
             const float s = fmaf(a, pos > 0 ? *sp : 0.f, bb);
             *sp = s;
@@ -382,8 +387,8 @@ b200_status kq_norm_prep(const KqNormPrep &p, int64_t rows, int K, float *h32, i
                          cudaStream_t st) {
     KQ_REQUIRE(p.x && rows >= 1 && K >= 1, "norm_prep: bad call");
     const uintptr_t al = (uintptr_t)p.x | (uintptr_t)p.sub | (uintptr_t)p.sub_w | (uintptr_t)p.norm_w | (uintptr_t)p.x_out | (uintptr_t)h32 |
-                         (uintptr_t)h16;
-    const bool vec = K % 4 == 0 && (al & 15) == 0 && ((p.ldx | p.ld_sub | p.ld_out | ld32 | ld16) & 3) == 0;
+                         (uintptr_t)h16 | (uintptr_t)p.gate;
+    const bool vec = K % 4 == 0 && (al & 15) == 0 && ((p.ldx | p.ld_sub | p.ld_out | ld32 | ld16 | p.ld_gate) & 3) == 0;
     if (vec) kq_launch(norm_prep_kernel<true>, (unsigned)rows, NT, 0, st, p, K, h32, ld32, h16, ld16);
     else kq_launch(norm_prep_kernel<false>, (unsigned)rows, NT, 0, st, p, K, h32, ld32, h16, ld16);
     KQ_COUNT_LAUNCH();

@@ -747,8 +747,10 @@ b200_status b200_stage_generate(b200_stage *st, uint64_t seed) {
     for (auto &t : st->tensors) {
         const uint64_t key = mix64_host(seed ^ name_hash(t.name.c_str()));
         // plain norm weights around one, everything else (zero-centred norm weights included) around zero
-        const bool is_norm = t.name.find("norm.weight") != std::string::npos || t.name.find("dkv.norm") != std::string::npos;
-        KQ_TRY(kq_synth_weights(t.type, t.dev, t.ne[1] * t.ne[2], t.ne[0], key, is_norm ? 1.0f : 0.0f, 0.02f,
+        const bool is_norm = t.name.find("norm.weight") != std::string::npos || t.name.find("dkv.norm") != std::string::npos ||
+                             (st->layers_desc && t.type == B200_TYPE_F32 && kq_layers_plain_norm(st, t.name));
+        const bool is_decay = t.name.find("mix.decay") != std::string::npos;
+        KQ_TRY(kq_synth_weights(t.type, t.dev, t.ne[1] * t.ne[2], t.ne[0], key, is_norm ? 1.0f : is_decay ? 0.95f : 0.0f, is_decay ? 0.005f : 0.02f,
                                 nullptr));
         t.loaded = true;
     }
@@ -776,6 +778,7 @@ b200_status b200_stage_forward(b200_stage *st, const int32_t *tokens, const floa
     KQ_REQUIRE(pos0 >= 0 && pos0 + T <= c.n_ctx, "stage_forward: positions [%d,%d) exceed n_ctx=%d", pos0,
                pos0 + T, c.n_ctx);
     KQ_REQUIRE(c.has_embd ? tokens != nullptr : hidden_in != nullptr, "stage_forward: missing input");
+    KQ_REQUIRE(tokens || !st->layers_desc || !kq_layers_read_tokens(st), "stage_forward: the layers of this stage read the token ids");
     KQ_REQUIRE(c.has_output || hidden_out, "stage_forward: missing hidden_out");
     KqDevGuard dev_guard(c.device);
     KQ_TRY(resolve(st));

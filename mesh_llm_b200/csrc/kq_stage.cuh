@@ -87,12 +87,6 @@ struct b200_stage {
 // kernel classes of a decode step, selectable for timing (b200_stage_profile_decode)
 enum { CLS_GEMV = 1, CLS_ATTN = 2, CLS_OTHER = 4, CLS_ALL = 7 };
 
-#define KQ_TRY(expr)                      \
-    do {                                  \
-        b200_status rc__ = (expr);        \
-        if (rc__ != B200_OK) return rc__; \
-    } while (0)
-
 b200_status kq_stage_alloc(b200_stage *st, void **p, size_t bytes);
 void kq_stage_add_tensor(b200_stage *st, const std::string &name, uint32_t type, int64_t ne0, int64_t ne1, int64_t ne2);
 StTensor *kq_stage_find(b200_stage *st, const std::string &name);
@@ -106,4 +100,6 @@ b200_status kq_layers_forward(b200_stage *st, const int32_t *tokens, const float
 b200_status kq_layers_check_pos(b200_stage *st, int seq0, int n_seq, int T, int pos0);
 void kq_layers_advance(b200_stage *st, int seq0, int n_seq, int pos); // pos < 0: the state is no longer usable
 bool kq_layers_tracing(const b200_stage *st);
+bool kq_layers_read_tokens(const b200_stage *st); // every stage of such a model takes the token ids, next to hidden_in
+bool kq_layers_plain_norm(const b200_stage *st, const std::string &name); // a norm weight around one, not around zero
 b200_status kq_layers_peek(b200_stage *st, const char *which, float *host_out, size_t n_floats);
