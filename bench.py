@@ -301,6 +301,14 @@ ARCH_SIZES = {
     "gonetar-4b": dict(width=3072, rec=3072, blocks=12, ff=9216, heads=24, kv=6, n_layer=32),
     "gonetar-9b": dict(width=4096, rec=4096, blocks=16, ff=12288, heads=32, kv=8, n_layer=38),
 }
+# Lomodra-shaped models (gated delta rule, linear attention under fixed decays, chunked attention whose keys every second
+# attention layer shares, experts) next to a K-quant mixture-of-experts decoder of the same width, depth, experts and vocabulary
+LOMODRA_SIZES = {
+    "lomodra-2048": dict(width=2048, heads=16, kv=4, experts=64, top=6, ff=768, shared=1536, side=256, n_layer=24),
+    "lomodra-3072": dict(width=3072, heads=24, kv=6, experts=64, top=6, ff=1024, shared=2048, side=256, n_layer=24),
+    "lomodra-4096": dict(width=4096, heads=32, kv=8, experts=32, top=4, ff=1536, shared=4096, side=256, n_layer=18),
+}
+LOMODRA_DIM, LOMODRA_RANK, LOMODRA_CHUNK = 128, 128, 2048
 ARCH_VOCAB, ARCH_WINDOW, ARCH_RANK, ARCH_DIM, ARCH_ROT, ARCH_VDIM = 128256, 2048, 512, 128, 64, 128
 
 
@@ -340,8 +348,48 @@ def arch_work(z, n_layer):
     return 2 * proj, 2 * gates, 2 * n_att * lat, 2 * (n_rec * rec + n_att * att + n_layer * ff) + 3 * 2 * gates // 2 + 2 * n_att * lat
 
 
+def lomodra_stage(z, n_layer, n_ctx, ubatch, local, precision=0):
+    """a stage of that size with random weights; pattern: delta rule, fixed decays, attention"""
+    from mesh_llm_b200 import capi
+    from mesh_llm_b200.stage import Stage
+
+    layers = []
+    for i in range(n_layer):
+        l = capi.LayerConfig(ffn=capi.FFN_MOE, n_expert=z["experts"], n_expert_used=z["top"], n_ff_exp=z["ff"], n_ff_shared=z["shared"],
+                             n_head=z["heads"], qk_dim=LOMODRA_DIM, v_dim=LOMODRA_DIM)
+        if i % 3 == 0:
+            l.mixer, l.n_head_kv, l.conv_taps, l.decay_rank, l.gate_rank = capi.MIXER_DELTA_STATE, z["heads"], 4, LOMODRA_RANK, LOMODRA_RANK
+        elif i % 3 == 1:
+            l.mixer = capi.MIXER_DECAY_STATE
+        else:
+            l.mixer, l.n_head_kv, l.chunk, l.attn_scale = capi.MIXER_GQA, z["kv"], LOMODRA_CHUNK, LOMODRA_DIM ** -0.5
+            if i % 6 == 5:
+                l.kv_shared, l.kv_layer = 1, i - 3
+        layers.append(l)
+    stack = capi.StackConfig(loop_times=1, precision=precision, embd_scale=1.0, norm_offset=0.0, norm_place=capi.NORM_OUTPUT, side_dim=z["side"],
+                             logit_softcap=30.0)
+    st = Stage(stack=stack, layers=layers, n_layer=n_layer, n_embd=z["width"], n_vocab=ARCH_VOCAB, n_ctx=n_ctx, n_seq=1,
+               n_ubatch=ubatch, device=local)
+    st.generate(20251125)
+    return st
+
+
+def lomodra_work(z, n_layer):
+    """per token: (bytes of projection weights a decode step reads, bytes of low-rank matrices and states it moves, flops of a
+    prompt's matrix products)"""
+    h, D, H, d = z["width"], z["heads"] * LOMODRA_DIM, z["heads"], LOMODRA_DIM
+    r, kv = LOMODRA_RANK, z["kv"] * LOMODRA_DIM
+    n = [sum(1 for i in range(n_layer) if i % 3 == j) for j in range(3)]
+    shared = sum(1 for i in range(n_layer) if i % 6 == 5)
+    proj = n[0] * h * (4 * D + H + 2 * r) + n[1] * h * 5 * D + n[2] * h * 2 * D + (n[2] - shared) * h * 2 * kv
+    low = n[0] * 2 * r * D
+    ff = n_layer * (h * (z["experts"] + 3 * z["shared"]) + 3 * z["top"] * h * z["ff"] + 2 * h * z["side"])
+    state = (n[0] + n[1]) * 2 * 4 * H * d * d
+    return 2 * (proj + ff + ARCH_VOCAB * h), 2 * low + state, 2 * (proj + ff + low)
+
+
 def run_arch(args):
-    """--arch: prefill and decode of Gonetar-shaped models and of the K-quant decoder of equal size; one JSON line each"""
+    """--arch: prefill and decode of Gonetar- and Lomodra-shaped models and of the K-quant decoder of equal size; one JSON line each"""
     import ctypes as C
 
     import torch
@@ -358,20 +406,26 @@ def run_arch(args):
     except Exception:
         tf = 1400.0
     prompt, steps = 4096, max(16, args.steps)
-    names = sorted(ARCH_SIZES) if args.arch == "all" else [args.arch]
+    sizes = dict(ARCH_SIZES, **LOMODRA_SIZES)
+    names = sorted(sizes) if args.arch == "all" else [args.arch]
     for name in names:
-        z = ARCH_SIZES[name]
+        z = sizes[name]
         L = args.layers or z["n_layer"]
-        for kind in ("gonetar", "kquant"):
+        own = "gonetar" if name in ARCH_SIZES else "lomodra"
+        moe = dict(n_expert=z["experts"], n_expert_used=z["top"], n_ff_exp=z["ff"]) if own == "lomodra" else {}
+        for kind in (own, "kquant"):
             n_ctx = prompt + 4 * steps + 64
             if kind == "gonetar":
                 st = arch_stage(z, L, n_ctx, 2048, local)
+            elif kind == "lomodra":
+                st = lomodra_stage(z, L, n_ctx, 2048, local)
             else:
-                st = Stage(n_layer=L, n_embd=z["width"], n_head=z["heads"], n_head_kv=z["kv"], head_dim=128, n_ff=z["ff"],
-                           n_vocab=ARCH_VOCAB, n_ctx=n_ctx, n_seq=1, n_ubatch=2048, device=local)
+                st = Stage(n_layer=L, n_embd=z["width"], n_head=z["heads"], n_head_kv=z["kv"], head_dim=128, n_ff=0 if moe else z["ff"],
+                           n_vocab=ARCH_VOCAB, n_ctx=n_ctx, n_seq=1, n_ubatch=2048, device=local, **moe)
                 st.generate(20251125)
             out = {"arch": kind, "size": name, "layers": L, "weight_bytes": st.weight_bytes(), "data": "synthetic, random weights",
-                   "prompt": prompt, "window": ARCH_WINDOW if kind == "gonetar" else None}
+                   "prompt": prompt, "window": ARCH_WINDOW if kind == "gonetar" else None,
+                   "chunk": LOMODRA_CHUNK if kind == "lomodra" else None}
             toks = torch.from_numpy(np.random.default_rng(1).integers(0, ARCH_VOCAB, prompt).astype(np.int32)).to(dev)
             logits = torch.empty((1, ARCH_VOCAB), dtype=torch.float32, device=dev)
             nxt = torch.zeros(1, dtype=torch.int32, device=dev)
@@ -407,13 +461,18 @@ def run_arch(args):
                 out[f"{label}_ms"], out[f"{label}_launches"] = ms.value, int(n.value)
             out["clocks"] = sampler.stop(t0, time.time())
             st.synchronize()
-            if kind == "gonetar":
+            if kind == "lomodra":
+                proj, state, flops = lomodra_work(z, L)
+                out["gemv_frac_of_hbm_peak"] = proj / (out["gemv_ms"] * 1e-3) / 1e9 / hbm
+                out["step_frac_of_hbm_peak"] = (proj + state) / (out["step_ms"] * 1e-3) / 1e9 / hbm
+                out["prefill_frac_of_bf16_peak"] = out["prefill_ubatch2048_tok_s"] * flops / 1e12 / tf
+            elif kind == "gonetar":
                 proj, gates, lat, flops = arch_work(z, L)
                 out["gemv_frac_of_hbm_peak"] = proj / (out["gemv_ms"] * 1e-3) / 1e9 / hbm
                 out["step_frac_of_hbm_peak"] = (proj + gates + lat) / (out["step_ms"] * 1e-3) / 1e9 / hbm
                 out["prefill_frac_of_bf16_peak"] = out["prefill_ubatch2048_tok_s"] * flops / 1e12 / tf
             else:
-                w = dict(n_embd=z["width"], n_head=z["heads"], n_head_kv=z["kv"], head_dim=128, n_ff=z["ff"], n_vocab=ARCH_VOCAB)
+                w = dict(n_embd=z["width"], n_head=z["heads"], n_head_kv=z["kv"], head_dim=128, n_ff=z["ff"], n_vocab=ARCH_VOCAB, **moe)
                 b = step_gemv_bytes(w, 0, L, True)
                 out["gemv_frac_of_hbm_peak"] = b / (out["gemv_ms"] * 1e-3) / 1e9 / hbm
                 out["step_frac_of_hbm_peak"] = b / (out["step_ms"] * 1e-3) / 1e9 / hbm
@@ -455,8 +514,8 @@ def main():
     ap.add_argument("--no-extras", action="store_true", help="N = 1: skip the cfg3 / cfg4 / cfg1-against-CPU measurements "
                     "that follow the headline workload in the same run")
     ap.add_argument("--sweep", action="store_true", help="the isolated matmul sweep: all shapes x types x M")
-    ap.add_argument("--arch", default="", choices=["", "all"] + sorted(ARCH_SIZES), help="prefill and decode of a Gonetar-shaped "
-                    "model (random weights) next to the K-quant decoder of equal size; one JSON line each")
+    ap.add_argument("--arch", default="", choices=["", "all"] + sorted(ARCH_SIZES) + sorted(LOMODRA_SIZES), help="prefill and decode of a Gonetar- or "
+                    "Lomodra-shaped model (random weights) next to the K-quant decoder of equal size; one JSON line each")
     args = ap.parse_args()
     if args.arch:
         return run_arch(args)

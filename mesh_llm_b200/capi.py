@@ -51,8 +51,9 @@ class StageConfig(C.Structure):
     ]
 
 
-MIXER_LATENT_ATTN, MIXER_LINEAR_REC = 1, 2
-FFN_NONE, FFN_CLAMPED_GLU = 0, 1
+MIXER_LATENT_ATTN, MIXER_LINEAR_REC, MIXER_GQA, MIXER_DECAY_STATE, MIXER_DELTA_STATE = 1, 2, 3, 4, 5
+FFN_NONE, FFN_CLAMPED_GLU, FFN_MOE = 0, 1, 2
+NORM_SANDWICH, NORM_OUTPUT = 0, 1
 PRECISION_BF16, PRECISION_F32 = 0, 1
 
 
