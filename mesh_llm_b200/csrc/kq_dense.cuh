@@ -276,21 +276,24 @@ struct KqMatState {
     float *s, *conv;                          // first sequence of the call
 };
 constexpr int KQ_STATE_MAX_DIM = 256;
-static inline int kq_state_ld(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 96 ? 96 : dim <= 128 ? 128 : dim <= 192 ? 192 : 256; }
+static inline __host__ __device__ int kq_state_ld(int dim) { return dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
 static inline __host__ __device__ int64_t kq_state_channels(const KqMatState &m) { return 2 * (int64_t)m.kv_heads * m.dim + (int64_t)m.heads * m.vdim; }
 // Columns of the fused projection's rows
 struct KqStateIn {
     const float *q, *k, *v, *b, *z; // z: decay projection [rows][ldz], bias not added yet; b: write strengths before the sigmoid
     int64_t ld, ldz;
 };
-// What the token loop reads: q, k after convolution, SiLU, unit norm (delta) and scaling, v after convolution and SiLU,
-// decays g, and per head (beta, q.k).  Buffers of the caller.
+// Records of blocks of four tokens (kq_state_ops.cu): for every sequence kq_state_blocks(T) times kq_state_rec_floats and
+// kq_state_val_floats floats, 16-byte aligned
 struct KqStateTok {
-    float *q, *k, *v, *g, *b; // [rows][kq_f32_ld(kv_heads dim)], same, [rows][kq_f32_ld(heads vdim)], [rows][kq_f32_ld(heads dim)], [rows][2 heads]
+    float *rec, *val;
 };
+static inline int64_t kq_state_blocks(int64_t T) { return (T + 3) / 4; }
+int64_t kq_state_rec_floats(const KqMatState &m);
+int64_t kq_state_val_floats(const KqMatState &m);
 b200_status kq_state_tokens(const KqMatState &m, const KqStateIn &in, const KqStateTok &t, int n_seq, int T, const int32_t *pos0_dev, int pos0,
                             cudaStream_t st);
-// the token loop over T positions: o [rows][ldo] f32; also moves the convolution's ring forward (in: its inputs)
+// the walk over T positions: o [rows][ldo] f32; also moves the convolution's ring forward (in: its inputs)
 b200_status kq_state_scan(const KqMatState &m, const KqStateIn &in, const KqStateTok &t, int n_seq, int T, const int32_t *pos0_dev, int pos0,
                           float *o, int64_t ldo, cudaStream_t st);
 // every head's o over its rms times norm_w [vdim] times sigmoid(gate); f32 or bf16 rows (padded with zeros)

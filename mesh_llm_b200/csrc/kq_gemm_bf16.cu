@@ -54,7 +54,16 @@ struct Col4 {
 #pragma unroll
         for (int e = 0; e < 4; e++) bias[e] = s.bias && e < valid && (c.groups > 1 || n + e < s.n_rows) ? s.bias[n + e] : 0.f;
     }
-    __device__ __forceinline__ void store(const KqDense &c, const KqDenseSeg &s, int64_t m, int g, const float4 &v) const {
+    // the factors of row m: eight bytes where the row allows it
+    __device__ __forceinline__ uint2 factors(const KqDense &c, int64_t m) const {
+        const uint16_t *f = c.row_mul + (int64_t)c.mul_row[m] * c.ld_mul + n;
+        if (n_mul >= 4 && ((uintptr_t)f & 7) == 0) return *reinterpret_cast<const uint2 *>(f);
+        uint32_t w[4];
+#pragma unroll
+        for (int e = 0; e < 4; e++) w[e] = e < n_mul ? f[e] : 0;
+        return make_uint2(w[0] | (w[1] << 16), w[2] | (w[3] << 16));
+    }
+    __device__ __forceinline__ void store(const KqDense &c, const KqDenseSeg &s, int64_t m, int g, const float4 &v, const uint2 f = make_uint2(0, 0)) const {
         float o[4] = {v.x + bias[0], v.y + bias[1], v.z + bias[2], v.w + bias[3]};
         if (s.act == KQ_ACT_GELU_TANH) {
 #pragma unroll
@@ -70,10 +79,8 @@ struct Col4 {
             for (int e = 0; e < 4; e++) o[e] *= f;
         }
         if (c.row_mul) {
-            const uint16_t *f = c.row_mul + (int64_t)c.mul_row[m] * c.ld_mul + n;
-#pragma unroll
-            for (int e = 0; e < 4; e++)
-                if (e < n_mul) o[e] *= kq_bf2f(f[e]);
+            o[0] *= kq_bf2f((uint16_t)f.x), o[1] *= kq_bf2f((uint16_t)(f.x >> 16));
+            o[2] *= kq_bf2f((uint16_t)f.y), o[3] *= kq_bf2f((uint16_t)(f.y >> 16));
         }
         if (vec) {
             const int64_t i = m * s.ldy + col;
@@ -259,10 +266,20 @@ __global__ void __launch_bounds__(NTHREADS, 1) gemm_bf16_kernel(const __grid_con
                 const int n = n0 + j + c4, n_valid = std::min(4, lim - n);
                 if (n_valid > 0) {
                     const Col4 col(p.c, s, (p.c.experts ? 0 : (int64_t)w.g * n_rows) + n, n_valid);
+                    if (p.c.row_mul) { // the factors of all of a lane's rows are requested together: they may come from anywhere
+                        uint2 f[8];
+#pragma unroll
+                        for (int i = 0; i < 8; i++) f[i] = m0 + r4 + 4 * i < m_end ? col.factors(p.c, m0 + r4 + 4 * i) : make_uint2(0, 0);
+#pragma unroll
+                        for (int i = 0; i < 8; i++)
+                            if (m0 + r4 + 4 * i < m_end)
+                                col.store(p.c, s, m0 + r4 + 4 * i, w.g, *reinterpret_cast<const float4 *>(stage + (r4 + 4 * i) * EP + c4), f[i]);
+                    } else {
 #pragma unroll 2
-                    for (int r = r4; m0 + r < m_end; r += 4) {
-                        const float4 v = *reinterpret_cast<const float4 *>(stage + r * EP + c4);
-                        col.store(p.c, s, m0 + r, w.g, v);
+                        for (int r = r4; m0 + r < m_end; r += 4) {
+                            const float4 v = *reinterpret_cast<const float4 *>(stage + r * EP + c4);
+                            col.store(p.c, s, m0 + r, w.g, v);
+                        }
                     }
                 }
                 __syncwarp();

@@ -4,7 +4,8 @@
 // A CTA takes a range of one row's visible keys for up to RT query heads of one key / value head.  Lanes split the
 // dimensions two by two, so that a warp reads whole key rows; a warp takes four keys at a time, their scores are reduced
 // across the warp together.  Scores of a tile of keys sit in shared memory, the softmax is online over tiles, all in f32.
-// The ranges' results (maximum, sum, weighted values) are merged by the last CTA of a row to arrive.  In a decode step the
+// The ranges' results (maximum, sum, weighted values) are merged by the last CTA of a row to arrive; ranges without keys
+// take no part.  In a decode step the
 // same launch norms the queries and the new key and stores the new row: only the CTA whose range ends with the new
 // position reads that row, and it is the one that stores it.
 #include "kq_dense.cuh"
@@ -14,6 +15,7 @@
 namespace {
 
 constexpr int NT = 128, NW = NT / 32, KT = 128; // threads, warps, keys per tile
+constexpr int MAX_SPLITS = KT, MIN_RANGE = 32;  // ranges of a row's keys, keys of a range
 
 struct Params {
     KqGqa a;
@@ -25,7 +27,8 @@ struct Params {
     int64_t ldo;
     uint16_t *out16;
     int64_t ldo16;
-    float *part;        // [row][head][split][2 + vdim]: maximum, sum, weighted values
+    float *part;        // [row][head][split][vdim padded to 4]: weighted values
+    float2 *ml;         // [row][head][split]: maximum, sum
     unsigned *counters; // [row][head group], zero between launches
     int32_t splits, groups;
 };
@@ -86,11 +89,13 @@ __global__ void __launch_bounds__(NT) gqa_attn_kernel(const __grid_constant__ Pa
     const int g = blockIdx.y / gpk, h0 = g * rep + blockIdx.y % gpk * RT, nh = min(RT, (g + 1) * rep - h0);
     const int64_t r = blockIdx.z, seq = r / p.T;
     const int pos = (p.pos0_dev ? *p.pos0_dev : p.pos0) + (int)(r % p.T);
-    const int lo = kq_first_key(pos, a.window, a.chunk), n = pos - lo + 1, per = (n + S - 1) / S;
+    const int lo = kq_first_key(pos, a.window, a.chunk), n = pos - lo + 1, per = max((n + S - 1) / S, MIN_RANGE);
     const int j0 = min(n, split * per), j1 = min(n, j0 + per); // keys lo + j0 .. lo + j1 - 1
+    const int live = (n + per - 1) / per;                      // ranges that have any
+    if (j0 >= j1) return;
     const int ldk = (a.dim + 63) / 64 * 64, ldv = (a.vdim + 63) / 64 * 64;
 
-    if (j0 < j1) {
+    {
         if (FUSED && a.own_kv && j1 == n && warp == NW - 1) // head groups of one key head store the same values
             store_row<CT>(a, p.k + r * p.ldp + (int64_t)g * a.dim, p.v + r * p.ldp + (int64_t)g * a.vdim, seq, pos, g, lane);
         for (int t = warp; t < RT; t += NW) {
@@ -212,7 +217,7 @@ __global__ void __launch_bounds__(NT) gqa_attn_kernel(const __grid_constant__ Pa
         s_p[tid][0] = mt, s_p[tid][1] = lt;
     }
     __syncthreads();
-    const int64_t rec = 2 + a.vdim;
+    const int64_t rec = (a.vdim + 3) / 4 * 4;
     auto emit = [&](int h, int d, float v) {
         const int64_t c = (int64_t)h * a.vdim + d;
         if (p.out) p.out[r * p.ldo + c] = v;
@@ -223,52 +228,63 @@ __global__ void __launch_bounds__(NT) gqa_attn_kernel(const __grid_constant__ Pa
         float v = 0.f;
 #pragma unroll
         for (int w = 0; w < NW; w++) v += reinterpret_cast<const float *>(s_o[w][t])[d];
-        if (S == 1) emit(h0 + t, d, v / s_p[t][1]);
-        else __stcg(p.part + ((r * a.n_head + h0 + t) * S + split) * rec + 2 + d, v);
+        if (live == 1) emit(h0 + t, d, v / s_p[t][1]);
+        else __stcg(p.part + ((r * a.n_head + h0 + t) * S + split) * rec + d, v);
     }
-    if (S == 1) return;
-    if (tid < nh) {
-        float *d = p.part + ((r * a.n_head + h0 + tid) * S + split) * rec;
-        __stcg(d, s_p[tid][0]);
-        __stcg(d + 1, s_p[tid][1]);
-    }
+    if (live == 1) return;
+    if (tid < nh) __stcg(p.ml + (r * a.n_head + h0 + tid) * S + split, make_float2(s_p[tid][0], s_p[tid][1]));
     __threadfence();
     __syncthreads();
     if (tid == 0) {
         unsigned *c = p.counters + r * p.groups + blockIdx.y;
-        s_last = atomicAdd(c, 1u) == (unsigned)S - 1;
+        s_last = atomicAdd(c, 1u) == (unsigned)live - 1;
         if (s_last) *c = 0u;
     }
     __syncthreads();
     if (!s_last) return;
     __threadfence();
     for (int t = warp; t < nh; t += NW) { // weights of the ranges, by a warp per head
-        const float *d = p.part + (r * a.n_head + h0 + t) * S * rec;
+        const float2 *d = p.ml + (r * a.n_head + h0 + t) * S;
+        float2 x[MAX_SPLITS / 32];
         float mx = -INFINITY, sum = 0.f;
-        for (int s = lane; s < S; s += 32) mx = fmaxf(mx, __ldcg(d + s * rec));
+#pragma unroll
+        for (int i = 0; i < MAX_SPLITS / 32; i++) {
+            x[i] = lane + 32 * i < live ? __ldcg(d + lane + 32 * i) : make_float2(-INFINITY, 0.f);
+            mx = fmaxf(mx, x[i].x);
+        }
         mx = kq_warp_max(mx);
-        for (int s = lane; s < S; s += 32) sum += __ldcg(d + s * rec + 1) * expf(__ldcg(d + s * rec) - mx);
+#pragma unroll
+        for (int i = 0; i < MAX_SPLITS / 32; i++) sum += x[i].y * expf(x[i].x - mx);
         sum = kq_warp_sum(sum);
-        for (int s = lane; s < S; s += 32) s_p[t][s] = expf(__ldcg(d + s * rec) - mx) / sum;
+#pragma unroll
+        for (int i = 0; i < MAX_SPLITS / 32; i++) s_p[t][lane + 32 * i] = expf(x[i].x - mx) / sum;
     }
     __syncthreads();
-    for (int i = tid; i < nh * a.vdim; i += NT) {
-        const int t = i / a.vdim, d = i % a.vdim;
-        const float *src = p.part + (r * a.n_head + h0 + t) * S * rec + 2 + d;
-        float v = 0.f;
-#pragma unroll 8
-        for (int s = 0; s < S; s++) v = fmaf(s_p[t][s], __ldcg(src + s * rec), v);
-        emit(h0 + t, d, v);
+    const int n4 = (int)rec / 4;
+    for (int i = tid; i < nh * n4; i += NT) { // what lies behind vdim is not written out
+        const int t = i / n4, d = i % n4 * 4;
+        const float4 *src = reinterpret_cast<const float4 *>(p.part + (r * a.n_head + h0 + t) * S * rec + d);
+        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 16
+        for (int s = 0; s < live; s++) {
+            const float w = s_p[t][s];
+            const float4 x = __ldcg(src + s * n4);
+            v.x = fmaf(w, x.x, v.x), v.y = fmaf(w, x.y, v.y), v.z = fmaf(w, x.z, v.z), v.w = fmaf(w, x.w, v.w);
+        }
+        const float o4[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int e = 0; e < 4; e++)
+            if (d + e < a.vdim) emit(h0 + t, d + e, o4[e]);
     }
 }
 
-constexpr int MAX_SPLITS = KT, SPLIT_ROWS = 8; // up to SPLIT_ROWS rows are split
+constexpr int SPLIT_ROWS = 8; // up to SPLIT_ROWS rows are split
 
 int splits_of(const KqGqa &a, int rows, int max_keys) {
     if (rows > SPLIT_ROWS) return 1;
     const int64_t ctas = (int64_t)rows * a.kv_heads * kq_div_up(a.n_head / a.kv_heads, 4);
     const int64_t fill = kq_div_up(4 * (int64_t)kq_sm_count(), ctas);
-    return (int)std::max<int64_t>(1, std::min<int64_t>({kq_div_up(max_keys, 32), fill, MAX_SPLITS}));
+    return (int)std::max<int64_t>(1, std::min<int64_t>({kq_div_up(max_keys, MIN_RANGE), fill, MAX_SPLITS}));
 }
 
 template <typename CT, bool FUSED>
@@ -304,8 +320,8 @@ b200_status kq_gqa_store(const KqGqa &a, float *q, const float *k, const float *
 size_t kq_gqa_scratch_bytes(const KqGqa &a, int max_rows, int max_keys) {
     size_t n = 0;
     for (int r = 1; r <= std::min(max_rows, SPLIT_ROWS); r++)
-        n = std::max(n, (size_t)r * a.n_head * splits_of(a, r, max_keys) * (2 + a.vdim) * 4);
-    return n;
+        n = std::max(n, (size_t)r * a.n_head * splits_of(a, r, max_keys) * (2 + (size_t)kq_pad(a.vdim, 4)) * 4);
+    return n + 16;
 }
 int64_t kq_gqa_counters(const KqGqa &a) { return (int64_t)SPLIT_ROWS * a.n_head; }
 
@@ -323,8 +339,10 @@ b200_status kq_gqa_attention(const KqGqa &a, bool fused, const float *q, const f
     p.splits = splits_of(a, rows, max_keys);
     p.groups = (int)(a.kv_heads * kq_div_up(rep, rt));
     p.counters = counters;
+    const int64_t records = (int64_t)rows * a.n_head * p.splits, per = kq_pad(a.vdim, 4);
     p.part = scratch;
-    KQ_REQUIRE(p.splits == 1 || (counters && scratch_bytes >= (size_t)rows * a.n_head * p.splits * (2 + a.vdim) * 4), "gqa_attention: scratch");
+    p.ml = (float2 *)(scratch + records * per);
+    KQ_REQUIRE(p.splits == 1 || (counters && scratch_bytes >= (size_t)records * (2 + per) * 4), "gqa_attention: scratch");
     const dim3 grid((unsigned)p.splits, (unsigned)p.groups, (unsigned)rows);
     KQ_REQUIRE(p.groups <= 65535, "gqa_attention: %d heads", a.n_head);
     if (a.f32) return fused ? launch<float, true>(p, grid, n, rt == 1, st) : launch<float, false>(p, grid, n, rt == 1, st);

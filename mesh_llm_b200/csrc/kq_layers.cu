@@ -82,6 +82,7 @@ struct KqLayers {
     float *f[9] = {}; // projections of a mixer
     std::vector<Pack> packs;
     const uint16_t *side_embed = nullptr;
+    KqStateTok state_tok = {};
     // experts: activations of few rows; tiles of rows by expert
     float *moe_act = nullptr, *moe_y = nullptr;
     void *moe_x = nullptr, *moe_h = nullptr; // bf16, or f32 in the 32-bit mode
@@ -511,9 +512,8 @@ struct Pass {
                 OTHER_(kq_gemm_bf16(g, g16, kq_bf16_ld(c.gate_rank), 1, s));
             }
         }
-        const KqStateTok t = {k->f[1], k->f[2], k->f[3], k->f[4], k->f[7]};
-        OTHER_(kq_state_tokens(m, si, t, n_seq, T, pos_dev, pos0, s));
-        OTHER_(kq_state_scan(m, si, t, n_seq, T, pos_dev, pos0, o, ldv, s));
+        OTHER_(kq_state_tokens(m, si, k->state_tok, n_seq, T, pos_dev, pos0, s));
+        OTHER_(kq_state_scan(m, si, k->state_tok, n_seq, T, pos_dev, pos0, o, ldv, s));
         if (!m.delta) return close_normed(L.wo, K, o, ldv, L.o_norm, gate, ldp, L.post1);
         OTHER_(kq_head_norm_gate(o, ldv, k->f[5], ldv, L.o_norm, st->c.rms_eps, rows, m.heads, m.vdim, tc ? nullptr : z, ldv, tc ? k->z16 : nullptr, ld16, s));
         return close(L.wo, K, z, ldv, k->z16, L.post1);
@@ -836,7 +836,7 @@ b200_status b200_stage_create_layers(const b200_stage_config *cfg, const b200_st
     if (c.has_embd || c.has_output) kq_stage_add_tensor(st, "embed", B200_TYPE_BF16, h, c.n_vocab, 1);
     if (stack->side_dim) kq_stage_add_tensor(st, "side.embed", B200_TYPE_BF16, (int64_t)c.n_layer * stack->side_dim, c.n_vocab, 1);
     int64_t fmax[9] = {}, wmax16 = 0, u16max = 0, ffmax = 0, scratch = 0, rec_scratch = 0, prefill = 0;
-    int64_t gqa_counters = 0, few_act = 0, moe_rows = 0, moe_ff = 0, moe_pairs = 0, moe_tiles = 0;
+    int64_t gqa_counters = 0, state_rec = 0, state_val = 0, few_act = 0, moe_rows = 0, moe_ff = 0, moe_pairs = 0, moe_tiles = 0;
     const bool f32 = stack->precision == B200_PRECISION_F32;
     auto grow = [](int64_t &a, int64_t b) { a = std::max(a, b); };
     for (int i = c.layer_begin; i < c.layer_end; i++) {
@@ -901,11 +901,12 @@ b200_status b200_stage_create_layers(const b200_stage_config *cfg, const b200_st
             }
             mat("mix.o", K, h);
             L.in_pack = pack(in, 8);
-            grow(fmax[1], kq_f32_ld(G * l.qk_dim));
-            grow(fmax[2], kq_f32_ld(G * l.qk_dim));
             if (delta) grow(fmax[4], kq_f32_ld(H * l.qk_dim));
-            for (int f : {3, 5, 6, 8}) grow(fmax[f], kq_f32_ld(K));
-            grow(fmax[7], kq_f32_ld(2 * H));
+            for (int f : {5, 6, 8}) grow(fmax[f], kq_f32_ld(K));
+            KqMatState m = {};
+            m.heads = l.n_head, m.dim = l.qk_dim, m.vdim = l.v_dim, m.delta = delta;
+            grow(state_rec, kq_state_rec_floats(m));
+            grow(state_val, kq_state_val_floats(m));
             grow(wmax16, kq_bf16_ld(K));
         } else if (l.mixer == B200_MIXER_LINEAR_REC) {
             const int64_t W = l.rec_width, m = W / l.rec_blocks;
@@ -1078,6 +1079,11 @@ b200_status b200_stage_create_layers(const b200_stage_config *cfg, const b200_st
     if (wide) A(&k->u16, (size_t)(R * u16max * 2));
     if (ffmax) A(&k->act32, (size_t)((f32 ? R : std::min<int64_t>(R, SMALL_ROWS)) * kq_f32_ld(ffmax) * 4));
     if (ffmax && wide) A(&k->act16, (size_t)(R * kq_bf16_ld(ffmax) * 2));
+    if (state_rec) {
+        const int64_t blocks = R / 4 + std::min<int64_t>(R, c.n_seq) + 1; // of all sequences of a call
+        A(&k->state_tok.rec, (size_t)(blocks * state_rec * 4));
+        A(&k->state_tok.val, (size_t)(blocks * state_val * 4));
+    }
     if (gqa_counters) A(&k->gqa_counters, (size_t)gqa_counters * 4);
     if (moe_pairs) {
         A(&k->moe_act, (size_t)few_act * 4);

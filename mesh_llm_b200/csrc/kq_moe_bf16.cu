@@ -95,8 +95,8 @@ __global__ void __launch_bounds__(NT) moe_few_gate_up_kernel(const __grid_consta
     }
 }
 
-// grid (slices of output rows, rows); a warp takes two output rows over all chosen experts and the shared one
-constexpr int DOWN_ROWS = 2 * NW;
+// grid (slices of output rows, rows); a warp takes an output row over all chosen experts and the shared one
+constexpr int DOWN_ROWS = NW, DOWN_U = 8; // chunks in flight per lane
 __global__ void __launch_bounds__(NT) moe_few_down_kernel(const __grid_constant__ KqMoe m, const float *act, int64_t ld_act, const int32_t *ids, const float *wts,
                                                           const uint16_t *down, const uint16_t *sh_down, float *out, int64_t ldo) {
     extern __shared__ __align__(16) float sm[]; // [top][padded ff] activations times weight, [padded ff_shared]
@@ -104,6 +104,19 @@ __global__ void __launch_bounds__(NT) moe_few_down_kernel(const __grid_constant_
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = blockIdx.y;
     const int fp = (m.ff + 7) / 8 * 8, sp = (m.ff_shared + 7) / 8 * 8, per = fp / 8, n_ck = m.top * per, s_ck = sp / 8;
     float4 *p0 = reinterpret_cast<float4 *>(sm), *p1 = p0 + n_ck + s_ck; // two planes of float4
+    const int n = blockIdx.x * DOWN_ROWS + warp, all = n_ck + s_ck;
+    const int64_t ldw = kq_bf16_ld(m.ff), lds = kq_bf16_ld(m.ff_shared);
+    uint4 q[DOWN_U];
+    auto request = [&](int c0) {
+#pragma unroll
+        for (int u = 0; u < DOWN_U; u++) {
+            const int c = c0 + lane + 32 * u;
+            q[u] = make_uint4(0, 0, 0, 0);
+            if (n < m.h && c < n_ck) q[u] = kq_ld_stream(down + ((int64_t)ids[row * m.top + c / per] * m.h + n) * ldw + c % per * 8);
+            else if (n < m.h && c < all) q[u] = kq_ld_stream(sh_down + n * lds + (c - n_ck) * 8);
+        }
+    };
+    request(0);
     float *f0 = reinterpret_cast<float *>(p0), *f1 = reinterpret_cast<float *>(p1);
     for (int i = tid; i < m.top * fp; i += NT) {
         const int s = i / fp, j = i % fp;
@@ -115,48 +128,49 @@ __global__ void __launch_bounds__(NT) moe_few_down_kernel(const __grid_constant_
         ((j & 4) ? f1 : f0)[(n_ck + j / 8) * 4 + (j & 3)] = v;
     }
     __syncthreads();
-    const int n = blockIdx.x * DOWN_ROWS + warp * 2;
-    if (n >= m.h) return;
-    const int64_t ldw = kq_bf16_ld(m.ff), lds = kq_bf16_ld(m.ff_shared);
-    const int n1 = min(n + 1, m.h - 1);
-    float a0 = 0.f, a1 = 0.f;
-    const int all = n_ck + s_ck;
-    for (int c0 = lane; c0 < all; c0 += 128) {
-        uint4 q[4][2];
+    float a = 0.f;
+    for (int c0 = 0;;) {
 #pragma unroll
-        for (int u = 0; u < 4; u++) {
-            const int c = c0 + 32 * u;
-            q[u][0] = q[u][1] = make_uint4(0, 0, 0, 0);
-            if (c < n_ck) {
-                const uint16_t *w = down + (int64_t)ids[row * m.top + c / per] * m.h * ldw + c % per * 8;
-                q[u][0] = kq_ld_stream(w + n * ldw), q[u][1] = kq_ld_stream(w + n1 * ldw);
-            } else if (c < all) {
-                q[u][0] = kq_ld_stream(sh_down + n * lds + (c - n_ck) * 8), q[u][1] = kq_ld_stream(sh_down + n1 * lds + (c - n_ck) * 8);
-            }
+        for (int u = 0; u < DOWN_U; u++) {
+            const int c = c0 + lane + 32 * u;
+            if (c < all) a = kq_dot8(q[u], p0[c], p1[c], a);
         }
-#pragma unroll
-        for (int u = 0; u < 4; u++) {
-            const int c = c0 + 32 * u;
-            if (c < all) {
-                a0 = kq_dot8(q[u][0], p0[c], p1[c], a0);
-                a1 = kq_dot8(q[u][1], p0[c], p1[c], a1);
-            }
-        }
+        c0 += 32 * DOWN_U;
+        if (c0 >= all || n >= m.h) break;
+        request(c0);
     }
-    a0 = kq_warp_sum(a0);
-    a1 = kq_warp_sum(a1);
-    if (lane == 0) {
-        out[row * ldo + n] = a0;
-        if (n + 1 < m.h) out[row * ldo + n + 1] = a1;
-    }
+    a = kq_warp_sum(a);
+    if (lane == 0 && n < m.h) out[row * ldo + n] = a;
 }
 
-// a warp per row: choice; then the CTA forms the shared GLU of its rows
-__global__ void __launch_bounds__(NT) moe_route_kernel(const __grid_constant__ KqMoe m, int rows, KqMoeOrder o, float *sh32, int64_t ld32, uint16_t *sh16, int64_t ld16) {
+// the first CTAs: a warp per row chooses; the others form the shared GLU, a row and GLU_COLS columns each
+constexpr int GLU_COLS = 4 * NT;
+__global__ void __launch_bounds__(NT) moe_route_kernel(const __grid_constant__ KqMoe m, int rows, int route_ctas, int slices, KqMoeOrder o, float *sh32, int64_t ld32,
+                                                       uint16_t *sh16, int64_t ld16) {
     extern __shared__ __align__(16) float sm[]; // [NW][experts]
     __shared__ int32_t s_id[NW][KQ_MOE_MAX_TOP];
     __shared__ float s_w[NW][KQ_MOE_MAX_TOP];
     KQ_PDL_ENTER();
+    if ((int)blockIdx.x >= route_ctas) {
+        const int64_t i = blockIdx.x - route_ctas, r = i / slices;
+        const int j = (int)(i % slices) * GLU_COLS + threadIdx.x * 4, w = sh16 ? (int)ld16 : m.ff_shared;
+        const float *g = m.sh_gate + r * m.ldz, *u = m.sh_up + r * m.ldz;
+        if (j >= w) return;
+        float v[4];
+        if (j + 4 <= m.ff_shared && ((m.ldz & 3) == 0) && ((((uintptr_t)m.sh_gate | (uintptr_t)m.sh_up) & 15) == 0)) {
+            const float4 a = *reinterpret_cast<const float4 *>(g + j), b = *reinterpret_cast<const float4 *>(u + j);
+            v[0] = kq_silu(a.x) * b.x, v[1] = kq_silu(a.y) * b.y, v[2] = kq_silu(a.z) * b.z, v[3] = kq_silu(a.w) * b.w;
+        } else {
+#pragma unroll
+            for (int e = 0; e < 4; e++) v[e] = j + e < m.ff_shared ? kq_silu(g[j + e]) * u[j + e] : 0.f;
+        }
+        if (sh16) // rows of a multiple of 64 elements, padded with zeros
+            *reinterpret_cast<uint2 *>(sh16 + r * ld16 + j) = make_uint2((uint32_t)kq_f2bf(v[0]) | ((uint32_t)kq_f2bf(v[1]) << 16),
+                                                                         (uint32_t)kq_f2bf(v[2]) | ((uint32_t)kq_f2bf(v[3]) << 16));
+        else
+            for (int e = 0; e < 4 && j + e < w; e++) sh32[r * ld32 + j + e] = v[e];
+        return;
+    }
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int64_t row = (int64_t)blockIdx.x * NW + warp;
     if (row < rows) {
@@ -169,16 +183,6 @@ __global__ void __launch_bounds__(NT) moe_route_kernel(const __grid_constant__ K
             o.wts[row * m.top + s] = s_w[warp][s];
         }
     }
-    const int r0 = blockIdx.x * NW, nr = min(NW, rows - r0);
-    const int w = sh16 ? (int)ld16 : m.ff_shared;
-    if (m.ff_shared)
-        for (int i = threadIdx.x; i < nr * w; i += NT) {
-            const int64_t r = r0 + i / w;
-            const int j = i % w;
-            const float v = j < m.ff_shared ? kq_silu(m.sh_gate[r * m.ldz + j]) * m.sh_up[r * m.ldz + j] : 0.f;
-            if (sh16) sh16[r * ld16 + j] = kq_f2bf(v);
-            else sh32[r * ld32 + j] = v;
-        }
 }
 
 // one CTA: how many pairs every expert has, whole tiles for each, a place for every pair
@@ -305,7 +309,8 @@ b200_status kq_moe_route(const KqMoe &m, int rows, const KqMoeOrder &o, float *s
     const size_t smem = (size_t)NW * m.experts * 4;
     static size_t have[16];
     KQ_TRY(allow_smem(moe_route_kernel, smem + 8192, have));
-    kq_launch(moe_route_kernel, (unsigned)kq_div_up(rows, NW), NT, smem, st, m, rows, o, sh32, ld32, sh16, ld16);
+    const int route_ctas = (int)kq_div_up(rows, NW), slices = m.ff_shared ? (int)kq_div_up(sh16 ? ld16 : m.ff_shared, GLU_COLS) : 0;
+    kq_launch(moe_route_kernel, (unsigned)(route_ctas + rows * slices), NT, smem, st, m, rows, route_ctas, slices, o, sh32, ld32, sh16, ld16);
     KQ_COUNT_LAUNCH();
     KQ_LAUNCH_CHECK();
     return B200_OK;

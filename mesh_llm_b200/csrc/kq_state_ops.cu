@@ -1,26 +1,53 @@
 // Recurrences whose state is a matrix per head, all in f32: linear attention under a fixed decay, and the delta rule with a
 // decay per key channel behind short convolutions.
 //
-// Prompts: one launch prepares every token's q, k, v, decay and write strength (convolution, SiLU, unit norms); the token loop
-// then keeps the state in registers.  A column of the state (one value dimension) belongs to eight lanes that split the
-// key dimension in groups of four, so a token costs two multiply-adds per element for the products with k and q, one
-// for the decay and one for the write, and one exchange over eight lanes: the read-out of the new state is the read-out
-// of the decayed one plus (q.k) u, so both products wait for the same reduction.  A CTA has 16 columns of one head; tiles of
-// tokens come through shared memory by cp.async, two tiles in flight.
+// Prompts, in blocks of four tokens.  Written out over a block, with S the state in front of it, G_j the product of the
+// block's decays up to token j and P_ij that of the decays behind token i up to token j,
+//   u_j = beta_j (v_j - S^T (G_j k_j) - sum_(i<j) A_ji u_i),   A_ji = k_j . (P_ij k_i)
+//   o_j = S^T (G_j q_j) + sum_(i<=j) B_ji u_i,                 B_ji = q_j . (P_ij k_i)
+//   S  <- G_4 S + sum_i (P_i4 k_i) u_i^T
+// with products of decays only, no quotients.  One launch makes every block's vectors and scalars (convolution, SiLU, unit
+// norms, decays) and leaves them as one record per block and head; the second walks the blocks with the state in
+// registers, so that eight products with the state wait for one reduction and a record is read from shared memory once
+// per four columns.  A thread holds four key dimensions (or eight) of four columns (value dimensions).  Records come by bulk
+// copies, two tiles in flight; every wait is bounded.
+// The fixed decay is the same with u = v and scalar products of decays.
 // A decode step is one launch: a CTA per head convolves, norms, works out the low-rank decays and gates, updates the
 // state and norms and gates the head's output.
 #include "kq_gemv_grouped.cuh"
+#include "kq_tc.cuh"
 
 #include <algorithm>
 
 namespace {
 
-constexpr int COLS = 16, SCAN_NT = COLS * 8; // columns and threads of a CTA of the token loop
+__device__ int g_state_error;
 
 __device__ __forceinline__ float sum8(float v) { // over the eight lanes of a column
     v += __shfl_xor_sync(0xffffffffu, v, 4);
     v += __shfl_xor_sync(0xffffffffu, v, 2);
     return v + __shfl_xor_sync(0xffffffffu, v, 1);
+}
+// N values of every lane summed over groups of L lanes (powers of two).  Each exchange halves the values a lane still carries:
+// with p the lane's place in its group, v[i] ends as value p N / L + i (N >= L), v[0] as value p / (L / N) (N < L).
+template <int N, int L>
+__device__ __forceinline__ void spread_sum(float (&v)[N], int lane) {
+    int n = N;
+#pragma unroll
+    for (int m = L / 2; m >= 1; m /= 2) {
+        if (n > 1) {
+            n /= 2;
+            const bool up = lane & m;
+#pragma unroll
+            for (int i = 0; i < N / 2; i++)
+                if (i < n) {
+                    const float send = up ? v[i] : v[i + n], keep = up ? v[i + n] : v[i];
+                    v[i] = keep + __shfl_xor_sync(0xffffffffu, send, m);
+                }
+        } else {
+            v[0] += __shfl_xor_sync(0xffffffffu, v[0], m);
+        }
+    }
 }
 
 // the convolution's input at position pos0 + t: this call's rows, the ring, or zero before the start
@@ -37,160 +64,189 @@ struct ConvIn {
     }
 };
 
-// ---- tokens ------------------------------------------------------------------------------------------
-constexpr int TOK_NT = 256, TOK_NW = TOK_NT / 32, RUN = 16; // tokens a warp walks for one head
+// ---- records of blocks of tokens -----------------------------------------------------------------------
+constexpr int BT = 4, TOK_NT = 256, TOK_NW = TOK_NT / 32, RUN = 4; // tokens per block, blocks a warp walks
+constexpr int N_SCALAR = 32;                                       // beta (4), A (6, from 4), B (10, from 12)
+// floats of a record: decayed k, decayed q, k towards the block's end (four vectors each) and the block's decay; fixed decay: the
+// middle two
+__host__ __device__ constexpr int rec_floats(int dp, bool delta) { return (delta ? 13 : 8) * dp + N_SCALAR; }
+
 struct TokParams {
     KqMatState m;
     KqStateIn in;
-    KqStateTok t;
-    int32_t T, pos0;
+    float *rec, *val; // [seq][block][head][record], [seq][block][head][vdim][BT]
+    int32_t T, pos0, blocks, head_ctas;
     const int32_t *pos0_dev;
-    int64_t ldq, ldv, ldg;
 };
 
-// SiLU of the convolution of up to 32 C channels of one head for a run of tokens: f(t, values of the lane's channels)
-template <int C, typename F>
-__device__ __forceinline__ void conv_run(const TokParams &p, const float *x, const float *w, int64_t channel0, int n, int64_t seq, int t0, int t1, int pos0,
-                                         int lane, F f) {
+// SiLU of the convolution of channels lane + 32 c (< n) at the BT positions from t0 on; zero past the call's rows
+template <int C>
+__device__ __forceinline__ void conv_block(const TokParams &p, const float *x, const float *w, int64_t channel0, int n, int64_t seq, int t0, int pos0, int lane,
+                                           float (&out)[BT][C]) {
     const int taps = p.m.taps;
     const int64_t row0 = seq * p.T, channels = kq_state_channels(p.m);
-    if (taps == 4) { // the last inputs and the weights stay in registers
-        float cw[C][4], in[C][4];
 #pragma unroll
-        for (int c = 0; c < C; c++) {
-            const int d = lane + 32 * c;
-            const ConvIn ci = {x + row0 * p.in.ld + d, p.in.ld, p.m.conv + seq * taps * channels + channel0 + d, channels, taps, pos0};
+    for (int c = 0; c < C; c++) {
+        const int d = lane + 32 * c;
+        if (d >= n) {
 #pragma unroll
-            for (int k = 0; k < 4; k++) {
-                cw[c][k] = d < n ? w[d * 4 + k] : 0.f;
-                in[c][k] = d < n && k < 3 ? ci.at(t0 - 3 + k) : 0.f;
-            }
+            for (int j = 0; j < BT; j++) out[j][c] = 0.f;
+            continue;
         }
-        for (int t = t0; t < t1; t++) {
-            float v[C];
+        const ConvIn ci = {x + row0 * p.in.ld + d, p.in.ld, taps ? p.m.conv + seq * taps * channels + channel0 + d : nullptr, channels, taps, pos0};
+        if (taps == 4) {
+            float in[BT + 3];
 #pragma unroll
-            for (int c = 0; c < C; c++) {
-                const int d = lane + 32 * c;
-                in[c][3] = d < n ? x[(row0 + t) * p.in.ld + d] : 0.f;
+            for (int k = 0; k < BT + 3; k++) in[k] = t0 - 3 + k < p.T ? ci.at(t0 - 3 + k) : 0.f;
+            const float4 cw = *reinterpret_cast<const float4 *>(w + d * 4);
+#pragma unroll
+            for (int j = 0; j < BT; j++) out[j][c] = fmaf(cw.w, in[j + 3], fmaf(cw.z, in[j + 2], fmaf(cw.y, in[j + 1], cw.x * in[j])));
+        } else {
+#pragma unroll
+            for (int j = 0; j < BT; j++) {
                 float s = 0.f;
-#pragma unroll
-                for (int k = 0; k < 4; k++) s = fmaf(cw[c][k], in[c][k], s);
-                v[c] = kq_silu(s);
-                in[c][0] = in[c][1], in[c][1] = in[c][2], in[c][2] = in[c][3];
-            }
-            f(t, v);
-        }
-        return;
-    }
-    for (int t = t0; t < t1; t++) {
-        float v[C];
-#pragma unroll
-        for (int c = 0; c < C; c++) {
-            const int d = lane + 32 * c;
-            float s = 0.f;
-            if (d < n) {
-                if (taps == 0) {
-                    s = x[(row0 + t) * p.in.ld + d];
-                } else {
-                    const ConvIn ci = {x + row0 * p.in.ld + d, p.in.ld, p.m.conv + seq * taps * channels + channel0 + d, channels, taps, pos0};
-                    for (int k = 0; k < taps; k++) s = fmaf(w[(int64_t)d * taps + k], ci.at(t - (taps - 1) + k), s);
+                if (t0 + j < p.T) {
+                    if (taps == 0) s = ci.at(t0 + j);
+                    for (int k = 0; k < taps; k++) s = fmaf(w[(int64_t)d * taps + k], ci.at(t0 + j - (taps - 1) + k), s);
                 }
+                out[j][c] = s;
             }
-            v[c] = kq_silu(s);
         }
-        f(t, v);
+#pragma unroll
+        for (int j = 0; j < BT; j++) out[j][c] = t0 + j < p.T ? kq_silu(out[j][c]) : 0.f;
     }
 }
 
-// grid (jobs / warps, runs of tokens, sequences); a job is a query / key head pair, 32 C channels of the values, or the decays and
-// write strengths of a head
-template <int C>
-__global__ void __launch_bounds__(TOK_NT) state_tokens_kernel(const __grid_constant__ TokParams p, int v_jobs) {
+// grid (heads / warps, then values, runs of blocks, sequences)
+template <int C, bool DELTA>
+__global__ void __launch_bounds__(TOK_NT) state_tokens_kernel(const __grid_constant__ TokParams p) {
     KQ_PDL_ENTER();
+    constexpr int DP = 32 * C, REC = rec_floats(DP, DELTA);
     const KqMatState &m = p.m;
-    const int lane = threadIdx.x & 31, t0 = blockIdx.y * RUN, t1 = min(p.T, t0 + RUN);
-    const int64_t seq = blockIdx.z, row0 = seq * p.T;
+    const int lane = threadIdx.x & 31, b0 = blockIdx.y * RUN, b1 = min(p.blocks, b0 + RUN);
+    const int64_t seq = blockIdx.z, nq = (int64_t)m.kv_heads * m.dim;
     const int pos0 = p.pos0_dev ? *p.pos0_dev : p.pos0;
-    int job = blockIdx.x * TOK_NW + (threadIdx.x >> 5);
-    const int64_t nq = (int64_t)m.kv_heads * m.dim;
-    if (job < m.kv_heads) { // q, then k and their product
-        const int64_t c0 = (int64_t)job * m.dim;
-        conv_run<C>(p, p.in.q + c0, m.taps ? m.conv_q + c0 * m.taps : nullptr, c0, m.dim, seq, t0, t1, pos0, lane, [&](int t, const float (&v)[C]) {
-            float ss = 0.f;
-#pragma unroll
-            for (int c = 0; c < C; c++) ss += v[c] * v[c];
-            const float sc = m.delta ? 1.0f / sqrtf(kq_warp_sum(ss) + 1e-6f) / sqrtf((float)m.dim) : 1.f;
-#pragma unroll
-            for (int c = 0; c < C; c++)
-                if (lane + 32 * c < m.dim) p.t.q[(row0 + t) * p.ldq + c0 + lane + 32 * c] = v[c] * sc;
-        });
-        conv_run<C>(p, p.in.k + c0, m.taps ? m.conv_k + c0 * m.taps : nullptr, nq + c0, m.dim, seq, t0, t1, pos0, lane, [&](int t, const float (&v)[C]) {
-            float ss = 0.f, qk = 0.f;
-#pragma unroll
-            for (int c = 0; c < C; c++) ss += v[c] * v[c];
-            const float sc = m.delta ? 1.0f / sqrtf(kq_warp_sum(ss) + 1e-6f) : 1.f;
-#pragma unroll
-            for (int c = 0; c < C; c++)
-                if (lane + 32 * c < m.dim) {
-                    const int64_t i = (row0 + t) * p.ldq + c0 + lane + 32 * c;
-                    if (m.delta) qk = fmaf(p.t.q[i], v[c] * sc, qk); // this lane's own store
-                    p.t.k[i] = v[c] * sc;
-                }
-            if (m.delta) {
-                qk = kq_warp_sum(qk);
-                const int rep = m.heads / m.kv_heads;
-                for (int h = lane; h < rep; h += 32) p.t.b[((row0 + t) * m.heads + job * rep + h) * 2 + 1] = qk;
-            }
-        });
+    if ((int)blockIdx.x >= p.head_ctas) { // a lane per value channel
+        const int64_t c0 = ((int64_t)(blockIdx.x - p.head_ctas) * TOK_NW + (threadIdx.x >> 5)) * 32, nv = (int64_t)m.heads * m.vdim;
+        if (c0 >= nv) return;
+        const int n = (int)min((int64_t)32, nv - c0);
+        for (int b = b0; b < b1; b++) {
+            float v[BT][1];
+            conv_block<1>(p, p.in.v + c0, m.taps ? m.conv_v + c0 * m.taps : nullptr, 2 * nq + c0, n, seq, b * BT, pos0, lane, v);
+            if (lane < n) *reinterpret_cast<float4 *>(p.val + (((seq * p.blocks + b) * nv) + c0 + lane) * BT) = make_float4(v[0][0], v[1][0], v[2][0], v[3][0]);
+        }
         return;
     }
-    job -= m.kv_heads;
-    if (job < v_jobs) {
-        const int64_t c0 = (int64_t)job * 32 * C, nv = (int64_t)m.heads * m.vdim;
-        const int n = (int)min((int64_t)32 * C, nv - c0);
-        conv_run<C>(p, p.in.v + c0, m.taps ? m.conv_v + c0 * m.taps : nullptr, 2 * nq + c0, n, seq, t0, t1, pos0, lane, [&](int t, const float (&v)[C]) {
-#pragma unroll
-            for (int c = 0; c < C; c++)
-                if (lane + 32 * c < n) p.t.v[(row0 + t) * p.ldv + c0 + lane + 32 * c] = v[c];
-        });
-        return;
-    }
-    job -= v_jobs;
-    if (!m.delta || job >= m.heads) return;
-    const float a = expf(m.a_log[job]);
-    const int64_t c0 = (int64_t)job * m.dim;
+    const int h = blockIdx.x * TOK_NW + (threadIdx.x >> 5);
+    if (h >= m.heads) return;
+    const int kh = h / (m.heads / m.kv_heads);
+    const int64_t cq = (int64_t)kh * m.dim, cg = (int64_t)h * m.dim;
     float bias[C];
 #pragma unroll
-    for (int c = 0; c < C; c++) bias[c] = lane + 32 * c < m.dim ? m.dt_bias[c0 + lane + 32 * c] : 0.f;
-    for (int t = t0; t < t1; t++) {
+    for (int c = 0; c < C; c++) bias[c] = DELTA && lane + 32 * c < m.dim ? m.dt_bias[cg + lane + 32 * c] : 0.f;
+    const float a = DELTA ? expf(m.a_log[h]) : 0.f, decay = DELTA ? 1.f : m.decay[h];
+    const float q_scale = DELTA ? 1.0f / sqrtf((float)m.dim) : 1.f;
+    for (int b = b0; b < b1; b++) {
+        const int t0 = b * BT;
+        float *rec = p.rec + ((seq * p.blocks + b) * m.heads + h) * (int64_t)REC;
+        float q[BT][C], k[BT][C], g[BT][C];
+        conv_block<C>(p, p.in.q + cq, m.taps ? m.conv_q + cq * m.taps : nullptr, cq, m.dim, seq, t0, pos0, lane, q);
+        conv_block<C>(p, p.in.k + cq, m.taps ? m.conv_k + cq * m.taps : nullptr, nq + cq, m.dim, seq, t0, pos0, lane, k);
+        if (DELTA) {
+            float ss[2 * BT];
 #pragma unroll
-        for (int c = 0; c < C; c++)
-            if (lane + 32 * c < m.dim)
-                p.t.g[(row0 + t) * p.ldg + c0 + lane + 32 * c] = expf(-a * kq_softplus(p.in.z[(row0 + t) * p.in.ldz + c0 + lane + 32 * c] + bias[c]));
-        if (lane == 0) p.t.b[((row0 + t) * m.heads + job) * 2] = kq_sigmoid(p.in.b[(row0 + t) * p.in.ld + job]);
+            for (int j = 0; j < BT; j++) {
+                ss[j] = ss[BT + j] = 0.f;
+#pragma unroll
+                for (int c = 0; c < C; c++) ss[j] = fmaf(q[j][c], q[j][c], ss[j]), ss[BT + j] = fmaf(k[j][c], k[j][c], ss[BT + j]);
+            }
+            spread_sum<2 * BT, 32>(ss, lane); // lane holds sum lane / 4
+            const float sc = 1.0f / sqrtf(ss[0] + 1e-6f);
+#pragma unroll
+            for (int j = 0; j < BT; j++) {
+                const float sq = __shfl_sync(0xffffffffu, sc, 4 * j) * q_scale, sk = __shfl_sync(0xffffffffu, sc, 4 * (BT + j));
+#pragma unroll
+                for (int c = 0; c < C; c++) {
+                    const int d = lane + 32 * c;
+                    q[j][c] *= sq, k[j][c] *= sk;
+                    g[j][c] = d < m.dim && t0 + j < p.T ? expf(-a * kq_softplus(p.in.z[(seq * p.T + t0 + j) * p.in.ldz + cg + d] + bias[c])) : 1.f;
+                }
+            }
+        } else {
+#pragma unroll
+            for (int j = 0; j < BT; j++)
+#pragma unroll
+                for (int c = 0; c < C; c++) g[j][c] = t0 + j < p.T ? decay : 1.f;
+        }
+        float dot[16]; // A21 A31 A32 A41 A42 A43, B11 B21 B22 B31 B32 B33 B41 B42 B43 B44
+#pragma unroll
+        for (int i = 0; i < 16; i++) dot[i] = 0.f;
+#pragma unroll
+        for (int c = 0; c < C; c++) {
+            const float g2 = g[1][c], g3 = g[2][c], g4 = g[3][c];
+            const float k1 = k[0][c], k2 = k[1][c], k3 = k[2][c], k4 = k[3][c], q1 = q[0][c], q2 = q[1][c], q3 = q[2][c], q4 = q[3][c];
+            const float p12 = g2 * k1, p13 = g3 * p12, p14 = g4 * p13, p23 = g3 * k2, p24 = g4 * p23, p34 = g4 * k3;
+            if (DELTA) {
+                dot[0] = fmaf(k2, p12, dot[0]), dot[1] = fmaf(k3, p13, dot[1]), dot[2] = fmaf(k3, p23, dot[2]);
+                dot[3] = fmaf(k4, p14, dot[3]), dot[4] = fmaf(k4, p24, dot[4]), dot[5] = fmaf(k4, p34, dot[5]);
+            }
+            dot[6] = fmaf(q1, k1, dot[6]);
+            dot[7] = fmaf(q2, p12, dot[7]), dot[8] = fmaf(q2, k2, dot[8]);
+            dot[9] = fmaf(q3, p13, dot[9]), dot[10] = fmaf(q3, p23, dot[10]), dot[11] = fmaf(q3, k3, dot[11]);
+            dot[12] = fmaf(q4, p14, dot[12]), dot[13] = fmaf(q4, p24, dot[13]), dot[14] = fmaf(q4, p34, dot[14]), dot[15] = fmaf(q4, k4, dot[15]);
+            const float G1 = g[0][c], G2 = G1 * g2, G3 = G2 * g3, G4 = G3 * g4;
+            float *o = rec + lane + 32 * c;
+            if (DELTA) {
+                o[0] = G1 * k1, o[DP] = G2 * k2, o[2 * DP] = G3 * k3, o[3 * DP] = G4 * k4;
+                o += 4 * DP;
+            }
+            o[0] = G1 * q1, o[DP] = G2 * q2, o[2 * DP] = G3 * q3, o[3 * DP] = G4 * q4;
+            o[4 * DP] = p14, o[5 * DP] = p24, o[6 * DP] = p34, o[7 * DP] = k4;
+            if (DELTA) o[8 * DP] = G4;
+        }
+        spread_sum<16, 32>(dot, lane); // lane holds sum lane / 2
+        float *sc = rec + REC - N_SCALAR;
+        if ((lane & 1) == 0) sc[lane / 2 < 6 ? 4 + lane / 2 : 6 + lane / 2] = dot[0];
+        if (DELTA && lane < BT)
+            sc[lane] = t0 + lane < p.T ? kq_sigmoid(p.in.b[(seq * p.T + t0 + lane) * p.in.ld + h]) : 0.f;
     }
 }
 
-// ---- token loop --------------------------------------------------------------------------------------
-template <int DP>
-struct Scan {
-    static constexpr int R4 = DP / 32;                 // groups of four key dimensions per lane
-    static constexpr int TT = DP <= 128 ? 16 : 8;      // tokens per tile
-    static constexpr int TILE = TT * (3 * DP + COLS + 2); // floats: q, k, g, values of the CTA's columns, (beta, q.k)
-    static constexpr int SMEM = (2 * TILE + TT * COLS) * 4;
-};
+// ---- the walk over the blocks -----------------------------------------------------------------------------
+constexpr int NC = 4, TB = 4; // columns per thread, blocks per tile
+constexpr int MAX_WARPS = 8;
+constexpr uint64_t LIMIT = 5 * KQ_WAIT_LIMIT_NS;
 struct ScanParams {
     KqMatState m;
     KqStateIn in;
-    KqStateTok t;
-    int32_t T, pos0, vec;
+    const float *rec, *val;
+    int32_t T, pos0, blocks;
     const int32_t *pos0_dev;
-    int64_t ldq, ldv, ldg, ldo;
+    int64_t ldo;
     float *o;
 };
+__host__ __device__ constexpr int scan_tile_floats(int dp, bool delta, int cols) { return TB * (rec_floats(dp, delta) + cols * BT); }
 
-__device__ __forceinline__ void cp4(uint32_t dst, const void *src) { asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(dst), "l"(src) : "memory"); }
-__device__ __forceinline__ void cp16(uint32_t dst, const void *src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); }
+__device__ __forceinline__ uint64_t pack2(float a, float b) {
+    uint64_t r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+    uint64_t r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ float add2(uint64_t a) {
+    float x, y;
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(x), "=f"(y) : "l"(a));
+    return x + y;
+}
 
 // the last `taps` inputs of every channel into the ring, shared out over all CTAs of the grid
 __device__ __forceinline__ void move_ring(const KqMatState &m, const KqStateIn &in, int64_t n_seq, int T, int pos0, int64_t id, int64_t n_threads) {
@@ -204,123 +260,177 @@ __device__ __forceinline__ void move_ring(const KqMatState &m, const KqStateIn &
     }
 }
 
-// grid (blocks of columns, heads, sequences)
-template <int DP, bool DELTA>
-__global__ void __launch_bounds__(SCAN_NT) state_scan_kernel(const __grid_constant__ ScanParams p) {
+// grid (blocks of columns, heads, sequences).  LPC lanes share NC columns, each with R groups of four key dimensions.
+template <int LPC, int R, bool DELTA>
+__global__ void __launch_bounds__(MAX_WARPS * 32) state_scan_kernel(const __grid_constant__ ScanParams p) {
+    constexpr int DP = LPC * R * 4, REC = rec_floats(DP, DELTA), GW = 32 / LPC, NV = DELTA ? 32 : 16, LEFT = NV > LPC ? NV / LPC : 1;
+    extern __shared__ __align__(128) float sm[];
+    __shared__ uint64_t full[2];
+    __shared__ __align__(16) float s_red[MAX_WARPS][2][GW][NV], s_u[MAX_WARPS][2][GW][NC * BT];
+    __shared__ int s_abort;
     KQ_PDL_ENTER();
-    using S = Scan<DP>;
-    constexpr int R4 = S::R4, TT = S::TT;
-    extern __shared__ __align__(16) float sm[];
     const KqMatState &m = p.m;
-    const int tid = threadIdx.x, part = tid & 7, col = tid >> 3;
-    const int h = blockIdx.y, kh = h / (m.heads / m.kv_heads), e0 = blockIdx.x * COLS, ne = min(COLS, m.vdim - e0);
-    const int64_t seq = blockIdx.z, row0 = seq * p.T;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, part = lane % LPC, grp = lane / LPC;
+    const int cols = (int)(blockDim.x / 32) * GW * NC; // of the CTA
+    const int h = blockIdx.y, e0 = blockIdx.x * cols, ne = min(cols, m.vdim - e0);
+    const int64_t seq = blockIdx.z;
     const int pos0 = p.pos0_dev ? *p.pos0_dev : p.pos0;
     if (m.taps)
-        move_ring(m, p.in, gridDim.z, p.T, pos0, ((seq * gridDim.y + h) * gridDim.x + blockIdx.x) * SCAN_NT + tid,
-                  (int64_t)gridDim.x * gridDim.y * gridDim.z * SCAN_NT);
-    for (int i = tid; i < 2 * S::TILE; i += SCAN_NT) sm[i] = 0.f; // what no copy reaches stays zero
+        move_ring(m, p.in, gridDim.z, p.T, pos0, ((seq * gridDim.y + h) * gridDim.x + blockIdx.x) * blockDim.x + tid,
+                  (int64_t)gridDim.x * gridDim.y * gridDim.z * blockDim.x);
+    const int tile_floats = scan_tile_floats(DP, DELTA, cols), tiles = (p.blocks + TB - 1) / TB;
+    float *so = sm + 2 * tile_floats; // [TB * BT][cols]
+    if (tid == 0) {
+        for (int i = 0; i < 2; i++) asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;" ::"r"((uint32_t)__cvta_generic_to_shared(&full[i])));
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        s_abort = 0;
+    }
     __syncthreads();
-    const float *q = p.t.q + row0 * p.ldq + (int64_t)kh * m.dim, *k = p.t.k + row0 * p.ldq + (int64_t)kh * m.dim,
-                *g = DELTA ? p.t.g + row0 * p.ldg + (int64_t)h * m.dim : nullptr, *v = p.t.v + row0 * p.ldv + (int64_t)h * m.vdim + e0,
-                *b = DELTA ? p.t.b + (row0 * m.heads + h) * 2 : nullptr;
-    auto request = [&](int tile) {
-        float *dst = sm + (tile & 1) * S::TILE;
-        const int t0 = tile * TT, n = min(TT, p.T - t0);
-        const uint32_t d0 = (uint32_t)__cvta_generic_to_shared(dst);
-        if (p.vec) {
-            const int n4 = m.dim / 4, v4 = ne / 4;
-            for (int i = tid; i < n * n4; i += SCAN_NT) {
-                const int t = i / n4, c = i % n4 * 4;
-                const uint32_t d = d0 + (t * DP + c) * 4;
-                cp16(d, q + (int64_t)(t0 + t) * p.ldq + c);
-                cp16(d + TT * DP * 4, k + (int64_t)(t0 + t) * p.ldq + c);
-                if (DELTA) cp16(d + 2 * TT * DP * 4, g + (int64_t)(t0 + t) * p.ldg + c);
-            }
-            for (int i = tid; i < n * v4; i += SCAN_NT) {
-                const int t = i / v4, c = i % v4 * 4;
-                cp16(d0 + (3 * TT * DP + t * COLS + c) * 4, v + (int64_t)(t0 + t) * p.ldv + c);
-            }
-        } else {
-            for (int i = tid; i < n * m.dim; i += SCAN_NT) {
-                const int t = i / m.dim, c = i % m.dim;
-                const uint32_t d = d0 + (t * DP + c) * 4;
-                cp4(d, q + (int64_t)(t0 + t) * p.ldq + c);
-                cp4(d + TT * DP * 4, k + (int64_t)(t0 + t) * p.ldq + c);
-                if (DELTA) cp4(d + 2 * TT * DP * 4, g + (int64_t)(t0 + t) * p.ldg + c);
-            }
-            for (int i = tid; i < n * ne; i += SCAN_NT) cp4(d0 + (3 * TT * DP + i / ne * COLS + i % ne) * 4, v + (int64_t)(t0 + i / ne) * p.ldv + i % ne);
+    auto request = [&](int tile) { // by one thread: the records and the values of this CTA's columns
+        const uint32_t bar = (uint32_t)__cvta_generic_to_shared(&full[tile & 1]);
+        float *dst = sm + (tile & 1) * tile_floats;
+        const int b0 = tile * TB, n = min(TB, p.blocks - b0);
+        asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(n * (REC + ne * BT) * 4) : "memory");
+        for (int i = 0; i < n; i++) {
+            const int64_t at = (seq * p.blocks + b0 + i) * m.heads + h;
+            asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
+                             (uint32_t)__cvta_generic_to_shared(dst + i * REC)),
+                         "l"(p.rec + at * REC), "r"(REC * 4), "r"(bar)
+                         : "memory");
+            asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
+                             (uint32_t)__cvta_generic_to_shared(dst + TB * REC + i * cols * BT)),
+                         "l"(p.val + (at * m.vdim + e0) * BT), "r"(ne * BT * 4), "r"(bar)
+                         : "memory");
         }
-        if (DELTA)
-            for (int i = tid; i < 2 * n; i += SCAN_NT) cp4(d0 + (TT * (3 * DP + COLS) + i) * 4, b + (int64_t)(t0 + i / 2) * 2 * m.heads + (i & 1));
-        asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    // the column's state; a lane holds the dimensions 4 (part + 8 i) .. + 3
-    const bool live = col < ne;
-    float *sp = m.s + ((seq * m.heads + h) * m.vdim + e0 + (live ? col : 0)) * DP;
-    float4 s[R4];
+    if (tid == 0) {
+        request(0);
+        if (tiles > 1) request(1);
+    }
+    const int c0 = (warp * GW + grp) * NC; // this lane group's columns inside the CTA
+    uint64_t s[NC][R][2];
+    const int64_t ld = kq_state_ld(m.dim);
+    float *sp = m.s + ((seq * m.heads + h) * m.vdim + e0 + c0) * ld + 4 * part;
 #pragma unroll
-    for (int i = 0; i < R4; i++) s[i] = pos0 > 0 ? *reinterpret_cast<const float4 *>(sp + 4 * (part + 8 * i)) : make_float4(0.f, 0.f, 0.f, 0.f);
-    const float decay = DELTA ? 1.f : m.decay[h];
-    const int n_tiles = (p.T + TT - 1) / TT;
-    float *so = sm + 2 * S::TILE;
-    request(0);
-    for (int tile = 0; tile < n_tiles; tile++) {
-        if (tile + 1 < n_tiles) {
-            request(tile + 1);
-            asm volatile("cp.async.wait_group 1;" ::: "memory");
-        } else {
-            asm volatile("cp.async.wait_group 0;" ::: "memory");
+    for (int c = 0; c < NC; c++)
+#pragma unroll
+        for (int i = 0; i < R; i++) {
+            const ulonglong2 v = pos0 > 0 && c0 + c < ne ? *reinterpret_cast<const ulonglong2 *>(sp + c * ld + 4 * LPC * i) : make_ulonglong2(0, 0);
+            s[c][i][0] = v.x, s[c][i][1] = v.y;
         }
-        __syncthreads();
-        const float *src = sm + (tile & 1) * S::TILE;
-        const int n = min(TT, p.T - tile * TT);
-        for (int t = 0; t < n; t++) {
-            const float4 *sq = reinterpret_cast<const float4 *>(src + t * DP), *sk = sq + TT * DP / 4, *sg = sk + TT * DP / 4;
-            const float vt = src[3 * TT * DP + t * COLS + col];
-            if (DELTA) {
-                const float beta = src[TT * (3 * DP + COLS) + 2 * t], qk = src[TT * (3 * DP + COLS) + 2 * t + 1];
-                float4 kk[R4], dk = make_float4(0.f, 0.f, 0.f, 0.f), dq = dk;
+    float d_full = 1.f, d_last = 1.f; // fixed decay over a block; the last one may hold fewer tokens
+    if (!DELTA)
+        for (int j = 0; j < BT; j++) {
+            d_full *= m.decay[h];
+            if ((p.blocks - 1) * BT + j < p.T) d_last *= m.decay[h];
+        }
+    for (int tile = 0; tile < tiles; tile++) {
+        if (!tc_wait((uint32_t)__cvta_generic_to_shared(&full[tile & 1]), (uint32_t)((tile >> 1) & 1), &s_abort, &g_state_error, 1, LIMIT)) {
+            s_abort = 1;
+        }
+        const float *src = sm + (tile & 1) * tile_floats;
+        const int nb = min(TB, p.blocks - tile * TB);
+        for (int b = 0; b < nb; b++) {
+            const float *rec = src + b * REC, *sc = rec + REC - N_SCALAR;
+            const ulonglong2 *vec = reinterpret_cast<const ulonglong2 *>(rec) + part; // vector v, group i: vec[v * DP / 4 + LPC * i]
+            float val[NV];
 #pragma unroll
-                for (int i = 0; i < R4; i++) {
-                    const float4 gg = sg[part + 8 * i], qq = sq[part + 8 * i];
-                    kk[i] = sk[part + 8 * i];
-                    s[i].x *= gg.x, s[i].y *= gg.y, s[i].z *= gg.z, s[i].w *= gg.w;
-                    dk.x = fmaf(s[i].x, kk[i].x, dk.x), dk.y = fmaf(s[i].y, kk[i].y, dk.y), dk.z = fmaf(s[i].z, kk[i].z, dk.z), dk.w = fmaf(s[i].w, kk[i].w, dk.w);
-                    dq.x = fmaf(s[i].x, qq.x, dq.x), dq.y = fmaf(s[i].y, qq.y, dq.y), dq.z = fmaf(s[i].z, qq.z, dq.z), dq.w = fmaf(s[i].w, qq.w, dq.w);
-                }
-                const float rk = sum8((dk.x + dk.y) + (dk.z + dk.w)), rq = sum8((dq.x + dq.y) + (dq.z + dq.w));
-                const float u = beta * (vt - rk);
+            for (int v = 0; v < NV / NC; v++) { // products with the state: [decayed k,] decayed q of the four tokens
+                uint64_t acc[NC];
 #pragma unroll
-                for (int i = 0; i < R4; i++) {
-                    s[i].x = fmaf(kk[i].x, u, s[i].x), s[i].y = fmaf(kk[i].y, u, s[i].y);
-                    s[i].z = fmaf(kk[i].z, u, s[i].z), s[i].w = fmaf(kk[i].w, u, s[i].w);
-                }
-                if (part == 0) so[t * COLS + col] = fmaf(qk, u, rq);
-            } else {
-                float4 dq = make_float4(0.f, 0.f, 0.f, 0.f);
+                for (int i = 0; i < R; i++) {
+                    const ulonglong2 x = vec[v * DP / 4 + LPC * i];
 #pragma unroll
-                for (int i = 0; i < R4; i++) {
-                    const float4 kk = sk[part + 8 * i], qq = sq[part + 8 * i];
-                    s[i].x = fmaf(kk.x, vt, decay * s[i].x), s[i].y = fmaf(kk.y, vt, decay * s[i].y);
-                    s[i].z = fmaf(kk.z, vt, decay * s[i].z), s[i].w = fmaf(kk.w, vt, decay * s[i].w);
-                    dq.x = fmaf(s[i].x, qq.x, dq.x), dq.y = fmaf(s[i].y, qq.y, dq.y), dq.z = fmaf(s[i].z, qq.z, dq.z), dq.w = fmaf(s[i].w, qq.w, dq.w);
+                    for (int c = 0; c < NC; c++) acc[c] = fma2(s[c][i][1], x.y, i == 0 ? mul2(s[c][i][0], x.x) : fma2(s[c][i][0], x.x, acc[c]));
                 }
-                const float rq = sum8((dq.x + dq.y) + (dq.z + dq.w));
-                if (part == 0) so[t * COLS + col] = rq;
+#pragma unroll
+                for (int c = 0; c < NC; c++) val[v / BT * 16 + c * BT + v % BT] = add2(acc[c]);
+            }
+            spread_sum<NV, LPC>(val, lane);
+            float *red = s_red[warp][b & 1][grp], *us = s_u[warp][b & 1][grp];
+            if (NV >= LPC) {
+#pragma unroll
+                for (int i = 0; i < LEFT; i++) red[part * LEFT + i] = val[i];
+            } else if (part % (LPC / NV) == 0) {
+                red[part / (LPC / NV)] = val[0];
+            }
+            __syncwarp();
+            { // every lane solves one of the group's columns; the first four lanes pass theirs on
+                const int c = part & (NC - 1);
+                const float4 vt = *reinterpret_cast<const float4 *>(src + TB * REC + (b * cols + c0 + c) * BT);
+                const float4 dq = *reinterpret_cast<const float4 *>(red + (DELTA ? 16 : 0) + c * BT);
+                float4 u = vt;
+                if (DELTA) {
+                    const float4 dk = *reinterpret_cast<const float4 *>(red + c * BT), be = *reinterpret_cast<const float4 *>(sc),
+                                 A0 = *reinterpret_cast<const float4 *>(sc + 4), A1 = *reinterpret_cast<const float4 *>(sc + 8);
+                    u.x = be.x * (vt.x - dk.x);
+                    u.y = be.y * (vt.y - dk.y - A0.x * u.x);
+                    u.z = be.z * (vt.z - dk.z - A0.y * u.x - A0.z * u.y);
+                    u.w = be.w * (vt.w - dk.w - A0.w * u.x - A1.x * u.y - A1.y * u.z);
+                }
+                if (part < NC) {
+                    *reinterpret_cast<float4 *>(us + c * BT) = u;
+                    const float4 B0 = *reinterpret_cast<const float4 *>(sc + 12), B1 = *reinterpret_cast<const float4 *>(sc + 16);
+                    const float2 B2 = *reinterpret_cast<const float2 *>(sc + 20);
+                    float *o = so + b * BT * cols + c0 + c;
+                    o[0] = fmaf(B0.x, u.x, dq.x);
+                    o[cols] = fmaf(B0.z, u.y, fmaf(B0.y, u.x, dq.y));
+                    o[2 * cols] = fmaf(B1.y, u.z, fmaf(B1.x, u.y, fmaf(B0.w, u.x, dq.z)));
+                    o[3 * cols] = fmaf(B2.y, u.w, fmaf(B2.x, u.z, fmaf(B1.w, u.y, fmaf(B1.z, u.x, dq.w))));
+                }
+            }
+            __syncwarp();
+            constexpr int KH = DELTA ? 8 : 4; // first of the vectors that are written
+#pragma unroll
+            for (int i = 0; i < R; i++) {
+                ulonglong2 gg;
+                if (DELTA) gg = vec[12 * DP / 4 + LPC * i];
+                else gg.x = gg.y = tile * TB + b == p.blocks - 1 ? pack2(d_last, d_last) : pack2(d_full, d_full);
+#pragma unroll
+                for (int c = 0; c < NC; c++) s[c][i][0] = mul2(s[c][i][0], gg.x), s[c][i][1] = mul2(s[c][i][1], gg.y);
+            }
+#pragma unroll
+            for (int c = 0; c < NC; c++) {
+                const float4 u = *reinterpret_cast<const float4 *>(us + c * BT);
+                const float uv[BT] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+                for (int j = 0; j < BT; j++) {
+                    const uint64_t uu = pack2(uv[j], uv[j]);
+#pragma unroll
+                    for (int i = 0; i < R; i++) {
+                        const ulonglong2 kk = vec[(KH + j) * DP / 4 + LPC * i];
+                        s[c][i][0] = fma2(kk.x, uu, s[c][i][0]), s[c][i][1] = fma2(kk.y, uu, s[c][i][1]);
+                    }
+                }
             }
         }
         __syncthreads(); // the tile's buffer is free, its outputs are complete
-        for (int i = tid; i < n * COLS; i += SCAN_NT)
-            if (i % COLS < ne) p.o[(row0 + tile * TT + i / COLS) * p.ldo + (int64_t)h * m.vdim + e0 + i % COLS] = so[i];
+        if (s_abort) break;
+        if (tid == 0 && tile + 2 < tiles) request(tile + 2);
+        const int n = min(TB * BT, p.T - tile * TB * BT);
+        for (int i = tid; i < n * cols; i += blockDim.x)
+            if (i % cols < ne) p.o[(seq * p.T + tile * TB * BT + i / cols) * p.ldo + (int64_t)h * m.vdim + e0 + i % cols] = so[i];
+        __syncthreads();
     }
-    if (live) {
+    if (s_abort) { // copies in flight must land before the CTA goes away
+        if (tid == 0)
+            for (int i = 0; i < 2; i++) {
+                kq_mbar_wait((uint32_t)__cvta_generic_to_shared(&full[i]), 0u, KQ_WAIT_LIMIT_NS);
+                kq_mbar_wait((uint32_t)__cvta_generic_to_shared(&full[i]), 1u, KQ_WAIT_LIMIT_NS);
+            }
+        __syncthreads();
+        return;
+    }
 #pragma unroll
-        for (int i = 0; i < R4; i++) *reinterpret_cast<float4 *>(sp + 4 * (part + 8 * i)) = s[i];
-    }
+    for (int c = 0; c < NC; c++)
+#pragma unroll
+        for (int i = 0; i < R; i++)
+            if (c0 + c < ne) *reinterpret_cast<ulonglong2 *>(sp + c * ld + 4 * LPC * i) = make_ulonglong2(s[c][i][0], s[c][i][1]);
 }
 
 // ---- output of a prompt --------------------------------------------------------------------------------
+// a warp per row and head; VEC: four elements per access
+template <bool VEC>
 __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float *o, int64_t ldo, const float *gate, int64_t ldg, const float *w, float eps, int64_t rows,
                                                              int heads, int vdim, float *out32, int64_t ld32, uint16_t *out16, int64_t ld16) {
     KQ_PDL_ENTER();
@@ -328,30 +438,49 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float *o, int
     const int h = (int)(id % heads), lane = threadIdx.x & 31;
     if (r >= rows) return;
     const float *x = o + r * ldo + (int64_t)h * vdim, *gt = gate + r * ldg + (int64_t)h * vdim;
-    constexpr int KEEP = 8;
-    float v[KEEP], ss = 0.f;
+    float ss = 0.f;
+    if (VEC) {
+        constexpr int KEEP = 2;
+        float4 v[KEEP], g[KEEP];
+        const int n = vdim / 4;
 #pragma unroll
-    for (int i = 0; i < KEEP; i++) {
-        v[i] = lane + 32 * i < vdim ? x[lane + 32 * i] : 0.f;
-        ss += v[i] * v[i];
+        for (int i = 0; i < KEEP; i++) {
+            v[i] = g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (lane + 32 * i < n) v[i] = reinterpret_cast<const float4 *>(x)[lane + 32 * i], g[i] = reinterpret_cast<const float4 *>(gt)[lane + 32 * i];
+            ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+        }
+        for (int d = lane + 32 * KEEP; d < n; d += 32) {
+            const float4 a = reinterpret_cast<const float4 *>(x)[d];
+            ss += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+        }
+        const float sc = 1.0f / sqrtf(kq_warp_sum(ss) / (float)vdim + eps);
+        auto emit = [&](int d, float4 a, const float4 &b) {
+            const float4 wv = reinterpret_cast<const float4 *>(w)[d];
+            a.x *= sc * wv.x * kq_sigmoid(b.x), a.y *= sc * wv.y * kq_sigmoid(b.y), a.z *= sc * wv.z * kq_sigmoid(b.z), a.w *= sc * wv.w * kq_sigmoid(b.w);
+            if (out32) *reinterpret_cast<float4 *>(out32 + r * ld32 + (int64_t)h * vdim + 4 * d) = a;
+            if (out16)
+                *reinterpret_cast<uint2 *>(out16 + r * ld16 + (int64_t)h * vdim + 4 * d) =
+                    make_uint2((uint32_t)kq_f2bf(a.x) | ((uint32_t)kq_f2bf(a.y) << 16), (uint32_t)kq_f2bf(a.z) | ((uint32_t)kq_f2bf(a.w) << 16));
+        };
+#pragma unroll
+        for (int i = 0; i < KEEP; i++)
+            if (lane + 32 * i < n) emit(lane + 32 * i, v[i], g[i]);
+        for (int d = lane + 32 * KEEP; d < n; d += 32) emit(d, reinterpret_cast<const float4 *>(x)[d], reinterpret_cast<const float4 *>(gt)[d]);
+    } else {
+        for (int d = lane; d < vdim; d += 32) ss += x[d] * x[d];
+        const float sc = 1.0f / sqrtf(kq_warp_sum(ss) / (float)vdim + eps);
+        for (int d = lane; d < vdim; d += 32) {
+            const float a = x[d] * sc * w[d] * kq_sigmoid(gt[d]);
+            if (out32) out32[r * ld32 + (int64_t)h * vdim + d] = a;
+            if (out16) out16[r * ld16 + (int64_t)h * vdim + d] = kq_f2bf(a);
+        }
     }
-    for (int d = lane + 32 * KEEP; d < vdim; d += 32) ss += x[d] * x[d];
-    const float sc = 1.0f / sqrtf(kq_warp_sum(ss) / (float)vdim + eps);
-    auto emit = [&](int d, float a) {
-        a *= sc * w[d] * kq_sigmoid(gt[d]);
-        if (out32) out32[r * ld32 + (int64_t)h * vdim + d] = a;
-        if (out16) out16[r * ld16 + (int64_t)h * vdim + d] = kq_f2bf(a);
-    };
-#pragma unroll
-    for (int i = 0; i < KEEP; i++)
-        if (lane + 32 * i < vdim) emit(lane + 32 * i, v[i]);
-    for (int d = lane + 32 * KEEP; d < vdim; d += 32) emit(d, x[d]);
     if (out16 && h == heads - 1)
         for (int64_t d = (int64_t)heads * vdim + lane; d < ld16; d += 32) out16[r * ld16 + d] = 0;
 }
 
 // ---- one token -----------------------------------------------------------------------------------------
-constexpr int STEP_NT = 256, STEP_NW = STEP_NT / 32;
+constexpr int STEP_NT = 512, STEP_NW = STEP_NT / 32;
 struct StepParams {
     KqMatState m;
     KqStateIn in;
@@ -362,24 +491,36 @@ struct StepParams {
     int64_t ldz;
 };
 
-// y[i] = W[i] . x for n rows of bf16 weights (16-byte chunks of padded rows), x in shared memory; groups of lanes share rows
-__device__ __forceinline__ void small_matvec(const uint16_t *W, int64_t ldw, int n, int K, const float *x, float *y, int warp, int lane) {
-    const int nck = (K + 7) / 8;
-    int w = 1; // lanes per row
-    while (w < nck && w < 32) w *= 2;
-    const int per = 32 / w, sub = lane / w, l = lane % w;
-    for (int r0 = warp * per; r0 < n; r0 += STEP_NW * per) {
-        const int r = r0 + sub;
-        float s = 0.f;
+// y[i] = W[i] . x for n rows of bf16 weights (16-byte chunks of padded rows), x in shared memory; groups of lanes share rows.  The
+// first chunk of the first rows is requested ahead.
+struct SmallMatvec {
+    static constexpr int PRE = 4;
+    const uint16_t *W;
+    int64_t ldw;
+    int n, nck, w, l, r0, step;
+    uint4 q[PRE];
+    __device__ __forceinline__ SmallMatvec(const uint16_t *W_, int64_t ldw_, int n_, int K, int warp, int lane) : W(W_), ldw(ldw_), n(n_), nck((K + 7) / 8) {
+        w = 1; // lanes per row
+        while (w < nck && w < 32) w *= 2;
+        l = lane % w, r0 = warp * (32 / w) + lane / w, step = STEP_NW * (32 / w);
+#pragma unroll
+        for (int u = 0; u < PRE; u++) q[u] = r0 + u * step < n && l < nck ? kq_ld_stream(W + (int64_t)(r0 + u * step) * ldw + 8 * l) : make_uint4(0, 0, 0, 0);
+    }
+    __device__ __forceinline__ float dot(const uint4 &v, const float *x, int c, float s) const {
+        return kq_dot8(v, *reinterpret_cast<const float4 *>(x + 8 * c), *reinterpret_cast<const float4 *>(x + 8 * c + 4), s);
+    }
+    __device__ __forceinline__ void row(int r, float s, int c0, const float *x, float *y) const {
         if (r < n)
-            for (int c = l; c < nck; c += w) {
-                const uint4 q = *reinterpret_cast<const uint4 *>(W + (int64_t)r * ldw + 8 * c);
-                s = kq_dot8(q, *reinterpret_cast<const float4 *>(x + 8 * c), *reinterpret_cast<const float4 *>(x + 8 * c + 4), s);
-            }
+            for (int c = c0; c < nck; c += w) s = dot(kq_ld_stream(W + (int64_t)r * ldw + 8 * c), x, c, s);
         for (int o = w / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
         if (r < n && l == 0) y[r] = s;
     }
-}
+    __device__ __forceinline__ void run(const float *x, float *y) const {
+#pragma unroll
+        for (int u = 0; u < PRE; u++) row(r0 + u * step, l < nck ? dot(q[u], x, l, 0.f) : 0.f, l + w, x, y);
+        for (int t = PRE * step; t < n; t += step) row(r0 + t, 0.f, l, x, y); // whole warps: n is the same for all
+    }
+};
 // SiLU of the convolution of one head's channels; the CTA that owns them (`owns`) also stores the new input.  The slot of the
 // current position is read by nobody in this launch.
 __device__ __forceinline__ void conv_step(const KqMatState &m, const float *x, const float *w, float *ring, int64_t channels, int n, int pos, bool owns, float *out) {
@@ -398,7 +539,7 @@ __device__ __forceinline__ void conv_step(const KqMatState &m, const float *x, c
 // grid (heads, sequences)
 template <int DP, bool DELTA>
 __global__ void __launch_bounds__(STEP_NT) state_step_kernel(const __grid_constant__ StepParams p) {
-    constexpr int R4 = DP / 32, PC = STEP_NT / 8; // columns of a pass
+    constexpr int R4 = DP / 32, PC = STEP_NT / 8, KEEP = 2; // PC: columns of a pass
     extern __shared__ __align__(16) float sm[];
     __shared__ float s_red[4];
     KQ_PDL_TRIGGER();
@@ -408,22 +549,25 @@ __global__ void __launch_bounds__(STEP_NT) state_step_kernel(const __grid_consta
     const int64_t seq = blockIdx.y;
     const int ra = (p.x.a_rank + 7) / 8 * 8, rg = (p.x.g_rank + 7) / 8 * 8, vp = (m.vdim + 3) / 4 * 4;
     float *sq = sm, *sk = sq + DP, *sg = sk + DP, *sv = sg + DP, *sgate = sv + vp, *so = sgate + vp, *sa = so + vp, *sg1 = sa + ra;
-    if (DELTA) { // the low-rank matrices come towards this SM while the predecessor finishes
-        const int64_t lda = kq_bf16_ld(p.x.a_rank), ldg = kq_bf16_ld(p.x.g_rank);
-        for (int i = tid * 128; i < m.dim * lda * 2; i += STEP_NT * 128)
-            asm volatile("prefetch.global.L2 [%0];" ::"l"((const uint8_t *)(p.x.a2 + (int64_t)h * m.dim * lda) + i));
-        for (int i = tid * 128; i < m.vdim * ldg * 2; i += STEP_NT * 128)
-            asm volatile("prefetch.global.L2 [%0];" ::"l"((const uint8_t *)(p.x.g2 + (int64_t)h * m.vdim * ldg) + i));
-    }
-    {
-        const uint8_t *s0 = (const uint8_t *)(m.s + (seq * m.heads + h) * (int64_t)m.vdim * DP);
-        for (int i = tid * 128; i < m.vdim * DP * 4; i += STEP_NT * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(s0 + i));
-    }
+    const int64_t lda = kq_bf16_ld(p.x.a_rank), ldg = kq_bf16_ld(p.x.g_rank);
+    const SmallMatvec wa(p.x.a2 + (int64_t)h * m.dim * lda, lda, DELTA ? m.dim : 0, p.x.a_rank, warp, lane);
+    const SmallMatvec wg(p.x.g2 + (int64_t)h * m.vdim * ldg, ldg, DELTA ? m.vdim : 0, p.x.g_rank, warp, lane);
+    float *base = m.s + (seq * m.heads + h) * (int64_t)m.vdim * DP;
+    for (int i = tid * 32; i < m.vdim * DP; i += STEP_NT * 32) asm volatile("prefetch.global.L2 [%0];" ::"l"(base + i));
     KQ_PDL_WAIT();
     const int pos = p.pos_dev ? *p.pos_dev : p.pos;
     const int64_t channels = kq_state_channels(m), nq = (int64_t)m.kv_heads * m.dim, cq = (int64_t)kh * m.dim, cv = (int64_t)h * m.vdim;
     float *ring = m.taps ? m.conv + seq * m.taps * channels : nullptr;
     const bool owns = h % rep == 0;
+    // the first columns of the state come while the vectors are made
+    float4 first[KEEP][R4];
+    auto load = [&](int e, float4 (&s)[R4]) {
+#pragma unroll
+        for (int i = 0; i < R4; i++)
+            s[i] = pos > 0 && e < m.vdim ? *reinterpret_cast<const float4 *>(base + (int64_t)e * DP + 4 * (part + 8 * i)) : make_float4(0.f, 0.f, 0.f, 0.f);
+    };
+#pragma unroll
+    for (int u = 0; u < KEEP; u++) load(u * PC + col, first[u]);
     conv_step(m, p.in.q + seq * p.in.ld + cq, m.conv_q + cq * m.taps, ring + cq, channels, m.dim, pos, owns, sq);
     conv_step(m, p.in.k + seq * p.in.ld + cq, m.conv_k + cq * m.taps, ring + nq + cq, channels, m.dim, pos, owns, sk);
     conv_step(m, p.in.v + seq * p.in.ld + cv, m.conv_v + cv * m.taps, ring + 2 * nq + cv, channels, m.vdim, pos, true, sv);
@@ -440,8 +584,8 @@ __global__ void __launch_bounds__(STEP_NT) state_step_kernel(const __grid_consta
             ss = 1.0f / sqrtf(kq_warp_sum(ss) + 1e-6f);
             if (lane == 0) s_red[warp] = warp ? ss : ss / sqrtf((float)m.dim);
         }
-        small_matvec(p.x.a2 + (int64_t)h * m.dim * kq_bf16_ld(p.x.a_rank), kq_bf16_ld(p.x.a_rank), m.dim, p.x.a_rank, sa, sg, warp, lane);
-        small_matvec(p.x.g2 + (int64_t)h * m.vdim * kq_bf16_ld(p.x.g_rank), kq_bf16_ld(p.x.g_rank), m.vdim, p.x.g_rank, sg1, sgate, warp, lane);
+        wa.run(sa, sg);
+        wg.run(sg1, sgate);
         __syncthreads();
         const float a = expf(m.a_log[h]);
         for (int d = tid; d < m.dim; d += STEP_NT) {
@@ -459,16 +603,10 @@ __global__ void __launch_bounds__(STEP_NT) state_step_kernel(const __grid_consta
         if (DELTA) gg[i] = reinterpret_cast<const float4 *>(sg)[part + 8 * i];
     }
     const float beta = DELTA ? kq_sigmoid(p.in.b[seq * p.in.ld + h]) : 0.f, decay = DELTA ? 1.f : m.decay[h];
-    float *base = m.s + (seq * m.heads + h) * (int64_t)m.vdim * DP;
-#pragma unroll 2
-    for (int e0 = 0; e0 < m.vdim; e0 += PC) {
-        const int e = e0 + col;
+    auto column = [&](int e, float4 (&s)[R4]) {
         const bool live = e < m.vdim;
         float *sp = base + (int64_t)(live ? e : 0) * DP;
         const float vt = live ? sv[e] : 0.f;
-        float4 s[R4];
-#pragma unroll
-        for (int i = 0; i < R4; i++) s[i] = pos > 0 ? *reinterpret_cast<const float4 *>(sp + 4 * (part + 8 * i)) : make_float4(0.f, 0.f, 0.f, 0.f);
         float w = vt;
         if (DELTA) {
             float rk = 0.f;
@@ -489,6 +627,14 @@ __global__ void __launch_bounds__(STEP_NT) state_step_kernel(const __grid_consta
         }
         rq = sum8(rq);
         if (live && part == 0) so[e] = rq;
+    };
+#pragma unroll
+    for (int u = 0; u < KEEP; u++)
+        if (u * PC < m.vdim) column(u * PC + col, first[u]);
+    for (int e0 = KEEP * PC; e0 < m.vdim; e0 += PC) {
+        float4 s[R4];
+        load(e0 + col, s);
+        column(e0 + col, s);
     }
     __syncthreads();
     float *z = p.z + seq * p.ldz + cv;
@@ -530,16 +676,34 @@ b200_status check_state(const KqMatState &m, int n_seq, int T) {
     return B200_OK;
 }
 
-template <int DP, bool DELTA>
+template <int LPC, int R, bool DELTA>
 b200_status launch_scan(const ScanParams &p, int n_seq, cudaStream_t st) {
-    static bool attr[16];
+    constexpr int DP = LPC * R * 4, per_warp = 32 / LPC * NC;
+    // warps per CTA: as few as possible on the busiest SM, then as many as possible in a CTA, which share a record
+    int warps = 1;
+    int64_t best = INT64_MAX;
+    for (int w = 1; w <= MAX_WARPS; w++) {
+        const int64_t ctas = kq_div_up(p.m.vdim, w * per_warp) * p.m.heads * n_seq, load = kq_div_up(ctas, kq_sm_count()) * w;
+        if (load <= best && (w == 1 || (w - 1) * per_warp < p.m.vdim)) best = load, warps = w;
+    }
+    const int cols = warps * per_warp;
+    const size_t smem = (size_t)(2 * scan_tile_floats(DP, DELTA, cols) + TB * BT * cols) * 4;
+    static size_t attr[16];
     int dev = 0;
     KQ_CUDA(cudaGetDevice(&dev));
-    if (dev < 0 || dev >= 16 || !attr[dev]) {
-        KQ_CUDA(cudaFuncSetAttribute(state_scan_kernel<DP, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, Scan<DP>::SMEM));
-        if (dev >= 0 && dev < 16) attr[dev] = true;
+    if (dev < 0 || dev >= 16 || attr[dev] < smem) {
+        KQ_CUDA(cudaFuncSetAttribute(state_scan_kernel<LPC, R, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        if (dev >= 0 && dev < 16) attr[dev] = smem;
     }
-    kq_launch(state_scan_kernel<DP, DELTA>, dim3((unsigned)kq_div_up(p.m.vdim, COLS), (unsigned)p.m.heads, (unsigned)n_seq), SCAN_NT, Scan<DP>::SMEM, st, p);
+    kq_launch(state_scan_kernel<LPC, R, DELTA>, dim3((unsigned)kq_div_up(p.m.vdim, cols), (unsigned)p.m.heads, (unsigned)n_seq), warps * 32, smem, st, p);
+    KQ_COUNT_LAUNCH();
+    KQ_LAUNCH_CHECK();
+    return B200_OK;
+}
+template <int C, bool DELTA>
+b200_status launch_tokens(const TokParams &p, int n_seq, cudaStream_t st) {
+    const dim3 grid((unsigned)(p.head_ctas + kq_div_up((int64_t)p.m.heads * p.m.vdim, 32 * TOK_NW)), (unsigned)kq_div_up(p.blocks, RUN), (unsigned)n_seq);
+    kq_launch(state_tokens_kernel<C, DELTA>, grid, TOK_NT, 0, st, p);
     KQ_COUNT_LAUNCH();
     KQ_LAUNCH_CHECK();
     return B200_OK;
@@ -558,52 +722,52 @@ b200_status launch_step(const StepParams &p, int n_seq, size_t smem, cudaStream_
     KQ_LAUNCH_CHECK();
     return B200_OK;
 }
-#define BY_DIM(FN, ...)                                                                              \
-    switch (kq_state_ld(m.dim)) {                                                                    \
-    case 32: return m.delta ? FN<32, true>(__VA_ARGS__) : FN<32, false>(__VA_ARGS__);                \
-    case 64: return m.delta ? FN<64, true>(__VA_ARGS__) : FN<64, false>(__VA_ARGS__);                \
-    case 96: return m.delta ? FN<96, true>(__VA_ARGS__) : FN<96, false>(__VA_ARGS__);                \
-    case 128: return m.delta ? FN<128, true>(__VA_ARGS__) : FN<128, false>(__VA_ARGS__);             \
-    case 192: return m.delta ? FN<192, true>(__VA_ARGS__) : FN<192, false>(__VA_ARGS__);             \
-    default: return m.delta ? FN<256, true>(__VA_ARGS__) : FN<256, false>(__VA_ARGS__);              \
+#define BY_DIM(FN, ARGS32, ARGS64, ARGS128, ARGS256, ...)                                                          \
+    switch (kq_state_ld(m.dim)) {                                                                                  \
+    case 32: return m.delta ? FN<ARGS32, true>(__VA_ARGS__) : FN<ARGS32, false>(__VA_ARGS__);                      \
+    case 64: return m.delta ? FN<ARGS64, true>(__VA_ARGS__) : FN<ARGS64, false>(__VA_ARGS__);                      \
+    case 128: return m.delta ? FN<ARGS128, true>(__VA_ARGS__) : FN<ARGS128, false>(__VA_ARGS__);                   \
+    default: return m.delta ? FN<ARGS256, true>(__VA_ARGS__) : FN<ARGS256, false>(__VA_ARGS__);                    \
     }
+#define TWO(a, b) a, b
 
 } // namespace
+
+int kq_state_error_fetch() {
+    int v = 0, zero = 0;
+    if (cudaMemcpyFromSymbol(&v, g_state_error, sizeof(int)) != cudaSuccess) return -1;
+    if (v) cudaMemcpyToSymbol(g_state_error, &zero, sizeof(int));
+    return v;
+}
+
+int64_t kq_state_rec_floats(const KqMatState &m) { return (int64_t)m.heads * rec_floats(kq_state_ld(m.dim), m.delta != 0); }
+int64_t kq_state_val_floats(const KqMatState &m) { return (int64_t)m.heads * m.vdim * BT; }
 
 b200_status kq_state_tokens(const KqMatState &m, const KqStateIn &in, const KqStateTok &t, int n_seq, int T, const int32_t *pos0_dev, int pos0,
                             cudaStream_t st) {
     KQ_TRY(check_state(m, n_seq, T));
+    KQ_REQUIRE((((uintptr_t)t.rec | (uintptr_t)t.val) & 15) == 0, "matrix state: records");
     TokParams p;
-    p.m = m, p.in = in, p.t = t, p.T = T, p.pos0 = pos0, p.pos0_dev = pos0_dev;
-    p.ldq = kq_f32_ld((int64_t)m.kv_heads * m.dim), p.ldv = kq_f32_ld((int64_t)m.heads * m.vdim), p.ldg = kq_f32_ld((int64_t)m.heads * m.dim);
-    const int c = (int)kq_div_up(m.dim, 32), C = c <= 1 ? 1 : c <= 2 ? 2 : c <= 4 ? 4 : 8;
-    const int v_jobs = (int)kq_div_up((int64_t)m.heads * m.vdim, 32 * C);
-    const dim3 grid((unsigned)kq_div_up(m.kv_heads + v_jobs + (m.delta ? m.heads : 0), TOK_NW), (unsigned)kq_div_up(T, RUN), (unsigned)n_seq);
-    if (C == 1) kq_launch(state_tokens_kernel<1>, grid, TOK_NT, 0, st, p, v_jobs);
-    else if (C == 2) kq_launch(state_tokens_kernel<2>, grid, TOK_NT, 0, st, p, v_jobs);
-    else if (C == 4) kq_launch(state_tokens_kernel<4>, grid, TOK_NT, 0, st, p, v_jobs);
-    else kq_launch(state_tokens_kernel<8>, grid, TOK_NT, 0, st, p, v_jobs);
-    KQ_COUNT_LAUNCH();
-    KQ_LAUNCH_CHECK();
-    return B200_OK;
+    p.m = m, p.in = in, p.rec = t.rec, p.val = t.val, p.T = T, p.pos0 = pos0, p.pos0_dev = pos0_dev;
+    p.blocks = (int)kq_div_up(T, BT), p.head_ctas = (int)kq_div_up(m.heads, TOK_NW);
+    BY_DIM(launch_tokens, 1, 2, 4, 8, p, n_seq, st)
 }
 
 b200_status kq_state_scan(const KqMatState &m, const KqStateIn &in, const KqStateTok &t, int n_seq, int T, const int32_t *pos0_dev, int pos0,
                           float *o, int64_t ldo, cudaStream_t st) {
     KQ_TRY(check_state(m, n_seq, T));
     ScanParams p;
-    p.m = m, p.in = in, p.t = t, p.T = T, p.pos0 = pos0, p.pos0_dev = pos0_dev, p.o = o, p.ldo = ldo;
-    p.ldq = kq_f32_ld((int64_t)m.kv_heads * m.dim), p.ldv = kq_f32_ld((int64_t)m.heads * m.vdim), p.ldg = kq_f32_ld((int64_t)m.heads * m.dim);
-    const uintptr_t al = (uintptr_t)t.q | (uintptr_t)t.k | (uintptr_t)t.v | (uintptr_t)t.g;
-    p.vec = m.dim % 4 == 0 && m.vdim % 4 == 0 && (al & 15) == 0;
-    BY_DIM(launch_scan, p, n_seq, st)
+    p.m = m, p.in = in, p.rec = t.rec, p.val = t.val, p.T = T, p.pos0 = pos0, p.pos0_dev = pos0_dev, p.blocks = (int)kq_div_up(T, BT), p.o = o, p.ldo = ldo;
+    BY_DIM(launch_scan, TWO(8, 1), TWO(16, 1), TWO(32, 1), TWO(32, 2), p, n_seq, st)
 }
 
 b200_status kq_head_norm_gate(const float *o, int64_t ldo, const float *gate, int64_t ldg, const float *norm_w, float eps, int64_t rows, int heads,
                               int vdim, float *out32, int64_t ld32, uint16_t *out16, int64_t ld16, cudaStream_t st) {
     KQ_REQUIRE(o && gate && norm_w && rows >= 1 && heads >= 1 && vdim >= 1, "head_norm_gate: bad call");
-    kq_launch(head_norm_gate_kernel, (unsigned)kq_div_up(rows * heads, 8), 256, 0, st, o, ldo, gate, ldg, norm_w, eps, rows, heads, vdim, out32, ld32, out16,
-              ld16);
+    const uintptr_t al = (uintptr_t)o | (uintptr_t)gate | (uintptr_t)norm_w | (uintptr_t)out32 | (uintptr_t)out16;
+    const bool vec = vdim % 4 == 0 && ((ldo | ldg | ld32 | ld16) & 3) == 0 && (al & 15) == 0;
+    kq_launch(vec ? head_norm_gate_kernel<true> : head_norm_gate_kernel<false>, (unsigned)kq_div_up(rows * heads, 8), 256, 0, st, o, ldo, gate, ldg, norm_w, eps,
+              rows, heads, vdim, out32, ld32, out16, ld16);
     KQ_COUNT_LAUNCH();
     KQ_LAUNCH_CHECK();
     return B200_OK;
@@ -616,7 +780,7 @@ b200_status kq_state_step(const KqMatState &m, const KqStateIn &in, const KqStat
     p.m = m, p.in = in, p.x = x, p.pos_dev = pos_dev, p.pos = pos, p.z = z, p.ldz = ldz;
     const size_t smem = (size_t)(3 * kq_state_ld(m.dim) + 3 * kq_pad(m.vdim, 4) + kq_pad(x.a_rank, 8) + kq_pad(x.g_rank, 8)) * 4;
     KQ_REQUIRE(smem <= 200 * 1024, "matrix state: %d value dimensions", m.vdim);
-    BY_DIM(launch_step, p, n_seq, smem, st)
+    BY_DIM(launch_step, 32, 64, 128, 256, p, n_seq, smem, st)
 }
 
 b200_status kq_rank_operands(const float *a, int n, uint16_t *a16, const float *g, int m, uint16_t *g16, int64_t ld, int64_t rows, cudaStream_t st) {
