@@ -9,8 +9,8 @@
 // with products of decays only, no quotients.  One launch makes every block's vectors and scalars (convolution, SiLU, unit
 // norms, decays) and leaves them as one record per block and head; the second walks the blocks with the state in
 // registers, so that eight products with the state wait for one reduction and a record is read from shared memory once
-// per four columns.  A thread holds four key dimensions (or eight) of four columns (value dimensions).  Records come by bulk
-// copies, two tiles in flight; every wait is bounded.
+// per pair of columns.  A thread holds some key dimensions of two columns (value dimensions).  A warp of its own brings the
+// records by bulk copies into a ring, the others walk through it without waiting for one another; every wait is bounded.
 // The fixed decay is the same with u = v and scalar products of decays.
 // A decode step is one launch: a CTA per head convolves, norms, works out the low-rank decays and gates, updates the
 // state and norms and gates the head's output.
@@ -65,8 +65,8 @@ struct ConvIn {
 };
 
 // ---- records of blocks of tokens -----------------------------------------------------------------------
-constexpr int BT = 4, TOK_NT = 256, TOK_NW = TOK_NT / 32, RUN = 4; // tokens per block, blocks a warp walks
-constexpr int N_SCALAR = 32;                                       // beta (4), A (6, from 4), B (10, from 12)
+constexpr int BT = 4, TOK_NT = 128, TOK_NW = TOK_NT / 32, RUN = 4; // tokens per block, blocks a warp walks
+constexpr int N_SCALAR = 32;                                       // beta (4), A (6, from 4), B (four rows of four, from 12)
 // floats of a record: decayed k, decayed q, k towards the block's end (four vectors each) and the block's decay; fixed decay: the
 // middle two
 __host__ __device__ constexpr int rec_floats(int dp, bool delta) { return (delta ? 13 : 8) * dp + N_SCALAR; }
@@ -79,47 +79,63 @@ struct TokParams {
     const int32_t *pos0_dev;
 };
 
-// SiLU of the convolution of channels lane + 32 c (< n) at the BT positions from t0 on; zero past the call's rows
+// The convolution of channels lane + 32 c (< n) at the BT positions from t0 on, with SiLU; zero past the call's rows.  Four taps: what
+// is read is requested by the constructor.
 template <int C>
-__device__ __forceinline__ void conv_block(const TokParams &p, const float *x, const float *w, int64_t channel0, int n, int64_t seq, int t0, int pos0, int lane,
-                                           float (&out)[BT][C]) {
-    const int taps = p.m.taps;
-    const int64_t row0 = seq * p.T, channels = kq_state_channels(p.m);
+struct ConvBlock {
+    float in[C][BT + 3];
+    __device__ __forceinline__ ConvIn input(const TokParams &p, const float *x, int64_t channel0, int64_t seq, int pos0, int d) const {
+        const int64_t channels = kq_state_channels(p.m);
+        return {x + seq * p.T * p.in.ld + d, p.in.ld, p.m.taps ? p.m.conv + seq * p.m.taps * channels + channel0 + d : nullptr, channels, p.m.taps, pos0};
+    }
+    __device__ __forceinline__ ConvBlock(const TokParams &p, const float *x, int64_t channel0, int n, int64_t seq, int t0, int pos0, int lane) {
+        if (p.m.taps != 4) return;
+        if (t0 >= 3 && t0 + BT <= p.T) { // all of this call
+            const float *r = x + (seq * p.T + t0 - 3) * p.in.ld + lane;
 #pragma unroll
-    for (int c = 0; c < C; c++) {
-        const int d = lane + 32 * c;
-        if (d >= n) {
+            for (int k = 0; k < BT + 3; k++)
 #pragma unroll
-            for (int j = 0; j < BT; j++) out[j][c] = 0.f;
-            continue;
-        }
-        const ConvIn ci = {x + row0 * p.in.ld + d, p.in.ld, taps ? p.m.conv + seq * taps * channels + channel0 + d : nullptr, channels, taps, pos0};
-        if (taps == 4) {
-            float in[BT + 3];
-#pragma unroll
-            for (int k = 0; k < BT + 3; k++) in[k] = t0 - 3 + k < p.T ? ci.at(t0 - 3 + k) : 0.f;
-            const float4 cw = *reinterpret_cast<const float4 *>(w + d * 4);
-#pragma unroll
-            for (int j = 0; j < BT; j++) out[j][c] = fmaf(cw.w, in[j + 3], fmaf(cw.z, in[j + 2], fmaf(cw.y, in[j + 1], cw.x * in[j])));
+                for (int c = 0; c < C; c++) in[c][k] = lane + 32 * c < n ? r[k * p.in.ld + 32 * c] : 0.f;
         } else {
 #pragma unroll
-            for (int j = 0; j < BT; j++) {
-                float s = 0.f;
-                if (t0 + j < p.T) {
-                    if (taps == 0) s = ci.at(t0 + j);
-                    for (int k = 0; k < taps; k++) s = fmaf(w[(int64_t)d * taps + k], ci.at(t0 + j - (taps - 1) + k), s);
-                }
-                out[j][c] = s;
+            for (int c = 0; c < C; c++) {
+                const ConvIn ci = input(p, x, channel0, seq, pos0, lane + 32 * c);
+#pragma unroll
+                for (int k = 0; k < BT + 3; k++) in[c][k] = lane + 32 * c < n && t0 - 3 + k < p.T ? ci.at(t0 - 3 + k) : 0.f;
             }
         }
-#pragma unroll
-        for (int j = 0; j < BT; j++) out[j][c] = t0 + j < p.T ? kq_silu(out[j][c]) : 0.f;
     }
-}
+    __device__ __forceinline__ void run(const TokParams &p, const float *x, const float *w, int64_t channel0, int n, int64_t seq, int t0, int pos0, int lane,
+                                        float (&out)[BT][C]) const {
+        const int taps = p.m.taps;
+#pragma unroll
+        for (int c = 0; c < C; c++) {
+            const int d = lane + 32 * c;
+            if (taps == 4) {
+                const float4 cw = d < n ? *reinterpret_cast<const float4 *>(w + d * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+                for (int j = 0; j < BT; j++) out[j][c] = fmaf(cw.w, in[c][j + 3], fmaf(cw.z, in[c][j + 2], fmaf(cw.y, in[c][j + 1], cw.x * in[c][j])));
+            } else {
+                const ConvIn ci = input(p, x, channel0, seq, pos0, d);
+#pragma unroll
+                for (int j = 0; j < BT; j++) {
+                    float s = 0.f;
+                    if (d < n && t0 + j < p.T) {
+                        if (taps == 0) s = ci.at(t0 + j);
+                        for (int k = 0; k < taps; k++) s = fmaf(w[(int64_t)d * taps + k], ci.at(t0 + j - (taps - 1) + k), s);
+                    }
+                    out[j][c] = s;
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < BT; j++) out[j][c] = t0 + j < p.T ? kq_silu(out[j][c]) : 0.f;
+        }
+    }
+};
 
 // grid (heads / warps, then values, runs of blocks, sequences)
 template <int C, bool DELTA>
-__global__ void __launch_bounds__(TOK_NT) state_tokens_kernel(const __grid_constant__ TokParams p) {
+__global__ void __launch_bounds__(TOK_NT, C > 4 ? 2 : DELTA ? 3 : 6) state_tokens_kernel(const __grid_constant__ TokParams p) {
     KQ_PDL_ENTER();
     constexpr int DP = 32 * C, REC = rec_floats(DP, DELTA);
     const KqMatState &m = p.m;
@@ -132,7 +148,8 @@ __global__ void __launch_bounds__(TOK_NT) state_tokens_kernel(const __grid_const
         const int n = (int)min((int64_t)32, nv - c0);
         for (int b = b0; b < b1; b++) {
             float v[BT][1];
-            conv_block<1>(p, p.in.v + c0, m.taps ? m.conv_v + c0 * m.taps : nullptr, 2 * nq + c0, n, seq, b * BT, pos0, lane, v);
+            const ConvBlock<1> cv(p, p.in.v + c0, 2 * nq + c0, n, seq, b * BT, pos0, lane);
+            cv.run(p, p.in.v + c0, m.conv_v + c0 * m.taps, 2 * nq + c0, n, seq, b * BT, pos0, lane, v);
             if (lane < n) *reinterpret_cast<float4 *>(p.val + (((seq * p.blocks + b) * nv) + c0 + lane) * BT) = make_float4(v[0][0], v[1][0], v[2][0], v[3][0]);
         }
         return;
@@ -150,8 +167,18 @@ __global__ void __launch_bounds__(TOK_NT) state_tokens_kernel(const __grid_const
         const int t0 = b * BT;
         float *rec = p.rec + ((seq * p.blocks + b) * m.heads + h) * (int64_t)REC;
         float q[BT][C], k[BT][C], g[BT][C];
-        conv_block<C>(p, p.in.q + cq, m.taps ? m.conv_q + cq * m.taps : nullptr, cq, m.dim, seq, t0, pos0, lane, q);
-        conv_block<C>(p, p.in.k + cq, m.taps ? m.conv_k + cq * m.taps : nullptr, nq + cq, m.dim, seq, t0, pos0, lane, k);
+        {
+            const ConvBlock<C> a(p, p.in.q + cq, cq, m.dim, seq, t0, pos0, lane), b(p, p.in.k + cq, nq + cq, m.dim, seq, t0, pos0, lane);
+            if (DELTA) {
+#pragma unroll
+                for (int j = 0; j < BT; j++)
+#pragma unroll
+                    for (int c = 0; c < C; c++)
+                        g[j][c] = lane + 32 * c < m.dim && t0 + j < p.T ? p.in.z[(seq * p.T + t0 + j) * p.in.ldz + cg + lane + 32 * c] : 0.f;
+            }
+            a.run(p, p.in.q + cq, m.conv_q + cq * m.taps, cq, m.dim, seq, t0, pos0, lane, q);
+            b.run(p, p.in.k + cq, m.conv_k + cq * m.taps, nq + cq, m.dim, seq, t0, pos0, lane, k);
+        }
         if (DELTA) {
             float ss[2 * BT];
 #pragma unroll
@@ -169,7 +196,7 @@ __global__ void __launch_bounds__(TOK_NT) state_tokens_kernel(const __grid_const
                 for (int c = 0; c < C; c++) {
                     const int d = lane + 32 * c;
                     q[j][c] *= sq, k[j][c] *= sk;
-                    g[j][c] = d < m.dim && t0 + j < p.T ? expf(-a * kq_softplus(p.in.z[(seq * p.T + t0 + j) * p.in.ldz + cg + d] + bias[c])) : 1.f;
+                    g[j][c] = d < m.dim && t0 + j < p.T ? expf(-a * kq_softplus(g[j][c] + bias[c])) : 1.f;
                 }
             }
         } else {
@@ -206,14 +233,16 @@ __global__ void __launch_bounds__(TOK_NT) state_tokens_kernel(const __grid_const
         }
         spread_sum<16, 32>(dot, lane); // lane holds sum lane / 2
         float *sc = rec + REC - N_SCALAR;
-        if ((lane & 1) == 0) sc[lane / 2 < 6 ? 4 + lane / 2 : 6 + lane / 2] = dot[0];
+        const int i = lane / 2, bi = i - 6, row = bi < 1 ? 0 : bi < 3 ? 1 : bi < 6 ? 2 : 3;
+        if ((lane & 1) == 0) sc[i < 6 ? 4 + i : 12 + 4 * row + bi - row * (row + 1) / 2] = dot[0];
+        else if (i < 6) sc[12 + (i < 3 ? 1 + i : i < 5 ? 3 + i : 11)] = 0.f; // above B's diagonal
         if (DELTA && lane < BT)
             sc[lane] = t0 + lane < p.T ? kq_sigmoid(p.in.b[(seq * p.T + t0 + lane) * p.in.ld + h]) : 0.f;
     }
 }
 
 // ---- the walk over the blocks -----------------------------------------------------------------------------
-constexpr int NC = 4, TB = 4; // columns per thread, blocks per tile
+constexpr int TB = 4, STAGES = 3; // blocks per tile, tiles in the ring
 constexpr int MAX_WARPS = 8;
 constexpr uint64_t LIMIT = 5 * KQ_WAIT_LIMIT_NS;
 struct ScanParams {
@@ -260,18 +289,19 @@ __device__ __forceinline__ void move_ring(const KqMatState &m, const KqStateIn &
     }
 }
 
-// grid (blocks of columns, heads, sequences).  LPC lanes share NC columns, each with R groups of four key dimensions.
+// grid (blocks of columns, heads, sequences).  LPC lanes share NC columns, each with R groups of four key dimensions, so that under
+// the delta rule the 8 NC sums of a block are one per lane.  The last warp brings the records.
 template <int LPC, int R, bool DELTA>
-__global__ void __launch_bounds__(MAX_WARPS * 32) state_scan_kernel(const __grid_constant__ ScanParams p) {
-    constexpr int DP = LPC * R * 4, REC = rec_floats(DP, DELTA), GW = 32 / LPC, NV = DELTA ? 32 : 16, LEFT = NV > LPC ? NV / LPC : 1;
+__global__ void __launch_bounds__((MAX_WARPS + 1) * 32) state_scan_kernel(const __grid_constant__ ScanParams p) {
+    constexpr int DP = LPC * R * 4, REC = rec_floats(DP, DELTA), GW = 32 / LPC, NC = LPC / (2 * BT), WC = GW * NC, NV = (DELTA ? 2 : 1) * NC * BT;
     extern __shared__ __align__(128) float sm[];
-    __shared__ uint64_t full[2];
-    __shared__ __align__(16) float s_red[MAX_WARPS][2][GW][NV], s_u[MAX_WARPS][2][GW][NC * BT];
+    __shared__ uint64_t full[STAGES], empty[STAGES];
+    __shared__ __align__(16) float s_o[MAX_WARPS][TB * BT][WC];
     __shared__ int s_abort;
     KQ_PDL_ENTER();
     const KqMatState &m = p.m;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, part = lane % LPC, grp = lane / LPC;
-    const int cols = (int)(blockDim.x / 32) * GW * NC; // of the CTA
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, part = lane % LPC, grp = lane / LPC, warps = (int)(blockDim.x / 32) - 1;
+    const int cols = warps * WC; // of the CTA
     const int h = blockIdx.y, e0 = blockIdx.x * cols, ne = min(cols, m.vdim - e0);
     const int64_t seq = blockIdx.z;
     const int pos0 = p.pos0_dev ? *p.pos0_dev : p.pos0;
@@ -279,153 +309,175 @@ __global__ void __launch_bounds__(MAX_WARPS * 32) state_scan_kernel(const __grid
         move_ring(m, p.in, gridDim.z, p.T, pos0, ((seq * gridDim.y + h) * gridDim.x + blockIdx.x) * blockDim.x + tid,
                   (int64_t)gridDim.x * gridDim.y * gridDim.z * blockDim.x);
     const int tile_floats = scan_tile_floats(DP, DELTA, cols), tiles = (p.blocks + TB - 1) / TB;
-    float *so = sm + 2 * tile_floats; // [TB * BT][cols]
     if (tid == 0) {
-        for (int i = 0; i < 2; i++) asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;" ::"r"((uint32_t)__cvta_generic_to_shared(&full[i])));
+        for (int i = 0; i < STAGES; i++) {
+            asm volatile("mbarrier.init.shared::cta.b64 [%0], 1;" ::"r"(smem_u32(&full[i])));
+            asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(smem_u32(&empty[i])), "r"(warps));
+        }
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
         s_abort = 0;
     }
     __syncthreads();
-    auto request = [&](int tile) { // by one thread: the records and the values of this CTA's columns
-        const uint32_t bar = (uint32_t)__cvta_generic_to_shared(&full[tile & 1]);
-        float *dst = sm + (tile & 1) * tile_floats;
-        const int b0 = tile * TB, n = min(TB, p.blocks - b0);
-        asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(n * (REC + ne * BT) * 4) : "memory");
-        for (int i = 0; i < n; i++) {
-            const int64_t at = (seq * p.blocks + b0 + i) * m.heads + h;
-            asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
-                             (uint32_t)__cvta_generic_to_shared(dst + i * REC)),
-                         "l"(p.rec + at * REC), "r"(REC * 4), "r"(bar)
-                         : "memory");
-            asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
-                             (uint32_t)__cvta_generic_to_shared(dst + TB * REC + i * cols * BT)),
-                         "l"(p.val + (at * m.vdim + e0) * BT), "r"(ne * BT * 4), "r"(bar)
-                         : "memory");
-        }
-    };
-    if (tid == 0) {
-        request(0);
-        if (tiles > 1) request(1);
-    }
-    const int c0 = (warp * GW + grp) * NC; // this lane group's columns inside the CTA
-    uint64_t s[NC][R][2];
-    const int64_t ld = kq_state_ld(m.dim);
-    float *sp = m.s + ((seq * m.heads + h) * m.vdim + e0 + c0) * ld + 4 * part;
-#pragma unroll
-    for (int c = 0; c < NC; c++)
-#pragma unroll
-        for (int i = 0; i < R; i++) {
-            const ulonglong2 v = pos0 > 0 && c0 + c < ne ? *reinterpret_cast<const ulonglong2 *>(sp + c * ld + 4 * LPC * i) : make_ulonglong2(0, 0);
-            s[c][i][0] = v.x, s[c][i][1] = v.y;
-        }
-    float d_full = 1.f, d_last = 1.f; // fixed decay over a block; the last one may hold fewer tokens
-    if (!DELTA)
-        for (int j = 0; j < BT; j++) {
-            d_full *= m.decay[h];
-            if ((p.blocks - 1) * BT + j < p.T) d_last *= m.decay[h];
-        }
-    for (int tile = 0; tile < tiles; tile++) {
-        if (!tc_wait((uint32_t)__cvta_generic_to_shared(&full[tile & 1]), (uint32_t)((tile >> 1) & 1), &s_abort, &g_state_error, 1, LIMIT)) {
-            s_abort = 1;
-        }
-        const float *src = sm + (tile & 1) * tile_floats;
-        const int nb = min(TB, p.blocks - tile * TB);
-        for (int b = 0; b < nb; b++) {
-            const float *rec = src + b * REC, *sc = rec + REC - N_SCALAR;
-            const ulonglong2 *vec = reinterpret_cast<const ulonglong2 *>(rec) + part; // vector v, group i: vec[v * DP / 4 + LPC * i]
-            float val[NV];
-#pragma unroll
-            for (int v = 0; v < NV / NC; v++) { // products with the state: [decayed k,] decayed q of the four tokens
-                uint64_t acc[NC];
-#pragma unroll
-                for (int i = 0; i < R; i++) {
-                    const ulonglong2 x = vec[v * DP / 4 + LPC * i];
-#pragma unroll
-                    for (int c = 0; c < NC; c++) acc[c] = fma2(s[c][i][1], x.y, i == 0 ? mul2(s[c][i][0], x.x) : fma2(s[c][i][0], x.x, acc[c]));
-                }
-#pragma unroll
-                for (int c = 0; c < NC; c++) val[v / BT * 16 + c * BT + v % BT] = add2(acc[c]);
-            }
-            spread_sum<NV, LPC>(val, lane);
-            float *red = s_red[warp][b & 1][grp], *us = s_u[warp][b & 1][grp];
-            if (NV >= LPC) {
-#pragma unroll
-                for (int i = 0; i < LEFT; i++) red[part * LEFT + i] = val[i];
-            } else if (part % (LPC / NV) == 0) {
-                red[part / (LPC / NV)] = val[0];
+    if (warp == warps) {
+        for (int tile = 0; tile < tiles; tile++) {
+            const int st = tile % STAGES, round = tile / STAGES;
+            if (round > 0 && !__all_sync(0xffffffffu, tc_wait(smem_u32(&empty[st]), (uint32_t)((round - 1) & 1), &s_abort, &g_state_error, 1, LIMIT))) break;
+            float *dst = sm + st * tile_floats;
+            const int b0 = tile * TB, n = min(TB, p.blocks - b0);
+            const uint32_t bar = smem_u32(&full[st]);
+            if (lane == 0) asm volatile("mbarrier.arrive.expect_tx.shared::cta.b64 _, [%0], %1;" ::"r"(bar), "r"(n * (REC + ne * BT) * 4) : "memory");
+            __syncwarp();
+            if (lane < 2 * n) { // a lane per copy: the records, and the values of this CTA's columns
+                const int i = lane / 2;
+                const int64_t at = (seq * p.blocks + b0 + i) * m.heads + h;
+                const float *src = lane & 1 ? p.val + (at * m.vdim + e0) * BT : p.rec + at * REC;
+                asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(
+                                 smem_u32(dst + (lane & 1 ? TB * REC + i * cols * BT : i * REC))),
+                             "l"(src), "r"((lane & 1 ? ne * BT : REC) * 4), "r"(bar)
+                             : "memory");
             }
             __syncwarp();
-            { // every lane solves one of the group's columns; the first four lanes pass theirs on
-                const int c = part & (NC - 1);
-                const float4 vt = *reinterpret_cast<const float4 *>(src + TB * REC + (b * cols + c0 + c) * BT);
-                const float4 dq = *reinterpret_cast<const float4 *>(red + (DELTA ? 16 : 0) + c * BT);
-                float4 u = vt;
-                if (DELTA) {
-                    const float4 dk = *reinterpret_cast<const float4 *>(red + c * BT), be = *reinterpret_cast<const float4 *>(sc),
-                                 A0 = *reinterpret_cast<const float4 *>(sc + 4), A1 = *reinterpret_cast<const float4 *>(sc + 8);
-                    u.x = be.x * (vt.x - dk.x);
-                    u.y = be.y * (vt.y - dk.y - A0.x * u.x);
-                    u.z = be.z * (vt.z - dk.z - A0.y * u.x - A0.z * u.y);
-                    u.w = be.w * (vt.w - dk.w - A0.w * u.x - A1.x * u.y - A1.y * u.z);
-                }
-                if (part < NC) {
-                    *reinterpret_cast<float4 *>(us + c * BT) = u;
-                    const float4 B0 = *reinterpret_cast<const float4 *>(sc + 12), B1 = *reinterpret_cast<const float4 *>(sc + 16);
-                    const float2 B2 = *reinterpret_cast<const float2 *>(sc + 20);
-                    float *o = so + b * BT * cols + c0 + c;
-                    o[0] = fmaf(B0.x, u.x, dq.x);
-                    o[cols] = fmaf(B0.z, u.y, fmaf(B0.y, u.x, dq.y));
-                    o[2 * cols] = fmaf(B1.y, u.z, fmaf(B1.x, u.y, fmaf(B0.w, u.x, dq.z)));
-                    o[3 * cols] = fmaf(B2.y, u.w, fmaf(B2.x, u.z, fmaf(B1.w, u.y, fmaf(B1.z, u.x, dq.w))));
-                }
-            }
-            __syncwarp();
-            constexpr int KH = DELTA ? 8 : 4; // first of the vectors that are written
+        }
+    } else {
+        const int c0 = warp * WC + grp * NC; // this lane group's columns inside the CTA
+        uint64_t s[NC][R][2];
+        const int64_t ld = kq_state_ld(m.dim);
+        float *sp = m.s + ((seq * m.heads + h) * m.vdim + e0 + c0) * ld + 4 * part;
+#pragma unroll
+        for (int c = 0; c < NC; c++)
 #pragma unroll
             for (int i = 0; i < R; i++) {
-                ulonglong2 gg;
-                if (DELTA) gg = vec[12 * DP / 4 + LPC * i];
-                else gg.x = gg.y = tile * TB + b == p.blocks - 1 ? pack2(d_last, d_last) : pack2(d_full, d_full);
-#pragma unroll
-                for (int c = 0; c < NC; c++) s[c][i][0] = mul2(s[c][i][0], gg.x), s[c][i][1] = mul2(s[c][i][1], gg.y);
+                const ulonglong2 v = pos0 > 0 && c0 + c < ne ? *reinterpret_cast<const ulonglong2 *>(sp + c * ld + 4 * LPC * i) : make_ulonglong2(0, 0);
+                s[c][i][0] = v.x, s[c][i][1] = v.y;
             }
+        float d_full = 1.f, d_last = 1.f; // fixed decay over a block; the last one may hold fewer tokens
+        if (!DELTA)
+            for (int j = 0; j < BT; j++) {
+                d_full *= m.decay[h];
+                if ((p.blocks - 1) * BT + j < p.T) d_last *= m.decay[h];
+            }
+        float *out = p.o + seq * p.T * p.ldo + (int64_t)h * m.vdim + e0 + warp * WC;
+        const int wn = min(WC, ne - warp * WC); // columns of this warp
+        const bool vec = WC == 4 && wn == 4 && (p.ldo & 3) == 0 && ((uintptr_t)out & 15) == 0;
+        bool ok = true;
+        for (int tile = 0; tile < tiles; tile++) {
+            const int st = tile % STAGES;
+            ok = __all_sync(0xffffffffu, tc_wait(smem_u32(&full[st]), (uint32_t)((tile / STAGES) & 1), &s_abort, &g_state_error, 2, LIMIT));
+            if (!ok) break;
+            const float *src = sm + st * tile_floats;
+            const int nb = min(TB, p.blocks - tile * TB);
+            constexpr int KH = DELTA ? 8 : 4; // first of the vectors that are written
+            const ulonglong2 *vec2 = reinterpret_cast<const ulonglong2 *>(src) + part; // vector v, group i: vec2[v * DP / 4 + LPC * i]
+            constexpr bool AHEAD = R == 1; // vectors wait in registers, where there are few
+            ulonglong2 x[KH][R];
+            auto load_x = [&](int v) {
 #pragma unroll
-            for (int c = 0; c < NC; c++) {
-                const float4 u = *reinterpret_cast<const float4 *>(us + c * BT);
-                const float uv[BT] = {u.x, u.y, u.z, u.w};
+                for (int i = 0; i < R; i++) x[v][i] = vec2[v * DP / 4 + LPC * i];
+            };
+            if (AHEAD) {
 #pragma unroll
-                for (int j = 0; j < BT; j++) {
-                    const uint64_t uu = pack2(uv[j], uv[j]);
+                for (int v = 0; v < KH; v++) load_x(v);
+            }
+            for (int b = 0; b < nb; b++) {
+                const float *sc = src + b * REC + REC - N_SCALAR, *vals = src + TB * REC + (b * cols + c0) * BT;
+                float val[NV];
+#pragma unroll
+                for (int v = 0; v < KH; v++) { // products with the state: [decayed k,] decayed q of the four tokens
+                    uint64_t acc[NC];
+                    if (!AHEAD) load_x(v);
+#pragma unroll
+                    for (int i = 0; i < R; i++)
+#pragma unroll
+                        for (int c = 0; c < NC; c++) acc[c] = fma2(s[c][i][1], x[v][i].y, i == 0 ? mul2(s[c][i][0], x[v][i].x) : fma2(s[c][i][0], x[v][i].x, acc[c]));
+#pragma unroll
+                    for (int c = 0; c < NC; c++) val[v / BT * NC * BT + c * BT + v % BT] = add2(acc[c]);
+                }
+                // requested ahead of the reduction: what the rest of the block reads
+                ulonglong2 kk[BT][R], gg[R];
+                auto load_k = [&]() {
 #pragma unroll
                     for (int i = 0; i < R; i++) {
-                        const ulonglong2 kk = vec[(KH + j) * DP / 4 + LPC * i];
-                        s[c][i][0] = fma2(kk.x, uu, s[c][i][0]), s[c][i][1] = fma2(kk.y, uu, s[c][i][1]);
+#pragma unroll
+                        for (int j = 0; j < BT; j++) kk[j][i] = vec2[(KH + j) * DP / 4 + LPC * i];
+                        if (DELTA) gg[i] = vec2[(KH + BT) * DP / 4 + LPC * i];
                     }
+                };
+                if (AHEAD) load_k();
+                // the sum that ends in this lane: column c, token j, of k (lower half of the lanes) or q
+                const int idx = part / (LPC / NV), c = idx / BT % NC, j = idx % BT;
+                const float4 vt = *reinterpret_cast<const float4 *>(vals + c * BT), B = *reinterpret_cast<const float4 *>(sc + 12 + 4 * j);
+                float4 u = vt, be, A0, A1;
+                if (DELTA) be = *reinterpret_cast<const float4 *>(sc), A0 = *reinterpret_cast<const float4 *>(sc + 4), A1 = *reinterpret_cast<const float4 *>(sc + 8);
+                spread_sum<NV, LPC>(val, lane);
+                if (DELTA) { // every lane solves for its column
+                    float dk[BT];
+#pragma unroll
+                    for (int i = 0; i < BT; i++) dk[i] = __shfl_sync(0xffffffffu, val[0], c * BT + i, LPC);
+                    u.x = be.x * (vt.x - dk[0]);
+                    u.y = be.y * (vt.y - dk[1] - A0.x * u.x);
+                    u.z = be.z * (vt.z - dk[2] - A0.y * u.x - A0.z * u.y);
+                    u.w = be.w * (vt.w - dk[3] - A0.w * u.x - A1.x * u.y - A1.y * u.z);
                 }
+                if (DELTA ? part >= LPC / 2 : part % 2 == 0)
+                    s_o[warp][b * BT + j][grp * NC + c] = fmaf(B.w, u.w, fmaf(B.z, u.z, fmaf(B.y, u.y, fmaf(B.x, u.x, val[0]))));
+                float4 w[NC];
+                if (NC == 1) {
+                    w[0] = u;
+                } else if (DELTA) { // the other column's, from the lane that solves for it
+                    const float4 o = make_float4(__shfl_xor_sync(0xffffffffu, u.x, BT), __shfl_xor_sync(0xffffffffu, u.y, BT),
+                                                 __shfl_xor_sync(0xffffffffu, u.z, BT), __shfl_xor_sync(0xffffffffu, u.w, BT));
+                    w[0] = c ? o : u, w[NC - 1] = c ? u : o;
+                } else {
+#pragma unroll
+                    for (int e = 0; e < NC; e++) w[e] = *reinterpret_cast<const float4 *>(vals + e * BT);
+                }
+                if (!AHEAD) load_k();
+                vec2 += REC / 4;
+                if (AHEAD && b + 1 < nb) { // the next block's first vectors
+#pragma unroll
+                    for (int v = 0; v < KH; v++) load_x(v);
+                }
+#pragma unroll
+                for (int i = 0; i < R; i++) {
+                    if (!DELTA) gg[i].x = gg[i].y = tile * TB + b == p.blocks - 1 ? pack2(d_last, d_last) : pack2(d_full, d_full);
+#pragma unroll
+                    for (int e = 0; e < NC; e++) s[e][i][0] = mul2(s[e][i][0], gg[i].x), s[e][i][1] = mul2(s[e][i][1], gg[i].y);
+                }
+#pragma unroll
+                for (int t = 0; t < BT; t++)
+#pragma unroll
+                    for (int e = 0; e < NC; e++) {
+                        const float f = t == 0 ? w[e].x : t == 1 ? w[e].y : t == 2 ? w[e].z : w[e].w;
+                        const uint64_t ff = pack2(f, f);
+#pragma unroll
+                        for (int i = 0; i < R; i++) s[e][i][0] = fma2(kk[t][i].x, ff, s[e][i][0]), s[e][i][1] = fma2(kk[t][i].y, ff, s[e][i][1]);
+                    }
             }
+            __syncwarp(); // this warp is done with the tile, its outputs are complete
+            if (lane == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(&empty[st])) : "memory");
+            const int t0 = tile * TB * BT, n = min(TB * BT, p.T - t0);
+            if (vec) {
+                if (lane < n) *reinterpret_cast<float4 *>(out + (int64_t)(t0 + lane) * p.ldo) = *reinterpret_cast<const float4 *>(s_o[warp][lane]);
+            } else {
+                for (int i = lane; i < n * WC; i += 32)
+                    if (i % WC < wn) out[(int64_t)(t0 + i / WC) * p.ldo + i % WC] = s_o[warp][i / WC][i % WC];
+            }
+            __syncwarp();
         }
-        __syncthreads(); // the tile's buffer is free, its outputs are complete
-        if (s_abort) break;
-        if (tid == 0 && tile + 2 < tiles) request(tile + 2);
-        const int n = min(TB * BT, p.T - tile * TB * BT);
-        for (int i = tid; i < n * cols; i += blockDim.x)
-            if (i % cols < ne) p.o[(seq * p.T + tile * TB * BT + i / cols) * p.ldo + (int64_t)h * m.vdim + e0 + i % cols] = so[i];
-        __syncthreads();
-    }
-    if (s_abort) { // copies in flight must land before the CTA goes away
-        if (tid == 0)
-            for (int i = 0; i < 2; i++) {
-                kq_mbar_wait((uint32_t)__cvta_generic_to_shared(&full[i]), 0u, KQ_WAIT_LIMIT_NS);
-                kq_mbar_wait((uint32_t)__cvta_generic_to_shared(&full[i]), 1u, KQ_WAIT_LIMIT_NS);
-            }
-        __syncthreads();
-        return;
-    }
+        if (ok) {
 #pragma unroll
-    for (int c = 0; c < NC; c++)
+            for (int c = 0; c < NC; c++)
 #pragma unroll
-        for (int i = 0; i < R; i++)
-            if (c0 + c < ne) *reinterpret_cast<ulonglong2 *>(sp + c * ld + 4 * LPC * i) = make_ulonglong2(s[c][i][0], s[c][i][1]);
+                for (int i = 0; i < R; i++)
+                    if (c0 + c < ne) *reinterpret_cast<ulonglong2 *>(sp + c * ld + 4 * LPC * i) = make_ulonglong2(s[c][i][0], s[c][i][1]);
+        }
+    }
+    __syncthreads();
+    if (s_abort && tid == 0) // copies in flight must land before the CTA goes away
+        for (int i = 0; i < STAGES; i++) {
+            kq_mbar_wait(smem_u32(&full[i]), 0u, KQ_WAIT_LIMIT_NS);
+            kq_mbar_wait(smem_u32(&full[i]), 1u, KQ_WAIT_LIMIT_NS);
+        }
 }
 
 // ---- output of a prompt --------------------------------------------------------------------------------
@@ -678,16 +730,17 @@ b200_status check_state(const KqMatState &m, int n_seq, int T) {
 
 template <int LPC, int R, bool DELTA>
 b200_status launch_scan(const ScanParams &p, int n_seq, cudaStream_t st) {
-    constexpr int DP = LPC * R * 4, per_warp = 32 / LPC * NC;
+    constexpr int DP = LPC * R * 4, per_warp = 32 / LPC * (LPC / (2 * BT));
     // warps per CTA: as few as possible on the busiest SM, then as many as possible in a CTA, which share a record
     int warps = 1;
     int64_t best = INT64_MAX;
-    for (int w = 1; w <= MAX_WARPS; w++) {
+    const int most = std::min<int>(MAX_WARPS, (int)((200 * 1024 / 4 / STAGES / TB - rec_floats(DP, DELTA)) / (per_warp * BT)));
+    for (int w = 1; w <= most; w++) {
         const int64_t ctas = kq_div_up(p.m.vdim, w * per_warp) * p.m.heads * n_seq, load = kq_div_up(ctas, kq_sm_count()) * w;
         if (load <= best && (w == 1 || (w - 1) * per_warp < p.m.vdim)) best = load, warps = w;
     }
     const int cols = warps * per_warp;
-    const size_t smem = (size_t)(2 * scan_tile_floats(DP, DELTA, cols) + TB * BT * cols) * 4;
+    const size_t smem = (size_t)STAGES * scan_tile_floats(DP, DELTA, cols) * 4;
     static size_t attr[16];
     int dev = 0;
     KQ_CUDA(cudaGetDevice(&dev));
@@ -695,7 +748,7 @@ b200_status launch_scan(const ScanParams &p, int n_seq, cudaStream_t st) {
         KQ_CUDA(cudaFuncSetAttribute(state_scan_kernel<LPC, R, DELTA>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         if (dev >= 0 && dev < 16) attr[dev] = smem;
     }
-    kq_launch(state_scan_kernel<LPC, R, DELTA>, dim3((unsigned)kq_div_up(p.m.vdim, cols), (unsigned)p.m.heads, (unsigned)n_seq), warps * 32, smem, st, p);
+    kq_launch(state_scan_kernel<LPC, R, DELTA>, dim3((unsigned)kq_div_up(p.m.vdim, cols), (unsigned)p.m.heads, (unsigned)n_seq), (warps + 1) * 32, smem, st, p);
     KQ_COUNT_LAUNCH();
     KQ_LAUNCH_CHECK();
     return B200_OK;
@@ -758,7 +811,7 @@ b200_status kq_state_scan(const KqMatState &m, const KqStateIn &in, const KqStat
     KQ_TRY(check_state(m, n_seq, T));
     ScanParams p;
     p.m = m, p.in = in, p.rec = t.rec, p.val = t.val, p.T = T, p.pos0 = pos0, p.pos0_dev = pos0_dev, p.blocks = (int)kq_div_up(T, BT), p.o = o, p.ldo = ldo;
-    BY_DIM(launch_scan, TWO(8, 1), TWO(16, 1), TWO(32, 1), TWO(32, 2), p, n_seq, st)
+    BY_DIM(launch_scan, TWO(8, 1), TWO(16, 1), TWO(16, 2), TWO(16, 4), p, n_seq, st)
 }
 
 b200_status kq_head_norm_gate(const float *o, int64_t ldo, const float *gate, int64_t ldg, const float *norm_w, float eps, int64_t rows, int heads,
