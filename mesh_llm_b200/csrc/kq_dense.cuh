@@ -49,9 +49,8 @@ struct KqDense {
     const float *head_gate = nullptr;
     int64_t ld_gate = 0;
     float cap = 0.f; // KQ_ACT_SOFT_CAP
-    // row_mul: y *= row_mul[mul_row[m] * ld_mul + n] (bf16), after the activation
+    // row_mul: y *= row_mul[m * ld_mul + n] (bf16), after the activation
     const uint16_t *row_mul = nullptr;
-    const int32_t *mul_row = nullptr;
     int64_t ld_mul = 0;
     // experts > 0 (matrix products): every segment holds `experts` matrices of n_rows rows one after the other; the rows of
     // x come in tiles of KQ_TILE_M, tile i belongs to expert tile_expert[i], *n_tiles of them (device) hold anything
@@ -120,7 +119,7 @@ __device__ __forceinline__ void kq_dense_store(const KqDense &c, const KqDenseSe
     if (s.act == KQ_ACT_GELU_TANH) v = kq_gelu_tanh(v);
     if (s.act == KQ_ACT_SOFT_CAP) v = c.cap * tanhf(v / c.cap);
     if (c.head_gate) v *= kq_sigmoid(c.head_gate[m * c.ld_gate + g]);
-    if (c.row_mul) v *= kq_bf2f(c.row_mul[(int64_t)c.mul_row[m] * c.ld_mul + n]);
+    if (c.row_mul) v *= kq_bf2f(c.row_mul[m * c.ld_mul + n]);
     kq_dense_put(s, m, n, v);
 }
 #endif
@@ -138,6 +137,8 @@ b200_status kq_gemm_f32(const KqDense &c, const float *x, int64_t ldx, cudaStrea
 // embedding rows of a bf16 table times `scale`
 b200_status kq_embed_bf16(const uint16_t *W, int64_t ldw, const int32_t *ids, int64_t rows, int K, float scale, float *y,
                           int64_t ldy, cudaStream_t st);
+// rows `ids` of a bf16 table as they are
+b200_status kq_gather_bf16(const uint16_t *W, const int32_t *ids, int64_t rows, uint16_t *y, int64_t ld, cudaStream_t st);
 // the prologue above as a kernel of its own; h as f32 (h32) and / or as a bf16 staging copy (h16), either may be null
 b200_status kq_norm_prep(const KqNormPrep &p, int64_t rows, int K, float *h32, int64_t ld32, uint16_t *h16, int64_t ld16,
                          cudaStream_t st);

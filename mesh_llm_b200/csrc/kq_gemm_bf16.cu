@@ -56,7 +56,7 @@ struct Col4 {
     }
     // the factors of row m: eight bytes where the row allows it
     __device__ __forceinline__ uint2 factors(const KqDense &c, int64_t m) const {
-        const uint16_t *f = c.row_mul + (int64_t)c.mul_row[m] * c.ld_mul + n;
+        const uint16_t *f = c.row_mul + m * c.ld_mul + n;
         if (n_mul >= 4 && ((uintptr_t)f & 7) == 0) return *reinterpret_cast<const uint2 *>(f);
         uint32_t w[4];
 #pragma unroll
@@ -266,7 +266,7 @@ __global__ void __launch_bounds__(NTHREADS, 1) gemm_bf16_kernel(const __grid_con
                 const int n = n0 + j + c4, n_valid = std::min(4, lim - n);
                 if (n_valid > 0) {
                     const Col4 col(p.c, s, (p.c.experts ? 0 : (int64_t)w.g * n_rows) + n, n_valid);
-                    if (p.c.row_mul) { // the factors of all of a lane's rows are requested together: they may come from anywhere
+                    if (p.c.row_mul) { // the factors of all of a lane's rows are requested together
                         uint2 f[8];
 #pragma unroll
                         for (int i = 0; i < 8; i++) f[i] = m0 + r4 + 4 * i < m_end ? col.factors(p.c, m0 + r4 + 4 * i) : make_uint2(0, 0);

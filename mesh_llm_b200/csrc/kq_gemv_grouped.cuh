@@ -96,6 +96,6 @@ static inline KqDense kq_rows_of(const KqDense &c, int m0, int m) {
     for (int i = 0; i < d.nseg; i++)
         d.seg[i].y = (uint8_t *)c.seg[i].y + m0 * c.seg[i].ldy * (c.seg[i].out == KQ_OUT_F32 ? 4 : 2);
     if (d.head_gate) d.head_gate += m0 * d.ld_gate;
-    if (d.mul_row) d.mul_row += m0;
+    if (d.row_mul) d.row_mul += m0 * d.ld_mul;
     return d;
 }

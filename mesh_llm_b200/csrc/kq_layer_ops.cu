@@ -34,6 +34,13 @@ __global__ void embed_bf16_kernel(const uint16_t *W, int64_t ldw, const int32_t 
     }
 }
 
+// a thread per eight values; rows of a multiple of 64 elements
+__global__ void gather_bf16_kernel(const uint16_t *W, const int32_t *ids, uint16_t *y, int64_t ld) {
+    KQ_PDL_ENTER();
+    const int64_t k = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * 8, r = blockIdx.y;
+    if (k < ld) *reinterpret_cast<uint4 *>(y + r * ld + k) = *reinterpret_cast<const uint4 *>(W + (int64_t)ids[r] * ld + k);
+}
+
 constexpr int NT = 256;
 __device__ __forceinline__ float block_sum(float v, float *red) {
     v = kq_warp_sum(v);
@@ -378,6 +385,14 @@ b200_status kq_embed_bf16(const uint16_t *W, int64_t ldw, const int32_t *ids, in
     KQ_REQUIRE(W && ids && y && rows >= 1 && K >= 1, "embed_bf16: bad call");
     KQ_REQUIRE(rows <= 65535 && ((uintptr_t)y & 15) == 0, "embed_bf16: %lld rows", (long long)rows);
     kq_launch(embed_bf16_kernel, dim3((unsigned)kq_div_up(K, 8 * 128), (unsigned)rows), 128, 0, st, W, ldw, ids, rows, K, scale, y, ldy);
+    KQ_COUNT_LAUNCH();
+    KQ_LAUNCH_CHECK();
+    return B200_OK;
+}
+
+b200_status kq_gather_bf16(const uint16_t *W, const int32_t *ids, int64_t rows, uint16_t *y, int64_t ld, cudaStream_t st) {
+    KQ_REQUIRE(W && ids && y && rows >= 1 && rows <= 65535 && ld % 64 == 0, "gather_bf16: bad call");
+    kq_launch(gather_bf16_kernel, dim3((unsigned)kq_div_up(ld, 8 * 128), (unsigned)rows), 128, 0, st, W, ids, y, ld);
     KQ_COUNT_LAUNCH();
     KQ_LAUNCH_CHECK();
     return B200_OK;

@@ -82,6 +82,7 @@ struct KqLayers {
     float *f[9] = {}; // projections of a mixer
     std::vector<Pack> packs;
     const uint16_t *side_embed = nullptr;
+    uint16_t *side_rows = nullptr; // the rows of a call's tokens, all layers
     KqStateTok state_tok = {};
     // experts: activations of few rows; tiles of rows by expert
     float *moe_act = nullptr, *moe_y = nullptr;
@@ -236,7 +237,7 @@ struct Pass {
     b200_stage *st;
     KqLayers *k;
     int seq0, n_seq, T, pos0, rows;
-    const int32_t *pos_dev, *tokens;
+    const int32_t *pos_dev;
     bool small, f32;
     unsigned classes;
     cudaStream_t s;
@@ -579,9 +580,8 @@ struct Pass {
         c.seg[0] = tc ? seg(L.side_gate, sd, k->u16, kq_bf16_ld(sd), nullptr, KQ_ACT_GELU_TANH, KQ_OUT_BF16)
                       : seg(L.side_gate, sd, k->f[1], kq_f32_ld(sd), nullptr, KQ_ACT_GELU_TANH);
         if (tc) c.seg[0].pad_cols = (int32_t)kq_bf16_ld(sd);
-        c.row_mul = k->side_embed + (int64_t)layer * sd;
+        c.row_mul = k->side_rows + (int64_t)layer * sd;
         c.ld_mul = kq_bf16_ld((int64_t)st->c.n_layer * sd);
-        c.mul_row = tokens;
         KQ_TRY(project(c, nullptr));
         return close(L.side_proj, sd, k->f[1], kq_f32_ld(sd), k->u16, L.side_norm);
     }
@@ -650,7 +650,6 @@ b200_status kq_layers_forward(b200_stage *st, const int32_t *tokens, const float
     Pass P;
     P.st = st, P.k = k, P.seq0 = seq0, P.n_seq = n_seq, P.T = T, P.pos0 = pos0, P.rows = n_seq * T;
     P.pos_dev = pos_from_dev ? st->pos0_dev : nullptr;
-    P.tokens = tokens;
     P.small = P.rows <= SMALL_ROWS;
     P.f32 = k->s.precision == B200_PRECISION_F32;
     P.classes = classes;
@@ -660,6 +659,8 @@ b200_status kq_layers_forward(b200_stage *st, const int32_t *tokens, const float
         if (classes & CLS_OTHER) KQ_TRY(kq_embed_bf16(k->embed, kq_bf16_ld(c.n_embd), tokens, P.rows, c.n_embd, k->s.embd_scale, k->x[0], k->ldx, s));
         P.x = {k->x[0], k->ldx, nullptr, 1};
     }
+    if (k->s.side_dim && (classes & CLS_OTHER))
+        KQ_TRY(kq_gather_bf16(k->side_embed, tokens, P.rows, k->side_rows, kq_bf16_ld((int64_t)c.n_layer * k->s.side_dim), s));
     int run = 0;
     for (const RunState &r : k->runs) {
         const LayerDesc &L = k->layers[r.layer - c.layer_begin];
@@ -1098,6 +1099,7 @@ b200_status b200_stage_create_layers(const b200_stage_config *cfg, const b200_st
         A(&k->moe_h, (size_t)(moe_rows * (f32 ? kq_f32_ld(moe_ff) * 4 : kq_bf16_ld(moe_ff) * 2)));
         A(&k->moe_y, (size_t)(moe_rows * k->ldx * 4));
     }
+    if (stack->side_dim) A(&k->side_rows, (size_t)(R * kq_bf16_ld((int64_t)c.n_layer * stack->side_dim) * 2));
     k->rec_scratch_bytes = (size_t)rec_scratch;
     A(&k->rec_scratch, (size_t)rec_scratch);
     k->att_scratch_bytes = (size_t)scratch;

@@ -95,52 +95,54 @@ __global__ void __launch_bounds__(NT) moe_few_gate_up_kernel(const __grid_consta
     }
 }
 
-// grid (slices of output rows, rows); a warp takes an output row over all chosen experts and the shared one
-constexpr int DOWN_ROWS = NW, DOWN_U = 8; // chunks in flight per lane
+// grid (slices of output rows, rows).  The chosen experts' and the shared one's hidden values are one long row, in chunks of eight;
+// warps split the chunks, every warp for all of the CTA's output rows, so that a lane makes its activations once and has
+// many weights in flight.
+constexpr int DOWN_ROWS = 8;
 __global__ void __launch_bounds__(NT) moe_few_down_kernel(const __grid_constant__ KqMoe m, const float *act, int64_t ld_act, const int32_t *ids, const float *wts,
                                                           const uint16_t *down, const uint16_t *sh_down, float *out, int64_t ldo) {
-    extern __shared__ __align__(16) float sm[]; // [top][padded ff] activations times weight, [padded ff_shared]
+    __shared__ float part[NW][DOWN_ROWS];
     KQ_PDL_ENTER();
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = blockIdx.y;
-    const int fp = (m.ff + 7) / 8 * 8, sp = (m.ff_shared + 7) / 8 * 8, per = fp / 8, n_ck = m.top * per, s_ck = sp / 8;
-    float4 *p0 = reinterpret_cast<float4 *>(sm), *p1 = p0 + n_ck + s_ck; // two planes of float4
-    const int n = blockIdx.x * DOWN_ROWS + warp, all = n_ck + s_ck;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, row = blockIdx.y, n0 = blockIdx.x * DOWN_ROWS;
+    const int per = (m.ff + 7) / 8, n_ck = m.top * per, all = n_ck + (m.ff_shared + 7) / 8;
     const int64_t ldw = kq_bf16_ld(m.ff), lds = kq_bf16_ld(m.ff_shared);
-    uint4 q[DOWN_U];
-    auto request = [&](int c0) {
+    const bool vec = (m.ldz & 3) == 0 && ((((uintptr_t)m.sh_gate | (uintptr_t)m.sh_up) & 15) == 0);
+    float acc[DOWN_ROWS] = {};
+#pragma unroll 2
+    for (int c = tid; c < all; c += NT) {
+        const bool shared = c >= n_ck;
+        const int s = shared ? 0 : c / per, k = 8 * (shared ? c - n_ck : c - s * per);
+        const int64_t step = shared ? lds : ldw;
+        const uint16_t *w = (shared ? sh_down + n0 * lds : down + ((int64_t)ids[row * m.top + s] * m.h + n0) * ldw) + k;
+        uint4 q[DOWN_ROWS];
 #pragma unroll
-        for (int u = 0; u < DOWN_U; u++) {
-            const int c = c0 + lane + 32 * u;
-            q[u] = make_uint4(0, 0, 0, 0);
-            if (n < m.h && c < n_ck) q[u] = kq_ld_stream(down + ((int64_t)ids[row * m.top + c / per] * m.h + n) * ldw + c % per * 8);
-            else if (n < m.h && c < all) q[u] = kq_ld_stream(sh_down + n * lds + (c - n_ck) * 8);
+        for (int r = 0; r < DOWN_ROWS; r++) q[r] = kq_ld_stream(w + min(r, m.h - 1 - n0) * step);
+        float4 a, b;
+        if (shared) {
+            const float4 g0 = kq_load4(m.sh_gate + row * m.ldz, k, m.ff_shared, vec), g1 = kq_load4(m.sh_gate + row * m.ldz, k + 4, m.ff_shared, vec);
+            a = kq_load4(m.sh_up + row * m.ldz, k, m.ff_shared, vec), b = kq_load4(m.sh_up + row * m.ldz, k + 4, m.ff_shared, vec);
+            a.x *= kq_silu(g0.x), a.y *= kq_silu(g0.y), a.z *= kq_silu(g0.z), a.w *= kq_silu(g0.w);
+            b.x *= kq_silu(g1.x), b.y *= kq_silu(g1.y), b.z *= kq_silu(g1.z), b.w *= kq_silu(g1.w);
+        } else {
+            const float *x = act + ((int64_t)row * m.top + s) * ld_act, wt = wts[row * m.top + s];
+            a = kq_load4(x, k, m.ff, true), b = kq_load4(x, k + 4, m.ff, true);
+            a.x *= wt, a.y *= wt, a.z *= wt, a.w *= wt, b.x *= wt, b.y *= wt, b.z *= wt, b.w *= wt;
         }
-    };
-    request(0);
-    float *f0 = reinterpret_cast<float *>(p0), *f1 = reinterpret_cast<float *>(p1);
-    for (int i = tid; i < m.top * fp; i += NT) {
-        const int s = i / fp, j = i % fp;
-        const float v = j < m.ff ? act[((int64_t)row * m.top + s) * ld_act + j] * wts[row * m.top + s] : 0.f;
-        ((j & 4) ? f1 : f0)[(s * per + j / 8) * 4 + (j & 3)] = v;
+#pragma unroll
+        for (int r = 0; r < DOWN_ROWS; r++) acc[r] = kq_dot8(q[r], a, b, acc[r]);
     }
-    for (int j = tid; j < sp; j += NT) {
-        const float v = j < m.ff_shared ? kq_silu(m.sh_gate[row * m.ldz + j]) * m.sh_up[row * m.ldz + j] : 0.f;
-        ((j & 4) ? f1 : f0)[(n_ck + j / 8) * 4 + (j & 3)] = v;
+#pragma unroll
+    for (int r = 0; r < DOWN_ROWS; r++) {
+        const float v = kq_warp_sum(acc[r]);
+        if (lane == 0) part[warp][r] = v;
     }
     __syncthreads();
-    float a = 0.f;
-    for (int c0 = 0;;) {
+    if (tid < DOWN_ROWS && n0 + tid < m.h) {
+        float v = 0.f;
 #pragma unroll
-        for (int u = 0; u < DOWN_U; u++) {
-            const int c = c0 + lane + 32 * u;
-            if (c < all) a = kq_dot8(q[u], p0[c], p1[c], a);
-        }
-        c0 += 32 * DOWN_U;
-        if (c0 >= all || n >= m.h) break;
-        request(c0);
+        for (int i = 0; i < NW; i++) v += part[i][tid];
+        out[row * ldo + n0 + tid] = v;
     }
-    a = kq_warp_sum(a);
-    if (lane == 0 && n < m.h) out[row * ldo + n] = a;
 }
 
 // the first CTAs: a warp per row chooses; the others form the shared GLU, a row and GLU_COLS columns each
@@ -292,11 +294,8 @@ b200_status kq_moe_few_gate_up(const KqMoe &m, const float *x, int64_t ldx, int 
 b200_status kq_moe_few_down(const KqMoe &m, const float *act, int64_t ld_act, const int32_t *ids, const float *wts, int rows, const uint16_t *down,
                             const uint16_t *sh_down, float *out, int64_t ldo, cudaStream_t st) {
     KQ_TRY(check_moe(m, rows));
-    const size_t smem = (size_t)(m.top * kq_pad(m.ff, 8) + kq_pad(m.ff_shared, 8)) * 4;
-    KQ_REQUIRE(smem <= MAX_SMEM, "experts: %d of %d hidden values in one step", m.top, m.ff);
-    static size_t have[16];
-    KQ_TRY(allow_smem(moe_few_down_kernel, smem, have));
-    kq_launch(moe_few_down_kernel, dim3((unsigned)kq_div_up(m.h, DOWN_ROWS), (unsigned)rows), NT, smem, st, m, act, ld_act, ids, wts, down, sh_down, out, ldo);
+    KQ_REQUIRE(ld_act % 4 == 0 && ((uintptr_t)act & 15) == 0, "experts: activations");
+    kq_launch(moe_few_down_kernel, dim3((unsigned)kq_div_up(m.h, DOWN_ROWS), (unsigned)rows), NT, 0, st, m, act, ld_act, ids, wts, down, sh_down, out, ldo);
     KQ_COUNT_LAUNCH();
     KQ_LAUNCH_CHECK();
     return B200_OK;
