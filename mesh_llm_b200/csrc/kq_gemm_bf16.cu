@@ -1,7 +1,7 @@
 // Prefill products with bf16 weights, y[m][n] = sum_k W[n][k] x[m][k]: the tensor-core form (tcgen05.mma
 // kind::f16 on bf16 operands, f32 accumulators in TMEM) and the f32 form on CUDA cores of the 32-bit mode.
 //
-// Tensor cores: a persistent CTA per SM walks tiles of 128 tokens (TMEM lanes) x 256 or 128 weight rows (columns), token
+// Tensor cores: a persistent CTA per SM walks tiles of 128 tokens (TMEM lanes) x 256, 128 or 64 weight rows (columns), token
 // tiles innermost, so that the CTAs at work share the weight rows they read.  K runs in slices of 64 (one
 // 128-byte-swizzled row per operand row); a producer thread brings the slices in by tiled TMA copies through a ring
 // of stages, one thread issues the MMAs into one of two accumulators in TMEM, four warps drain the other one meanwhile,
@@ -379,7 +379,7 @@ b200_status kq_gemm_bf16(const KqDense &c, const uint16_t *a, int64_t lda, int p
     p.parts = parts;
     p.nk = (int)kq_div_up(c.K, BK);
     p.mt = (int)kq_div_up(c.M, TM);
-    // 256-row tiles read less per product, 128-row tiles fill the last wave of CTAs better
+    // larger tiles read less per product, smaller ones fill the last wave of CTAs better
     auto n_tiles = [&](int tn) {
         int t = 0;
         if (c.glu) t = (int)kq_div_up(std::max(c.seg[0].n_rows, c.seg[0].pad_cols), tn / 2);
@@ -388,8 +388,9 @@ b200_status kq_gemm_bf16(const KqDense &c, const uint16_t *a, int64_t lda, int p
         return t;
     };
     const int64_t sms = kq_sm_count();
-    const int64_t w256 = kq_div_up((int64_t)p.mt * n_tiles(256) * c.groups, sms) * 20, w128 = kq_div_up((int64_t)p.mt * n_tiles(128) * c.groups, sms) * 13;
-    const int tn = w256 <= w128 ? 256 : 128;
+    const int64_t w256 = kq_div_up((int64_t)p.mt * n_tiles(256) * c.groups, sms) * 20, w128 = kq_div_up((int64_t)p.mt * n_tiles(128) * c.groups, sms) * 13,
+                  w64 = kq_div_up((int64_t)p.mt * n_tiles(64) * c.groups, sms) * 9;
+    const int tn = w256 <= w128 && w256 <= w64 ? 256 : w128 <= w64 ? 128 : 64;
     p.nt = n_tiles(tn);
     {
         const uint64_t dims[3] = {(uint64_t)lda, (uint64_t)c.M, (uint64_t)parts};
@@ -415,9 +416,11 @@ b200_status kq_gemm_bf16(const KqDense &c, const uint16_t *a, int64_t lda, int p
     if (dev < 0 || dev >= 16 || !attr[dev]) {
         KQ_CUDA(cudaFuncSetAttribute(gemm_bf16_kernel<256>, cudaFuncAttributeMaxDynamicSharedMemorySize, Tile<256>::SMEM_TOTAL));
         KQ_CUDA(cudaFuncSetAttribute(gemm_bf16_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, Tile<128>::SMEM_TOTAL));
+        KQ_CUDA(cudaFuncSetAttribute(gemm_bf16_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, Tile<64>::SMEM_TOTAL));
         if (dev >= 0 && dev < 16) attr[dev] = true;
     }
     if (tn == 256) kq_launch(gemm_bf16_kernel<256>, grid, NTHREADS, Tile<256>::SMEM_TOTAL, st, p);
+    else if (tn == 64) kq_launch(gemm_bf16_kernel<64>, grid, NTHREADS, Tile<64>::SMEM_TOTAL, st, p);
     else kq_launch(gemm_bf16_kernel<128>, grid, NTHREADS, Tile<128>::SMEM_TOTAL, st, p);
     KQ_COUNT_LAUNCH();
     KQ_LAUNCH_CHECK();
