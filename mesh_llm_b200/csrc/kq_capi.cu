@@ -37,7 +37,7 @@ int kq_sm_count() {
 // one code per bounded wait that gave up since the last call, 0 when none did
 int kq_device_wait_errors() {
     return kq_stream_error_fetch() | (kq_gemm_error_fetch() << 4) | (kq_attn_tc_error_fetch() << 8) | (kq_gemm_bf16_error_fetch() << 12) |
-           (kq_prompt_attn_error_fetch() << 16) | (kq_state_error_fetch() << 20);
+           (kq_prompt_attn_error_fetch() << 16) | ((kq_state_error_fetch() | kq_state_chunk_error_fetch()) << 20);
 }
 
 extern "C" {

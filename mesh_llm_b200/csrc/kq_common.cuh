@@ -319,6 +319,7 @@ int kq_attn_tc_error_fetch();
 int kq_gemm_bf16_error_fetch();
 int kq_prompt_attn_error_fetch();
 int kq_state_error_fetch();
+int kq_state_chunk_error_fetch();
 int kq_device_wait_errors(); // all of the above in one code
 b200_status kq_launch_gemm(uint32_t type, const uint8_t *W, const int8_t *q, const float *d,
                            const int16_t *bs, int64_t M, int64_t N, int64_t K, float *y,

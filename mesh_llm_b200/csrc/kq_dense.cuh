@@ -76,10 +76,9 @@ struct KqNormPrep {
 };
 
 #ifdef __CUDACC__
-__device__ __forceinline__ float kq_gelu_tanh(float z) {
-    return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
-}
-__device__ __forceinline__ float kq_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+__device__ __forceinline__ float kq_sigmoid(float z) { return __fdividef(1.0f, 1.0f + expf(-z)); }
+// 0.5 z (1 + tanh(u)) = z sigmoid(2 u)
+__device__ __forceinline__ float kq_gelu_tanh(float z) { return z * kq_sigmoid(1.5957691216057308f * (z + 0.044715f * z * z * z)); }
 __device__ __forceinline__ float kq_clamped_glu(float g, float u, float limit, float alpha) {
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
@@ -284,12 +283,12 @@ struct KqStateIn {
     const float *q, *k, *v, *b, *z; // z: decay projection [rows][ldz], bias not added yet; b: write strengths before the sigmoid
     int64_t ld, ldz;
 };
-// Records of blocks of four tokens (kq_state_ops.cu): for every sequence kq_state_blocks(T) times kq_state_rec_floats and
-// kq_state_val_floats floats, 16-byte aligned
+// Records of blocks of tokens: for every sequence kq_state_groups(T) times kq_state_rec_floats and kq_state_val_floats floats,
+// 16-byte aligned; a launch of kq_state_tokens or kq_state_chunks writes them, the walk that goes with it reads them
 struct KqStateTok {
     float *rec, *val;
 };
-static inline int64_t kq_state_blocks(int64_t T) { return (T + 3) / 4; }
+static inline int64_t kq_state_groups(int64_t T) { return (T + 15) / 16; }
 int64_t kq_state_rec_floats(const KqMatState &m);
 int64_t kq_state_val_floats(const KqMatState &m);
 b200_status kq_state_tokens(const KqMatState &m, const KqStateIn &in, const KqStateTok &t, int n_seq, int T, const int32_t *pos0_dev, int pos0,
@@ -297,6 +296,15 @@ b200_status kq_state_tokens(const KqMatState &m, const KqStateIn &in, const KqSt
 // the walk over T positions: o [rows][ldo] f32; also moves the convolution's ring forward (in: its inputs)
 b200_status kq_state_scan(const KqMatState &m, const KqStateIn &in, const KqStateTok &t, int n_seq, int T, const int32_t *pos0_dev, int pos0,
                           float *o, int64_t ldo, cudaStream_t st);
+// ---- kq_state_chunk.cu: the same in chunks of 16 tokens, the products with the state on tensor cores (f32 operands in two parts),
+// for heads of up to 128 key dimensions
+bool kq_state_chunks_fit(const KqMatState &m);
+int64_t kq_state_chunk_rec_floats(const KqMatState &m); // per head and chunk
+b200_status kq_state_chunks(const KqMatState &m, const KqStateIn &in, const KqStateTok &t, int n_seq, int T, const int32_t *pos0_dev, int pos0,
+                            cudaStream_t st);
+b200_status kq_state_chunk_walk(const KqMatState &m, const KqStateIn &in, const KqStateTok &t, int n_seq, int T, const int32_t *pos0_dev, int pos0,
+                                float *o, int64_t ldo, cudaStream_t st);
+// ---- kq_state_ops.cu
 // every head's o over its rms times norm_w [vdim] times sigmoid(gate); f32 or bf16 rows (padded with zeros)
 b200_status kq_head_norm_gate(const float *o, int64_t ldo, const float *gate, int64_t ldg, const float *norm_w, float eps, int64_t rows, int heads,
                               int vdim, float *out32, int64_t ld32, uint16_t *out16, int64_t ld16, cudaStream_t st);

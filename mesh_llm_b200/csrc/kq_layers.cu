@@ -513,8 +513,13 @@ struct Pass {
                 OTHER_(kq_gemm_bf16(g, g16, kq_bf16_ld(c.gate_rank), 1, s));
             }
         }
-        OTHER_(kq_state_tokens(m, si, k->state_tok, n_seq, T, pos_dev, pos0, s));
-        OTHER_(kq_state_scan(m, si, k->state_tok, n_seq, T, pos_dev, pos0, o, ldv, s));
+        if (tc && kq_state_chunks_fit(m)) {
+            OTHER_(kq_state_chunks(m, si, k->state_tok, n_seq, T, pos_dev, pos0, s));
+            OTHER_(kq_state_chunk_walk(m, si, k->state_tok, n_seq, T, pos_dev, pos0, o, ldv, s));
+        } else {
+            OTHER_(kq_state_tokens(m, si, k->state_tok, n_seq, T, pos_dev, pos0, s));
+            OTHER_(kq_state_scan(m, si, k->state_tok, n_seq, T, pos_dev, pos0, o, ldv, s));
+        }
         if (!m.delta) return close_normed(L.wo, K, o, ldv, L.o_norm, gate, ldp, L.post1);
         OTHER_(kq_head_norm_gate(o, ldv, k->f[5], ldv, L.o_norm, st->c.rms_eps, rows, m.heads, m.vdim, tc ? nullptr : z, ldv, tc ? k->z16 : nullptr, ld16, s));
         return close(L.wo, K, z, ldv, k->z16, L.post1);
@@ -1081,7 +1086,7 @@ b200_status b200_stage_create_layers(const b200_stage_config *cfg, const b200_st
     if (ffmax) A(&k->act32, (size_t)((f32 ? R : std::min<int64_t>(R, SMALL_ROWS)) * kq_f32_ld(ffmax) * 4));
     if (ffmax && wide) A(&k->act16, (size_t)(R * kq_bf16_ld(ffmax) * 2));
     if (state_rec) {
-        const int64_t blocks = R / 4 + std::min<int64_t>(R, c.n_seq) + 1; // of all sequences of a call
+        const int64_t blocks = R / 16 + std::min<int64_t>(R, c.n_seq) + 1; // groups of 16 positions of all sequences of a call
         A(&k->state_tok.rec, (size_t)(blocks * state_rec * 4));
         A(&k->state_tok.val, (size_t)(blocks * state_val * 4));
     }

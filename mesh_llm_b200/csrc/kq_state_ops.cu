@@ -11,11 +11,11 @@
 // registers, so that eight products with the state wait for one reduction and a record is read from shared memory once
 // per pair of columns.  A thread holds some key dimensions of two columns (value dimensions).  A warp of its own brings the
 // records by bulk copies into a ring, the others walk through it without waiting for one another; every wait is bounded.
-// The fixed decay is the same with u = v and scalar products of decays.
+// The fixed decay is the same with u = v and scalar products of decays.  (kq_state_chunk.cu has the form on tensor cores.)
 // A decode step is one launch: a CTA per head convolves, norms, works out the low-rank decays and gates, updates the
 // state and norms and gates the head's output.
 #include "kq_gemv_grouped.cuh"
-#include "kq_tc.cuh"
+#include "kq_state.cuh"
 
 #include <algorithm>
 
@@ -28,42 +28,6 @@ __device__ __forceinline__ float sum8(float v) { // over the eight lanes of a co
     v += __shfl_xor_sync(0xffffffffu, v, 2);
     return v + __shfl_xor_sync(0xffffffffu, v, 1);
 }
-// N values of every lane summed over groups of L lanes (powers of two).  Each exchange halves the values a lane still carries:
-// with p the lane's place in its group, v[i] ends as value p N / L + i (N >= L), v[0] as value p / (L / N) (N < L).
-template <int N, int L>
-__device__ __forceinline__ void spread_sum(float (&v)[N], int lane) {
-    int n = N;
-#pragma unroll
-    for (int m = L / 2; m >= 1; m /= 2) {
-        if (n > 1) {
-            n /= 2;
-            const bool up = lane & m;
-#pragma unroll
-            for (int i = 0; i < N / 2; i++)
-                if (i < n) {
-                    const float send = up ? v[i] : v[i + n], keep = up ? v[i + n] : v[i];
-                    v[i] = keep + __shfl_xor_sync(0xffffffffu, send, m);
-                }
-        } else {
-            v[0] += __shfl_xor_sync(0xffffffffu, v[0], m);
-        }
-    }
-}
-
-// the convolution's input at position pos0 + t: this call's rows, the ring, or zero before the start
-struct ConvIn {
-    const float *x; // column of row 0 of the sequence
-    int64_t ld;
-    const float *ring; // column of slot 0
-    int64_t channels;
-    int taps, pos0;
-    __device__ __forceinline__ float at(int t) const {
-        if (t >= 0) return x[t * ld];
-        const int pos = pos0 + t;
-        return pos >= 0 ? ring[(int64_t)(pos % taps) * channels] : 0.f;
-    }
-};
-
 // ---- records of blocks of tokens -----------------------------------------------------------------------
 constexpr int BT = 4, TOK_NT = 128, TOK_NW = TOK_NT / 32, RUN = 4; // tokens per block, blocks a warp walks
 constexpr int N_SCALAR = 32;                                       // beta (4), A (6, from 4), B (four rows of four, from 12)
@@ -84,7 +48,7 @@ struct TokParams {
 template <int C>
 struct ConvBlock {
     float in[C][BT + 3];
-    __device__ __forceinline__ ConvIn input(const TokParams &p, const float *x, int64_t channel0, int64_t seq, int pos0, int d) const {
+    __device__ __forceinline__ KqConvIn input(const TokParams &p, const float *x, int64_t channel0, int64_t seq, int pos0, int d) const {
         const int64_t channels = kq_state_channels(p.m);
         return {x + seq * p.T * p.in.ld + d, p.in.ld, p.m.taps ? p.m.conv + seq * p.m.taps * channels + channel0 + d : nullptr, channels, p.m.taps, pos0};
     }
@@ -99,7 +63,7 @@ struct ConvBlock {
         } else {
 #pragma unroll
             for (int c = 0; c < C; c++) {
-                const ConvIn ci = input(p, x, channel0, seq, pos0, lane + 32 * c);
+                const KqConvIn ci = input(p, x, channel0, seq, pos0, lane + 32 * c);
 #pragma unroll
                 for (int k = 0; k < BT + 3; k++) in[c][k] = lane + 32 * c < n && t0 - 3 + k < p.T ? ci.at(t0 - 3 + k) : 0.f;
             }
@@ -116,7 +80,7 @@ struct ConvBlock {
 #pragma unroll
                 for (int j = 0; j < BT; j++) out[j][c] = fmaf(cw.w, in[c][j + 3], fmaf(cw.z, in[c][j + 2], fmaf(cw.y, in[c][j + 1], cw.x * in[c][j])));
             } else {
-                const ConvIn ci = input(p, x, channel0, seq, pos0, d);
+                const KqConvIn ci = input(p, x, channel0, seq, pos0, d);
 #pragma unroll
                 for (int j = 0; j < BT; j++) {
                     float s = 0.f;
@@ -187,7 +151,7 @@ __global__ void __launch_bounds__(TOK_NT, C > 4 ? 2 : DELTA ? 3 : 6) state_token
 #pragma unroll
                 for (int c = 0; c < C; c++) ss[j] = fmaf(q[j][c], q[j][c], ss[j]), ss[BT + j] = fmaf(k[j][c], k[j][c], ss[BT + j]);
             }
-            spread_sum<2 * BT, 32>(ss, lane); // lane holds sum lane / 4
+            kq_spread_sum<2 * BT, 32>(ss, lane); // lane holds sum lane / 4
             const float sc = 1.0f / sqrtf(ss[0] + 1e-6f);
 #pragma unroll
             for (int j = 0; j < BT; j++) {
@@ -231,7 +195,7 @@ __global__ void __launch_bounds__(TOK_NT, C > 4 ? 2 : DELTA ? 3 : 6) state_token
             o[4 * DP] = p14, o[5 * DP] = p24, o[6 * DP] = p34, o[7 * DP] = k4;
             if (DELTA) o[8 * DP] = G4;
         }
-        spread_sum<16, 32>(dot, lane); // lane holds sum lane / 2
+        kq_spread_sum<16, 32>(dot, lane); // lane holds sum lane / 2
         float *sc = rec + REC - N_SCALAR;
         const int i = lane / 2, bi = i - 6, row = bi < 1 ? 0 : bi < 3 ? 1 : bi < 6 ? 2 : 3;
         if ((lane & 1) == 0) sc[i < 6 ? 4 + i : 12 + 4 * row + bi - row * (row + 1) / 2] = dot[0];
@@ -277,18 +241,6 @@ __device__ __forceinline__ float add2(uint64_t a) {
     return x + y;
 }
 
-// the last `taps` inputs of every channel into the ring, shared out over all CTAs of the grid
-__device__ __forceinline__ void move_ring(const KqMatState &m, const KqStateIn &in, int64_t n_seq, int T, int pos0, int64_t id, int64_t n_threads) {
-    const int64_t channels = kq_state_channels(m), nq = (int64_t)m.kv_heads * m.dim;
-    const int keep = min(T, m.taps);
-    for (int64_t i = id; i < n_seq * keep * channels; i += n_threads) {
-        const int64_t c = i % channels, rest = i / channels, seq = rest / keep;
-        const int t = T - keep + (int)(rest % keep);
-        const float *x = c < nq ? in.q + c : c < 2 * nq ? in.k + (c - nq) : in.v + (c - 2 * nq);
-        m.conv[(seq * m.taps + (pos0 + t) % m.taps) * channels + c] = x[(seq * T + t) * in.ld];
-    }
-}
-
 // grid (blocks of columns, heads, sequences).  LPC lanes share NC columns, each with R groups of four key dimensions, so that under
 // the delta rule the 8 NC sums of a block are one per lane.  The last warp brings the records.
 template <int LPC, int R, bool DELTA>
@@ -306,7 +258,7 @@ __global__ void __launch_bounds__((MAX_WARPS + 1) * 32) state_scan_kernel(const 
     const int64_t seq = blockIdx.z;
     const int pos0 = p.pos0_dev ? *p.pos0_dev : p.pos0;
     if (m.taps)
-        move_ring(m, p.in, gridDim.z, p.T, pos0, ((seq * gridDim.y + h) * gridDim.x + blockIdx.x) * blockDim.x + tid,
+        kq_move_ring(m, p.in, gridDim.z, p.T, pos0, ((seq * gridDim.y + h) * gridDim.x + blockIdx.x) * blockDim.x + tid,
                   (int64_t)gridDim.x * gridDim.y * gridDim.z * blockDim.x);
     const int tile_floats = scan_tile_floats(DP, DELTA, cols), tiles = (p.blocks + TB - 1) / TB;
     if (tid == 0) {
@@ -408,7 +360,7 @@ __global__ void __launch_bounds__((MAX_WARPS + 1) * 32) state_scan_kernel(const 
                 const float4 vt = *reinterpret_cast<const float4 *>(vals + c * BT), B = *reinterpret_cast<const float4 *>(sc + 12 + 4 * j);
                 float4 u = vt, be, A0, A1;
                 if (DELTA) be = *reinterpret_cast<const float4 *>(sc), A0 = *reinterpret_cast<const float4 *>(sc + 4), A1 = *reinterpret_cast<const float4 *>(sc + 8);
-                spread_sum<NV, LPC>(val, lane);
+                kq_spread_sum<NV, LPC>(val, lane);
                 if (DELTA) { // every lane solves for its column
                     float dk[BT];
 #pragma unroll
@@ -580,7 +532,7 @@ __device__ __forceinline__ void conv_step(const KqMatState &m, const float *x, c
         float s = x[d];
         if (m.taps) {
             s = 0.f;
-            const ConvIn ci = {x + d, 0, ring + d, channels, m.taps, pos};
+            const KqConvIn ci = {x + d, 0, ring + d, channels, m.taps, pos};
             for (int k = 0; k < m.taps; k++) s = fmaf(w[(int64_t)d * m.taps + k], ci.at(k - (m.taps - 1)), s);
             if (owns) ring[(int64_t)(pos % m.taps) * channels + d] = x[d];
         }
@@ -720,14 +672,6 @@ __global__ void __launch_bounds__(256) rank_operands_kernel(const float *a, int 
     for (int64_t i = threadIdx.x; i < ldg; i += blockDim.x) g16[r * ldg + i] = i < m ? kq_f2bf(g[r * ld + i]) : 0;
 }
 
-b200_status check_state(const KqMatState &m, int n_seq, int T) {
-    KQ_REQUIRE(m.heads >= 1 && m.kv_heads >= 1 && m.heads % m.kv_heads == 0 && m.dim >= 1 && m.vdim >= 1 && m.taps >= 0 && n_seq >= 1 && T >= 1 &&
-                   m.s && (m.taps == 0 || m.conv),
-               "matrix state: bad shape");
-    KQ_REQUIRE(m.dim <= KQ_STATE_MAX_DIM && m.heads <= 65535 && n_seq <= 65535, "matrix state: %d heads of %d key dimensions", m.heads, m.dim);
-    return B200_OK;
-}
-
 template <int LPC, int R, bool DELTA>
 b200_status launch_scan(const ScanParams &p, int n_seq, cudaStream_t st) {
     constexpr int DP = LPC * R * 4, per_warp = 32 / LPC * (LPC / (2 * BT));
@@ -793,12 +737,14 @@ int kq_state_error_fetch() {
     return v;
 }
 
-int64_t kq_state_rec_floats(const KqMatState &m) { return (int64_t)m.heads * rec_floats(kq_state_ld(m.dim), m.delta != 0); }
-int64_t kq_state_val_floats(const KqMatState &m) { return (int64_t)m.heads * m.vdim * BT; }
+int64_t kq_state_rec_floats(const KqMatState &m) {
+    return (int64_t)m.heads * std::max<int64_t>(16 / BT * rec_floats(kq_state_ld(m.dim), m.delta != 0), kq_state_chunk_rec_floats(m));
+}
+int64_t kq_state_val_floats(const KqMatState &m) { return (int64_t)m.heads * m.vdim * 32; }
 
 b200_status kq_state_tokens(const KqMatState &m, const KqStateIn &in, const KqStateTok &t, int n_seq, int T, const int32_t *pos0_dev, int pos0,
                             cudaStream_t st) {
-    KQ_TRY(check_state(m, n_seq, T));
+    KQ_TRY(kq_check_state(m, n_seq, T));
     KQ_REQUIRE((((uintptr_t)t.rec | (uintptr_t)t.val) & 15) == 0, "matrix state: records");
     TokParams p;
     p.m = m, p.in = in, p.rec = t.rec, p.val = t.val, p.T = T, p.pos0 = pos0, p.pos0_dev = pos0_dev;
@@ -808,7 +754,7 @@ b200_status kq_state_tokens(const KqMatState &m, const KqStateIn &in, const KqSt
 
 b200_status kq_state_scan(const KqMatState &m, const KqStateIn &in, const KqStateTok &t, int n_seq, int T, const int32_t *pos0_dev, int pos0,
                           float *o, int64_t ldo, cudaStream_t st) {
-    KQ_TRY(check_state(m, n_seq, T));
+    KQ_TRY(kq_check_state(m, n_seq, T));
     ScanParams p;
     p.m = m, p.in = in, p.rec = t.rec, p.val = t.val, p.T = T, p.pos0 = pos0, p.pos0_dev = pos0_dev, p.blocks = (int)kq_div_up(T, BT), p.o = o, p.ldo = ldo;
     BY_DIM(launch_scan, TWO(8, 1), TWO(16, 1), TWO(16, 2), TWO(16, 4), p, n_seq, st)
@@ -828,7 +774,7 @@ b200_status kq_head_norm_gate(const float *o, int64_t ldo, const float *gate, in
 
 b200_status kq_state_step(const KqMatState &m, const KqStateIn &in, const KqStateStep &x, int n_seq, const int32_t *pos_dev, int pos, float *z,
                           int64_t ldz, cudaStream_t st) {
-    KQ_TRY(check_state(m, n_seq, 1));
+    KQ_TRY(kq_check_state(m, n_seq, 1));
     StepParams p;
     p.m = m, p.in = in, p.x = x, p.pos_dev = pos_dev, p.pos = pos, p.z = z, p.ldz = ldz;
     const size_t smem = (size_t)(3 * kq_state_ld(m.dim) + 3 * kq_pad(m.vdim, 4) + kq_pad(x.a_rank, 8) + kq_pad(x.g_rank, 8)) * 4;
