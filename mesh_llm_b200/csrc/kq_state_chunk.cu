@@ -378,6 +378,16 @@ __global__ void __launch_bounds__((MAX_GROUPS * SPLIT + 1) * 32) state_chunk_wal
             float2 uv[2][2];
 #pragma unroll
             for (int n = 0; n < 2; n++) uv[n][0] = *reinterpret_cast<const float2 *>(val + 8 * n), uv[n][1] = *reinterpret_cast<const float2 *>(val + 8 * 2 * CT + 8 * n);
+            // what does not wait for the other quarters: G S, and the parts of P k
+            const float dc = c == p.chunks - 1 ? d_last : d_full;
+            uint32_t kh[TILES][4], kl[TILES][4];
+#pragma unroll
+            for (int i = 0; i < TILES; i++) {
+                const float2 gg = DELTA ? *reinterpret_cast<const float2 *>(gc + 8 * i + 2 * t) : make_float2(dc, dc);
+                const float4 x = fk[i * 32];
+                s[i][0] *= gg.x, s[i][1] *= gg.y, s[i][2] *= gg.x, s[i][3] *= gg.y;
+                split2(x.x, kh[i][0], kl[i][0]), split2(x.y, kh[i][1], kl[i][1]), split2(x.z, kh[i][2], kl[i][2]), split2(x.w, kh[i][3], kl[i][3]);
+            }
             asm volatile("bar.sync %0, %1;" ::"r"(1 + group), "n"(SPLIT * 32) : "memory");
             // ---- u = U - S^T W of tokens 8 n + 2 t and the next, as the first operand of the product over the tokens
             uint32_t uh[2][4], ul[2][4];
@@ -394,6 +404,16 @@ __global__ void __launch_bounds__((MAX_GROUPS * SPLIT + 1) * 32) state_chunk_wal
                 // columns past the call's share hold anything: they stay apart and are not written
                 split2(u[0], uh[n][0], ul[n][0]), split2(u[2], uh[n][1], ul[n][1]), split2(u[1], uh[n][2], ul[n][2]), split2(u[3], uh[n][3], ul[n][3]);
             }
+            // ---- S <- G S + (P k) u^T, tiles side by side
+#pragma unroll
+            for (int n = 0; n < 2; n++) {
+#pragma unroll
+                for (int i = 0; i < TILES; i++) mma8(s[i], uh[n], kl[i][2 * n], kl[i][2 * n + 1]);
+#pragma unroll
+                for (int i = 0; i < TILES; i++) mma8(s[i], ul[n], kh[i][2 * n], kh[i][2 * n + 1]);
+#pragma unroll
+                for (int i = 0; i < TILES; i++) mma8(s[i], uh[n], kh[i][2 * n], kh[i][2 * n + 1]);
+            }
             { // outputs: a warp takes tile quarter / 2, and of it the lower or upper eight columns
                 const int n = quarter / 2, up = quarter % 2, t0 = c * CT + 8 * n + 2 * t;
                 float2 o = *reinterpret_cast<const float2 *>(val + up * 8 * 2 * CT + CT + 8 * n);
@@ -407,19 +427,6 @@ __global__ void __launch_bounds__((MAX_GROUPS * SPLIT + 1) * 32) state_chunk_wal
                     if (t0 < p.T) d[0] = o.x;
                     if (t0 + 1 < p.T) d[p.ldo] = o.y;
                 }
-            }
-            // ---- S <- G S + (P k) u^T
-            const float dc = c == p.chunks - 1 ? d_last : d_full;
-#pragma unroll
-            for (int i = 0; i < TILES; i++) {
-                const float2 gg = DELTA ? *reinterpret_cast<const float2 *>(gc + 8 * i + 2 * t) : make_float2(dc, dc);
-                s[i][0] *= gg.x, s[i][1] *= gg.y, s[i][2] *= gg.x, s[i][3] *= gg.y;
-                const float4 x = fk[i * 32];
-                uint32_t h0, h1, l0, l1;
-                split2(x.x, h0, l0), split2(x.y, h1, l1);
-                mma8(s[i], uh[0], l0, l1), mma8(s[i], ul[0], h0, h1), mma8(s[i], uh[0], h0, h1);
-                split2(x.z, h0, l0), split2(x.w, h1, l1);
-                mma8(s[i], uh[1], l0, l1), mma8(s[i], ul[1], h0, h1), mma8(s[i], uh[1], h0, h1);
             }
             __syncwarp(); // this warp is done with the stage
             if (lane == 0) asm volatile("mbarrier.arrive.shared::cta.b64 _, [%0];" ::"r"(smem_u32(&empty[st])) : "memory");
