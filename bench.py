@@ -308,7 +308,7 @@ LOMODRA_SIZES = {
     "lomodra-3072": dict(width=3072, heads=24, kv=6, experts=64, top=6, ff=1024, shared=2048, side=256, n_layer=24),
     "lomodra-4096": dict(width=4096, heads=32, kv=8, experts=32, top=4, ff=1536, shared=4096, side=256, n_layer=18),
 }
-LOMODRA_DIM, LOMODRA_RANK, LOMODRA_CHUNK = 128, 128, 2048
+LOMODRA_DIM, LOMODRA_RANK, LOMODRA_CHUNK = 128, 128, 8192
 ARCH_VOCAB, ARCH_WINDOW, ARCH_RANK, ARCH_DIM, ARCH_ROT, ARCH_VDIM = 128256, 2048, 512, 128, 64, 128
 
 

@@ -5,9 +5,9 @@
 // dimensions two by two, so that a warp reads whole key rows; a warp takes four keys at a time, their scores are reduced
 // across the warp together.  Scores of a tile of keys sit in shared memory, the softmax is online over tiles, all in f32.
 // The ranges' results (maximum, sum, weighted values) are merged by the last CTA of a row to arrive; ranges without keys
-// take no part.  In a decode step the
-// same launch norms the queries and the new key and stores the new row: only the CTA whose range ends with the new
-// position reads that row, and it is the one that stores it.
+// take no part.  In a decode step the same launch norms the queries and the new key and stores the new row: only the CTA
+// whose range ends with the new position reads that row, and it is the one that stores it.  The ranges' rows are prefetched
+// into L2 ahead of the dependency wait: they are of earlier steps, and loads see the latest values wherever they lie.
 #include "kq_dense.cuh"
 
 #include <algorithm>
@@ -15,7 +15,7 @@
 namespace {
 
 constexpr int NT = 128, NW = NT / 32, KT = 128; // threads, warps, keys per tile
-constexpr int MAX_SPLITS = KT, MIN_RANGE = 32;  // ranges of a row's keys, keys of a range
+constexpr int MAX_SPLITS = KT, MIN_RANGE = 64;  // ranges of a row's keys, keys of a range
 
 struct Params {
     KqGqa a;
@@ -78,7 +78,7 @@ __global__ void __launch_bounds__(NT) gqa_store_kernel(const __grid_constant__ K
 // N: pairs of dimensions per lane (dims up to 64 N); RT: query heads per CTA
 template <typename CT, int N, int RT, bool FUSED>
 __global__ void __launch_bounds__(NT) gqa_attn_kernel(const __grid_constant__ Params p) {
-    KQ_PDL_ENTER();
+    KQ_PDL_TRIGGER();
     const KqGqa &a = p.a;
     __shared__ __align__(16) float s_p[RT][KT];
     __shared__ __align__(16) float2 s_o[NW][RT][N * 32];
@@ -88,12 +88,28 @@ __global__ void __launch_bounds__(NT) gqa_attn_kernel(const __grid_constant__ Pa
     const int split = blockIdx.x, S = p.splits, rep = a.n_head / a.kv_heads, gpk = (rep + RT - 1) / RT;
     const int g = blockIdx.y / gpk, h0 = g * rep + blockIdx.y % gpk * RT, nh = min(RT, (g + 1) * rep - h0);
     const int64_t r = blockIdx.z, seq = r / p.T;
+    const int ldk = (a.dim + 63) / 64 * 64, ldv = (a.vdim + 63) / 64 * 64;
+    const CT *kc = (const CT *)a.k + (seq * a.cap * a.kv_heads + g) * (int64_t)ldk, *vc = (const CT *)a.v + (seq * a.cap * a.kv_heads + g) * (int64_t)ldv;
+    const int64_t rk = (int64_t)a.kv_heads * ldk, rv = (int64_t)a.kv_heads * ldv;
+    if (S > 1) { // the position may still be the one before
+        int pos = p.pos0;
+        if (p.pos0_dev) pos = __ldcg(p.pos0_dev);
+        pos = max(0, pos + (int)(r % p.T));
+        const int lo = kq_first_key(pos, a.window, a.chunk), n = pos - lo + 1, per = max((n + S - 1) / S, MIN_RANGE);
+        const int j0 = min(n, split * per), j1 = min(n, j0 + per), k_lines = (ldk * (int)sizeof(CT) + 127) / 128, v_lines = (ldv * (int)sizeof(CT) + 127) / 128;
+        for (int i = tid; i < (j1 - j0) * (k_lines + v_lines); i += NT) {
+            const int j = i / (k_lines + v_lines), l = i % (k_lines + v_lines);
+            const int64_t row = (lo + j0 + j) % a.cap;
+            const uint8_t *line = l < k_lines ? (const uint8_t *)(kc + row * rk) + l * 128 : (const uint8_t *)(vc + row * rv) + (l - k_lines) * 128;
+            asm volatile("prefetch.global.L2 [%0];" ::"l"(line));
+        }
+    }
+    KQ_PDL_WAIT();
     const int pos = (p.pos0_dev ? *p.pos0_dev : p.pos0) + (int)(r % p.T);
     const int lo = kq_first_key(pos, a.window, a.chunk), n = pos - lo + 1, per = max((n + S - 1) / S, MIN_RANGE);
     const int j0 = min(n, split * per), j1 = min(n, j0 + per); // keys lo + j0 .. lo + j1 - 1
     const int live = (n + per - 1) / per;                      // ranges that have any
     if (j0 >= j1) return;
-    const int ldk = (a.dim + 63) / 64 * 64, ldv = (a.vdim + 63) / 64 * 64;
 
     {
         if (FUSED && a.own_kv && j1 == n && warp == NW - 1) // head groups of one key head store the same values
@@ -114,21 +130,25 @@ __global__ void __launch_bounds__(NT) gqa_attn_kernel(const __grid_constant__ Pa
 #pragma unroll
         for (int i = 0; i < N; i++) o[t][i] = make_float2(0.f, 0.f);
     }
-    const CT *kc = (const CT *)a.k + (seq * a.cap * a.kv_heads + g) * (int64_t)ldk, *vc = (const CT *)a.v + (seq * a.cap * a.kv_heads + g) * (int64_t)ldv;
-    const int64_t rk = (int64_t)a.kv_heads * ldk, rv = (int64_t)a.kv_heads * ldv;
+    const int row0 = (lo + j0) % a.cap; // of the first key; a range wraps at most once
+    auto row_of = [&](int j) {
+        const int x = row0 + j - j0;
+        return (int64_t)(x >= a.cap ? x - a.cap : x);
+    };
     for (int t0 = j0; t0 < j1; t0 += KT) {
-        const int nk = min(KT, j1 - t0), base = lo + t0;
+        const int nk = min(KT, j1 - t0);
 #pragma unroll
         for (int t = 0; t < RT; t++)
 #pragma unroll
             for (int i = 0; i < N; i++) q[t][i] = *reinterpret_cast<const float2 *>(&s_q[t][2 * lane + 64 * i]);
+#pragma unroll 2
         for (int j = warp * 4; j < nk; j += NW * 4) {
             float2 kv[4][N];
 #pragma unroll
             for (int e = 0; e < 4; e++)
 #pragma unroll
                 for (int i = 0; i < N; i++)
-                    kv[e][i] = 64 * i < ldk ? ld2(kc + (int64_t)((base + min(j + e, nk - 1)) % a.cap) * rk + 2 * lane + 64 * i) : make_float2(0.f, 0.f);
+                    kv[e][i] = 64 * i < ldk ? ld2(kc + row_of(t0 + min(j + e, nk - 1)) * rk + 2 * lane + 64 * i) : make_float2(0.f, 0.f);
 #pragma unroll
             for (int t = 0; t < RT; t++) {
                 float s[4];
@@ -182,13 +202,14 @@ __global__ void __launch_bounds__(NT) gqa_attn_kernel(const __grid_constant__ Pa
 #pragma unroll
             for (int i = 0; i < N; i++) o[t][i].x *= al[t], o[t][i].y *= al[t];
         }
+#pragma unroll 2
         for (int j = warp * 4; j < nk; j += NW * 4) {
             float2 vv[4][N];
 #pragma unroll
             for (int e = 0; e < 4; e++)
 #pragma unroll
                 for (int i = 0; i < N; i++)
-                    vv[e][i] = 64 * i < ldv ? ld2(vc + (int64_t)((base + min(j + e, nk - 1)) % a.cap) * rv + 2 * lane + 64 * i) : make_float2(0.f, 0.f);
+                    vv[e][i] = 64 * i < ldv ? ld2(vc + row_of(t0 + min(j + e, nk - 1)) * rv + 2 * lane + 64 * i) : make_float2(0.f, 0.f);
 #pragma unroll
             for (int t = 0; t < RT; t++) {
                 const float4 w = *reinterpret_cast<const float4 *>(&s_p[t][j]); // zero past the tile's keys
