@@ -4,7 +4,7 @@
  * This is a plain-C restatement of the arithmetic that mesh-llm's serving stages execute
  * inside llama.cpp/ggml (the dependency pinned at third_party/llama.cpp/upstream.txt:1,
  * 45155597aa23243c5f6d10064bd9bca3eaddee16, which is NOT vendored in the reference tree).
- * It is the checker for the CUDA path and the timed CPU baseline; nothing in the product
+ * It is what the CUDA path is compared with and the timed CPU baseline; nothing in the product
  * library links, imports or calls it.
  *
  * PARITY STATUS: the block formats (Q4_K / Q6_K decode) are pinned against gguf-py's
